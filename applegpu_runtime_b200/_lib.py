@@ -197,6 +197,17 @@ EXT_SYMBOLS = {
     "applegpu_gpt2_decoder_uses_graph": (i32, [u64]),
     "applegpu_gpt2_decoder_set_engine": (i32, [u64, i32]),
     "applegpu_gpt2_decoder_destroy": (None, [u64]),
+    "applegpu_seq_create": (u64, [vp, vp, u64p, u32, u32, u32]),
+    "applegpu_seq_forward": (i32, [u64, u32, u32, vp, u32, vp, u32, vp, vp, vp]),
+    "applegpu_seq_decode": (i32, [u64, u32, u32, u32, vp, cbool]),
+    "applegpu_seq_reset": (i32, [u64, u32, u32]),
+    "applegpu_seq_length": (i32, [u64, u32]),
+    "applegpu_seq_info": (i32, [u64, i32]),
+    "applegpu_seq_destroy": (None, [u64]),
+    "applegpu_ffi_rms_norm": (u64, [u64, u64, f32, i8]),
+    "applegpu_ffi_clamped_glu": (u64, [u64, f32]),
+    "applegpu_ffi_mlstm": (u64, [u64, u64, u64, u64, u64, u32, u32, u32, f32, f32, i32]),
+    "applegpu_ffi_latent_attention": (u64, [u64, u64, u64, u64, u64, u64, u32, u32, u32, u32, u32, u32, f32, f32, i32]),
     "applegpu_test_wait_runs_out": (i32, [i32, u32]),
 }
 

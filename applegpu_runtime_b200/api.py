@@ -435,6 +435,30 @@ def matmul_int8(x, q, scales):
     return _wrap(_L().applegpu_ffi_matmul_int8(x.id, q.id, scales.id), x)
 
 
+def rms_norm(x, weight, eps=1e-5, dtype="bfloat16"):
+    """x / sqrt(mean(x^2) + eps) * weight over the last dimension of a float32 tensor, stored as `dtype`. Evaluated at once, like the
+    other mechanisms of the sequence models below."""
+    return GpuTensor(_L().applegpu_ffi_rms_norm(x.id, weight.id, float(eps), _DTYPE_CODES[_canon_dtype(dtype)]))
+
+
+def clamped_glu(gate_up, limit):
+    """[.., 2 n] (gate | up) -> g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    return GpuTensor(_L().applegpu_ffi_clamped_glu(gate_up.id, float(limit)))
+
+
+def mlstm(proj, gates, gate_bias, norm, state, heads, dim, vdim, gate_cap, eps=1e-5, chunked=True):
+    """The mLSTM recurrence over proj [B, T, cols] (q | k | v | output gate) and float32 gates [B, T, 2 heads] (input | forget,
+    without bias); `state` (float32 [B, n]) is updated in place. `chunked=False` goes token by token. Returns [B, T, heads * vdim]."""
+    return GpuTensor(_L().applegpu_ffi_mlstm(proj.id, gates.id, gate_bias.id, norm.id, state.id, heads, dim, vdim, float(gate_cap), float(eps), 0 if chunked else 1))
+
+
+def latent_attention(proj, norm, up, rot_table, cache, pos, past, heads, dim, rot_dim, vdim, kv_rank, scale, eps=1e-5, expanded=True):
+    """Causal latent attention of T new rows per sequence; the cache is appended in place and proj's queries may be rotated in place.
+    `expanded=False` attends in the latent space. Returns [B, T, heads * vdim]."""
+    return GpuTensor(_L().applegpu_ffi_latent_attention(proj.id, norm.id, up.id, 0 if rot_table is None else rot_table.id, cache.id, pos.id, int(past), heads, dim, rot_dim, vdim,
+                                                        kv_rank, float(scale), float(eps), 0 if expanded else 1))
+
+
 _ACT_CODES = {None: 0, "none": 0, "gelu": 1, "gelu_exact": 2, "relu": 3}
 
 

@@ -5,6 +5,8 @@
 #include "../../../include/applegpu_b200_ffi.h"
 #include "../../../include/applegpu_b200_ext.h"
 #include "../core/runtime.h"
+#include "../core/seqmodel.h"
+#include "../kernels/seq_kernels.h"
 #include "../kernels/kernels.h"
 #include <algorithm>
 #include <cmath>
@@ -1349,6 +1351,193 @@ int32_t applegpu_gpt2_decoder_set_engine(uint64_t decoder, int32_t engine) {
   return 0;
 }
 void applegpu_gpt2_decoder_destroy(uint64_t decoder) { decoder_destroy(decoder); }
+
+// ── sequence models ─────────────────────────────────────────────────────────
+static Status materialised_or_empty(LazyRuntime& rt, uint64_t id, TensorRec* out) { return id ? materialised(rt, id, out) : Status::OK(); }
+uint64_t applegpu_seq_create(const applegpu_seq_model* m, const applegpu_seq_layer* layers, const uint64_t* weight_ids, uint32_t n_weights, uint32_t slots, uint32_t max_len) {
+  if (!ffi_ready("seq_create")) return 0;
+  if (!m || !layers || !weight_ids) { set_ffi_error("seq_create failed: null argument"); return 0; }
+  LazyState& st = lazy_state();
+  std::lock_guard<std::mutex> g(st.mu);
+  SeqModelCfg cfg;
+  cfg.vocab = m->vocab; cfg.width = m->width; cfg.eps = m->eps; cfg.loop_start = m->loop_start; cfg.loop_stop = m->loop_stop; cfg.loop_times = m->loop_times;
+  for (int32_t i = 0; i < m->n_layers; i++) {
+    const applegpu_seq_layer& l = layers[i];
+    SeqLayerCfg c;
+    c.mixer = (MixerKind)l.mixer; c.heads = l.heads; c.dim = l.dim; c.vdim = l.vdim; c.rot_dim = l.rot_dim; c.rot_pairs = l.rot_pairs; c.kv_rank = l.kv_rank;
+    c.gate_cap = l.gate_cap; c.score_scale = l.score_scale; c.ff = l.ff; c.ff_limit = l.ff_limit;
+    cfg.layers.push_back(c);
+  }
+  std::vector<TensorRec> w(n_weights);
+  uint64_t h = 0;
+  Status s = Status::OK();
+  for (uint32_t i = 0; i < n_weights && s.ok(); i++) s = materialised_or_empty(st.rt, weight_ids[i], &w[i]);
+  if (s.ok()) s = seq_create(cfg, w, (int)slots, (int)max_len, &h);
+  if (!s.ok()) { set_ffi_error("seq_create failed: " + s.to_string()); return 0; }
+  return h;
+}
+int32_t applegpu_seq_forward(uint64_t engine, uint32_t slot0, uint32_t n_seq, const int32_t* tokens, uint32_t n_tokens, const int32_t* want, uint32_t n_want,
+                             float* host_logits, int32_t* picked, float* host_layers) {
+  if (!ffi_ready("seq_forward")) return -1;
+  std::lock_guard<std::mutex> g(lazy_state().mu);
+  Status s = seq_forward(engine, (int)slot0, (int)n_seq, tokens, (int)n_tokens, want, (int)n_want, host_logits, picked, host_layers);
+  if (!s.ok()) { set_ffi_error("seq_forward failed: " + s.to_string()); return -1; }
+  return 0;
+}
+int32_t applegpu_seq_decode(uint64_t engine, uint32_t slot0, uint32_t n_seq, uint32_t n_steps, int32_t* host_tokens, bool use_graph) {
+  if (!ffi_ready("seq_decode")) return -1;
+  std::lock_guard<std::mutex> g(lazy_state().mu);
+  Status s = seq_decode(engine, (int)slot0, (int)n_seq, (int)n_steps, host_tokens, use_graph);
+  if (!s.ok()) { set_ffi_error("seq_decode failed: " + s.to_string()); return -1; }
+  return 0;
+}
+int32_t applegpu_seq_reset(uint64_t engine, uint32_t slot, uint32_t n) {
+  if (!ffi_ready("seq_reset")) return -1;
+  std::lock_guard<std::mutex> g(lazy_state().mu);
+  Status s = seq_reset(engine, (int)slot, (int)n);
+  if (!s.ok()) { set_ffi_error("seq_reset failed: " + s.to_string()); return -1; }
+  return 0;
+}
+int32_t applegpu_seq_length(uint64_t engine, uint32_t slot) { return seq_length(engine, (int)slot); }
+int32_t applegpu_seq_info(uint64_t engine, int32_t what) { return seq_info(engine, what); }
+void applegpu_seq_destroy(uint64_t engine) { seq_destroy(engine); }
+
+static Status new_tensor(const Dims& shape, DType dt, TensorRec* out) {
+  out->shape = shape; out->strides = contiguous_strides(shape); out->dtype = dt; out->has_meta = true;
+  return Shared::get().pool.acquire(out->nbytes() ? out->nbytes() : 4, &out->buf);
+}
+// Looks the operands of an immediate op up; each must be contiguous (empty records for id 0).
+static Status immediate_operands(LazyRuntime& rt, const uint64_t* ids, TensorRec* out, int n) {
+  if (DeviceCtx::get().dry) return Status::compute("no CUDA device (dry-run mode)");
+  for (int i = 0; i < n; i++) {
+    AG_RETURN_IF_ERROR(materialised_or_empty(rt, ids[i], &out[i]));
+    if (ids[i] && !out[i].contiguous()) return Status::invalid("operand " + std::to_string(i) + " must be contiguous");
+  }
+  return DeviceCtx::get().make_current();
+}
+static uint64_t immediate_result(const char* what, LazyRuntime& rt, const Status& s, const TensorRec& out) {
+  if (!s.ok()) { set_ffi_error(std::string(what) + " failed: " + s.to_string()); return 0; }
+  note_launches(1);
+  const uint64_t id = next_tensor_id();
+  rt.insert_tensor(id, out);
+  return id;
+}
+uint64_t applegpu_ffi_rms_norm(uint64_t x_id, uint64_t weight_id, float eps, int8_t out_dtype) {
+  if (!ffi_ready("rms_norm")) return 0;
+  LazyState& st = lazy_state();
+  std::lock_guard<std::mutex> g(st.mu);
+  const uint64_t ids[2] = {x_id, weight_id};
+  TensorRec t[2], out;
+  DType dt = DType::Invalid;
+  auto run = [&]() -> Status {
+    AG_RETURN_IF_ERROR(immediate_operands(st.rt, ids, t, 2));
+    if (!dtype_from_wire(out_dtype, &dt)) return Status::invalid("unknown dtype");
+    if (t[0].dtype != DType::F32 || t[1].dtype != DType::F32 || t[0].shape.empty() || numel_of(t[1].shape) != t[0].shape.back()) return Status::invalid("float32 rows and a weight of their length");
+    const int64_t wd = t[0].shape.back();
+    AG_RETURN_IF_ERROR(new_tensor(t[0].shape, dt, &out));
+    k::RmsRowsDesc d;
+    d.dtype = dt; d.x = static_cast<float*>(t[0].data()); d.rows = numel_of(t[0].shape) / wd; d.width = (int)wd; d.eps = eps;
+    d.w1 = static_cast<const float*>(t[1].data()); d.out1 = out.data(); d.ld1 = wd;
+    return k::rms_rows(DeviceCtx::get().stream, d);
+  };
+  const Status s = run();
+  return immediate_result("rms_norm", st.rt, s, out);
+}
+uint64_t applegpu_ffi_clamped_glu(uint64_t gate_up_id, float limit) {
+  if (!ffi_ready("clamped_glu")) return 0;
+  LazyState& st = lazy_state();
+  std::lock_guard<std::mutex> g(st.mu);
+  TensorRec t, out;
+  auto run = [&]() -> Status {
+    AG_RETURN_IF_ERROR(immediate_operands(st.rt, &gate_up_id, &t, 1));
+    if (t.shape.empty() || t.shape.back() % 2) return Status::invalid("gate and up columns side by side");
+    Dims o = t.shape;
+    const int64_t c = o.back(), rows = numel_of(o) / (c ? c : 1);
+    o.back() = c / 2;
+    AG_RETURN_IF_ERROR(new_tensor(o, t.dtype, &out));
+    return k::clamped_glu(DeviceCtx::get().stream, t.dtype, t.data(), c, out.data(), c / 2, rows, (int)(c / 2), limit);
+  };
+  const Status s = run();
+  return immediate_result("clamped_glu", st.rt, s, out);
+}
+uint64_t applegpu_ffi_mlstm(uint64_t proj_id, uint64_t gates_id, uint64_t gate_bias_id, uint64_t norm_id, uint64_t state_id, uint32_t heads, uint32_t dim, uint32_t vdim,
+                            float gate_cap, float eps, int32_t form) {
+  if (!ffi_ready("mlstm")) return 0;
+  LazyState& st = lazy_state();
+  std::lock_guard<std::mutex> g(st.mu);
+  const uint64_t ids[5] = {proj_id, gates_id, gate_bias_id, norm_id, state_id};
+  TensorRec t[5], out, work;
+  auto run = [&]() -> Status {
+    AG_RETURN_IF_ERROR(immediate_operands(st.rt, ids, t, 5));
+    if (t[0].shape.size() != 3 || !heads || !dim || !vdim) return Status::invalid("proj must be [sequences, tokens, columns]");
+    const int64_t B = t[0].shape[0], T = t[0].shape[1], H = heads, sf = k::mlstm_state_floats((int)heads, (int)dim, (int)vdim);
+    if (t[0].shape[2] < 2 * H * (dim + vdim) || t[1].shape != Dims{B, T, 2 * H} || numel_of(t[2].shape) != 2 * H || numel_of(t[3].shape) != H * vdim || t[4].shape != Dims{B, sf})
+      return Status::invalid("operand shapes");
+    for (int i = 1; i < 5; i++) if (t[i].dtype != DType::F32) return Status::invalid("gates, bias, norm and state are float32");
+    AG_RETURN_IF_ERROR(new_tensor({B, T, H * vdim}, t[0].dtype, &out));
+    k::MlstmDesc d;
+    d.dtype = t[0].dtype; d.n_seq = (int)B; d.T = (int)T; d.heads = (int)heads; d.dim = (int)dim; d.vdim = (int)vdim; d.gate_cap = gate_cap; d.eps = eps;
+    d.proj = t[0].data(); d.ld = t[0].shape[2]; d.gates = static_cast<const float*>(t[1].data()); d.gates_ld = 2 * H;
+    d.gate_bias = static_cast<const float*>(t[2].data()); d.norm = static_cast<const float*>(t[3].data()); d.state = static_cast<float*>(t[4].data()); d.state_stride = sf;
+    d.y = out.data(); d.y_ld = H * vdim;
+    if (form == 1) return k::mlstm_step(DeviceCtx::get().stream, d);
+    AG_RETURN_IF_ERROR(new_tensor({(int64_t)k::mlstm_work_bytes((int)B, (int)T, (int)heads, (int)dim, (int)vdim)}, DType::U8, &work));
+    d.work = work.data();
+    return k::mlstm_prefill(DeviceCtx::get().stream, d);
+  };
+  const Status s = run();
+  return immediate_result("mlstm", st.rt, s, out);
+}
+uint64_t applegpu_ffi_latent_attention(uint64_t proj_id, uint64_t norm_id, uint64_t up_id, uint64_t rot_id, uint64_t cache_id, uint64_t pos_id, uint32_t past, uint32_t heads,
+                                       uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint32_t kv_rank, float scale, float eps, int32_t form) {
+  if (!ffi_ready("latent_attention")) return 0;
+  LazyState& st = lazy_state();
+  std::lock_guard<std::mutex> g(st.mu);
+  const uint64_t ids[6] = {proj_id, norm_id, up_id, rot_id, cache_id, pos_id};
+  TensorRec t[6], out, work;
+  auto run = [&]() -> Status {
+    AG_RETURN_IF_ERROR(immediate_operands(st.rt, ids, t, 6));
+    if (t[0].shape.size() != 3 || t[4].shape.size() != 3 || !heads || !dim || !vdim || !kv_rank) return Status::invalid("proj [sequences, tokens, columns], cache [sequences, positions, columns]");
+    const int64_t B = t[0].shape[0], T = t[0].shape[1], H = heads, cld = k::latent_cache_ld((int)kv_rank, (int)rot_dim), w_ld = k::pad8(kv_rank), v_off = k::pad8(H * dim);
+    const DType dt = t[0].dtype;
+    if (t[0].shape[2] < H * (dim + rot_dim) + kv_rank + rot_dim || t[4].shape[0] != B || t[4].shape[2] != cld || (int64_t)past + T > t[4].shape[1] || numel_of(t[1].shape) != kv_rank ||
+        t[2].shape != Dims{v_off + k::pad8(H * vdim), w_ld} || numel_of(t[5].shape) != B)
+      return Status::invalid("operand shapes");
+    if (t[1].dtype != DType::F32 || t[2].dtype != dt || t[4].dtype != dt || t[5].dtype != DType::I32) return Status::invalid("operand dtypes");
+    if (t[3].buf && (t[3].dtype != DType::F32 || t[3].shape.size() != 3 || t[3].shape[0] < t[4].shape[1] || t[3].shape[2] != 2)) return Status::invalid("rotation table");
+    AG_RETURN_IF_ERROR(new_tensor({B, T, H * vdim}, dt, &out));
+    const size_t esz = dtype_size(dt);
+    cudaStream_t cs = DeviceCtx::get().stream;
+    k::LatentDesc d;
+    d.dtype = dt; d.n_seq = (int)B; d.T = (int)T; d.heads = (int)heads; d.dim = (int)dim; d.rot_dim = (int)rot_dim; d.vdim = (int)vdim; d.kv_rank = (int)kv_rank;
+    d.rot_pairs = t[3].buf ? (int)t[3].shape[1] : 0; d.scale = scale; d.eps = eps; d.proj = t[0].data(); d.ld = t[0].shape[2]; d.c_norm = static_cast<const float*>(t[1].data());
+    d.rot_table = static_cast<const float2*>(t[3].data()); d.cache = t[4].data(); d.seq_stride = t[4].shape[1] * cld; d.pos = static_cast<const int*>(t[5].data());
+    d.max_len = (int)t[4].shape[1]; d.w_uk = t[2].data(); d.w_uv = static_cast<uint8_t*>(t[2].data()) + (size_t)v_off * w_ld * esz; d.w_ld = w_ld;
+    d.y = out.data(); d.y_ld = H * vdim;
+    if (form == 1) {
+      AG_RETURN_IF_ERROR(new_tensor({(int64_t)k::latent_decode_work_bytes((int)(B * T), (int)heads, (int)kv_rank, (int)rot_dim, d.max_len)}, DType::U8, &work));
+      return k::latent_decode(cs, d, work.data());
+    }
+    AG_RETURN_IF_ERROR(k::latent_append(cs, d));
+    const int64_t cols = v_off + k::pad8(H * vdim), keys = (int64_t)past + T;
+    AG_RETURN_IF_ERROR(new_tensor({keys, cols}, dt, &work));
+    for (int64_t i = 0; i < B; i++) {
+      uint8_t* cache = static_cast<uint8_t*>(d.cache) + (size_t)i * d.seq_stride * esz;
+      k::GemmDesc m;
+      m.dtype = dt; m.b_dtype = dt; m.a = cache; m.b = d.w_uk; m.c = work.data(); m.m = keys; m.n = cols; m.k = kv_rank; m.batch = 1;
+      m.a_row = cld; m.a_col = 1; m.a_batch = 0; m.b_row = 1; m.b_col = w_ld; m.b_batch = 0; m.c_row = cols; m.c_batch = 0;
+      AG_RETURN_IF_ERROR(k::matmul(cs, m));
+      k::LatentPrefillDesc p;
+      p.dtype = dt; p.T = (int)T; p.past = (int)past; p.heads = (int)heads; p.dim = (int)dim; p.rot_dim = (int)rot_dim; p.vdim = (int)vdim; p.scale = scale;
+      p.q = static_cast<uint8_t*>(d.proj) + (size_t)i * T * d.ld * esz; p.q_ld = d.ld; p.kv = work.data(); p.kv_ld = cols; p.v_off = v_off;
+      p.k_rot = cache + (size_t)k::pad8(kv_rank) * esz; p.k_rot_ld = cld; p.y = static_cast<uint8_t*>(out.data()) + (size_t)i * T * d.y_ld * esz; p.y_ld = d.y_ld;
+      AG_RETURN_IF_ERROR(k::latent_prefill(cs, p));
+    }
+    return Status::OK();
+  };
+  const Status s = run();
+  return immediate_result("latent_attention", st.rt, s, out);
+}
 
 int32_t applegpu_test_wait_runs_out(int32_t code, uint32_t limit_us) {
   DeviceCtx& ctx = DeviceCtx::get();

@@ -156,6 +156,13 @@ __device__ __forceinline__ float apply_act(float x, Act a) {
   }
 }
 
+// Gated activation with clamped operands: g sigmoid(1.702 g) (u + 1), g clipped from above, u on both sides.
+__device__ __forceinline__ float clamped_glu_f(float gate, float up, float limit) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
+
 inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
 
 inline Status cuda_status(cudaError_t e, const char* what) {

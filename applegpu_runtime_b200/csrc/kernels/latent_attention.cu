@@ -1,0 +1,405 @@
+// Latent attention: keys and values of all heads are linear images of one normed latent per token, plus one rotated
+// key part shared by the heads; the cache holds only those two.
+//
+//   append    one row per CTA: rotates the query parts, norms the latent, rotates the key part, writes the cache row
+//   prefill   attention of a prompt portion over keys and values expanded from the cache (the GEMM that expands them is
+//             the caller's). The form here runs on CUDA cores in float32 arithmetic and takes any sizes.
+//   decode    short portions stay in the latent space: W_uk is applied to the query instead of to every key, W_uv to the
+//             attended latent instead of to every value, so that a step reads each cached row once for all heads.
+//             prepare -> attend over splits of the keys -> merge the splits and apply W_uv.
+// Scores, their maximum and the weights are float32 throughout.
+#include "common.cuh"
+#include "seq_kernels.h"
+
+namespace ag { namespace k {
+
+struct LaParams {
+  void* proj; const float* c_norm; const float2* rot; void* cache; const int* pos; const void* uk; const void* uv; void* y;
+  long long ld, seq_stride, w_ld, y_ld;
+  int n_seq, T, heads, dim, rot_dim, vdim, rank, pairs, max_len, cld, coff;   // cld: cache pitch, coff: column of the rotated part
+  float scale, eps;
+  float* q_eff; float* part; int splits;
+};
+
+static Status la_params(const LatentDesc& d, LaParams* out) {
+  if (d.n_seq < 1 || d.T < 1 || d.heads < 1 || d.dim < 1 || d.rot_dim < 0 || d.vdim < 1 || d.kv_rank < 1 || 2 * d.rot_pairs > d.rot_dim)
+    return Status::invalid("latent attention: bad sizes");
+  if (!d.proj || !d.cache || !d.pos || !d.c_norm || (d.rot_pairs && !d.rot_table)) return Status::invalid("latent attention: missing operand");
+  LaParams& p = *out;
+  p.proj = d.proj; p.c_norm = d.c_norm; p.rot = d.rot_table; p.cache = d.cache; p.pos = d.pos; p.uk = d.w_uk; p.uv = d.w_uv; p.y = d.y;
+  p.ld = d.ld; p.seq_stride = d.seq_stride; p.w_ld = d.w_ld; p.y_ld = d.y_ld;
+  p.n_seq = d.n_seq; p.T = d.T; p.heads = d.heads; p.dim = d.dim; p.rot_dim = d.rot_dim; p.vdim = d.vdim; p.rank = d.kv_rank; p.pairs = d.rot_pairs;
+  p.max_len = d.max_len; p.cld = (int)latent_cache_ld(d.kv_rank, d.rot_dim); p.coff = (int)pad8(d.kv_rank);
+  p.scale = d.scale; p.eps = d.eps; p.q_eff = nullptr; p.part = nullptr; p.splits = 1;
+  return Status::OK();
+}
+
+// The latent and the rotated key part of one row into its cache row (whole block).
+template <typename T>
+__device__ __forceinline__ void la_cache_row(const LaParams& p, const T* row, T* crow, int position, float* red) {
+  const T* c = row + (long long)p.heads * (p.dim + p.rot_dim);
+  float sq = 0.f;
+  for (int i = threadIdx.x; i < p.rank; i += blockDim.x) { const float v = Cvt<T>::to(c[i]); sq = fmaf(v, v, sq); }
+  const float rs = 1.0f / sqrtf(block_sum(sq, red) / (float)p.rank + p.eps);
+  for (int i = threadIdx.x; i < p.rank; i += blockDim.x) crow[i] = Cvt<T>::from(Cvt<T>::to(c[i]) * rs * p.c_norm[i]);
+  const T* kr = c + p.rank;
+  T* dst = crow + p.coff;
+  for (int i = threadIdx.x; i < p.pairs; i += blockDim.x) {
+    const float2 cs = p.rot[(long long)position * p.pairs + i];
+    const float u = Cvt<T>::to(kr[2 * i]), v = Cvt<T>::to(kr[2 * i + 1]);
+    dst[2 * i] = Cvt<T>::from(u * cs.x - v * cs.y);
+    dst[2 * i + 1] = Cvt<T>::from(v * cs.x + u * cs.y);
+  }
+  for (int i = 2 * p.pairs + threadIdx.x; i < p.rot_dim; i += blockDim.x) dst[i] = kr[i];
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) latent_append_kernel(const LaParams p) {
+  __shared__ float red[33];
+  pdl_wait();
+  pdl_trigger();
+  const int r = blockIdx.x, s = r / p.T, t = r % p.T;
+  const int position = p.pos[s] + t;
+  if (position < 0 || position >= p.max_len) return;
+  T* row = reinterpret_cast<T*>(p.proj) + (long long)r * p.ld;
+  T* crow = reinterpret_cast<T*>(p.cache) + (long long)s * p.seq_stride + (long long)position * p.cld;
+  la_cache_row<T>(p, row, crow, position, red);
+  for (int i = threadIdx.x; i < p.heads * p.pairs; i += 256) {
+    const int h = i / p.pairs, j = i % p.pairs;
+    T* q = row + (long long)h * (p.dim + p.rot_dim) + p.dim + 2 * j;
+    const float2 cs = p.rot[(long long)position * p.pairs + j];
+    const float u = Cvt<T>::to(q[0]), v = Cvt<T>::to(q[1]);
+    q[0] = Cvt<T>::from(u * cs.x - v * cs.y);
+    q[1] = Cvt<T>::from(v * cs.x + u * cs.y);
+  }
+}
+
+Status latent_append(cudaStream_t s, const LatentDesc& d) {
+  LaParams p;
+  AG_RETURN_IF_ERROR(la_params(d, &p));
+  cudaError_t e = cudaSuccess;
+  AG_DISPATCH_FLOAT(d.dtype, T, (e = launch_pdl(latent_append_kernel<T>, dim3((unsigned)(d.n_seq * d.T)), dim3(256), 0, s, p)));
+  return cuda_status(e, "latent append");
+}
+
+// ── prefill, CUDA cores ─────────────────────────────────────────────────────
+struct LpParams {
+  const void* q; const void* kv; const void* kr; void* y;
+  long long q_ld, kv_ld, v_off, kr_ld, y_ld;
+  int T, past, heads, dim, rot, vdim;
+  float scale;
+};
+template <typename T, int TQ>
+__global__ void __launch_bounds__(256) latent_prefill_kernel(const LpParams p) {
+  extern __shared__ __align__(16) float sm[];
+  const int D = p.dim + p.rot, E = p.vdim;
+  float* sq = sm;                        // [TQ][D]
+  float* sk = sq + TQ * D;               // [TQ][D + 1]
+  float* sv = sk + TQ * (D + 1);         // [TQ][E]
+  float* so = sv + TQ * E;               // [TQ][E]
+  float* sp = so + TQ * E;               // [TQ][TQ + 1]
+  float* s_m = sp + TQ * (TQ + 1);       // [TQ] running maximum, sum, rescale factor
+  float* s_l = s_m + TQ;
+  float* s_a = s_l + TQ;
+  pdl_wait();
+  pdl_trigger();
+  const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * TQ, h = blockIdx.y;     // longest rows first
+  const int rows = min(TQ, p.T - q0);
+  const T* Q = reinterpret_cast<const T*>(p.q) + (long long)h * D;
+  const T* KV = reinterpret_cast<const T*>(p.kv);
+  const T* KR = reinterpret_cast<const T*>(p.kr);
+  for (int i = threadIdx.x; i < TQ * D; i += 256) {
+    const int t = i / D;
+    sq[i] = t < rows ? Cvt<T>::to(Q[(long long)(q0 + t) * p.q_ld + i % D]) * p.scale : 0.f;
+  }
+  for (int i = threadIdx.x; i < TQ * E; i += 256) so[i] = 0.f;
+  if (threadIdx.x < TQ) { s_m[threadIdx.x] = -INFINITY; s_l[threadIdx.x] = 0.f; }
+  const int n_keys = p.past + q0 + rows;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int k0 = 0; k0 < n_keys; k0 += TQ) {
+    const int nk = min(TQ, n_keys - k0);
+    __syncthreads();
+    for (int i = threadIdx.x; i < nk * D; i += 256) {
+      const int j = i / D, c = i % D;
+      sk[j * (D + 1) + c] = c < p.dim ? Cvt<T>::to(KV[(long long)(k0 + j) * p.kv_ld + h * p.dim + c]) : Cvt<T>::to(KR[(long long)(k0 + j) * p.kr_ld + c - p.dim]);
+    }
+    for (int i = threadIdx.x; i < nk * E; i += 256) sv[i] = Cvt<T>::to(KV[(long long)(k0 + i / E) * p.kv_ld + p.v_off + h * E + i % E]);
+    __syncthreads();
+    for (int i = threadIdx.x; i < TQ * TQ; i += 256) {
+      const int t = i / TQ, j = i % TQ;
+      float v = -INFINITY;
+      if (t < rows && j < nk && k0 + j <= p.past + q0 + t) {
+        v = 0.f;
+        for (int c = 0; c < D; c++) v = fmaf(sq[t * D + c], sk[j * (D + 1) + c], v);
+      }
+      sp[t * (TQ + 1) + j] = v;
+    }
+    __syncthreads();
+    for (int t = warp; t < rows; t += 8) {
+      const float v = lane < TQ ? sp[t * (TQ + 1) + lane] : -INFINITY;
+      const float m1 = fmaxf(s_m[t], warp_max(v));
+      const float e = v == -INFINITY ? 0.f : expf(v - m1);
+      const float sum = warp_sum(e);
+      if (lane < TQ) sp[t * (TQ + 1) + lane] = e;
+      __syncwarp();
+      if (lane == 0) {
+        const float a = m1 == -INFINITY ? 1.f : expf(s_m[t] - m1);
+        s_a[t] = a; s_l[t] = s_l[t] * a + sum; s_m[t] = m1;
+      }
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < rows * E; i += 256) {
+      const int t = i / E, e = i % E;
+      float a = so[i] * s_a[t];
+      for (int j = 0; j < nk; j++) a = fmaf(sp[t * (TQ + 1) + j], sv[j * E + e], a);
+      so[i] = a;
+    }
+  }
+  __syncthreads();
+  T* Y = reinterpret_cast<T*>(p.y) + (long long)h * E;
+  for (int i = threadIdx.x; i < rows * E; i += 256) Y[(long long)(q0 + i / E) * p.y_ld + i % E] = Cvt<T>::from(so[i] / s_l[i / E]);
+}
+
+template <typename T, int TQ>
+static cudaError_t launch_lp(cudaStream_t s, const LpParams& p, size_t smem) {
+  static bool attr = false;
+  if (!attr) {
+    cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel<T, TQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+    if (e != cudaSuccess) return e;
+    attr = true;
+  }
+  return launch_pdl(latent_prefill_kernel<T, TQ>, dim3((unsigned)((p.T + TQ - 1) / TQ), (unsigned)p.heads), dim3(256), smem, s, p);
+}
+
+Status latent_prefill(cudaStream_t s, const LatentPrefillDesc& d) {
+  if (d.T < 1 || d.past < 0 || d.heads < 1 || d.heads > 65535 || d.dim < 1 || d.rot_dim < 0 || d.vdim < 1 || !d.q || !d.kv || !d.y) return Status::invalid("latent prefill: bad description");
+  LpParams p;
+  p.q = d.q; p.kv = d.kv; p.kr = d.k_rot; p.y = d.y; p.q_ld = d.q_ld; p.kv_ld = d.kv_ld; p.v_off = d.v_off; p.kr_ld = d.k_rot_ld; p.y_ld = d.y_ld;
+  p.T = d.T; p.past = d.past; p.heads = d.heads; p.dim = d.dim; p.rot = d.rot_dim; p.vdim = d.vdim; p.scale = d.scale;
+  auto smem = [&](int tq) { return ((size_t)tq * (2 * (d.dim + d.rot_dim) + 1) + 2 * (size_t)tq * d.vdim + (size_t)tq * (tq + 1) + 3 * tq) * sizeof(float); };
+  const size_t lim = 220 * 1024;
+  if (smem(8) > lim) return Status::unsupported("latent prefill: head too large");
+  cudaError_t e = cudaSuccess;
+  AG_DISPATCH_FLOAT(d.dtype, T, (e = smem(32) <= lim ? launch_lp<T, 32>(s, p, smem(32)) : smem(16) <= lim ? launch_lp<T, 16>(s, p, smem(16)) : launch_lp<T, 8>(s, p, smem(8))));
+  return cuda_status(e, "latent prefill");
+}
+
+// ── decode ──────────────────────────────────────────────────────────────────
+// prepare: CTA h < heads: the query of head h in cache-row coordinates, scaled: (q W_uk | 0 | rotated part | 0); CTA `heads`
+// appends the row to the cache.
+template <typename T>
+__global__ void __launch_bounds__(256) latent_decode_prepare_kernel(const LaParams p) {
+  extern __shared__ __align__(16) float sq[];            // [dim]
+  __shared__ float red[33];
+  const int h = blockIdx.x, r = blockIdx.y, s = r / p.T, t = r % p.T;
+  pdl_wait();
+  pdl_trigger();
+  const int position = p.pos[s] + t;
+  if (position < 0 || position >= p.max_len) return;
+  const T* row = reinterpret_cast<const T*>(p.proj) + (long long)r * p.ld;
+  if (h == p.heads) {
+    la_cache_row<T>(p, row, reinterpret_cast<T*>(p.cache) + (long long)s * p.seq_stride + (long long)position * p.cld, position, red);
+    return;
+  }
+  const T* q = row + (long long)h * (p.dim + p.rot_dim);
+  float* out = p.q_eff + ((long long)r * p.heads + h) * p.cld;
+  for (int i = threadIdx.x; i < p.dim; i += 256) sq[i] = Cvt<T>::to(q[i]);
+  for (int i = threadIdx.x; i < p.cld - p.coff; i += 256) {
+    float v = 0.f;
+    if (i < 2 * p.pairs) {
+      const float2 cs = p.rot[(long long)position * p.pairs + i / 2];
+      const float a = Cvt<T>::to(q[p.dim + (i & ~1)]), b = Cvt<T>::to(q[p.dim + (i | 1)]);
+      v = (i & 1) ? b * cs.x + a * cs.y : a * cs.x - b * cs.y;
+    } else if (i < p.rot_dim) v = Cvt<T>::to(q[p.dim + i]);
+    out[p.coff + i] = v * p.scale;
+  }
+  __syncthreads();
+  const T* uk = reinterpret_cast<const T*>(p.uk) + (long long)h * p.dim * p.w_ld;
+  for (int i = threadIdx.x; i < p.coff; i += 256) {
+    float a = 0.f;
+    if (i < p.rank) {
+#pragma unroll 8
+      for (int d = 0; d < p.dim; d++) a = fmaf(sq[d], Cvt<T>::to(uk[(long long)d * p.w_ld + i]), a);
+    }
+    out[i] = a * p.scale;
+  }
+}
+
+// attend: CTA = (split of the keys, eight heads, row); a warp per head. Lane = key for the scores, lanes across the latent
+// for the weighted sum. Leaves (maximum, sum, unnormalised latent) per split.
+constexpr int kLdKeys = 32, kLdHeads = 8;
+template <typename T, int NR>
+__global__ void __launch_bounds__(256) latent_decode_attend_kernel(const LaParams p) {
+  extern __shared__ __align__(16) float sm[];
+  constexpr int PADE = sizeof(T) == 4 ? 1 : 2;           // keeps the row pitch an odd number of 32-bit words
+  const int cp = p.cld + PADE;
+  float* sq = sm;                                        // [kLdHeads][cld]
+  T* sk = reinterpret_cast<T*>(sq + kLdHeads * p.cld);   // [kLdKeys][cp]
+  const int split = blockIdx.x, r = blockIdx.z, s = r / p.T, t = r % p.T;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = (int)blockIdx.y * kLdHeads + warp;
+  pdl_wait();
+  pdl_trigger();
+  const int n_keys = min(p.pos[s] + t + 1, p.max_len);
+  const int per = ((n_keys + p.splits - 1) / p.splits + kLdKeys - 1) / kLdKeys * kLdKeys;
+  const int k_lo = split * per, k_hi = min(n_keys, k_lo + per);
+  const bool live = h < p.heads;
+  for (int i = threadIdx.x; i < kLdHeads * p.cld; i += 256) {
+    const int hh = (int)blockIdx.y * kLdHeads + i / p.cld;
+    sq[i] = hh < p.heads && k_lo < k_hi ? p.q_eff[((long long)r * p.heads + hh) * p.cld + i % p.cld] : 0.f;
+  }
+  float m = -INFINITY, l = 0.f, o[NR];
+#pragma unroll
+  for (int j = 0; j < NR; j++) o[j] = 0.f;
+  const T* cache = reinterpret_cast<const T*>(p.cache) + (long long)s * p.seq_stride;
+  constexpr int N = Pack<T>::N;
+  const float* qh = sq + warp * p.cld;
+  for (int k0 = k_lo; k0 < k_hi; k0 += kLdKeys) {
+    const int nk = min(kLdKeys, k_hi - k0);
+    __syncthreads();
+    for (int i = threadIdx.x; i < nk * (p.cld / N); i += 256) {
+      const int j = i / (p.cld / N), c = i % (p.cld / N) * N;
+      const Pack<T> v = ld16(cache + (long long)(k0 + j) * p.cld + c);
+      uint32_t* dst = reinterpret_cast<uint32_t*>(sk + j * cp + c);
+      const uint32_t* src = reinterpret_cast<const uint32_t*>(&v);
+      dst[0] = src[0]; dst[1] = src[1]; dst[2] = src[2]; dst[3] = src[3];
+    }
+    __syncthreads();
+    if (!live) continue;
+    float sc = -INFINITY;
+    if (lane < nk) {
+      const T* kr = sk + lane * cp;
+      float a0 = 0.f, a1 = 0.f;
+      for (int c = 0; c < p.rank; c += 2) {
+        a0 = fmaf(qh[c], Cvt<T>::to(kr[c]), a0);
+        if (c + 1 < p.rank) a1 = fmaf(qh[c + 1], Cvt<T>::to(kr[c + 1]), a1);
+      }
+      for (int c = p.coff; c < p.coff + p.rot_dim; c += 2) {
+        a0 = fmaf(qh[c], Cvt<T>::to(kr[c]), a0);
+        if (c + 1 < p.coff + p.rot_dim) a1 = fmaf(qh[c + 1], Cvt<T>::to(kr[c + 1]), a1);
+      }
+      sc = a0 + a1;
+    }
+    const float m1 = fmaxf(m, warp_max(sc));
+    const float e = lane < nk ? expf(sc - m1) : 0.f;
+    const float a = m == -INFINITY ? 0.f : expf(m - m1);
+    l = l * a + warp_sum(e);
+    m = m1;
+#pragma unroll
+    for (int j = 0; j < NR; j++) o[j] *= a;
+    for (int key = 0; key < nk; key++) {
+      const float w = __shfl_sync(0xffffffffu, e, key);
+      const T* kr = sk + key * cp;
+#pragma unroll
+      for (int j = 0; j < NR; j++) {
+        const int c = lane + 32 * j;
+        if (c < p.rank) o[j] = fmaf(w, Cvt<T>::to(kr[c]), o[j]);
+      }
+    }
+  }
+  if (!live) return;
+  float* dst = p.part + (((long long)r * p.heads + h) * p.splits + split) * (p.rank + 2);
+  if (lane == 0) { dst[0] = m; dst[1] = l; }
+#pragma unroll
+  for (int j = 0; j < NR; j++) {
+    const int c = lane + 32 * j;
+    if (c < p.rank) dst[2 + c] = o[j];
+  }
+}
+
+// merge: the splits of one head combined, then the head's slice of W_uv.
+template <typename T>
+__global__ void __launch_bounds__(256) latent_decode_merge_kernel(const LaParams p) {
+  extern __shared__ __align__(16) float so[];            // [rank]
+  __shared__ float s_w[128];
+  const int h = blockIdx.x, r = blockIdx.y;
+  pdl_wait();
+  pdl_trigger();
+  const float* part = p.part + ((long long)r * p.heads + h) * p.splits * (p.rank + 2);
+  if (threadIdx.x < 32) {
+    float m = -INFINITY;
+    for (int i = threadIdx.x; i < p.splits; i += 32) m = fmaxf(m, part[(long long)i * (p.rank + 2)]);
+    m = warp_max(m);
+    float l = 0.f;
+    for (int i = threadIdx.x; i < p.splits; i += 32) {
+      const float mi = part[(long long)i * (p.rank + 2)];
+      const float w = mi == -INFINITY ? 0.f : expf(mi - m);
+      s_w[i] = w;
+      l += w * part[(long long)i * (p.rank + 2) + 1];
+    }
+    l = warp_sum(l);
+    __syncwarp();
+    for (int i = threadIdx.x; i < p.splits; i += 32) s_w[i] /= l;
+  }
+  __syncthreads();
+  for (int c = threadIdx.x; c < p.rank; c += 256) {
+    float a = 0.f;
+#pragma unroll 4
+    for (int i = 0; i < p.splits; i++) if (s_w[i] != 0.f) a = fmaf(s_w[i], part[(long long)i * (p.rank + 2) + 2 + c], a);
+    so[c] = a;
+  }
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* uv = reinterpret_cast<const T*>(p.uv) + (long long)h * p.vdim * p.w_ld;
+  T* y = reinterpret_cast<T*>(p.y) + (long long)r * p.y_ld + (long long)h * p.vdim;
+  for (int e = warp; e < p.vdim; e += 8) {
+    float a = 0.f;
+    for (int c = lane; c < p.rank; c += 32) a = fmaf(so[c], Cvt<T>::to(uv[(long long)e * p.w_ld + c]), a);
+    a = warp_sum(a);
+    if (lane == 0) y[e] = Cvt<T>::from(a);
+  }
+}
+
+static int la_splits(int rows, int heads, int max_len) {
+  const int groups = rows * ((heads + kLdHeads - 1) / kLdHeads);
+  int want = (2 * 148 + groups - 1) / groups, cap = (max_len + 63) / 64;
+  if (want > cap) want = cap;
+  return want < 1 ? 1 : (want > 128 ? 128 : want);
+}
+size_t latent_decode_work_bytes(int rows, int heads, int kv_rank, int rot_dim, int max_len) {
+  int worst = 0;                                          // fewer rows may use more splits each
+  for (int r = 1; r <= rows; r++) { const int v = r * la_splits(r, heads, max_len); if (v > worst) worst = v; }
+  return ((size_t)rows * heads * latent_cache_ld(kv_rank, rot_dim) + 64 + (size_t)worst * heads * (kv_rank + 2)) * sizeof(float) + 512;
+}
+
+template <typename T, int NR>
+static cudaError_t launch_ld(cudaStream_t s, const LaParams& p, dim3 grid, size_t smem) {
+  static bool attr = false;
+  if (!attr) {
+    cudaError_t e = cudaFuncSetAttribute(latent_decode_attend_kernel<T, NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+    if (e != cudaSuccess) return e;
+    attr = true;
+  }
+  return launch_pdl(latent_decode_attend_kernel<T, NR>, grid, dim3(256), smem, s, p);
+}
+template <typename T>
+static cudaError_t latent_decode_t(cudaStream_t s, const LaParams& p) {
+  const int rows = p.n_seq * p.T;
+  cudaError_t e = launch_pdl(latent_decode_prepare_kernel<T>, dim3((unsigned)(p.heads + 1), (unsigned)rows), dim3(256), (size_t)p.dim * sizeof(float), s, p);
+  if (e != cudaSuccess) return e;
+  const size_t smem = (size_t)kLdHeads * p.cld * sizeof(float) + (size_t)kLdKeys * (p.cld + 2) * sizeof(T);
+  const dim3 grid((unsigned)p.splits, (unsigned)((p.heads + kLdHeads - 1) / kLdHeads), (unsigned)rows);
+  if (p.rank <= 64) e = launch_ld<T, 2>(s, p, grid, smem);
+  else if (p.rank <= 128) e = launch_ld<T, 4>(s, p, grid, smem);
+  else if (p.rank <= 256) e = launch_ld<T, 8>(s, p, grid, smem);
+  else if (p.rank <= 512) e = launch_ld<T, 16>(s, p, grid, smem);
+  else e = launch_ld<T, 32>(s, p, grid, smem);
+  if (e != cudaSuccess) return e;
+  return launch_pdl(latent_decode_merge_kernel<T>, dim3((unsigned)p.heads, (unsigned)rows), dim3(256), (size_t)p.rank * sizeof(float), s, p);
+}
+
+Status latent_decode(cudaStream_t s, const LatentDesc& d, void* work) {
+  LaParams p;
+  AG_RETURN_IF_ERROR(la_params(d, &p));
+  if (!work || !d.w_uk || !d.w_uv || !d.y) return Status::invalid("latent decode: missing operand");
+  if (d.n_seq * d.T > 65535 || d.kv_rank > 1024) return Status::unsupported("latent decode: latent rank above 1024");
+  const int rows = d.n_seq * d.T;
+  p.splits = la_splits(rows, d.heads, d.max_len);
+  p.q_eff = static_cast<float*>(work);
+  p.part = p.q_eff + ((size_t)rows * d.heads * p.cld + 63) / 64 * 64;
+  cudaError_t e = cudaSuccess;
+  AG_DISPATCH_FLOAT(d.dtype, T, (e = latent_decode_t<T>(s, p)));
+  return cuda_status(e, "latent decode");
+}
+
+}}  // namespace ag::k

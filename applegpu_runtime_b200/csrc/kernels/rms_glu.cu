@@ -1,0 +1,168 @@
+// RMS norms over a float32 residual stream and the clamped gated activation of a feed-forward.
+//
+// rms_rows is the only kernel that touches the stream between two layers: it starts it from the embedding table, adds
+// what a repeated pass adds ahead of its first layer (the embedding output and a step vector), and writes the two
+// normalised copies a parallel layer feeds to its mixer and its feed-forward, all in one pass over the row.
+#include "common.cuh"
+#include "seq_kernels.h"
+
+namespace ag { namespace k {
+
+constexpr int kRmsThreads = 256;
+constexpr int kRmsRegs = 32;          // values per thread kept in registers: rows up to 8192 wide are read once
+
+struct RmsParams {
+  float* x; const int32_t* tok; const void* embed; const float* step; const float* w1; const float* w2; const int32_t* row_map;
+  void* out1; void* out2;
+  long long ld1, ld2, embed_ld;
+  int width, vocab, load_x, write_x;
+  float eps;
+};
+
+// VEC elements per thread and access (4 when width and pitches allow it)
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kRmsThreads) rms_rows_kernel(const RmsParams p) {
+  __shared__ float red[33];
+  pdl_wait();
+  pdl_trigger();
+  const long long r = blockIdx.x;
+  const long long src = p.row_map ? p.row_map[r] : r;
+  float* x = p.x + src * p.width;
+  const T* e = nullptr;
+  if (p.embed) {
+    int t = p.tok[r];
+    t = t < 0 ? 0 : (t >= p.vocab ? p.vocab - 1 : t);
+    e = reinterpret_cast<const T*>(p.embed) + (long long)t * p.embed_ld;
+  }
+  constexpr int NREG = kRmsRegs / VEC;
+  float v[NREG][VEC];
+  float sq = 0.f;
+  const int packs = p.width / VEC;
+  auto fetch = [&](int i, float (&o)[VEC]) {
+    const int c = i * VEC;
+    if (p.load_x) {
+      if constexpr (VEC == 4) { const float4 q = *reinterpret_cast<const float4*>(x + c); o[0] = q.x; o[1] = q.y; o[2] = q.z; o[3] = q.w; }
+      else o[0] = x[c];
+    } else {
+#pragma unroll
+      for (int j = 0; j < VEC; j++) o[j] = 0.f;
+    }
+    if (e) {
+#pragma unroll
+      for (int j = 0; j < VEC; j++) o[j] += Cvt<T>::to(e[c + j]);
+    }
+    if (p.step) {
+#pragma unroll
+      for (int j = 0; j < VEC; j++) o[j] += p.step[c + j];
+    }
+  };
+  auto put = [&](int i, const float (&o)[VEC]) {
+    const int c = i * VEC;
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(x + c) = make_float4(o[0], o[1], o[2], o[3]);
+    else x[c] = o[0];
+  };
+#pragma unroll
+  for (int it = 0; it < NREG; it++) {
+    const int i = threadIdx.x + it * kRmsThreads;
+    if (i < packs) {
+      fetch(i, v[it]);
+      if (p.write_x) put(i, v[it]);
+#pragma unroll
+      for (int j = 0; j < VEC; j++) sq = fmaf(v[it][j], v[it][j], sq);
+    }
+  }
+  for (int i = threadIdx.x + NREG * kRmsThreads; i < packs; i += kRmsThreads) {   // rows too wide for the registers
+    float o[VEC];
+    fetch(i, o);
+    if (p.write_x) put(i, o);
+#pragma unroll
+    for (int j = 0; j < VEC; j++) sq = fmaf(o[j], o[j], sq);
+  }
+  if (!p.out1) return;
+  const float rs = 1.0f / sqrtf(block_sum(sq, red) / (float)p.width + p.eps);
+  T* o1 = reinterpret_cast<T*>(p.out1) + r * p.ld1;
+  T* o2 = p.out2 ? reinterpret_cast<T*>(p.out2) + r * p.ld2 : nullptr;
+  auto emit = [&](int i, const float (&o)[VEC]) {
+    const int c = i * VEC;
+    auto one = [&](T* dst, const float* w) {
+      alignas(16) T t[VEC];
+#pragma unroll
+      for (int j = 0; j < VEC; j++) t[j] = Cvt<T>::from(o[j] * rs * w[c + j]);
+      if constexpr (VEC == 4 && sizeof(T) == 4) *reinterpret_cast<uint4*>(dst + c) = *reinterpret_cast<const uint4*>(t);
+      else if constexpr (VEC == 4) *reinterpret_cast<uint2*>(dst + c) = *reinterpret_cast<const uint2*>(t);
+      else dst[c] = t[0];
+    };
+    one(o1, p.w1);
+    if (o2) one(o2, p.w2);
+  };
+#pragma unroll
+  for (int it = 0; it < NREG; it++) {
+    const int i = threadIdx.x + it * kRmsThreads;
+    if (i < packs) emit(i, v[it]);
+  }
+  for (int i = threadIdx.x + NREG * kRmsThreads; i < packs; i += kRmsThreads) {
+    float o[VEC];
+    if (p.write_x) {                                                 // the sum is in x already
+#pragma unroll
+      for (int j = 0; j < VEC; j++) o[j] = x[i * VEC + j];
+    } else fetch(i, o);
+    emit(i, o);
+  }
+}
+
+Status rms_rows(cudaStream_t s, const RmsRowsDesc& d) {
+  if (d.rows <= 0) return Status::OK();
+  if (d.width < 1 || !d.x || (d.embed && !d.tok) || (d.out1 && !d.w1) || (d.out2 && !d.w2)) return Status::invalid("rms_rows: missing operand");
+  if (d.row_map && (d.embed || d.step || !d.load_x)) return Status::invalid("rms_rows: a gathered row is read only");
+  RmsParams p;
+  p.x = d.x; p.tok = d.tok; p.embed = d.embed; p.step = d.step; p.w1 = d.w1; p.w2 = d.w2; p.row_map = d.row_map;
+  p.out1 = d.out1; p.out2 = d.out2; p.ld1 = d.ld1; p.ld2 = d.ld2; p.embed_ld = d.embed_ld;
+  p.width = d.width; p.vocab = d.vocab; p.load_x = d.load_x ? 1 : 0; p.write_x = (!d.load_x || d.embed || d.step) ? 1 : 0; p.eps = d.eps;
+  const bool vec = d.width % 4 == 0 && d.ld1 % 4 == 0 && d.ld2 % 4 == 0 && aligned16(d.x) && (!d.out1 || aligned16(d.out1)) && (!d.out2 || aligned16(d.out2));
+  cudaError_t e = cudaSuccess;
+  AG_DISPATCH_FLOAT(d.dtype, T, {
+    if (vec) e = launch_pdl(rms_rows_kernel<T, 4>, dim3((unsigned)d.rows), dim3(kRmsThreads), 0, s, p);
+    else e = launch_pdl(rms_rows_kernel<T, 1>, dim3((unsigned)d.rows), dim3(kRmsThreads), 0, s, p);
+  });
+  return cuda_status(e, "rms_rows");
+}
+
+// ── clamped gated activation ────────────────────────────────────────────────
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ gu, long long ld_in, T* __restrict__ out, long long ld_out, long long rows, int ff, float limit) {
+  pdl_wait();
+  pdl_trigger();
+  const int packs = ff / VEC;
+  const long long total = rows * packs;
+  for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < total; i += (long long)gridDim.x * 256) {
+    const long long r = i / packs;
+    const int c = (int)(i - r * packs) * VEC;
+    const T* g = gu + r * ld_in + c;
+    if constexpr (VEC > 1) {
+      const Pack<T> a = ld16(g), b = ld16(g + ff);
+      Pack<T> o;
+      float t[VEC];
+#pragma unroll
+      for (int j = 0; j < VEC; j++) t[j] = clamped_glu_f(Cvt<T>::to(a.v[j]), Cvt<T>::to(b.v[j]), limit);
+      pack_from_floats<T>(o, t);
+      st16(out + r * ld_out + c, o);
+    } else {
+      out[r * ld_out + c] = Cvt<T>::from(clamped_glu_f(Cvt<T>::to(g[0]), Cvt<T>::to(g[ff]), limit));
+    }
+  }
+}
+
+Status clamped_glu(cudaStream_t s, DType dt, const void* gu, int64_t ld_in, void* out, int64_t ld_out, int64_t rows, int ff, float limit) {
+  if (rows <= 0 || ff <= 0) return Status::OK();
+  cudaError_t e = cudaSuccess;
+  AG_DISPATCH_FLOAT(dt, T, {
+    constexpr int N = Pack<T>::N;
+    const bool vec = ff % N == 0 && ld_in % N == 0 && ld_out % N == 0 && aligned16(gu) && aligned16(out);
+    const int64_t work = rows * (ff / (vec ? N : 1));
+    if (vec) e = launch_pdl(clamped_glu_kernel<T, N>, dim3((unsigned)grid_for(work, 256)), dim3(256), 0, s, (const T*)gu, (long long)ld_in, (T*)out, (long long)ld_out, (long long)rows, ff, limit);
+    else e = launch_pdl(clamped_glu_kernel<T, 1>, dim3((unsigned)grid_for(work, 256)), dim3(256), 0, s, (const T*)gu, (long long)ld_in, (T*)out, (long long)ld_out, (long long)rows, ff, limit);
+  });
+  return cuda_status(e, "clamped_glu");
+}
+
+}}  // namespace ag::k

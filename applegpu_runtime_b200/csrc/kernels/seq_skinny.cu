@@ -1,0 +1,205 @@
+// Linears of a step that carries at most 16 rows (a generated token per sequence, or a prompt portion of a few tokens).
+//
+// Such a product is bound by reading its K-major weight once. A warp owns RW weight rows (for the gated form RW / 2
+// gate rows and their up rows), its lanes split K in 16-byte pieces, and the input rows wait in shared memory as floats.
+// One launch serves up to three weights that read the same stream: the projections of a mixer and of the feed-forward
+// beside it depend on nothing but x, so a layer starts with a single launch whose prologue takes the RMS norms. The
+// float32 residual is updated in the epilogue of the output product.
+#include "common.cuh"
+#include "seq_kernels.h"
+
+namespace ag { namespace k {
+
+constexpr int kSsThreads = 256;
+constexpr int kSsWarps = kSsThreads / 32;
+constexpr size_t kSsMaxSmem = 200 * 1024;
+
+struct SsSeg {
+  const void* w; void* out; const float* norm_w;
+  long long ld, out_ld;
+  int n, mode, block0;               // block0: first block of this segment
+  float limit;
+};
+struct SsParams {
+  const float* x; const void* a; long long a_ld; float eps;
+  int rows, k, kp, n_seg;            // kp: k rounded up to whole 8-element packs (the weights hold zeros there)
+  SsSeg seg[kSeqSegs];
+};
+
+template <typename T, int MR, int RW>
+__global__ void __launch_bounds__(kSsThreads) seq_skinny_kernel(const SsParams p) {
+  extern __shared__ __align__(16) float s_in[];       // [MR][kp]
+  constexpr int VEC = 16 / (int)sizeof(T);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int si = 0;
+#pragma unroll
+  for (int i = 1; i < kSeqSegs; i++) if (i < p.n_seg && (int)blockIdx.x >= p.seg[i].block0) si = i;
+  const SsSeg sg = p.seg[si];
+  const bool glu = sg.mode == (int)SeqOut::Glu;
+  constexpr int GW = RW >= 2 ? RW / 2 : 1;
+  const int n0 = (((int)blockIdx.x - sg.block0) * kSsWarps + warp) * (glu ? GW : RW);
+  const T* W = reinterpret_cast<const T*>(sg.w);
+  // weight row of register slot r: gate rows in the first half of the slots, their up rows in the second
+  auto row_of = [&](int r) -> long long {
+    if (!glu) return n0 + r < sg.n ? n0 + r : -1;
+    const int c = n0 + r % GW;
+    return c < sg.n ? (long long)c + (r / GW) * (long long)sg.n : -1;
+  };
+  const T* wp[RW];
+#pragma unroll
+  for (int r = 0; r < RW; r++) { const long long q = row_of(r); wp[r] = q < 0 ? nullptr : W + q * sg.ld; }
+  // model weights are not written by the step: start them towards the L2 before waiting for the previous kernel
+#pragma unroll
+  for (int r = 0; r < RW; r++)
+    if (wp[r]) for (int kc = lane * 128 / (int)sizeof(T); kc < p.kp; kc += 32 * 128 / (int)sizeof(T)) asm volatile("prefetch.global.L2 [%0];" ::"l"(wp[r] + kc));
+  pdl_wait();
+  pdl_trigger();
+  const int m0 = (int)blockIdx.y * MR;
+  const int mrows = min(MR, p.rows - m0);
+  if (p.x) {
+    for (int m = warp; m < MR; m += kSsWarps) {
+      float* dst = s_in + (long long)m * p.kp;
+      if (m >= mrows) { for (int c = lane; c < p.kp; c += 32) dst[c] = 0.f; continue; }
+      const float* xr = p.x + (long long)(m0 + m) * p.k;
+      float sq = 0.f;
+      for (int c = lane; c < p.kp; c += 32) { const float v = c < p.k ? xr[c] : 0.f; dst[c] = v; sq = fmaf(v, v, sq); }
+      const float rs = 1.0f / sqrtf(warp_sum(sq) / (float)p.k + p.eps);
+      for (int c = lane; c < p.k; c += 32) dst[c] *= rs * sg.norm_w[c];
+    }
+  } else {
+    const T* A = reinterpret_cast<const T*>(p.a);
+    for (int i = threadIdx.x; i < MR * p.kp; i += kSsThreads) {
+      const int m = i / p.kp, c = i - m * p.kp;
+      s_in[i] = (m < mrows && c < p.k) ? Cvt<T>::to(A[(long long)(m0 + m) * p.a_ld + c]) : 0.f;
+    }
+  }
+  __syncthreads();
+  if (n0 >= sg.n) return;
+  float acc[MR][RW];
+#pragma unroll
+  for (int m = 0; m < MR; m++)
+#pragma unroll
+    for (int r = 0; r < RW; r++) acc[m][r] = 0.f;
+#pragma unroll 2
+  for (int kc = lane * VEC; kc < p.kp; kc += 32 * VEC) {
+    Pack<T> raw[RW];
+#pragma unroll
+    for (int r = 0; r < RW; r++) {
+      if (wp[r]) raw[r] = ld16_stream(wp[r] + kc);
+      else {
+#pragma unroll
+        for (int e = 0; e < VEC; e++) raw[r].v[e] = Cvt<T>::from(0.f);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < MR; m++) {
+      float af[VEC];
+#pragma unroll
+      for (int q = 0; q < VEC / 4; q++) {
+        const float4 a4 = *reinterpret_cast<const float4*>(s_in + (long long)m * p.kp + kc + q * 4);
+        af[q * 4] = a4.x; af[q * 4 + 1] = a4.y; af[q * 4 + 2] = a4.z; af[q * 4 + 3] = a4.w;
+      }
+#pragma unroll
+      for (int r = 0; r < RW; r++)
+#pragma unroll
+        for (int e = 0; e < VEC; e++) acc[m][r] = fmaf(af[e], Cvt<T>::to(raw[r].v[e]), acc[m][r]);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < MR; m++)
+#pragma unroll
+    for (int r = 0; r < RW; r++) acc[m][r] = warp_sum(acc[m][r]);
+  // every lane holds all sums; lane l finishes results l, l + 32, ...
+#pragma unroll
+  for (int m = 0; m < MR; m++) {
+    if (m >= mrows) continue;
+    const long long row = m0 + m;
+    if (glu) {
+      if constexpr (RW >= 2) {
+#pragma unroll
+        for (int r = 0; r < GW; r++) {
+          if (((m * GW + r) & 31) != lane || n0 + r >= sg.n) continue;
+          reinterpret_cast<T*>(sg.out)[row * sg.out_ld + n0 + r] = Cvt<T>::from(clamped_glu_f(acc[m][r], acc[m][GW + r], sg.limit));
+        }
+      }
+      continue;
+    }
+#pragma unroll
+    for (int r = 0; r < RW; r++) {
+      if (((m * RW + r) & 31) != lane || n0 + r >= sg.n) continue;
+      const long long o = row * sg.out_ld + n0 + r;
+      if (sg.mode == (int)SeqOut::Store) reinterpret_cast<T*>(sg.out)[o] = Cvt<T>::from(acc[m][r]);
+      else if (sg.mode == (int)SeqOut::StoreF32) reinterpret_cast<float*>(sg.out)[o] = acc[m][r];
+      else reinterpret_cast<float*>(sg.out)[o] += acc[m][r];
+    }
+  }
+}
+
+bool seq_skinny_fits(int64_t k) { return pad8(k) * (int64_t)sizeof(float) <= (int64_t)kSsMaxSmem; }
+
+template <typename T, int MR, int RW>
+static cudaError_t launch_ss(cudaStream_t s, const SsParams& p, dim3 grid, size_t smem) {
+  static bool attr = false;
+  if (!attr) {
+    cudaError_t e = cudaFuncSetAttribute(seq_skinny_kernel<T, MR, RW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSsMaxSmem);
+    if (e != cudaSuccess) return e;
+    attr = true;
+  }
+  return launch_pdl(seq_skinny_kernel<T, MR, RW>, grid, dim3(kSsThreads), smem, s, p);
+}
+template <typename T, int MR>
+static cudaError_t launch_ss_rw(cudaStream_t s, const SsParams& p, dim3 grid, size_t smem, int rw) {
+  return rw == 4 ? launch_ss<T, MR, 4>(s, p, grid, smem) : launch_ss<T, MR, 2>(s, p, grid, smem);
+}
+
+Status seq_skinny(cudaStream_t s, const SeqSkinnyDesc& d) {
+  if (d.rows < 1 || d.rows > kSeqSkinnyRows || d.n_seg < 1 || d.n_seg > kSeqSegs || (!d.x == !d.a)) return Status::invalid("seq_skinny: bad description");
+  if (!seq_skinny_fits(d.k)) return Status::unsupported("seq_skinny: input rows too long");
+  SsParams p;
+  p.x = d.x; p.a = d.a; p.a_ld = d.a_ld; p.eps = d.eps; p.rows = d.rows; p.k = d.k; p.kp = (int)pad8(d.k); p.n_seg = d.n_seg;
+  int mr = 1;
+  while (mr < d.rows && (size_t)(2 * mr) * p.kp * sizeof(float) <= kSsMaxSmem) mr *= 2;
+  int64_t total = 0;
+  for (int i = 0; i < d.n_seg; i++) total += d.seg[i].n * (d.seg[i].mode == SeqOut::Glu ? 2 : 1);
+  const int rw = total / 4 >= (int64_t)sm_count() * 16 ? 4 : 2;    // enough warps to fill the machine either way
+  int blocks = 0;
+  for (int i = 0; i < d.n_seg; i++) {
+    const SeqSeg& g = d.seg[i];
+    if (!g.w || !g.out || g.n < 1 || g.ld % 8 != 0 || g.ld < d.k || !aligned16(g.w) || (d.x && !g.norm_w)) return Status::invalid("seq_skinny: bad segment");
+    SsSeg& q = p.seg[i];
+    q.w = g.w; q.out = g.out; q.norm_w = g.norm_w; q.ld = g.ld; q.out_ld = g.out_ld; q.n = g.n; q.mode = (int)g.mode; q.limit = g.limit; q.block0 = blocks;
+    const int per = (g.mode == SeqOut::Glu ? rw / 2 : rw) * kSsWarps;
+    blocks += (g.n + per - 1) / per;
+  }
+  const size_t smem = (size_t)mr * p.kp * sizeof(float);
+  dim3 grid((unsigned)blocks, (unsigned)((d.rows + mr - 1) / mr));
+  cudaError_t e = cudaSuccess;
+  AG_DISPATCH_FLOAT(d.dtype, T, {
+    switch (mr) {
+      case 1: e = launch_ss_rw<T, 1>(s, p, grid, smem, rw); break;
+      case 2: e = launch_ss_rw<T, 2>(s, p, grid, smem, rw); break;
+      case 4: e = launch_ss_rw<T, 4>(s, p, grid, smem, rw); break;
+      case 8: e = launch_ss_rw<T, 8>(s, p, grid, smem, rw); break;
+      default: e = launch_ss_rw<T, 16>(s, p, grid, smem, rw); break;
+    }
+  });
+  return cuda_status(e, "seq_skinny");
+}
+
+__global__ void seq_advance_kernel(int* pos, int n_seq, int T, const int32_t* tok, int32_t* history, int* step, int max_steps) {
+  pdl_wait();
+  pdl_trigger();
+  const int st = history ? *step : 0;
+  __syncthreads();
+  for (int i = threadIdx.x; i < n_seq; i += blockDim.x) {
+    pos[i] += T;
+    if (history && st < max_steps) history[(long long)st * n_seq + i] = tok[i];
+  }
+  if (history && threadIdx.x == 0) *step = st + 1;
+}
+Status seq_advance(cudaStream_t s, int* pos, int n_seq, int T, const int32_t* tok, int32_t* history, int* step, int max_steps) {
+  cudaError_t e = launch_pdl(seq_advance_kernel, dim3(1), dim3(128), 0, s, pos, n_seq, T, tok, history, step, max_steps);
+  return cuda_status(e, "seq_advance");
+}
+
+}}  // namespace ag::k

@@ -10,6 +10,7 @@ import numpy as np
 
 from . import api as gpu
 from .gpt2 import gpt2_forward
+from . import seqmodel
 
 
 def _sample_token(logits_np, temperature=1.0, top_k=0, top_p=0.0, rng=None):
@@ -117,7 +118,14 @@ def greedy_generate(model, input_ids, max_tokens=50, use_cache=True, compiled=Tr
     step as one cooperative kernel instead of one kernel per op). `engine="tape"` keeps the cache the reference's way
     (concatenation, models/gpt2.py:122-127) and replays an op tape per step (`compiled`), the picked token staying
     on the device between steps. Models the decoder does not take (int8 weights, head dimension other than 64,
-    more than 16 sequences) use the tape engine."""
+    more than 16 sequences) use the tape engine.
+
+    Sequence models (seqmodel.py) run on their own engine, with the captured step unless `engine="direct"`; their prompts may
+    have different lengths, and the result is then a list of token lists."""
+    if isinstance(model, seqmodel.SequenceModel):
+        prompts = [input_ids] if np.ndim(input_ids[0]) == 0 else list(input_ids)
+        out = seqmodel.greedy_generate(model, prompts, max_tokens, use_graph=engine != "direct")
+        return np.asarray(out, dtype=np.int64) if len({len(o) for o in out}) == 1 else out
     ids = np.asarray(input_ids, dtype=np.int64)
     if ids.ndim == 1:
         ids = ids.reshape(1, -1)
@@ -170,6 +178,8 @@ def generate(model, input_ids, max_tokens=50, use_cache=True, temperature=1.0, t
     ids = list(input_ids)
     if temperature <= 0:
         return greedy_generate(model, ids, max_tokens, use_cache)[0].tolist()
+    if isinstance(model, seqmodel.SequenceModel):
+        return seqmodel.sample_generate(model, ids, max_tokens, lambda row: _sample_token(row, temperature=temperature, top_k=top_k, top_p=top_p))
     kv = None
     gpu.pool_drain()
     for _ in range(max_tokens):

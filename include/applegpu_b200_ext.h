@@ -287,6 +287,60 @@ APPLEGPU_API int32_t applegpu_gpt2_decoder_uses_graph(uint64_t decoder);
 APPLEGPU_API int32_t applegpu_gpt2_decoder_set_engine(uint64_t decoder, int32_t engine);
 APPLEGPU_API void applegpu_gpt2_decoder_destroy(uint64_t decoder);
 
+/* ── sequence models: layers with per-sequence memory, prompt portions, generation ──
+ * No counterpart in the reference. An engine owns the weights of a decoder-only model given as a list of layers
+ *     x <- x + (mixer(rms(x) norm1) + ff(rms(x) norm2))
+ * over a float32 stream x, and `slots` sequences of at most max_len tokens. Each run of a layer keeps its own memory per
+ * slot: mixer 1 (mLSTM) a float32 state, mixer 2 (latent attention) one cached row per token. Layers loop_start ..
+ * loop_stop - 1 run loop_times times (0: no loop): before each pass but the first the embedding output is added to x, before
+ * every pass a step vector.
+ *   create:  weight_ids = embed [vocab, width], head [vocab, P(width)], final norm f32 [width], step vectors f32
+ *            [loop_times, width] (0 without a loop), then eight per layer: norm1, norm2 (f32 [width]; 0 without a
+ *            feed-forward), the mixer's input rows [cols, P(width)], the output rows [width, P(K)] with K = P(heads * vdim) + ff
+ *            (mixer columns, then feed-forward columns) or heads * vdim without a feed-forward, gate rows | up rows
+ *            [2 ff, P(width)] (or 0), and three of the mixer's own:
+ *              mLSTM    input rows q | k | v | g; own: i rows | f rows [2 heads, P(width)], f32 bias [2 heads], f32 norm [heads * vdim]
+ *              latent   input rows q (per head: dim, rot_dim) | latent | rotated key part; own: f32 latent norm [kv_rank],
+ *                       uk rows, padded to P(heads * dim), | uv rows, padded to P(heads * vdim), [.., P(kv_rank)], and
+ *                       f32 (cos, sin) [>= max_len, rot_pairs, 2]
+ *            P(n) rounds up to a multiple of 8; padding holds zeros. All matrices share one float dtype, which is the
+ *            storage type of activations and caches. Returns a handle, 0 on failure (applegpu_ffi_last_error).
+ *   forward: the next n_tokens tokens of the n_seq sequences in slots slot0 .. (row s * n_tokens + t is token t of sequence
+ *            s). want: rows whose logits are copied to host_logits [n_want, vocab] (may be NULL); picked [n_want] receives
+ *            their greedy choices (may be NULL); host_layers (may be NULL) the stream after every layer run.
+ *   decode:  n_steps greedy tokens per sequence, continuing from the last forward with `picked` and one wanted row per
+ *            sequence; host_tokens [n_steps, n_seq]. use_graph replays one captured step per token.
+ *   reset:   empties n slots. length: tokens a slot holds. info: 0 launches of the last one-token step, 1 whether it was
+ *            replayed as a graph, 2 layer runs. */
+typedef struct { int32_t vocab, width, n_layers, loop_start, loop_stop, loop_times; float eps; } applegpu_seq_model;
+typedef struct {
+  int32_t mixer, heads, dim, vdim, rot_dim, rot_pairs, kv_rank, ff;
+  float gate_cap, score_scale, ff_limit;
+} applegpu_seq_layer;
+APPLEGPU_API uint64_t applegpu_seq_create(const applegpu_seq_model* model, const applegpu_seq_layer* layers, const uint64_t* weight_ids, uint32_t n_weights, uint32_t slots, uint32_t max_len);
+APPLEGPU_API int32_t applegpu_seq_forward(uint64_t engine, uint32_t slot0, uint32_t n_seq, const int32_t* tokens, uint32_t n_tokens, const int32_t* want, uint32_t n_want,
+                                          float* host_logits, int32_t* picked, float* host_layers);
+APPLEGPU_API int32_t applegpu_seq_decode(uint64_t engine, uint32_t slot0, uint32_t n_seq, uint32_t n_steps, int32_t* host_tokens, bool use_graph);
+APPLEGPU_API int32_t applegpu_seq_reset(uint64_t engine, uint32_t slot, uint32_t n);
+APPLEGPU_API int32_t applegpu_seq_length(uint64_t engine, uint32_t slot);
+APPLEGPU_API int32_t applegpu_seq_info(uint64_t engine, int32_t what);
+APPLEGPU_API void applegpu_seq_destroy(uint64_t engine);
+/* The mechanisms one by one, evaluated at once (operands contiguous; 0 on failure).
+ *   rms_norm     float32 x [.., n], float32 weight [n] -> x / sqrt(mean(x^2) + eps) * weight in out_dtype
+ *   clamped_glu  [.., 2 n] (gate | up) -> g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)
+ *   mlstm        proj [B, T, cols] (q | k | v | g), gates f32 [B, T, 2 heads] (i | f without bias), state f32 [B, S floats: per
+ *                head dim * vdim, then heads * dim, then heads; S rounded up to 4], updated in place -> [B, T, heads * vdim];
+ *                form 0: chunk-parallel, 1: token by token
+ *   latent_attention  proj [B, T, cols], up and rotation table as in seq_create, cache [B, max_len, P(kv_rank) + P(rot_dim)]
+ *                appended in place at pos (int32 [B], all equal to `past`) -> [B, T, heads * vdim]; form 0: keys and values
+ *                expanded per head (rotates the queries of proj in place), 1: in the latent space */
+APPLEGPU_API uint64_t applegpu_ffi_rms_norm(uint64_t x_id, uint64_t weight_id, float eps, int8_t out_dtype);
+APPLEGPU_API uint64_t applegpu_ffi_clamped_glu(uint64_t gate_up_id, float limit);
+APPLEGPU_API uint64_t applegpu_ffi_mlstm(uint64_t proj_id, uint64_t gates_id, uint64_t gate_bias_id, uint64_t norm_id, uint64_t state_id, uint32_t heads, uint32_t dim,
+                                         uint32_t vdim, float gate_cap, float eps, int32_t form);
+APPLEGPU_API uint64_t applegpu_ffi_latent_attention(uint64_t proj_id, uint64_t norm_id, uint64_t up_id, uint64_t rot_id, uint64_t cache_id, uint64_t pos_id, uint32_t past,
+                                                    uint32_t heads, uint32_t dim, uint32_t rot_dim, uint32_t vdim, uint32_t kv_rank, float scale, float eps, int32_t form);
+
 /* ── attention without device allocation ───────────────────────────────────────
  * No counterpart in the reference.
  *
