@@ -452,11 +452,12 @@ def mlstm(proj, gates, gate_bias, norm, state, heads, dim, vdim, gate_cap, eps=1
     return GpuTensor(_L().applegpu_ffi_mlstm(proj.id, gates.id, gate_bias.id, norm.id, state.id, heads, dim, vdim, float(gate_cap), float(eps), 0 if chunked else 1))
 
 
-def latent_attention(proj, norm, up, rot_table, cache, pos, past, heads, dim, rot_dim, vdim, kv_rank, scale, eps=1e-5, expanded=True):
+def latent_attention(proj, norm, up, rot_table, cache, pos, past, heads, dim, rot_dim, vdim, kv_rank, scale, eps=1e-5, form="expanded"):
     """Causal latent attention of T new rows per sequence; the cache is appended in place and proj's queries may be rotated in place.
-    `expanded=False` attends in the latent space. Returns [B, T, heads * vdim]."""
+    form: "expanded" (keys and values per head), "latent" (attends in the latent space), "tensor" (expanded, on the tensor-core
+    kernel or an error). Returns [B, T, heads * vdim]."""
     return GpuTensor(_L().applegpu_ffi_latent_attention(proj.id, norm.id, up.id, 0 if rot_table is None else rot_table.id, cache.id, pos.id, int(past), heads, dim, rot_dim, vdim,
-                                                        kv_rank, float(scale), float(eps), 0 if expanded else 1))
+                                                        kv_rank, float(scale), float(eps), {"expanded": 0, "latent": 1, "tensor": 2}[form]))
 
 
 _ACT_CODES = {None: 0, "none": 0, "gelu": 1, "gelu_exact": 2, "relu": 3}

@@ -78,6 +78,21 @@ struct Scope {
     cudaEventRecord(g_spans[idx].b, DeviceCtx::get().stream);
   }
 };
+// Spans opened from other files: an index for end(), or -1 when nothing is being timed.
+long begin(const std::string& name, double work) {
+  if (!g_on || !wanted(name)) return -1;
+  Span sp; sp.name = name; sp.work = work;
+  std::lock_guard<std::mutex> g(g_mu);
+  if (!take_event(&sp.a) || !take_event(&sp.b)) return -1;
+  cudaEventRecord(sp.a, DeviceCtx::get().stream);
+  g_spans.push_back(sp);
+  return (long)g_spans.size() - 1;
+}
+void end(long i) {
+  if (i < 0) return;
+  std::lock_guard<std::mutex> g(g_mu);
+  if (i < (long)g_spans.size()) cudaEventRecord(g_spans[i].b, DeviceCtx::get().stream);
+}
 // "name count total_ms work" per line; work = algorithmic flops (GEMM, attention) or bytes (the rest).
 std::string report() {
   DeviceCtx& ctx = DeviceCtx::get();

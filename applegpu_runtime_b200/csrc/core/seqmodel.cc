@@ -22,8 +22,17 @@
 namespace ag {
 
 extern std::atomic<uint64_t> g_launch_count;
+namespace profile { long begin(const std::string& name, double work); void end(long i); bool enabled(); }
 
 namespace {
+
+// One timed launch (or group of launches) of a step; work is flops for products and prompt attention, bytes otherwise.
+struct Span {
+  long i;
+  Span(const char* name, double work) : i(profile::begin(name, work)) {}
+  ~Span() { profile::end(i); }
+};
+double product(double m, double n, double kdim) { return 2.0 * m * n * kdim; }
 
 constexpr int kShortT = 16;             // tokens per sequence up to which mixers run token by token
 constexpr int kMaxRows = 8192;          // rows of a step; longer portions are cut
@@ -57,7 +66,7 @@ struct Mixer {
   virtual size_t slot_bytes(int max_len) const = 0;
   virtual bool clear_on_reset() const = 0;
   virtual Status check(const SeqModelCfg& m, int max_len) const = 0;
-  virtual size_t kv_bytes(int) const { return 0; }   // expanded keys and values of a sequence
+  virtual size_t kv_bytes(const int*, int, int) const { return 0; }   // expanded keys and values of a step
   virtual size_t work_bytes(int n_seq, int T, int max_len) const = 0;
   virtual Status run(const StepCtx& x, void* proj, int64_t ld, const float* gates, void* mem, int max_len, const int* pos, void* y, int64_t y_ld, void* work, void* kv,
                      float eps, int* launches) const = 0;
@@ -101,6 +110,8 @@ struct MlstmMixer : Mixer {
     d.state_stride = (int64_t)(slot_bytes(max_len) / sizeof(float));
     d.state = static_cast<float*>(mem) + x.slot0 * d.state_stride;
     d.y = y; d.y_ld = y_ld; d.work = work;
+    const double row = (2.0 * c.dim + 3.0 * c.vdim) * dtype_size(dtype), mem_rw = 8.0 * c.dim * c.vdim;      // q k v g y; the state read and written once
+    Span span(x.T <= kShortT ? "mlstm_step" : "mlstm_prefill", c.heads * (row * x.rows() + mem_rw * x.n_seq));
     if (x.T <= kShortT) { *launches += 1; return k::mlstm_step(x.s, d); }
     *launches += 4;
     return k::mlstm_prefill(x.s, d);
@@ -121,7 +132,16 @@ struct LatentMixer : Mixer {
       return Status::invalid("rotation table");
     return Status::OK();
   }
-  size_t kv_bytes(int max_len) const override { return (size_t)max_len * kv_cols() * dtype_size(dtype); }
+  size_t kv_bytes(const int* host_len, int n_seq, int T) const override {
+    size_t worst = 0;
+    for (int i = 0; i < n_seq;) {
+      int n = 1;
+      while (i + n < n_seq && host_len[i + n] == host_len[i]) n++;
+      worst = std::max(worst, (size_t)n * (host_len[i] + T));
+      i += n;
+    }
+    return worst * kv_cols() * dtype_size(dtype);
+  }
   size_t work_bytes(int n_seq, int T, int max_len) const override {
     return T <= kShortT ? k::latent_decode_work_bytes(n_seq * T, c.heads, c.kv_rank, c.rot_dim, max_len) : 0;
   }
@@ -138,21 +158,40 @@ struct LatentMixer : Mixer {
     const uint8_t* wkv = static_cast<const uint8_t*>(w[kWAux1].data());
     const int64_t w_ld = pad8(c.kv_rank), v_off = pad8((int64_t)c.heads * c.dim);
     d.w_uk = wkv; d.w_uv = wkv + (size_t)v_off * w_ld * esz; d.w_ld = w_ld; d.y = y; d.y_ld = y_ld;
-    if (x.T <= kShortT) { *launches += 3; return k::latent_decode(x.s, d, work); }
-    AG_RETURN_IF_ERROR(k::latent_append(x.s, d));
+    if (x.T <= kShortT) {
+      double keys = 0;
+      for (int i = 0; i < x.n_seq; i++) keys += x.host_len[i] + x.T;
+      Span span("latent_decode", esz * (keys * cld() + (double)c.heads * (c.dim + c.vdim) * c.kv_rank));
+      *launches += 3;
+      return k::latent_decode(x.s, d, work);
+    }
+    {
+      Span span("latent_append", esz * (double)x.rows() * (2.0 * c.heads * c.rot_dim + 2.0 * (c.kv_rank + c.rot_dim)));
+      AG_RETURN_IF_ERROR(k::latent_append(x.s, d));
+    }
     *launches += 1;
-    for (int i = 0; i < x.n_seq; i++) {
+    // sequences that hold equally many tokens share the two launches
+    for (int i = 0; i < x.n_seq;) {
+      int n = 1;
+      while (i + n < x.n_seq && x.host_len[i + n] == x.host_len[i]) n++;
       const int past = x.host_len[i], keys = past + x.T;
       uint8_t* cache = static_cast<uint8_t*>(d.cache) + (size_t)i * slot_bytes(max_len);
-      AG_RETURN_IF_ERROR(k::matmul(x.s, linear_desc(dtype, cache, cld(), keys, c.kv_rank, wkv, w_ld, kv_cols(), kv, kv_cols(), false, nullptr)));
+      {
+        Span span("latent_expand", n * product(keys, kv_cols(), c.kv_rank));
+        k::GemmDesc g = linear_desc(dtype, cache, cld(), keys, c.kv_rank, wkv, w_ld, kv_cols(), kv, kv_cols(), false, nullptr);
+        g.batch = n; g.a_batch = d.seq_stride; g.c_batch = keys * kv_cols();
+        AG_RETURN_IF_ERROR(k::matmul(x.s, g));
+      }
       k::LatentPrefillDesc p;
-      p.dtype = dtype; p.T = x.T; p.past = past; p.heads = c.heads; p.dim = c.dim; p.rot_dim = c.rot_dim; p.vdim = c.vdim; p.scale = c.score_scale;
-      p.q = static_cast<uint8_t*>(proj) + (size_t)i * x.T * ld * esz; p.q_ld = ld;
-      p.kv = kv; p.kv_ld = kv_cols(); p.v_off = v_off;
-      p.k_rot = cache + (size_t)pad8(c.kv_rank) * esz; p.k_rot_ld = cld();
-      p.y = static_cast<uint8_t*>(y) + (size_t)i * x.T * y_ld * esz; p.y_ld = y_ld;
+      p.dtype = dtype; p.n_seq = n; p.T = x.T; p.past = past; p.heads = c.heads; p.dim = c.dim; p.rot_dim = c.rot_dim; p.vdim = c.vdim; p.scale = c.score_scale;
+      p.q = static_cast<uint8_t*>(proj) + (size_t)i * x.T * ld * esz; p.q_ld = ld; p.q_b = x.T * ld;
+      p.kv = kv; p.kv_ld = kv_cols(); p.v_off = v_off; p.kv_b = keys * kv_cols();
+      p.k_rot = cache + (size_t)pad8(c.kv_rank) * esz; p.k_rot_ld = cld(); p.k_rot_b = d.seq_stride;
+      p.y = static_cast<uint8_t*>(y) + (size_t)i * x.T * y_ld * esz; p.y_ld = y_ld; p.y_b = x.T * y_ld;
+      Span span("latent_prefill", 2.0 * n * c.heads * (c.dim + c.rot_dim + c.vdim) * (past * (double)x.T + 0.5 * x.T * (x.T + 1.0)));
       AG_RETURN_IF_ERROR(k::latent_prefill(x.s, p));
       *launches += 2;
+      i += n;
     }
     return Status::OK();
   }
@@ -183,17 +222,21 @@ struct SeqEngine {
   int64_t cat_k(const SeqLayerCfg& c) const { return c.ff ? y_cols(c) + c.ff : (int64_t)c.heads * c.vdim; }
   int64_t cat_ld(const SeqLayerCfg& c) const { return pad8(cat_k(c)); }
 
-  // Grows a buffer; graphs hold the old addresses, so they are dropped and recorded again.
-  Status ensure(Scratch* b, size_t bytes, bool zero = false) {
+  // Grows a buffer (by half at least); graphs hold the old addresses of the buffers their step uses, so they are dropped and
+  // recorded again.
+  Status ensure(Scratch* b, size_t bytes, bool zero = false, bool in_graphs = true) {
     if (b->buf && b->buf->capacity >= bytes) return Status::OK();
     cudaStream_t s = DeviceCtx::get().stream;
-    if (b->buf) { cudaStreamSynchronize(s); drop_graphs(); }
+    if (b->buf) {
+      bytes = std::max(bytes, b->buf->capacity + b->buf->capacity / 2);
+      if (in_graphs) { cudaStreamSynchronize(s); drop_graphs(); }
+    }
     b->buf.reset();
     AG_RETURN_IF_ERROR(Shared::get().pool.acquire(bytes, &b->buf));
     if (zero && cudaMemsetAsync(b->buf->ptr, 0, b->buf->capacity, s) != cudaSuccess) return Status::compute("sequence engine: clear");
     return Status::OK();
   }
-  Status reserve(int n_seq, int T, int n_want) {
+  Status reserve(int slot0, int n_seq, int T, int n_want) {
     const size_t R = (size_t)n_seq * T;
     int64_t pc = 0, gc = 1, fc = 1, cc = 0; size_t wb = 256, kb = 256;
     for (size_t l = 0; l < cfg.layers.size(); l++) {
@@ -201,14 +244,14 @@ struct SeqEngine {
       pc = std::max(pc, pad8(mixers[l]->proj_cols())); gc = std::max<int64_t>(gc, mixers[l]->gate_cols());
       fc = std::max(fc, pad8(2 * (int64_t)c.ff)); cc = std::max(cc, cat_ld(c));
       wb = std::max(wb, mixers[l]->work_bytes(n_seq, T, max_len));
-      if (T > kShortT) kb = std::max(kb, mixers[l]->kv_bytes(max_len));
+      if (T > kShortT) kb = std::max(kb, mixers[l]->kv_bytes(len.data() + slot0, n_seq, T));
     }
     AG_RETURN_IF_ERROR(ensure(&x, R * cfg.width * sizeof(float)));
     AG_RETURN_IF_ERROR(ensure(&proj, R * pc * esz()));
     AG_RETURN_IF_ERROR(ensure(&gates, R * gc * sizeof(float)));
     AG_RETURN_IF_ERROR(ensure(&cat, R * cc * esz(), true));
     AG_RETURN_IF_ERROR(ensure(&work, wb));
-    AG_RETURN_IF_ERROR(ensure(&kv, kb));
+    AG_RETURN_IF_ERROR(ensure(&kv, kb, false, false));
     const size_t hrows = std::max<size_t>(R > k::kSeqSkinnyRows || !skinny_ok() ? R : 1, (size_t)n_want);
     AG_RETURN_IF_ERROR(ensure(&h1, hrows * pad8(cfg.width) * esz()));
     AG_RETURN_IF_ERROR(ensure(&h2, hrows * pad8(cfg.width) * esz()));
@@ -257,17 +300,30 @@ struct SeqEngine {
         seg(W[kWIn], mx.proj_cols(), W[kWNorm1], k::SeqOut::Store, proj.ptr(), pl);
         if (mx.gate_cols()) seg(W[kWAux0], mx.gate_cols(), W[kWNorm1], k::SeqOut::StoreF32, gates.ptr(), mx.gate_cols());
         if (c.ff) seg(W[kWFf], c.ff, W[kWNorm2], k::SeqOut::Glu, ff_out, cl);
+        Span span("skinny_in", esz() * (double)wl * (mx.proj_cols() + mx.gate_cols() + 2.0 * c.ff));
         AG_RETURN_IF_ERROR(count(k::seq_skinny(st.s, d)));
       } else {
         n.w1 = f32(W[kWNorm1]); n.out1 = h1.ptr(); n.ld1 = wl;
         if (c.ff) { n.w2 = f32(W[kWNorm2]); n.out2 = h2.ptr(); n.ld2 = wl; }
-        AG_RETURN_IF_ERROR(count(k::rms_rows(st.s, n)));
-        AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h1.ptr(), wl, R, cfg.width, W[kWIn].data(), wl, mx.proj_cols(), proj.ptr(), pl, false, nullptr))));
-        if (mx.gate_cols())
+        {
+          Span span("rms_rows", (4.0 + (c.ff ? 2.0 : 1.0) * esz()) * R * cfg.width);
+          AG_RETURN_IF_ERROR(count(k::rms_rows(st.s, n)));
+        }
+        {
+          Span span("linear_in", product(R, mx.proj_cols(), cfg.width));
+          AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h1.ptr(), wl, R, cfg.width, W[kWIn].data(), wl, mx.proj_cols(), proj.ptr(), pl, false, nullptr))));
+        }
+        if (mx.gate_cols()) {
+          Span span("linear_gates", product(R, mx.gate_cols(), cfg.width));
           AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h1.ptr(), wl, R, cfg.width, W[kWAux0].data(), wl, mx.gate_cols(), gates.ptr(), mx.gate_cols(), true, nullptr))));
+        }
         if (c.ff) {
           const int64_t fl = pad8(2 * (int64_t)c.ff);
-          AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h2.ptr(), wl, R, cfg.width, W[kWFf].data(), wl, 2 * (int64_t)c.ff, gu.ptr(), fl, false, nullptr))));
+          {
+            Span span("linear_ff", product(R, 2.0 * c.ff, cfg.width));
+            AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h2.ptr(), wl, R, cfg.width, W[kWFf].data(), wl, 2 * (int64_t)c.ff, gu.ptr(), fl, false, nullptr))));
+          }
+          Span span("clamped_glu", 3.0 * esz() * R * c.ff);
           AG_RETURN_IF_ERROR(count(k::clamped_glu(st.s, dtype, gu.ptr(), fl, ff_out, cl, R, c.ff, c.ff_limit)));
         }
       }
@@ -276,8 +332,10 @@ struct SeqEngine {
         k::SeqSkinnyDesc d;
         d.dtype = dtype; d.rows = R; d.k = (int)cat_k(c); d.a = cat.ptr(); d.a_ld = cl; d.n_seg = 1;
         d.seg[0].w = W[kWOut].data(); d.seg[0].ld = cl; d.seg[0].n = cfg.width; d.seg[0].mode = k::SeqOut::AddF32; d.seg[0].out = X; d.seg[0].out_ld = cfg.width;
+        Span span("skinny_out", esz() * (double)cl * cfg.width);
         AG_RETURN_IF_ERROR(count(k::seq_skinny(st.s, d)));
       } else {
+        Span span("linear_out", product(R, cfg.width, cat_k(c)));
         AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, cat.ptr(), cl, R, cat_k(c), W[kWOut].data(), cl, cfg.width, X, cfg.width, true, X))));
       }
       if (layers_out) {
@@ -291,6 +349,7 @@ struct SeqEngine {
   // Logits of n rows of x: all of them in order (map null), or the ones listed in the device array `map`.
   Status enqueue_head(cudaStream_t s, int n, const int32_t* map) {
     const int64_t wl = pad8(cfg.width);
+    Span span(n <= k::kSeqSkinnyRows ? "skinny_head" : "linear_head", n <= k::kSeqSkinnyRows ? esz() * (double)wl * cfg.vocab : product(n, cfg.vocab, cfg.width));
     const bool skinny = n <= k::kSeqSkinnyRows && k::seq_skinny_fits(cfg.width);
     k::SeqSkinnyDesc d;
     d.dtype = dtype; d.rows = n; d.k = cfg.width; d.eps = cfg.eps; d.n_seg = 1;
@@ -323,7 +382,7 @@ struct SeqEngine {
   // capture), the second one is captured, later ones replay the graph.
   Status run_step(cudaStream_t s, int slot0, int n, bool use_graph) {
     last_graph = false;
-    if (!use_graph) { AG_RETURN_IF_ERROR(enqueue_step(s, slot0, n)); }
+    if (!use_graph || profile::enabled()) { AG_RETURN_IF_ERROR(enqueue_step(s, slot0, n)); }
     else {
       const auto key = std::make_pair(slot0, n);
       auto it = graphs.find(key);
@@ -479,7 +538,7 @@ Status seq_forward(uint64_t handle, int slot0, int n_seq, const int32_t* tokens,
     bool in_order = nw == n_seq * Ts;
     for (int i = 0; i < nw && in_order; i++) in_order = rows[i] == i;
     const bool one_token = T == 1 && !layers_out && (nw == 0 || in_order);
-    AG_RETURN_IF_ERROR(e->reserve(n_seq, Ts, one_token ? n_seq : nw));
+    AG_RETURN_IF_ERROR(e->reserve(slot0, n_seq, Ts, one_token ? n_seq : nw));
     AG_RETURN_IF_ERROR(copy_ok(cudaMemcpyAsync(e->tok.ptr(), toks.data(), toks.size() * 4, cudaMemcpyHostToDevice, s)));
     if (one_token) {
       // the step greedy generation replays; the picked token is ignored unless asked for
@@ -533,7 +592,7 @@ Status seq_decode(uint64_t handle, int slot0, int n_seq, int n_steps, int32_t* h
   DeviceCtx& ctx = DeviceCtx::get();
   AG_RETURN_IF_ERROR(ctx.make_current());
   cudaStream_t s = ctx.stream;
-  AG_RETURN_IF_ERROR(e->reserve(n_seq, 1, n_seq));
+  AG_RETURN_IF_ERROR(e->reserve(slot0, n_seq, 1, n_seq));
   if (cudaMemsetAsync(e->step.ptr(), 0, sizeof(int), s) != cudaSuccess) return Status::compute("sequence engine: step counter");
   for (int i = 0; i < n_steps; i++) AG_RETURN_IF_ERROR(e->run_step(s, slot0, n_seq, use_graph));
   const cudaError_t ce = cudaMemcpyAsync(host_tokens, e->history.ptr(), (size_t)n_steps * n_seq * 4, cudaMemcpyDeviceToHost, s);

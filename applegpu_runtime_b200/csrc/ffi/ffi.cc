@@ -1520,19 +1520,18 @@ uint64_t applegpu_ffi_latent_attention(uint64_t proj_id, uint64_t norm_id, uint6
     }
     AG_RETURN_IF_ERROR(k::latent_append(cs, d));
     const int64_t cols = v_off + k::pad8(H * vdim), keys = (int64_t)past + T;
-    AG_RETURN_IF_ERROR(new_tensor({keys, cols}, dt, &work));
-    for (int64_t i = 0; i < B; i++) {
-      uint8_t* cache = static_cast<uint8_t*>(d.cache) + (size_t)i * d.seq_stride * esz;
-      k::GemmDesc m;
-      m.dtype = dt; m.b_dtype = dt; m.a = cache; m.b = d.w_uk; m.c = work.data(); m.m = keys; m.n = cols; m.k = kv_rank; m.batch = 1;
-      m.a_row = cld; m.a_col = 1; m.a_batch = 0; m.b_row = 1; m.b_col = w_ld; m.b_batch = 0; m.c_row = cols; m.c_batch = 0;
-      AG_RETURN_IF_ERROR(k::matmul(cs, m));
-      k::LatentPrefillDesc p;
-      p.dtype = dt; p.T = (int)T; p.past = (int)past; p.heads = (int)heads; p.dim = (int)dim; p.rot_dim = (int)rot_dim; p.vdim = (int)vdim; p.scale = scale;
-      p.q = static_cast<uint8_t*>(d.proj) + (size_t)i * T * d.ld * esz; p.q_ld = d.ld; p.kv = work.data(); p.kv_ld = cols; p.v_off = v_off;
-      p.k_rot = cache + (size_t)k::pad8(kv_rank) * esz; p.k_rot_ld = cld; p.y = static_cast<uint8_t*>(out.data()) + (size_t)i * T * d.y_ld * esz; p.y_ld = d.y_ld;
-      AG_RETURN_IF_ERROR(k::latent_prefill(cs, p));
-    }
+    AG_RETURN_IF_ERROR(new_tensor({B, keys, cols}, dt, &work));
+    k::GemmDesc m;
+    m.dtype = dt; m.b_dtype = dt; m.a = d.cache; m.b = d.w_uk; m.c = work.data(); m.m = keys; m.n = cols; m.k = kv_rank; m.batch = B;
+    m.a_row = cld; m.a_col = 1; m.a_batch = d.seq_stride; m.b_row = 1; m.b_col = w_ld; m.b_batch = 0; m.c_row = cols; m.c_batch = keys * cols;
+    AG_RETURN_IF_ERROR(k::matmul(cs, m));
+    k::LatentPrefillDesc p;
+    p.dtype = dt; p.n_seq = (int)B; p.T = (int)T; p.past = (int)past; p.heads = (int)heads; p.dim = (int)dim; p.rot_dim = (int)rot_dim; p.vdim = (int)vdim; p.scale = scale;
+    p.q = d.proj; p.q_ld = d.ld; p.q_b = T * d.ld; p.kv = work.data(); p.kv_ld = cols; p.v_off = v_off; p.kv_b = keys * cols;
+    p.k_rot = static_cast<uint8_t*>(d.cache) + (size_t)k::pad8(kv_rank) * esz; p.k_rot_ld = cld; p.k_rot_b = d.seq_stride;
+    p.y = out.data(); p.y_ld = d.y_ld; p.y_b = T * d.y_ld;
+    if (form == 2) return k::latent_prefill_tc_eligible(p) ? k::latent_prefill_tc(cs, p) : Status::unsupported("these sizes do not take the tensor-core kernel");
+    AG_RETURN_IF_ERROR(k::latent_prefill(cs, p));
     return Status::OK();
   };
   const Status s = run();

@@ -21,6 +21,7 @@
 // latency nor the last product's latency leaves the softmax warps idle. All waits are bounded.
 #include "common.cuh"
 #include "sm100.cuh"
+#include "tc_math.cuh"
 #include <cuda.h>
 #include <cstdlib>
 #include <type_traits>
@@ -42,46 +43,6 @@ constexpr int kKVBytes = kKV * kD * 2;                   // 8 KB: one K or V blo
 constexpr int kKVStages = 4;                             // K and V rings: loads run up to four blocks ahead of the MMAs
 constexpr int kAttnSmem = 2 * kQBytes /*Q, two tiles*/ + kKVStages * kKVBytes /*K*/ + kKVStages * kKVBytes /*V*/ + 1024;
 constexpr int kAttnTmemCols = 256;                       // S: 2 x 64 (P over the head of each), O: 64
-
-__device__ __forceinline__ float ex2_approx(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-// Blackwell's packed fp32 pipe: two independent fp32 operations per instruction on a 64-bit register pair, and the
-// three-input maximum. The softmax below is bound by instruction issue and the MUFU pipe, not by arithmetic.
-__device__ __forceinline__ float max3_f32(float a, float b, float c) {
-  float d;
-  asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
-  return d;
-}
-__device__ __forceinline__ uint64_t pack_f32x2(float lo, float hi) {
-  uint64_t r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
-  return r;
-}
-__device__ __forceinline__ void unpack_f32x2(uint64_t v, float& lo, float& hi) {
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
-}
-__device__ __forceinline__ uint64_t fma_f32x2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ uint64_t add_f32x2(uint64_t a, uint64_t b) {
-  uint64_t d;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-template <typename T> __device__ __forceinline__ uint32_t pack2_t(float a, float b);
-template <> __device__ __forceinline__ uint32_t pack2_t<__nv_bfloat16>(float a, float b) {
-  __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-  return *reinterpret_cast<uint32_t*>(&v);
-}
-template <> __device__ __forceinline__ uint32_t pack2_t<__half>(float a, float b) {
-  __half2 v = __floats2half2_rn(a, b);
-  return *reinterpret_cast<uint32_t*>(&v);
-}
 
 struct AttnParams {
   void* o;

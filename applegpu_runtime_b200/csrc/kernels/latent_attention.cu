@@ -85,7 +85,7 @@ Status latent_append(cudaStream_t s, const LatentDesc& d) {
 // ── prefill, CUDA cores ─────────────────────────────────────────────────────
 struct LpParams {
   const void* q; const void* kv; const void* kr; void* y;
-  long long q_ld, kv_ld, v_off, kr_ld, y_ld;
+  long long q_ld, kv_ld, v_off, kr_ld, y_ld, q_b, kv_b, kr_b, y_b;
   int T, past, heads, dim, rot, vdim;
   float scale;
 };
@@ -105,9 +105,10 @@ __global__ void __launch_bounds__(256) latent_prefill_kernel(const LpParams p) {
   pdl_trigger();
   const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * TQ, h = blockIdx.y;     // longest rows first
   const int rows = min(TQ, p.T - q0);
-  const T* Q = reinterpret_cast<const T*>(p.q) + (long long)h * D;
-  const T* KV = reinterpret_cast<const T*>(p.kv);
-  const T* KR = reinterpret_cast<const T*>(p.kr);
+  const long long b = blockIdx.z;
+  const T* Q = reinterpret_cast<const T*>(p.q) + b * p.q_b + (long long)h * D;
+  const T* KV = reinterpret_cast<const T*>(p.kv) + b * p.kv_b;
+  const T* KR = reinterpret_cast<const T*>(p.kr) + b * p.kr_b;
   for (int i = threadIdx.x; i < TQ * D; i += 256) {
     const int t = i / D;
     sq[i] = t < rows ? Cvt<T>::to(Q[(long long)(q0 + t) * p.q_ld + i % D]) * p.scale : 0.f;
@@ -156,31 +157,34 @@ __global__ void __launch_bounds__(256) latent_prefill_kernel(const LpParams p) {
     }
   }
   __syncthreads();
-  T* Y = reinterpret_cast<T*>(p.y) + (long long)h * E;
+  T* Y = reinterpret_cast<T*>(p.y) + b * p.y_b + (long long)h * E;
   for (int i = threadIdx.x; i < rows * E; i += 256) Y[(long long)(q0 + i / E) * p.y_ld + i % E] = Cvt<T>::from(so[i] / s_l[i / E]);
 }
 
 template <typename T, int TQ>
-static cudaError_t launch_lp(cudaStream_t s, const LpParams& p, size_t smem) {
+static cudaError_t launch_lp(cudaStream_t s, const LpParams& p, int n_seq, size_t smem) {
   static bool attr = false;
   if (!attr) {
     cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel<T, TQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
     if (e != cudaSuccess) return e;
     attr = true;
   }
-  return launch_pdl(latent_prefill_kernel<T, TQ>, dim3((unsigned)((p.T + TQ - 1) / TQ), (unsigned)p.heads), dim3(256), smem, s, p);
+  return launch_pdl(latent_prefill_kernel<T, TQ>, dim3((unsigned)((p.T + TQ - 1) / TQ), (unsigned)p.heads, (unsigned)n_seq), dim3(256), smem, s, p);
 }
 
 Status latent_prefill(cudaStream_t s, const LatentPrefillDesc& d) {
-  if (d.T < 1 || d.past < 0 || d.heads < 1 || d.heads > 65535 || d.dim < 1 || d.rot_dim < 0 || d.vdim < 1 || !d.q || !d.kv || !d.y) return Status::invalid("latent prefill: bad description");
+  if (d.T < 1 || d.past < 0 || d.heads < 1 || d.heads > 65535 || d.dim < 1 || d.rot_dim < 0 || d.vdim < 1 || !d.q || !d.kv || !d.y || d.n_seq < 1 || d.n_seq > 65535)
+    return Status::invalid("latent prefill: bad description");
+  if (latent_prefill_tc_eligible(d)) return latent_prefill_tc(s, d);
   LpParams p;
   p.q = d.q; p.kv = d.kv; p.kr = d.k_rot; p.y = d.y; p.q_ld = d.q_ld; p.kv_ld = d.kv_ld; p.v_off = d.v_off; p.kr_ld = d.k_rot_ld; p.y_ld = d.y_ld;
+  p.q_b = d.q_b; p.kv_b = d.kv_b; p.kr_b = d.k_rot_b; p.y_b = d.y_b;
   p.T = d.T; p.past = d.past; p.heads = d.heads; p.dim = d.dim; p.rot = d.rot_dim; p.vdim = d.vdim; p.scale = d.scale;
   auto smem = [&](int tq) { return ((size_t)tq * (2 * (d.dim + d.rot_dim) + 1) + 2 * (size_t)tq * d.vdim + (size_t)tq * (tq + 1) + 3 * tq) * sizeof(float); };
   const size_t lim = 220 * 1024;
   if (smem(8) > lim) return Status::unsupported("latent prefill: head too large");
   cudaError_t e = cudaSuccess;
-  AG_DISPATCH_FLOAT(d.dtype, T, (e = smem(32) <= lim ? launch_lp<T, 32>(s, p, smem(32)) : smem(16) <= lim ? launch_lp<T, 16>(s, p, smem(16)) : launch_lp<T, 8>(s, p, smem(8))));
+  AG_DISPATCH_FLOAT(d.dtype, T, (e = smem(32) <= lim ? launch_lp<T, 32>(s, p, d.n_seq, smem(32)) : smem(16) <= lim ? launch_lp<T, 16>(s, p, d.n_seq, smem(16)) : launch_lp<T, 8>(s, p, d.n_seq, smem(8))));
   return cuda_status(e, "latent prefill");
 }
 

@@ -93,18 +93,21 @@ struct LatentDesc {
 inline int64_t latent_cache_ld(int kv_rank, int rot_dim) { return pad8(kv_rank) + pad8(rot_dim); }
 // Rotates q in place, norms the latent, rotates the key part and appends both to the cache (rows pos .. pos + T).
 Status latent_append(cudaStream_t s, const LatentDesc& d);
-// Attention of T new rows of ONE sequence over `keys` cached rows of which `past` lie before them, with keys and values
-// expanded per head: kv rows [keys, kv_ld] hold k (heads * dim) | v at column v_off (heads * vdim).
+// Attention of T new rows per sequence over past + T cached rows, with keys and values expanded per head: kv rows
+// [past + T, kv_ld] hold k (heads * dim) | v at column v_off (heads * vdim). The *_b strides step from sequence to sequence.
 struct LatentPrefillDesc {
   DType dtype;
-  int T, past, heads, dim, rot_dim, vdim;
+  int n_seq = 1, T, past, heads, dim, rot_dim, vdim;
   float scale;
   const void* q; int64_t q_ld;
   const void* kv; int64_t kv_ld; int64_t v_off;
   const void* k_rot; int64_t k_rot_ld;
   void* y; int64_t y_ld;
+  int64_t q_b = 0, kv_b = 0, k_rot_b = 0, y_b = 0;
 };
-Status latent_prefill(cudaStream_t s, const LatentPrefillDesc& d);
+Status latent_prefill(cudaStream_t s, const LatentPrefillDesc& d);      // picks one of the two below
+bool latent_prefill_tc_eligible(const LatentPrefillDesc& d);            // 16-bit, tensor cores (latent_attention_tc.cu)
+Status latent_prefill_tc(cudaStream_t s, const LatentPrefillDesc& d);
 // The same for short portions, attending in the latent space (the up-projections absorbed into query and output).
 // work: latent_decode_work_bytes.
 size_t latent_decode_work_bytes(int rows, int heads, int kv_rank, int rot_dim, int max_len);

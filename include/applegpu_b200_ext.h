@@ -333,7 +333,8 @@ APPLEGPU_API void applegpu_seq_destroy(uint64_t engine);
  *                form 0: chunk-parallel, 1: token by token
  *   latent_attention  proj [B, T, cols], up and rotation table as in seq_create, cache [B, max_len, P(kv_rank) + P(rot_dim)]
  *                appended in place at pos (int32 [B], all equal to `past`) -> [B, T, heads * vdim]; form 0: keys and values
- *                expanded per head (rotates the queries of proj in place), 1: in the latent space */
+ *                expanded per head (rotates the queries of proj in place), 1: in the latent space, 2: as 0, on the tensor-core
+ *                kernel or not at all */
 APPLEGPU_API uint64_t applegpu_ffi_rms_norm(uint64_t x_id, uint64_t weight_id, float eps, int8_t out_dtype);
 APPLEGPU_API uint64_t applegpu_ffi_clamped_glu(uint64_t gate_up_id, float limit);
 APPLEGPU_API uint64_t applegpu_ffi_mlstm(uint64_t proj_id, uint64_t gates_id, uint64_t gate_bias_id, uint64_t norm_id, uint64_t state_id, uint32_t heads, uint32_t dim,
