@@ -446,10 +446,11 @@ def clamped_glu(gate_up, limit):
     return GpuTensor(_L().applegpu_ffi_clamped_glu(gate_up.id, float(limit)))
 
 
-def mlstm(proj, gates, gate_bias, norm, state, heads, dim, vdim, gate_cap, eps=1e-5, chunked=True):
+def mlstm(proj, gates, gate_bias, norm, state, heads, dim, vdim, gate_cap, eps=1e-5, form="chunked"):
     """The mLSTM recurrence over proj [B, T, cols] (q | k | v | output gate) and float32 gates [B, T, 2 heads] (input | forget,
-    without bias); `state` (float32 [B, n]) is updated in place. `chunked=False` goes token by token. Returns [B, T, heads * vdim]."""
-    return GpuTensor(_L().applegpu_ffi_mlstm(proj.id, gates.id, gate_bias.id, norm.id, state.id, heads, dim, vdim, float(gate_cap), float(eps), 0 if chunked else 1))
+    without bias); `state` (float32 [B, n]) is updated in place. form: "chunked", "steps" (token by
+    token), "simple" (chunked, on CUDA cores only). Returns [B, T, heads * vdim]."""
+    return GpuTensor(_L().applegpu_ffi_mlstm(proj.id, gates.id, gate_bias.id, norm.id, state.id, heads, dim, vdim, float(gate_cap), float(eps), {"chunked": 0, "steps": 1, "simple": 2}[form]))
 
 
 def latent_attention(proj, norm, up, rot_table, cache, pos, past, heads, dim, rot_dim, vdim, kv_rank, scale, eps=1e-5, form="expanded"):

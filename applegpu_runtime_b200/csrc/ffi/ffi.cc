@@ -1483,6 +1483,7 @@ uint64_t applegpu_ffi_mlstm(uint64_t proj_id, uint64_t gates_id, uint64_t gate_b
     if (form == 1) return k::mlstm_step(DeviceCtx::get().stream, d);
     AG_RETURN_IF_ERROR(new_tensor({(int64_t)k::mlstm_work_bytes((int)B, (int)T, (int)heads, (int)dim, (int)vdim)}, DType::U8, &work));
     d.work = work.data();
+    d.simple = form == 2;
     return k::mlstm_prefill(DeviceCtx::get().stream, d);
   };
   const Status s = run();

@@ -11,56 +11,16 @@
 //   output   o_t = (q_t S_c) r_t + sum over the chunk's j <= t of w_tj (q_t k_j) v_j, the normaliser alike, the division
 //            by max(|n q|, exp(-m)) + 1e-6, the head's RMS norm, its weight and the output gate
 // A generated token (and a portion of a few) takes mlstm_step instead, which updates the state in place.
-#include "common.cuh"
-#include "seq_kernels.h"
+#include "mlstm.cuh"
 #include "sm100.cuh"
 
 namespace ag { namespace k {
 
-constexpr int kMlChunk = 256;          // tokens per chunk
-
-__device__ __forceinline__ float ml_log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float ml_cap(float z, float cap) { return cap * tanhf(z / cap); }
-
-// Scratch of a portion. F, log_i, m are [n_seq * heads, T]; m_start [n_seq * heads, chunks + 1]; states and normalisers of
-// the chunks [n_seq * heads, chunks, ...].
-struct MlWork {
-  double* F; float* log_i; float* m; float* m_start; float* S; float* n;
-  int chunks;
-};
-static size_t ml_align(size_t v) { return (v + 255) / 256 * 256; }
-static MlWork ml_layout(void* base, int n_seq, int T, int heads, int dim, int vdim, size_t* total) {
-  MlWork w;
-  const size_t sh = (size_t)n_seq * heads;
-  w.chunks = (T + kMlChunk - 1) / kMlChunk;
-  uint8_t* p = static_cast<uint8_t*>(base);
-  size_t o = 0;
-  auto take = [&](size_t bytes) { uint8_t* r = p + o; o += ml_align(bytes); return r; };
-  w.F = reinterpret_cast<double*>(take(sh * T * sizeof(double)));
-  w.log_i = reinterpret_cast<float*>(take(sh * T * sizeof(float)));
-  w.m = reinterpret_cast<float*>(take(sh * T * sizeof(float)));
-  w.m_start = reinterpret_cast<float*>(take(sh * (w.chunks + 1) * sizeof(float)));
-  w.S = reinterpret_cast<float*>(take(sh * w.chunks * (size_t)dim * vdim * sizeof(float)));
-  w.n = reinterpret_cast<float*>(take(sh * w.chunks * (size_t)dim * sizeof(float)));
-  if (total) *total = o;
-  return w;
-}
 size_t mlstm_work_bytes(int n_seq, int T, int heads, int dim, int vdim) {
   size_t total = 0;
   ml_layout(nullptr, n_seq, T, heads, dim, vdim, &total);
   return total;
 }
-
-struct MlParams {
-  const void* proj; const float* gates; const float* gate_bias; const float* norm; float* state; void* y;
-  long long ld, gates_ld, state_stride, y_ld;
-  int n_seq, T, heads, dim, vdim;
-  float cap, eps, q_scale;
-  MlWork w;
-  __device__ float* S_of(int s) const { return state + (long long)s * state_stride; }
-  __device__ float* n_of(int s) const { return S_of(s) + (long long)heads * dim * vdim; }
-  __device__ float* m_of(int s) const { return n_of(s) + (long long)heads * dim; }
-};
 
 // ── gates ───────────────────────────────────────────────────────────────────
 __global__ void __launch_bounds__(256) ml_gates_kernel(const MlParams p) {
@@ -93,10 +53,17 @@ __global__ void __launch_bounds__(256) ml_gates_kernel(const MlParams p) {
     __syncthreads();
     double bF = cF, bM = cM;                          // what lies before this warp
     for (int w = 0; w < warp; w++) { bM = fmax(bM + sF[w], sM[w]); bF += sF[w]; }
+    const double bF0 = cF;                            // the chunk starts here: 256 threads, 256 tokens
     M = fmax(bM + F, M);
     F += bF;
     if (t < p.T) {
       const long long o = (long long)sh * p.T + t;
+      constexpr double kLog2e = 1.4426950408889634;
+      const double a = (F - bF0) * kLog2e, b = (double)li * kLog2e - a;
+      float4 ab;
+      ab.x = (float)a; ab.y = (float)(a - (double)ab.x); ab.z = (float)b; ab.w = (float)(b - (double)ab.z);
+      p.w.ab[o] = ab;
+      p.w.m2[o] = (float)(M * kLog2e);
       p.w.F[o] = F; p.w.log_i[o] = li; p.w.m[o] = (float)M;
       if ((t + 1) % kMlChunk == 0 || t + 1 == p.T) p.w.m_start[(long long)sh * (p.w.chunks + 1) + (t + kMlChunk) / kMlChunk] = (float)M;
       if (t + 1 == p.T) *mp = (float)M;
@@ -163,6 +130,7 @@ __global__ void __launch_bounds__(256) ml_chunk_kernel(const MlParams p) {
 }
 
 // ── carry: the chunks' own states become the states in front of them ────────
+template <typename T>      // storage type of the planes the tensor-core output kernel reads; float: none, the states stay float32
 __global__ void __launch_bounds__(256) ml_carry_kernel(const MlParams p) {
   pdl_wait();
   pdl_trigger();
@@ -177,11 +145,18 @@ __global__ void __launch_bounds__(256) ml_carry_kernel(const MlParams p) {
   const double* F = p.w.F + (long long)sh * p.T;
   const float* ms = p.w.m_start + (long long)sh * (p.w.chunks + 1);
   float v = *home;
+#pragma unroll 4
   for (int c = 0; c < p.w.chunks; c++) {
     const int t1 = min(p.T, (c + 1) * kMlChunk);
     const double Fc = F[t1 - 1] - (c ? F[c * kMlChunk - 1] : 0.0);
     const float u = own[c * step];
-    own[c * step] = v;
+    if (sizeof(T) == 4 || is_n) own[c * step] = v;
+    else {
+      T* plane = reinterpret_cast<T*>(p.w.planes) + ((long long)sh * p.w.chunks + c) * 2 * n_state + i;
+      const T hi = Cvt<T>::from(v);
+      plane[0] = hi;
+      plane[n_state] = Cvt<T>::from(v - Cvt<T>::to(hi));
+    }
     v = fmaf(v, expf((float)Fc + ms[c] - ms[c + 1]), u);
   }
   *home = v;
@@ -316,12 +291,20 @@ Status mlstm_prefill(cudaStream_t s, const MlstmDesc& d) {
   if (sh > 65535 || p.w.chunks > 65535) return Status::unsupported("mlstm: too many heads or chunks for one launch");
   cudaError_t e = launch_pdl(ml_gates_kernel, dim3((unsigned)sh), dim3(256), 0, s, p);
   if (e != cudaSuccess) return cuda_status(e, "mlstm gates");
-  const int tiles = (d.dim + kMlCd - 1) / kMlCd * ((d.vdim + kMlCe - 1) / kMlCe);
-  AG_DISPATCH_FLOAT(d.dtype, T, (e = launch_pdl(ml_chunk_kernel<T>, dim3((unsigned)tiles, (unsigned)p.w.chunks, (unsigned)sh), dim3(256), 0, s, p)));
-  if (e != cudaSuccess) return cuda_status(e, "mlstm chunk states");
+  const bool tc = !d.simple && mlstm_tc_eligible(d);
+  if (tc) {
+    AG_RETURN_IF_ERROR(mlstm_chunk_tc(s, d.dtype, p));
+  } else {
+    const int tiles = (d.dim + kMlCd - 1) / kMlCd * ((d.vdim + kMlCe - 1) / kMlCe);
+    AG_DISPATCH_FLOAT(d.dtype, T, (e = launch_pdl(ml_chunk_kernel<T>, dim3((unsigned)tiles, (unsigned)p.w.chunks, (unsigned)sh), dim3(256), 0, s, p)));
+    if (e != cudaSuccess) return cuda_status(e, "mlstm chunk states");
+  }
   const long long per = (long long)d.dim * d.vdim + d.dim;
-  e = launch_pdl(ml_carry_kernel, dim3((unsigned)((per + 255) / 256), (unsigned)sh), dim3(256), 0, s, p);
+  const dim3 cgrid((unsigned)((per + 255) / 256), (unsigned)sh);
+  if (tc) e = d.dtype == DType::BF16 ? launch_pdl(ml_carry_kernel<__nv_bfloat16>, cgrid, dim3(256), 0, s, p) : launch_pdl(ml_carry_kernel<__half>, cgrid, dim3(256), 0, s, p);
+  else e = launch_pdl(ml_carry_kernel<float>, cgrid, dim3(256), 0, s, p);
   if (e != cudaSuccess) return cuda_status(e, "mlstm carry");
+  if (tc) return mlstm_output_tc(s, d.dtype, p);
   const size_t lim = 220 * 1024;
   const size_t s32 = ml_output_smem(32, d.dim, d.vdim), s16 = ml_output_smem(16, d.dim, d.vdim), s8 = ml_output_smem(8, d.dim, d.vdim);
   if (s8 > lim) return Status::unsupported("mlstm: head too large");

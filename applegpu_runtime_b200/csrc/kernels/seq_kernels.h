@@ -67,6 +67,7 @@ struct MlstmDesc {
   float* state; int64_t state_stride;  // floats between sequences
   void* y; int64_t y_ld;
   void* work = nullptr;              // mlstm_prefill only: mlstm_work_bytes
+  bool simple = false;               // keeps 16-bit portions on the CUDA-core kernels
 };
 inline int64_t mlstm_state_floats(int heads, int dim, int vdim) { return ((int64_t)heads * ((int64_t)dim * vdim + dim + 1) + 3) / 4 * 4; }
 size_t mlstm_work_bytes(int n_seq, int T, int heads, int dim, int vdim);

@@ -330,7 +330,7 @@ APPLEGPU_API void applegpu_seq_destroy(uint64_t engine);
  *   clamped_glu  [.., 2 n] (gate | up) -> g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)
  *   mlstm        proj [B, T, cols] (q | k | v | g), gates f32 [B, T, 2 heads] (i | f without bias), state f32 [B, S floats: per
  *                head dim * vdim, then heads * dim, then heads; S rounded up to 4], updated in place -> [B, T, heads * vdim];
- *                form 0: chunk-parallel, 1: token by token
+ *                form 0: chunk-parallel, 1: token by token, 2: chunk-parallel on CUDA cores
  *   latent_attention  proj [B, T, cols], up and rotation table as in seq_create, cache [B, max_len, P(kv_rank) + P(rot_dim)]
  *                appended in place at pos (int32 [B], all equal to `past`) -> [B, T, heads * vdim]; form 0: keys and values
  *                expanded per head (rotates the queries of proj in place), 1: in the latent space, 2: as 0, on the tensor-core

@@ -86,15 +86,15 @@ def state_parts(s, H, d, e):
     return s[:H * d * e].reshape(H, d, e), s[H * d * e:H * d * e + H * d].reshape(H, d), s[H * d * e + H * d:H * d * e + H * d + H]
 
 
-MLSTM_SIZES = [(1, 16, 16), (3, 20, 28), (2, 64, 128), (2, 8, 37), (1, 128, 256), (2, 72, 96)]
+MLSTM_SIZES = [(1, 16, 16), (3, 20, 28), (2, 64, 128), (2, 8, 37), (1, 128, 256), (2, 72, 96), (2, 200, 40), (1, 24, 264)]
 
 
 @pytest.mark.parametrize("H,d,e", MLSTM_SIZES)
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("chunked", [True, False])
-def test_mlstm_portions(gpu_dev, H, d, e, dtype, chunked):
+@pytest.mark.parametrize("form", ["chunked", "simple", "steps"])
+def test_mlstm_portions(gpu_dev, H, d, e, dtype, form):
     """Two sequences in portions around the borders of chunks and tiles, state carried from portion to portion."""
-    cuts = [2, 63, 1, 65, 130, 59, 257] if chunked else [1, 2, 16, 5]
+    cuts = [2, 63, 1, 65, 130, 59, 257] if form != "steps" else [1, 2, 16, 5]
     T, B, cap, eps = sum(cuts), 2, 9.0, 2e-5
     proj, gates, bias, norm = mlstm_case(T, H, d, e, seed=H * d + e, B=B)
     n = (H * (d * e + d + 1) + 3) // 4 * 4
@@ -103,7 +103,7 @@ def test_mlstm_portions(gpu_dev, H, d, e, dtype, chunked):
     bt, nt = g.from_numpy(bias), g.from_numpy(norm)
     out, lo = [], 0
     for c in cuts:
-        out.append(g.mlstm(put(g, proj[:, lo:lo + c], dtype), g.from_numpy(gates[:, lo:lo + c]), bt, nt, state, H, d, e, cap, eps, chunked=chunked).to_numpy())
+        out.append(g.mlstm(put(g, proj[:, lo:lo + c], dtype), g.from_numpy(gates[:, lo:lo + c]), bt, nt, state, H, d, e, cap, eps, form=form).to_numpy())
         lo += c
     got, st = np.concatenate(out, axis=1), state.to_numpy()
     for b in range(B):
