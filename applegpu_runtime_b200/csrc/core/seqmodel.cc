@@ -242,7 +242,7 @@ struct SeqEngine {
     for (size_t l = 0; l < cfg.layers.size(); l++) {
       const SeqLayerCfg& c = cfg.layers[l];
       pc = std::max(pc, pad8(mixers[l]->proj_cols())); gc = std::max<int64_t>(gc, mixers[l]->gate_cols());
-      fc = std::max(fc, pad8(2 * (int64_t)c.ff)); cc = std::max(cc, cat_ld(c));
+      fc = std::max(fc, k::glu_rows(c.ff)); cc = std::max(cc, cat_ld(c));
       wb = std::max(wb, mixers[l]->work_bytes(n_seq, T, max_len));
       if (T > kShortT) kb = std::max(kb, mixers[l]->kv_bytes(len.data() + slot0, n_seq, T));
     }
@@ -252,9 +252,9 @@ struct SeqEngine {
     AG_RETURN_IF_ERROR(ensure(&cat, R * cc * esz(), true));
     AG_RETURN_IF_ERROR(ensure(&work, wb));
     AG_RETURN_IF_ERROR(ensure(&kv, kb, false, false));
-    const size_t hrows = std::max<size_t>(R > k::kSeqSkinnyRows || !skinny_ok() ? R : 1, (size_t)n_want);
-    AG_RETURN_IF_ERROR(ensure(&h1, hrows * pad8(cfg.width) * esz()));
-    AG_RETURN_IF_ERROR(ensure(&h2, hrows * pad8(cfg.width) * esz()));
+    const size_t hrows = std::max<size_t>(R, (size_t)n_want);
+    AG_RETURN_IF_ERROR(ensure(&h1, hrows * pad8(cfg.width) * esz(), true));
+    AG_RETURN_IF_ERROR(ensure(&h2, hrows * pad8(cfg.width) * esz(), true));
     if (R > k::kSeqSkinnyRows || !skinny_ok()) AG_RETURN_IF_ERROR(ensure(&gu, R * fc * esz()));
     if (n_want) AG_RETURN_IF_ERROR(ensure(&logits, (size_t)n_want * cfg.vocab * sizeof(float)));
     AG_RETURN_IF_ERROR(ensure(&tok, std::max<size_t>(R, slots) * sizeof(int32_t)));
@@ -290,16 +290,24 @@ struct SeqEngine {
       n.load_x = !start;
       if (run.first) n.step = f32(w[3]) + (size_t)run.pass * cfg.width;
       if (skinny) {
-        if (start || n.step) AG_RETURN_IF_ERROR(count(k::rms_rows(st.s, n)));
+        // 16-bit: the norms are stored once and every product reads them; float32: the products take them in their prologue
+        const bool stored = dtype != DType::F32;
+        if (stored) {
+          n.w1 = f32(W[kWNorm1]); n.out1 = h1.ptr(); n.ld1 = wl;
+          if (c.ff) { n.w2 = f32(W[kWNorm2]); n.out2 = h2.ptr(); n.ld2 = wl; }
+        }
+        if (stored || start || n.step) AG_RETURN_IF_ERROR(count(k::rms_rows(st.s, n)));
         k::SeqSkinnyDesc d;
-        d.dtype = dtype; d.rows = R; d.k = cfg.width; d.x = X; d.eps = cfg.eps;
-        auto seg = [&](const TensorRec& wt, int64_t cols, const TensorRec& nw, k::SeqOut mode, void* out, int64_t ld) {
+        d.dtype = dtype; d.rows = R; d.k = cfg.width; d.eps = cfg.eps;
+        if (!stored) d.x = X;
+        auto seg = [&](const TensorRec& wt, int64_t cols, const TensorRec& nw, const Scratch& h, k::SeqOut mode, void* out, int64_t ld) {
           k::SeqSeg& g = d.seg[d.n_seg++];
-          g.w = wt.data(); g.ld = wl; g.n = (int)cols; g.norm_w = f32(nw); g.mode = mode; g.limit = c.ff_limit; g.out = out; g.out_ld = ld;
+          g.w = wt.data(); g.ld = wl; g.n = (int)cols; g.mode = mode; g.limit = c.ff_limit; g.out = out; g.out_ld = ld;
+          if (stored) { g.a = h.ptr(); g.a_ld = wl; } else g.norm_w = f32(nw);
         };
-        seg(W[kWIn], mx.proj_cols(), W[kWNorm1], k::SeqOut::Store, proj.ptr(), pl);
-        if (mx.gate_cols()) seg(W[kWAux0], mx.gate_cols(), W[kWNorm1], k::SeqOut::StoreF32, gates.ptr(), mx.gate_cols());
-        if (c.ff) seg(W[kWFf], c.ff, W[kWNorm2], k::SeqOut::Glu, ff_out, cl);
+        seg(W[kWIn], mx.proj_cols(), W[kWNorm1], h1, k::SeqOut::Store, proj.ptr(), pl);
+        if (mx.gate_cols()) seg(W[kWAux0], mx.gate_cols(), W[kWNorm1], h1, k::SeqOut::StoreF32, gates.ptr(), mx.gate_cols());
+        if (c.ff) seg(W[kWFf], c.ff, W[kWNorm2], h2, k::SeqOut::Glu, ff_out, cl);
         Span span("skinny_in", esz() * (double)wl * (mx.proj_cols() + mx.gate_cols() + 2.0 * c.ff));
         AG_RETURN_IF_ERROR(count(k::seq_skinny(st.s, d)));
       } else {
@@ -318,19 +326,27 @@ struct SeqEngine {
           AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h1.ptr(), wl, R, cfg.width, W[kWAux0].data(), wl, mx.gate_cols(), gates.ptr(), mx.gate_cols(), true, nullptr))));
         }
         if (c.ff) {
-          const int64_t fl = pad8(2 * (int64_t)c.ff);
-          {
+          const int64_t fn = k::glu_rows(c.ff);
+          k::GemmDesc g = linear_desc(dtype, h2.ptr(), wl, R, cfg.width, W[kWFf].data(), wl, fn, gu.ptr(), fn, false, nullptr);
+          if (k::matmul_tc_ready(g)) {                  // the gate rides in the product's epilogue
+            g.c = ff_out; g.c_row = cl; g.ep.glu_n = c.ff; g.ep.glu_limit = c.ff_limit;
             Span span("linear_ff", product(R, 2.0 * c.ff, cfg.width));
-            AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h2.ptr(), wl, R, cfg.width, W[kWFf].data(), wl, 2 * (int64_t)c.ff, gu.ptr(), fl, false, nullptr))));
+            AG_RETURN_IF_ERROR(count(k::matmul(st.s, g)));
+          } else {
+            {
+              Span span("linear_ff", product(R, 2.0 * c.ff, cfg.width));
+              AG_RETURN_IF_ERROR(count(k::matmul(st.s, g)));
+            }
+            Span span("clamped_glu", 3.0 * esz() * R * c.ff);
+            AG_RETURN_IF_ERROR(count(k::clamped_glu(st.s, dtype, gu.ptr(), fn, ff_out, cl, R, c.ff, k::kGluBlock, c.ff_limit)));
           }
-          Span span("clamped_glu", 3.0 * esz() * R * c.ff);
-          AG_RETURN_IF_ERROR(count(k::clamped_glu(st.s, dtype, gu.ptr(), fl, ff_out, cl, R, c.ff, c.ff_limit)));
         }
       }
       AG_RETURN_IF_ERROR(mx.run(st, proj.ptr(), pl, static_cast<const float*>(gates.ptr()), memory[r]->ptr, max_len, p, cat.ptr(), cl, work.ptr(), kv.ptr(), cfg.eps, &launches));
       if (skinny) {
         k::SeqSkinnyDesc d;
         d.dtype = dtype; d.rows = R; d.k = (int)cat_k(c); d.a = cat.ptr(); d.a_ld = cl; d.n_seg = 1;
+        d.seg[0].a = cat.ptr(); d.seg[0].a_ld = cl;
         d.seg[0].w = W[kWOut].data(); d.seg[0].ld = cl; d.seg[0].n = cfg.width; d.seg[0].mode = k::SeqOut::AddF32; d.seg[0].out = X; d.seg[0].out_ld = cfg.width;
         Span span("skinny_out", esz() * (double)cl * cfg.width);
         AG_RETURN_IF_ERROR(count(k::seq_skinny(st.s, d)));
@@ -355,11 +371,11 @@ struct SeqEngine {
     d.dtype = dtype; d.rows = n; d.k = cfg.width; d.eps = cfg.eps; d.n_seg = 1;
     d.seg[0].w = w[1].data(); d.seg[0].ld = wl; d.seg[0].n = cfg.vocab; d.seg[0].norm_w = f32(w[2]); d.seg[0].mode = k::SeqOut::StoreF32; d.seg[0].out = logits.ptr();
     d.seg[0].out_ld = cfg.vocab;
-    if (skinny && !map) { d.x = static_cast<const float*>(x.ptr()); return count(k::seq_skinny(s, d)); }
+    if (skinny && !map && dtype == DType::F32) { d.x = static_cast<const float*>(x.ptr()); return count(k::seq_skinny(s, d)); }
     k::RmsRowsDesc r;
     r.dtype = dtype; r.x = static_cast<float*>(x.ptr()); r.rows = n; r.width = cfg.width; r.eps = cfg.eps; r.row_map = map; r.w1 = f32(w[2]); r.out1 = h1.ptr(); r.ld1 = wl;
     AG_RETURN_IF_ERROR(count(k::rms_rows(s, r)));
-    if (skinny) { d.a = h1.ptr(); d.a_ld = wl; return count(k::seq_skinny(s, d)); }
+    if (skinny) { d.a = d.seg[0].a = h1.ptr(); d.a_ld = d.seg[0].a_ld = wl; return count(k::seq_skinny(s, d)); }
     return count(k::matmul(s, linear_desc(dtype, h1.ptr(), wl, n, cfg.width, w[1].data(), wl, cfg.vocab, logits.ptr(), cfg.vocab, true, nullptr)));
   }
   Status enqueue_pick(cudaStream_t s, int n, void* out) {
@@ -458,7 +474,7 @@ Status seq_create(const SeqModelCfg& cfg, const std::vector<TensorRec>& weights,
     else return Status::invalid(at + "unknown mixer");
     const Mixer& m = *e->mixers.back();
     if (!is_vector(t[kWNorm1], W) || !is_matrix(t[kWIn], dt, m.proj_cols(), wl) || !is_matrix(t[kWOut], dt, W, e->cat_ld(c))) return Status::invalid(at + "norm, input or output weights");
-    if (c.ff && (!is_vector(t[kWNorm2], W) || !is_matrix(t[kWFf], dt, 2 * (int64_t)c.ff, wl))) return Status::invalid(at + "feed-forward weights");
+    if (c.ff && (!is_vector(t[kWNorm2], W) || !is_matrix(t[kWFf], dt, k::glu_rows(c.ff), wl))) return Status::invalid(at + "feed-forward weights");
     const Status st = m.check(cfg, max_len);
     if (!st.ok()) return Status{st.kind, at + st.msg};
   }

@@ -1455,7 +1455,7 @@ uint64_t applegpu_ffi_clamped_glu(uint64_t gate_up_id, float limit) {
     const int64_t c = o.back(), rows = numel_of(o) / (c ? c : 1);
     o.back() = c / 2;
     AG_RETURN_IF_ERROR(new_tensor(o, t.dtype, &out));
-    return k::clamped_glu(DeviceCtx::get().stream, t.dtype, t.data(), c, out.data(), c / 2, rows, (int)(c / 2), limit);
+    return k::clamped_glu(DeviceCtx::get().stream, t.dtype, t.data(), c, out.data(), c / 2, rows, (int)(c / 2), (int)(c / 2), limit);
   };
   const Status s = run();
   return immediate_result("clamped_glu", st.rt, s, out);

@@ -56,6 +56,8 @@ struct TcParams {
   float ln_inv_k, ln_eps;
   long long* stats_out;              // folded layer_norm, producer side: row sums of what is stored (fixed point, integer atomics)
   long long* stats_zero;             // rows of the other statistics tensor to clear
+  int glu_n, glu_vec;                // gated result: B rows come in blocks of 16 gate | 16 up, C has glu_n columns (16-byte rows: glu_vec)
+  float glu_limit;
   int* status;
 #ifdef AG_GEMM_PROBE
   long long* probe;   // per CTA: [0] cycles the MMA thread waited for a free accumulator, [1] cycles in the k loops, [2] k steps, [3] cycles epilogue warp 2 waited for a full accumulator, [4] cycles it spent in the epilogue, [5] tiles, [6] kernel cycles
@@ -232,6 +234,36 @@ __device__ __forceinline__ void emit_row_stats(const TcParams& p, long long gm, 
     atomicAdd(reinterpret_cast<unsigned long long*>(p.stats_out) + 2 * gm + 1, (unsigned long long)__float2ll_rn(row_sq * kStatsScale));
   }
   if (p.stats_zero && clears) *reinterpret_cast<longlong2*>(p.stats_zero + 2 * gm) = make_longlong2(0, 0);
+}
+
+// Gated epilogue: the 32 accumulator columns are 16 gates and the 16 values they gate; each lane stores its row's 16 results.
+template <typename T>
+__device__ __forceinline__ void glu_group(const TcParams& p, uint32_t taddr, long long row0, int col0, int lane) {
+  uint32_t acc[32];
+  tmem_ld_32x32(taddr, acc);
+  tmem_ld_wait();
+  const long long gm = row0 + lane;
+  const int c0 = col0 / 2;
+  if (gm >= p.m || c0 >= p.glu_n) return;
+  uint32_t o[8];
+#pragma unroll
+  for (int w = 0; w < 8; w++) {
+    float r[2];
+#pragma unroll
+    for (int q = 0; q < 2; q++) {
+      const float g = fminf(__uint_as_float(acc[2 * w + q]), p.glu_limit), u = fminf(fmaxf(__uint_as_float(acc[16 + 2 * w + q]), -p.glu_limit), p.glu_limit);
+      r[q] = __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+    }
+    o[w] = pack2<T>(r[0], r[1]);
+  }
+  T* crow = reinterpret_cast<T*>(p.c) + gm * p.c_row + c0;
+  if (p.glu_vec && c0 + 16 <= p.glu_n) {
+    *reinterpret_cast<uint4*>(crow) = make_uint4(o[0], o[1], o[2], o[3]);
+    *reinterpret_cast<uint4*>(crow + 8) = make_uint4(o[4], o[5], o[6], o[7]);
+  } else {
+    const T* tv = reinterpret_cast<const T*>(o);
+    for (int e = 0; e < 16 && c0 + e < p.glu_n; e++) crow[e] = tv[e];
+  }
 }
 
 #ifdef AG_CHAIN_PROBE
@@ -874,6 +906,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant
       for (int g = pair, gi = 0; g < BN / 32; g += 2, gi++) {
         if (n0 + g * 32 >= p.n) break;  // uniform across the warp
         int next_col0 = (g + 2 < BN / 32 && n0 + (g + 2) * 32 < p.n) ? n0 + (g + 2) * 32 : -1;
+        if (p.glu_n) { glu_group<T>(p, taddr + (uint32_t)(g * 32), row0, n0 + g * 32, lane); continue; }
         epilogue_group<T>(p, taddr + (uint32_t)(g * 32), stg, (p.bias && !p.c_f32) ? bias_s + gi * 32 : nullptr, fsrc ? scale_s + gi * 32 : nullptr, rpre, row0, n0 + g * 32, next_col0,
                           c_off, lane, best_key, ln_mean, ln_rstd, row_sum, row_sq, packed_epi ? bias_f + gi * 32 : nullptr);
       }
@@ -1210,6 +1243,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
         for (int g = pair, gi = 0; g < BN / 32; g += 2, gi++) {
           if (n0 + g * 32 >= p.n) break;
           int next_col0 = (g + 2 < BN / 32 && n0 + (g + 2) * 32 < p.n) ? n0 + (g + 2) * 32 : -1;
+          if (p.glu_n) { glu_group<T>(p, taddr + (uint32_t)(g * 32), row0, n0 + g * 32, lane); continue; }
           epilogue_group<T>(p, taddr + (uint32_t)(g * 32), stg, (p.bias && !p.c_f32) ? bias_s + gi * 32 : nullptr, fsrc ? scale_s + gi * 32 : nullptr, rpre, row0, n0 + g * 32, next_col0,
                             c_off, lane, best_key, ln_mean, ln_rstd, row_sum, row_sq, packed_epi ? bias_f + gi * 32 : nullptr);
         }
@@ -1527,7 +1561,7 @@ gemm_tc_chain_kernel(const __grid_constant__ ChainMaps maps, const __grid_consta
         p.c = sp.c; p.bias = sp.bias; p.residual = sp.residual; p.b_scales = nullptr; p.alpha = sp.alpha; p.act = sp.act;
         p.m = sp.m; p.n = sp.n; p.k = sp.k; p.batch = 1; p.batch_inner = 1; p.c_row = sp.c_row; p.c_batch = 0; p.c_batch_inner = 0;
         p.a_bcast = 0; p.b_bcast = 0; p.tiles_m = sp.tiles_m; p.tiles_n = sp.tiles_n; p.vec_ok = 2 /* the only layout a link may have: the others compile out */; p.bias_vec = 0;
-        p.argmax_keys = nullptr; p.c_f32 = 0; p.ln_stats = sp.ln_stats; p.ln_colsum = sp.ln_colsum; p.ln_inv_k = sp.ln_inv_k; p.ln_eps = sp.ln_eps;
+        p.argmax_keys = nullptr; p.c_f32 = 0; p.glu_n = 0; p.ln_stats = sp.ln_stats; p.ln_colsum = sp.ln_colsum; p.ln_inv_k = sp.ln_inv_k; p.ln_eps = sp.ln_eps;
         p.stats_out = sp.stats_out; p.stats_zero = sp.stats_zero; p.status = status;
       }
       const int mi = lt / p.tiles_n, ni = lt - mi * p.tiles_n;
@@ -1935,6 +1969,8 @@ Status matmul_tc(cudaStream_t s, const GemmDesc& d, int* status_word) {
   p.c_f32 = d.c_f32 ? 1 : 0;
   p.ln_stats = d.ep.ln_stats; p.ln_colsum = d.ep.ln_colsum; p.ln_inv_k = d.k ? 1.0f / (float)d.k : 0.f; p.ln_eps = d.ep.ln_eps;
   p.stats_out = d.ep.stats_out; p.stats_zero = d.ep.stats_zero;
+  p.glu_n = d.ep.glu_n; p.glu_limit = d.ep.glu_limit;
+  p.glu_vec = (reinterpret_cast<uintptr_t>(d.c) & 15u) == 0 && d.c_row % 8 == 0 ? 1 : 0;
 #ifdef AG_GEMM_PROBE
   p.probe = g_tc_probe;
 #endif
@@ -2225,6 +2261,7 @@ static int initial_tile_override() {
 static const int g_tile_override_init = (g_tile_override = initial_tile_override());
 void set_gemm_tile(int code) { g_tile_override = code; }
 
+bool matmul_tc_ready(const GemmDesc& d) { return g_force_path != 1 && tc_eligible(d); }
 const char* matmul_path(const GemmDesc& d) {
   if (g_force_path == 1) return "simt";
   return tc_eligible(d) ? "tcgen05" : "simt";
@@ -2253,6 +2290,13 @@ Status matmul(cudaStream_t s, const GemmDesc& d) {
     return matmul_skinny_kmajor(s, d);
   }
   bool elig = tc_eligible(d);
+  if (d.ep.glu_n) {
+    if (!elig || g_force_path == 1 || d.batch != 1 || d.batch_inner != 1 || d.c_f32 || d.ep.bias || d.ep.residual || d.ep.argmax_keys || d.n % 32 || 2 * d.ep.glu_n > d.n)
+      return Status::invalid("matmul: the gated epilogue needs an unbatched 16-bit product on the tensor-core kernel");
+    int* st = matmul_status_word();
+    if (!st) return Status::compute("matmul: the kernel workspace is not initialised");
+    return matmul_tc(s, d, st);
+  }
   if (d.ep.argmax_keys && (!elig || g_force_path == 1)) return Status::invalid("matmul: the row-argmax epilogue needs the tensor-core kernel");
   if (d.ep.ln_stats || d.ep.stats_out || d.ep.stats_zero) {
     if (!elig || g_force_path == 1 || d.batch != 1 || d.batch_inner != 1 || d.c_f32 || d.ep.argmax_keys || d.ep.b_scales || (d.ep.ln_stats && !d.ep.ln_colsum))

@@ -83,6 +83,10 @@ struct GemmEpilogue {
   float ln_eps = 1e-5f;
   long long* stats_out = nullptr;
   long long* stats_zero = nullptr;
+  // Gated result (tensor-core kernels, unbatched, 16-bit C): B's columns come in blocks of 16 gates | 16 values, n a multiple of
+  // 32, and C gets glu_n <= n / 2 columns g sigmoid(1.702 g) (u + 1), g = min(gate, glu_limit), u = clamp(value, +-glu_limit).
+  int glu_n = 0;
+  float glu_limit = 0.f;
 };
 struct GemmDesc {
   DType dtype;            // dtype of A and C (f32/f16/bf16)
@@ -106,6 +110,7 @@ struct GemmDesc {
   GemmEpilogue ep;
 };
 Status matmul(cudaStream_t s, const GemmDesc& d);
+bool matmul_tc_ready(const GemmDesc& d);      // `matmul` would take a tensor-core kernel
 // Chained products: up to kChainMax unbatched 16-bit products with [K, N] weights, each reading the previous one's
 // result as its A operand, as ONE launch of the tensor-core kernel (a 256-row block of product g + 1 only needs the same
 // rows of product g, so tiles of consecutive products overlap and the pipeline fills and drains once).

@@ -53,8 +53,9 @@ __device__ __forceinline__ void la_cache_row(const LaParams& p, const T* row, T*
   for (int i = 2 * p.pairs + threadIdx.x; i < p.rot_dim; i += blockDim.x) dst[i] = kr[i];
 }
 
+constexpr int kLaThreads = 128;
 template <typename T>
-__global__ void __launch_bounds__(256) latent_append_kernel(const LaParams p) {
+__global__ void __launch_bounds__(kLaThreads) latent_append_kernel(const LaParams p) {
   __shared__ float red[33];
   pdl_wait();
   pdl_trigger();
@@ -64,13 +65,20 @@ __global__ void __launch_bounds__(256) latent_append_kernel(const LaParams p) {
   T* row = reinterpret_cast<T*>(p.proj) + (long long)r * p.ld;
   T* crow = reinterpret_cast<T*>(p.cache) + (long long)s * p.seq_stride + (long long)position * p.cld;
   la_cache_row<T>(p, row, crow, position, red);
-  for (int i = threadIdx.x; i < p.heads * p.pairs; i += 256) {
-    const int h = i / p.pairs, j = i % p.pairs;
-    T* q = row + (long long)h * (p.dim + p.rot_dim) + p.dim + 2 * j;
+  // a warp per head, a lane per pair (read and written as one word when pairs lie on words)
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, hd = p.dim + p.rot_dim;
+  const bool words = sizeof(T) == 2 && p.dim % 2 == 0 && hd % 2 == 0;
+  for (int j = lane; j < p.pairs; j += 32) {
     const float2 cs = p.rot[(long long)position * p.pairs + j];
-    const float u = Cvt<T>::to(q[0]), v = Cvt<T>::to(q[1]);
-    q[0] = Cvt<T>::from(u * cs.x - v * cs.y);
-    q[1] = Cvt<T>::from(v * cs.x + u * cs.y);
+    for (int h = warp; h < p.heads; h += kLaThreads / 32) {
+      T* q = row + (long long)h * hd + p.dim + 2 * j;
+      alignas(8) T t[2];
+      if (words) *reinterpret_cast<uint32_t*>(t) = *reinterpret_cast<const uint32_t*>(q); else { t[0] = q[0]; t[1] = q[1]; }
+      const float u = Cvt<T>::to(t[0]), v = Cvt<T>::to(t[1]);
+      t[0] = Cvt<T>::from(u * cs.x - v * cs.y);
+      t[1] = Cvt<T>::from(v * cs.x + u * cs.y);
+      if (words) *reinterpret_cast<uint32_t*>(q) = *reinterpret_cast<const uint32_t*>(t); else { q[0] = t[0]; q[1] = t[1]; }
+    }
   }
 }
 
@@ -78,7 +86,7 @@ Status latent_append(cudaStream_t s, const LatentDesc& d) {
   LaParams p;
   AG_RETURN_IF_ERROR(la_params(d, &p));
   cudaError_t e = cudaSuccess;
-  AG_DISPATCH_FLOAT(d.dtype, T, (e = launch_pdl(latent_append_kernel<T>, dim3((unsigned)(d.n_seq * d.T)), dim3(256), 0, s, p)));
+  AG_DISPATCH_FLOAT(d.dtype, T, (e = launch_pdl(latent_append_kernel<T>, dim3((unsigned)(d.n_seq * d.T)), dim3(kLaThreads), 0, s, p)));
   return cuda_status(e, "latent append");
 }
 

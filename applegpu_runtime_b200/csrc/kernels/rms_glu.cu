@@ -8,8 +8,7 @@
 
 namespace ag { namespace k {
 
-constexpr int kRmsThreads = 256;
-constexpr int kRmsRegs = 32;          // values per thread kept in registers: rows up to 8192 wide are read once
+constexpr int kRmsThreads = 128;      // small blocks: many rows in flight per SM
 
 struct RmsParams {
   float* x; const int32_t* tok; const void* embed; const float* step; const float* w1; const float* w2; const int32_t* row_map;
@@ -19,8 +18,9 @@ struct RmsParams {
   float eps;
 };
 
-// VEC elements per thread and access (4 when width and pitches allow it)
-template <typename T, int VEC>
+// VEC elements per thread and access (4 when width and pitches allow it), NREG accesses kept in registers (wider rows are read
+// twice)
+template <typename T, int VEC, int NREG>
 __global__ void __launch_bounds__(kRmsThreads) rms_rows_kernel(const RmsParams p) {
   __shared__ float red[33];
   pdl_wait();
@@ -34,7 +34,6 @@ __global__ void __launch_bounds__(kRmsThreads) rms_rows_kernel(const RmsParams p
     t = t < 0 ? 0 : (t >= p.vocab ? p.vocab - 1 : t);
     e = reinterpret_cast<const T*>(p.embed) + (long long)t * p.embed_ld;
   }
-  constexpr int NREG = kRmsRegs / VEC;
   float v[NREG][VEC];
   float sq = 0.f;
   const int packs = p.width / VEC;
@@ -48,8 +47,12 @@ __global__ void __launch_bounds__(kRmsThreads) rms_rows_kernel(const RmsParams p
       for (int j = 0; j < VEC; j++) o[j] = 0.f;
     }
     if (e) {
+      alignas(16) T t[VEC];
+      if constexpr (VEC == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(t) = *reinterpret_cast<const uint2*>(e + c);
+      else if constexpr (VEC == 4) *reinterpret_cast<uint4*>(t) = *reinterpret_cast<const uint4*>(e + c);
+      else t[0] = e[c];
 #pragma unroll
-      for (int j = 0; j < VEC; j++) o[j] += Cvt<T>::to(e[c + j]);
+      for (int j = 0; j < VEC; j++) o[j] += Cvt<T>::to(t[j]);
     }
     if (p.step) {
 #pragma unroll
@@ -87,7 +90,7 @@ __global__ void __launch_bounds__(kRmsThreads) rms_rows_kernel(const RmsParams p
     auto one = [&](T* dst, const float* w) {
       alignas(16) T t[VEC];
 #pragma unroll
-      for (int j = 0; j < VEC; j++) t[j] = Cvt<T>::from(o[j] * rs * w[c + j]);
+      for (int j = 0; j < VEC; j++) t[j] = Cvt<T>::from(o[j] * rs * __ldg(w + c + j));
       if constexpr (VEC == 4 && sizeof(T) == 4) *reinterpret_cast<uint4*>(dst + c) = *reinterpret_cast<const uint4*>(t);
       else if constexpr (VEC == 4) *reinterpret_cast<uint2*>(dst + c) = *reinterpret_cast<const uint2*>(t);
       else dst[c] = t[0];
@@ -118,18 +121,23 @@ Status rms_rows(cudaStream_t s, const RmsRowsDesc& d) {
   p.x = d.x; p.tok = d.tok; p.embed = d.embed; p.step = d.step; p.w1 = d.w1; p.w2 = d.w2; p.row_map = d.row_map;
   p.out1 = d.out1; p.out2 = d.out2; p.ld1 = d.ld1; p.ld2 = d.ld2; p.embed_ld = d.embed_ld;
   p.width = d.width; p.vocab = d.vocab; p.load_x = d.load_x ? 1 : 0; p.write_x = (!d.load_x || d.embed || d.step) ? 1 : 0; p.eps = d.eps;
-  const bool vec = d.width % 4 == 0 && d.ld1 % 4 == 0 && d.ld2 % 4 == 0 && aligned16(d.x) && (!d.out1 || aligned16(d.out1)) && (!d.out2 || aligned16(d.out2));
+  const bool vec = d.width % 4 == 0 && d.ld1 % 4 == 0 && d.ld2 % 4 == 0 && aligned16(d.x) && (!d.embed || (d.embed_ld % 4 == 0 && aligned16(d.embed))) && (!d.out1 || aligned16(d.out1)) && (!d.out2 || aligned16(d.out2));
   cudaError_t e = cudaSuccess;
   AG_DISPATCH_FLOAT(d.dtype, T, {
-    if (vec) e = launch_pdl(rms_rows_kernel<T, 4>, dim3((unsigned)d.rows), dim3(kRmsThreads), 0, s, p);
-    else e = launch_pdl(rms_rows_kernel<T, 1>, dim3((unsigned)d.rows), dim3(kRmsThreads), 0, s, p);
+    const dim3 grid((unsigned)d.rows), block(kRmsThreads);
+    if (!vec) e = launch_pdl(rms_rows_kernel<T, 1, 16>, grid, block, 0, s, p);
+    else if (d.width <= 2 * 4 * kRmsThreads) e = launch_pdl(rms_rows_kernel<T, 4, 2>, grid, block, 0, s, p);
+    else if (d.width <= 4 * 4 * kRmsThreads) e = launch_pdl(rms_rows_kernel<T, 4, 4>, grid, block, 0, s, p);
+    else if (d.width <= 8 * 4 * kRmsThreads) e = launch_pdl(rms_rows_kernel<T, 4, 8>, grid, block, 0, s, p);
+    else e = launch_pdl(rms_rows_kernel<T, 4, 16>, grid, block, 0, s, p);
   });
   return cuda_status(e, "rms_rows");
 }
 
 // ── clamped gated activation ────────────────────────────────────────────────
+// gate of column c at (c / block) * 2 * block + c % block, the value it gates `block` columns later
 template <typename T, int VEC>
-__global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ gu, long long ld_in, T* __restrict__ out, long long ld_out, long long rows, int ff, float limit) {
+__global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ gu, long long ld_in, T* __restrict__ out, long long ld_out, long long rows, int ff, int block, float limit) {
   pdl_wait();
   pdl_trigger();
   const int packs = ff / VEC;
@@ -137,9 +145,9 @@ __global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ 
   for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < total; i += (long long)gridDim.x * 256) {
     const long long r = i / packs;
     const int c = (int)(i - r * packs) * VEC;
-    const T* g = gu + r * ld_in + c;
+    const T* g = gu + r * ld_in + c / block * 2 * block + c % block;
     if constexpr (VEC > 1) {
-      const Pack<T> a = ld16(g), b = ld16(g + ff);
+      const Pack<T> a = ld16(g), b = ld16(g + block);
       Pack<T> o;
       float t[VEC];
 #pragma unroll
@@ -147,20 +155,21 @@ __global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ 
       pack_from_floats<T>(o, t);
       st16(out + r * ld_out + c, o);
     } else {
-      out[r * ld_out + c] = Cvt<T>::from(clamped_glu_f(Cvt<T>::to(g[0]), Cvt<T>::to(g[ff]), limit));
+      out[r * ld_out + c] = Cvt<T>::from(clamped_glu_f(Cvt<T>::to(g[0]), Cvt<T>::to(g[block]), limit));
     }
   }
 }
 
-Status clamped_glu(cudaStream_t s, DType dt, const void* gu, int64_t ld_in, void* out, int64_t ld_out, int64_t rows, int ff, float limit) {
+Status clamped_glu(cudaStream_t s, DType dt, const void* gu, int64_t ld_in, void* out, int64_t ld_out, int64_t rows, int ff, int block, float limit) {
   if (rows <= 0 || ff <= 0) return Status::OK();
+  if (block < 1) return Status::invalid("clamped_glu: block");
   cudaError_t e = cudaSuccess;
   AG_DISPATCH_FLOAT(dt, T, {
     constexpr int N = Pack<T>::N;
-    const bool vec = ff % N == 0 && ld_in % N == 0 && ld_out % N == 0 && aligned16(gu) && aligned16(out);
+    const bool vec = ff % N == 0 && block % N == 0 && ld_in % N == 0 && ld_out % N == 0 && aligned16(gu) && aligned16(out);
     const int64_t work = rows * (ff / (vec ? N : 1));
-    if (vec) e = launch_pdl(clamped_glu_kernel<T, N>, dim3((unsigned)grid_for(work, 256)), dim3(256), 0, s, (const T*)gu, (long long)ld_in, (T*)out, (long long)ld_out, (long long)rows, ff, limit);
-    else e = launch_pdl(clamped_glu_kernel<T, 1>, dim3((unsigned)grid_for(work, 256)), dim3(256), 0, s, (const T*)gu, (long long)ld_in, (T*)out, (long long)ld_out, (long long)rows, ff, limit);
+    if (vec) e = launch_pdl(clamped_glu_kernel<T, N>, dim3((unsigned)grid_for(work, 256)), dim3(256), 0, s, (const T*)gu, (long long)ld_in, (T*)out, (long long)ld_out, (long long)rows, ff, block, limit);
+    else e = launch_pdl(clamped_glu_kernel<T, 1>, dim3((unsigned)grid_for(work, 256)), dim3(256), 0, s, (const T*)gu, (long long)ld_in, (T*)out, (long long)ld_out, (long long)rows, ff, block, limit);
   });
   return cuda_status(e, "clamped_glu");
 }

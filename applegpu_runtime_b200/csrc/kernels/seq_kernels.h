@@ -27,16 +27,22 @@ struct RmsRowsDesc {
   float eps = 1e-5f;
 };
 Status rms_rows(cudaStream_t s, const RmsRowsDesc& d);
-// out[r, 0 .. ff) = g sigmoid(1.702 g) (u + 1), g = min(gu[r, c], limit), u = clamp(gu[r, ff + c], -limit, limit)
-Status clamped_glu(cudaStream_t s, DType dt, const void* gu, int64_t ld_in, void* out, int64_t ld_out, int64_t rows, int ff, float limit);
+// out[r, 0 .. ff) = g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit); the columns of gu come in
+// blocks of `block` gates followed by the values they gate (block = ff: two halves; kGluBlock: as the GEMM's gated epilogue
+// wants its weight rows).
+constexpr int kGluBlock = 16;
+inline int64_t glu_rows(int64_t ff) { return (ff + kGluBlock - 1) / kGluBlock * 2 * kGluBlock; }
+Status clamped_glu(cudaStream_t s, DType dt, const void* gu, int64_t ld_in, void* out, int64_t ld_out, int64_t rows, int ff, int block, float limit);
 
 // ── linears of a step with at most 16 rows (seq_skinny.cu) ──────────────────
-// One launch runs up to kSeqSegs products against K-major weights [n, ld] (rows of length k). The input rows are either
-// x (float32) normalised on the way into shared memory, rms(x) * norm_w, or `a` (storage type) as it lies.
+// One launch runs up to kSeqSegs products against K-major weights [n, ld] (rows of length k). 16-bit models hand each product
+// its stored input rows `a` (tensor cores); any model can hand all of them the float32 stream x, normalised on the way into shared
+// memory as rms(x) * norm_w, or one stored input (CUDA cores).
 enum class SeqOut : int { Store = 0, StoreF32 = 1, Glu = 2, AddF32 = 3 };
 struct SeqSeg {
-  const void* w = nullptr; int64_t ld = 0; int n = 0;      // Glu: w holds n gate rows, then n up rows
+  const void* w = nullptr; int64_t ld = 0; int n = 0;      // Glu: n results from glu_rows(n) weight rows in blocks of kGluBlock gates | values
   const float* norm_w = nullptr;
+  const void* a = nullptr; int64_t a_ld = 0;
   SeqOut mode = SeqOut::Store; float limit = 0.f;
   void* out = nullptr; int64_t out_ld = 0;
 };

@@ -1,6 +1,7 @@
 // Linears of a step that carries at most 16 rows (a generated token per sequence, or a prompt portion of a few tokens).
 //
-// Such a product is bound by reading its K-major weight once. A warp owns RW weight rows (for the gated form RW / 2
+// Such a product is bound by reading its K-major weight once. 16-bit models take the tensor-core form further down. In the other
+// one, a warp owns RW weight rows (for the gated form RW / 2
 // gate rows and their up rows), its lanes split K in 16-byte pieces, and the input rows wait in shared memory as floats.
 // One launch serves up to three weights that read the same stream: the projections of a mixer and of the feed-forward
 // beside it depend on nothing but x, so a layer starts with a single launch whose prologue takes the RMS norms. The
@@ -39,11 +40,11 @@ __global__ void __launch_bounds__(kSsThreads) seq_skinny_kernel(const SsParams p
   constexpr int GW = RW >= 2 ? RW / 2 : 1;
   const int n0 = (((int)blockIdx.x - sg.block0) * kSsWarps + warp) * (glu ? GW : RW);
   const T* W = reinterpret_cast<const T*>(sg.w);
-  // weight row of register slot r: gate rows in the first half of the slots, their up rows in the second
+  // weight row of register slot r: gate rows in the first half of the slots, the rows of the values they gate in the second
   auto row_of = [&](int r) -> long long {
     if (!glu) return n0 + r < sg.n ? n0 + r : -1;
     const int c = n0 + r % GW;
-    return c < sg.n ? (long long)c + (r / GW) * (long long)sg.n : -1;
+    return c < sg.n ? (long long)(c / kGluBlock * 2 * kGluBlock + c % kGluBlock + r / GW * kGluBlock) : -1;
   };
   const T* wp[RW];
 #pragma unroll
@@ -135,6 +136,123 @@ __global__ void __launch_bounds__(kSsThreads) seq_skinny_kernel(const SsParams p
   }
 }
 
+// ── the tensor-core form ────────────────────────────────────────────────────
+// 16-bit weights and inputs. A CTA owns 16 weight rows (for the gated form 8 gate rows and the 8 rows they gate), its eight
+// warps take every eighth 32-column block of K, and mma.m16n8k16 multiplies them with the input rows as the 8-wide
+// operand. The order of K inside a block is free as long as both operands agree on it, so a lane feeds two MMAs from one
+// 16-byte piece of each of its two weight rows and of its input row: no shared memory and no shuffles in the loop. The
+// first pieces of the weights are requested before the programmatic dependency wait. The warps' sums meet in shared memory.
+struct SmSeg { const void* w; const void* a; void* out; long long ld, a_ld, out_ld; int n, mode, block0; float limit; };
+struct SmParams { SmSeg seg[kSeqSegs]; int n_seg, rows, kp; };
+
+template <typename T> __device__ __forceinline__ void mma_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1);
+template <> __device__ __forceinline__ void mma_16816<__nv_bfloat16>(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+template <> __device__ __forceinline__ void mma_16816<__half>(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+template <typename T, int NT>        // NT groups of 8 input rows
+__global__ void __launch_bounds__(kSsThreads) seq_skinny_mma_kernel(const SmParams p) {
+  constexpr int U = 4;               // 32-column blocks in flight per warp
+  __shared__ float red[kSsWarps][NT * 8][17];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
+  int si = 0;
+#pragma unroll
+  for (int i = 1; i < kSeqSegs; i++) if (i < p.n_seg && (int)blockIdx.x >= p.seg[i].block0) si = i;
+  const SmSeg sg = p.seg[si];
+  const bool glu = sg.mode == (int)SeqOut::Glu;
+  const int group = (int)blockIdx.x - sg.block0;
+  const int c0 = group * (glu ? 8 : 16);                        // first result column
+  long long r0, r1;                                             // this lane's two weight rows
+  if (glu) { r0 = c0 / kGluBlock * 2 * kGluBlock + c0 % kGluBlock + g; r1 = r0 + kGluBlock; }
+  else { r0 = c0 + g; r1 = r0 + 8; }
+  const bool live0 = glu || r0 < sg.n, live1 = glu || r1 < sg.n;
+  const T* w0 = reinterpret_cast<const T*>(sg.w) + r0 * sg.ld;
+  const T* w1 = reinterpret_cast<const T*>(sg.w) + r1 * sg.ld;
+  const T* x[NT];
+#pragma unroll
+  for (int t = 0; t < NT; t++) x[t] = g + 8 * t < p.rows ? reinterpret_cast<const T*>(sg.a) + (long long)(g + 8 * t) * sg.a_ld : nullptr;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  float acc[NT][4];
+#pragma unroll
+  for (int t = 0; t < NT; t++) { acc[t][0] = 0.f; acc[t][1] = 0.f; acc[t][2] = 0.f; acc[t][3] = 0.f; }
+  uint4 a0[U], a1[U];
+  auto fetch = [&](int kb) {
+#pragma unroll
+    for (int u = 0; u < U; u++) {
+      const int kk = (kb + u * kSsWarps) * 32 + q * 8;
+      a0[u] = live0 && kk < p.kp ? __ldcs(reinterpret_cast<const uint4*>(w0 + kk)) : zero;
+      a1[u] = live1 && kk < p.kp ? __ldcs(reinterpret_cast<const uint4*>(w1 + kk)) : zero;
+    }
+  };
+  fetch(warp);
+  pdl_wait();
+  pdl_trigger();
+  for (int kb = warp; kb * 32 < p.kp;) {
+    uint4 b[U][NT];
+#pragma unroll
+    for (int u = 0; u < U; u++) {
+      const int kk = (kb + u * kSsWarps) * 32 + q * 8;
+#pragma unroll
+      for (int t = 0; t < NT; t++) b[u][t] = x[t] && kk < p.kp ? *reinterpret_cast<const uint4*>(x[t] + kk) : zero;
+    }
+#pragma unroll
+    for (int u = 0; u < U; u++)
+#pragma unroll
+      for (int t = 0; t < NT; t++) {
+        mma_16816<T>(acc[t], a0[u].x, a1[u].x, a0[u].y, a1[u].y, b[u][t].x, b[u][t].y);
+        mma_16816<T>(acc[t], a0[u].z, a1[u].z, a0[u].w, a1[u].w, b[u][t].z, b[u][t].w);
+      }
+    kb += U * kSsWarps;
+    if (kb * 32 < p.kp) fetch(kb);
+  }
+#pragma unroll
+  for (int t = 0; t < NT; t++) {      // lane: rows g and g + 8 of the weights, input rows 2 q and 2 q + 1
+    red[warp][t * 8 + 2 * q][g] = acc[t][0]; red[warp][t * 8 + 2 * q + 1][g] = acc[t][1];
+    red[warp][t * 8 + 2 * q][g + 8] = acc[t][2]; red[warp][t * 8 + 2 * q + 1][g + 8] = acc[t][3];
+  }
+  __syncthreads();
+  const int width = glu ? 8 : 16;
+  for (int i = threadIdx.x; i < NT * 8 * width; i += kSsThreads) {
+    const int m = i / width, n = i % width;
+    if (m >= p.rows || c0 + n >= sg.n) continue;
+    float v = 0.f, up = 0.f;
+#pragma unroll
+    for (int w = 0; w < kSsWarps; w++) { v += red[w][m][n]; if (glu) up += red[w][m][n + 8]; }
+    const long long o = (long long)m * sg.out_ld + c0 + n;
+    if (glu) reinterpret_cast<T*>(sg.out)[o] = Cvt<T>::from(clamped_glu_f(v, up, sg.limit));
+    else if (sg.mode == (int)SeqOut::Store) reinterpret_cast<T*>(sg.out)[o] = Cvt<T>::from(v);
+    else if (sg.mode == (int)SeqOut::StoreF32) reinterpret_cast<float*>(sg.out)[o] = v;
+    else reinterpret_cast<float*>(sg.out)[o] += v;
+  }
+}
+
+static Status seq_skinny_mma(cudaStream_t s, const SeqSkinnyDesc& d) {
+  SmParams p;
+  p.n_seg = d.n_seg; p.rows = d.rows; p.kp = (int)pad8(d.k);
+  int blocks = 0;
+  for (int i = 0; i < d.n_seg; i++) {
+    const SeqSeg& g = d.seg[i];
+    if (!g.w || !g.out || !g.a || g.n < 1 || g.ld % 8 != 0 || g.ld < d.k || g.a_ld % 8 != 0 || g.a_ld < p.kp || !aligned16(g.w) || !aligned16(g.a)) return Status::invalid("seq_skinny: bad segment");
+    SmSeg& q = p.seg[i];
+    q.w = g.w; q.a = g.a; q.out = g.out; q.ld = g.ld; q.a_ld = g.a_ld; q.out_ld = g.out_ld; q.n = g.n; q.mode = (int)g.mode; q.block0 = blocks; q.limit = g.limit;
+    const int per = g.mode == SeqOut::Glu ? 8 : 16;
+    blocks += (g.n + per - 1) / per;
+  }
+  cudaError_t e;
+  if (d.dtype == DType::BF16)
+    e = d.rows <= 8 ? launch_pdl(seq_skinny_mma_kernel<__nv_bfloat16, 1>, dim3((unsigned)blocks), dim3(kSsThreads), 0, s, p)
+                    : launch_pdl(seq_skinny_mma_kernel<__nv_bfloat16, 2>, dim3((unsigned)blocks), dim3(kSsThreads), 0, s, p);
+  else
+    e = d.rows <= 8 ? launch_pdl(seq_skinny_mma_kernel<__half, 1>, dim3((unsigned)blocks), dim3(kSsThreads), 0, s, p)
+                    : launch_pdl(seq_skinny_mma_kernel<__half, 2>, dim3((unsigned)blocks), dim3(kSsThreads), 0, s, p);
+  return cuda_status(e, "seq_skinny (tensor cores)");
+}
+
 bool seq_skinny_fits(int64_t k) { return pad8(k) * (int64_t)sizeof(float) <= (int64_t)kSsMaxSmem; }
 
 template <typename T, int MR, int RW>
@@ -153,7 +271,9 @@ static cudaError_t launch_ss_rw(cudaStream_t s, const SsParams& p, dim3 grid, si
 }
 
 Status seq_skinny(cudaStream_t s, const SeqSkinnyDesc& d) {
-  if (d.rows < 1 || d.rows > kSeqSkinnyRows || d.n_seg < 1 || d.n_seg > kSeqSegs || (!d.x == !d.a)) return Status::invalid("seq_skinny: bad description");
+  if (d.rows < 1 || d.rows > kSeqSkinnyRows || d.n_seg < 1 || d.n_seg > kSeqSegs) return Status::invalid("seq_skinny: bad description");
+  if (d.seg[0].a && d.dtype != DType::F32) return seq_skinny_mma(s, d);
+  if (!d.x == !d.a) return Status::invalid("seq_skinny: one input");
   if (!seq_skinny_fits(d.k)) return Status::unsupported("seq_skinny: input rows too long");
   SsParams p;
   p.x = d.x; p.a = d.a; p.a_ld = d.a_ld; p.eps = d.eps; p.rows = d.rows; p.k = d.k; p.kp = (int)pad8(d.k); p.n_seg = d.n_seg;

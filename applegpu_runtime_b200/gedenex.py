@@ -6,7 +6,7 @@ weights are [out, in].
 """
 import numpy as np
 
-from .seqmodel import Layer, Rotary, SequenceModel, rows, side_by_side
+from .seqmodel import Layer, Rotary, SequenceModel, interleaved, rows, side_by_side
 
 ARCHITECTURE = "Gedenex"
 
@@ -68,7 +68,7 @@ def load_gedenex(config, weights, dtype="bfloat16"):
                 raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']}")
             layer.ff, layer.ff_limit = int(mlp["ff"]), float(mlp["limit"])
             layer.norm2 = t.get(p + "norm2", width)
-            layer.w_ff = rows(t.get(p + "mlp.gate", layer.ff, width), t.get(p + "mlp.up", layer.ff, width))
+            layer.w_ff = interleaved(t.get(p + "mlp.gate", layer.ff, width), t.get(p + "mlp.up", layer.ff, width))
             down = t.get(p + "mlp.down", width, layer.ff)
         layer.w_out = side_by_side(out, down)
         layers.append(layer)

@@ -75,6 +75,17 @@ def rows(*parts, pad_rows=False):
     return np.concatenate(out, axis=0)
 
 
+def interleaved(gate, up, block=16):
+    """Gate and up rows in blocks of 16 gates and the 16 rows they gate, padded with zero rows to whole blocks."""
+    n = (gate.shape[0] + block - 1) // block
+    a = np.zeros((n, 2, block, gate.shape[1]), np.float32)
+    for i, p in enumerate((gate, up)):
+        q = np.zeros((n * block, gate.shape[1]), np.float32)
+        q[:p.shape[0]] = p
+        a[:, i] = q.reshape(n, block, -1)
+    return rows(a.reshape(2 * n * block, -1))
+
+
 def side_by_side(first, second):
     """Two [out, in] matrices with their inputs one after the other, the first one's padded to a multiple of 8."""
     if second is None:

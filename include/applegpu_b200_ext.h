@@ -297,8 +297,8 @@ APPLEGPU_API void applegpu_gpt2_decoder_destroy(uint64_t decoder);
  *   create:  weight_ids = embed [vocab, width], head [vocab, P(width)], final norm f32 [width], step vectors f32
  *            [loop_times, width] (0 without a loop), then eight per layer: norm1, norm2 (f32 [width]; 0 without a
  *            feed-forward), the mixer's input rows [cols, P(width)], the output rows [width, P(K)] with K = P(heads * vdim) + ff
- *            (mixer columns, then feed-forward columns) or heads * vdim without a feed-forward, gate rows | up rows
- *            [2 ff, P(width)] (or 0), and three of the mixer's own:
+ *            (mixer columns, then feed-forward columns) or heads * vdim without a feed-forward, feed-forward rows in
+ *            blocks of 16 gates | the 16 they gate (ff rounded up to 16, zero rows) [.., P(width)] (or 0), and three of the mixer's own:
  *              mLSTM    input rows q | k | v | g; own: i rows | f rows [2 heads, P(width)], f32 bias [2 heads], f32 norm [heads * vdim]
  *              latent   input rows q (per head: dim, rot_dim) | latent | rotated key part; own: f32 latent norm [kv_rank],
  *                       uk rows, padded to P(heads * dim), | uv rows, padded to P(heads * vdim), [.., P(kv_rank)], and

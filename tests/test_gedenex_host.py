@@ -50,7 +50,7 @@ def test_safetensors_round_trip(tmp_path):
 
 
 def test_packing():
-    from applegpu_runtime_b200.seqmodel import rows, side_by_side
+    from applegpu_runtime_b200.seqmodel import interleaved, rows, side_by_side
     a, b = np.ones((3, 5), np.float32), 2 * np.ones((2, 5), np.float32)
     m = rows(a, b)
     assert m.shape == (5, 8) and np.all(m[:3, :5] == 1) and np.all(m[3:, :5] == 2) and np.all(m[:, 5:] == 0)
@@ -58,6 +58,9 @@ def test_packing():
     assert m.shape == (16, 8) and np.all(m[8:10, :5] == 2) and m.sum() == 15 + 20
     m = side_by_side(np.ones((4, 3), np.float32), 2 * np.ones((4, 6), np.float32))
     assert m.shape == (4, 16) and np.all(m[:, :3] == 1) and np.all(m[:, 3:8] == 0) and np.all(m[:, 8:14] == 2) and np.all(m[:, 14:] == 0)
+    m = interleaved(np.arange(18, dtype=np.float32)[:, None], 100 + np.arange(18, dtype=np.float32)[:, None])
+    assert m.shape == (64, 8) and m[:16, 0].tolist() == list(range(16)) and m[16:32, 0].tolist() == list(range(100, 116)) and m[32:34, 0].tolist() == [16, 17]
+    assert m[48:50, 0].tolist() == [116, 117] and m[34:48].sum() == 0 and m[50:].sum() == 0
     with pytest.raises(ValueError):
         rows(a, np.ones((2, 4), np.float32))
 
