@@ -487,6 +487,8 @@ Status seq_create(const SeqModelCfg& cfg, const std::vector<TensorRec>& weights,
   for (const LayerRun& r : e->runs) {
     std::shared_ptr<Buffer> b;
     AG_RETURN_IF_ERROR(Shared::get().pool.acquire((size_t)slots * e->mixers[r.layer]->slot_bytes(max_len), &b));
+    // padding columns of caches take part in products with zeros: they must hold numbers
+    if (cudaMemsetAsync(b->ptr, 0, b->capacity, ctx.stream) != cudaSuccess) return Status::compute("sequence engine: clear");
     e->memory.push_back(b);
   }
   e->len.assign(slots, 0);

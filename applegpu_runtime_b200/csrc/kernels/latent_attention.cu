@@ -10,6 +10,7 @@
 // Scores, their maximum and the weights are float32 throughout.
 #include "common.cuh"
 #include "seq_kernels.h"
+#include "mma_sync.cuh"
 
 namespace ag { namespace k {
 
@@ -226,14 +227,31 @@ __global__ void __launch_bounds__(256) latent_decode_prepare_kernel(const LaPara
     out[p.coff + i] = v * p.scale;
   }
   __syncthreads();
+  // 16-byte pieces of the rows of W_uk: a thread owns one piece's columns and every G-th row, the G partial sums meet in
+  // shared memory
+  constexpr int N = Pack<T>::N;
   const T* uk = reinterpret_cast<const T*>(p.uk) + (long long)h * p.dim * p.w_ld;
+  float* part = sq + p.dim;
+  const int nv = p.coff / N, G = nv >= 256 ? 1 : 256 / nv, g = threadIdx.x / nv, col = threadIdx.x % nv;
+  if (g < G) {
+    float a[N];
+#pragma unroll
+    for (int e = 0; e < N; e++) a[e] = 0.f;
+#pragma unroll 8
+    for (int d = g; d < p.dim; d += G) {
+      const Pack<T> w = ld16(uk + (long long)d * p.w_ld + col * N);
+      const float x = sq[d];
+#pragma unroll
+      for (int e = 0; e < N; e++) a[e] = fmaf(x, Cvt<T>::to(w.v[e]), a[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < N; e++) part[g * p.coff + col * N + e] = a[e];
+  }
+  __syncthreads();
   for (int i = threadIdx.x; i < p.coff; i += 256) {
     float a = 0.f;
-    if (i < p.rank) {
-#pragma unroll 8
-      for (int d = 0; d < p.dim; d++) a = fmaf(sq[d], Cvt<T>::to(uk[(long long)d * p.w_ld + i]), a);
-    }
-    out[i] = a * p.scale;
+    for (int k = 0; k < G; k++) a += part[k * p.coff + i];
+    out[i] = i < p.rank ? a * p.scale : 0.f;
   }
 }
 
@@ -319,6 +337,155 @@ __global__ void __launch_bounds__(256) latent_decode_attend_kernel(const LaParam
   }
 }
 
+// The same on tensor cores for 16-bit caches: CTA = (split, sixteen heads, row), blocks of 64 keys in shared memory. The query
+// (float32) and the weights (float32) enter the products as high part and remainder. A warp takes 8 keys of the scores and
+// every eighth 8-column tile of the latent; each warp's two heads get their maximum, weights and sum in between.
+constexpr int kLmKeys = 64, kLmHeads = 16;
+__host__ __device__ inline int lm_k(int cld) { return (cld + 31) / 32 * 32; }
+__host__ __device__ inline int lm_pitch(int cld) { const int p = lm_k(cld) / 8; return (p % 2 ? p : p + 1) * 8; }   // odd number of 16-byte pieces: no bank conflicts
+static size_t lm_smem(int cld) { return ((size_t)kLmKeys + 2 * kLmHeads) * lm_pitch(cld) * 2 + (size_t)kLmHeads * (kLmKeys + 1) * 4 + 2 * (size_t)kLmHeads * (kLmKeys + 8) * 2 + 4 * kLmHeads * 4; }
+__device__ __forceinline__ uint32_t lm_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+template <typename T, int NW>          // NW: 8-column latent tiles per warp, rank <= 64 * NW
+__global__ void __launch_bounds__(256) latent_decode_attend_mma_kernel(const LaParams p) {
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  const int K = lm_k(p.cld), P = lm_pitch(p.cld);
+  T* sk = reinterpret_cast<T*>(smem_raw);              // [kLmKeys][P]
+  T* sqh = sk + kLmKeys * P;                           // [16][P] high parts of the queries, then their remainders
+  T* sql = sqh + kLmHeads * P;
+  float* ss = reinterpret_cast<float*>(sql + kLmHeads * P);          // [16][kLmKeys + 1]
+  T* sph = reinterpret_cast<T*>(ss + kLmHeads * (kLmKeys + 1));      // [16][kLmKeys + 8]
+  T* spl = sph + kLmHeads * (kLmKeys + 8);
+  float* sm_m = reinterpret_cast<float*>(spl + kLmHeads * (kLmKeys + 8));
+  float* sm_l = sm_m + kLmHeads;
+  float* sm_a = sm_l + kLmHeads;
+  const int split = blockIdx.x, r = blockIdx.z, s = r / p.T, t = r % p.T, h0 = (int)blockIdx.y * kLmHeads;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  pdl_wait();
+  pdl_trigger();
+  const int n_keys = min(p.pos[s] + t + 1, p.max_len);
+  const int per = ((n_keys + p.splits - 1) / p.splits + kLmKeys - 1) / kLmKeys * kLmKeys;
+  const int k_lo = split * per, k_hi = min(n_keys, k_lo + per);
+  const int live = min(kLmHeads, p.heads - h0);
+  if (k_lo >= k_hi) {                                  // nothing for this split: an empty partial
+    for (int i = threadIdx.x; i < live; i += 256) {
+      float* dst = p.part + (((long long)r * p.heads + h0 + i) * p.splits + split) * (p.rank + 2);
+      dst[0] = -INFINITY; dst[1] = 0.f;
+    }
+    for (int i = threadIdx.x; i < live * p.rank; i += 256)
+      p.part[(((long long)r * p.heads + h0 + i / p.rank) * p.splits + split) * (p.rank + 2) + 2 + i % p.rank] = 0.f;
+    return;
+  }
+  for (int i = threadIdx.x; i < kLmHeads * K; i += 256) {
+    const int hh = i / K, c = i % K;
+    const float v = hh < live && c < p.cld ? p.q_eff[((long long)r * p.heads + h0 + hh) * p.cld + c] : 0.f;
+    const T hi = Cvt<T>::from(v);
+    sqh[hh * P + c] = hi;
+    sql[hh * P + c] = Cvt<T>::from(v - Cvt<T>::to(hi));
+  }
+  for (int i = threadIdx.x; i < kLmKeys * (K - p.cld); i += 256) sk[i / (K - p.cld) * P + p.cld + i % (K - p.cld)] = Cvt<T>::from(0.f);
+  if (threadIdx.x < kLmHeads) { sm_m[threadIdx.x] = -INFINITY; sm_l[threadIdx.x] = 0.f; }
+  const T* cache = reinterpret_cast<const T*>(p.cache) + (long long)s * p.seq_stride;
+  float o[NW][4];
+#pragma unroll
+  for (int j = 0; j < NW; j++) { o[j][0] = 0.f; o[j][1] = 0.f; o[j][2] = 0.f; o[j][3] = 0.f; }
+  const int pieces = p.cld / 8;
+  for (int k0 = k_lo; k0 < k_hi; k0 += kLmKeys) {
+    const int nk = min(kLmKeys, k_hi - k0);
+    __syncthreads();
+    for (int i = threadIdx.x; i < kLmKeys * pieces; i += 256) {
+      const int j = i / pieces, c = i % pieces * 8;
+      T* dst = sk + j * P + c;
+      if (j < nk) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(lm_addr(dst)), "l"(cache + (long long)(k0 + j) * p.cld + c));
+      else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    {
+      // scores: 16 heads x 8 keys per warp
+      float c4[4] = {0.f, 0.f, 0.f, 0.f};
+      const uint32_t qa = lm_addr(sqh + (lane & 15) * P + (lane >> 4) * 8), la = lm_addr(sql + (lane & 15) * P + (lane >> 4) * 8);
+      const uint32_t ka = lm_addr(sk + (warp * 8 + (lane & 7)) * P + (lane >> 3) * 8);
+      for (int kk = 0; kk < K; kk += 32) {
+        uint32_t b[4], a0[4], a1[4];
+        ldsm_x4(b, ka + kk * 2);
+        ldsm_x4(a0, qa + kk * 2);
+        ldsm_x4(a1, qa + kk * 2 + 32);
+        mma_16816<T>(c4, a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
+        mma_16816<T>(c4, a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
+        ldsm_x4(a0, la + kk * 2);
+        ldsm_x4(a1, la + kk * 2 + 32);
+        mma_16816<T>(c4, a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
+        mma_16816<T>(c4, a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
+      }
+      const int g = lane >> 2, q = lane & 3, key = warp * 8 + 2 * q;
+      ss[g * (kLmKeys + 1) + key] = c4[0]; ss[g * (kLmKeys + 1) + key + 1] = c4[1];
+      ss[(g + 8) * (kLmKeys + 1) + key] = c4[2]; ss[(g + 8) * (kLmKeys + 1) + key + 1] = c4[3];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 2; i++) {
+      const int h = warp * 2 + i;
+      const float x0 = lane < nk ? ss[h * (kLmKeys + 1) + lane] : -INFINITY, x1 = lane + 32 < nk ? ss[h * (kLmKeys + 1) + lane + 32] : -INFINITY;
+      const float m0 = sm_m[h], m1 = fmaxf(m0, warp_max(fmaxf(x0, x1)));
+      const float e0 = lane < nk ? expf(x0 - m1) : 0.f, e1 = lane + 32 < nk ? expf(x1 - m1) : 0.f;
+      const float sum = warp_sum(e0 + e1);
+      const T p0 = Cvt<T>::from(e0), p1 = Cvt<T>::from(e1);
+      sph[h * (kLmKeys + 8) + lane] = p0; sph[h * (kLmKeys + 8) + lane + 32] = p1;
+      spl[h * (kLmKeys + 8) + lane] = Cvt<T>::from(e0 - Cvt<T>::to(p0)); spl[h * (kLmKeys + 8) + lane + 32] = Cvt<T>::from(e1 - Cvt<T>::to(p1));
+      if (lane == 0) {
+        const float a = m0 == -INFINITY ? 0.f : expf(m0 - m1);
+        sm_a[h] = a; sm_l[h] = sm_l[h] * a + sum; sm_m[h] = m1;
+      }
+    }
+    __syncthreads();
+    {
+      const int g = lane >> 2;
+      const float f0 = sm_a[g], f1 = sm_a[g + 8];
+#pragma unroll
+      for (int j = 0; j < NW; j++) { o[j][0] *= f0; o[j][1] *= f0; o[j][2] *= f1; o[j][3] *= f1; }
+      const uint32_t pa = lm_addr(sph + (lane & 15) * (kLmKeys + 8) + (lane >> 4) * 8), pl = lm_addr(spl + (lane & 15) * (kLmKeys + 8) + (lane >> 4) * 8);
+#pragma unroll
+      for (int kk = 0; kk < kLmKeys; kk += 32) {
+        uint32_t h0a[4], h1a[4], l0a[4], l1a[4];
+        ldsm_x4(h0a, pa + kk * 2); ldsm_x4(h1a, pa + kk * 2 + 32);
+        ldsm_x4(l0a, pl + kk * 2); ldsm_x4(l1a, pl + kk * 2 + 32);
+#pragma unroll
+        for (int j = 0; j < NW; j++) {
+          const int c = (j * 8 + warp) * 8;
+          if (c >= p.rank) break;
+          uint32_t b[4];                               // keys kk .. kk + 31 of eight latent columns
+          ldsm_x4_t(b, lm_addr(sk + (kk + lane) * P + c));
+          mma_16816<T>(o[j], h0a[0], h0a[1], h0a[2], h0a[3], b[0], b[1]);
+          mma_16816<T>(o[j], h1a[0], h1a[1], h1a[2], h1a[3], b[2], b[3]);
+          mma_16816<T>(o[j], l0a[0], l0a[1], l0a[2], l0a[3], b[0], b[1]);
+          mma_16816<T>(o[j], l1a[0], l1a[1], l1a[2], l1a[3], b[2], b[3]);
+        }
+      }
+    }
+  }
+  const int g = lane >> 2, q = lane & 3;
+#pragma unroll
+  for (int i = 0; i < 2; i++) {
+    const int h = g + 8 * i;
+    if (h >= live) continue;
+    float* dst = p.part + (((long long)r * p.heads + h0 + h) * p.splits + split) * (p.rank + 2);
+    if (warp == 0 && q == 0) { dst[0] = sm_m[h]; dst[1] = sm_l[h]; }
+#pragma unroll
+    for (int j = 0; j < NW; j++) {
+      const int c = (j * 8 + warp) * 8 + 2 * q;
+      if (c < p.rank) dst[2 + c] = o[j][2 * i];
+      if (c + 1 < p.rank) dst[2 + c + 1] = o[j][2 * i + 1];
+    }
+  }
+}
+
 // merge: the splits of one head combined, then the head's slice of W_uv.
 template <typename T>
 __global__ void __launch_bounds__(256) latent_decode_merge_kernel(const LaParams p) {
@@ -344,21 +511,39 @@ __global__ void __launch_bounds__(256) latent_decode_merge_kernel(const LaParams
     for (int i = threadIdx.x; i < p.splits; i += 32) s_w[i] /= l;
   }
   __syncthreads();
-  for (int c = threadIdx.x; c < p.rank; c += 256) {
+  for (int c = threadIdx.x; c < p.coff; c += 256) {
     float a = 0.f;
-#pragma unroll 4
-    for (int i = 0; i < p.splits; i++) if (s_w[i] != 0.f) a = fmaf(s_w[i], part[(long long)i * (p.rank + 2) + 2 + c], a);
+    if (c < p.rank)
+#pragma unroll 8
+      for (int i = 0; i < p.splits; i++) a = fmaf(s_w[i], part[(long long)i * (p.rank + 2) + 2 + c], a);
     so[c] = a;
   }
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const T* uv = reinterpret_cast<const T*>(p.uv) + (long long)h * p.vdim * p.w_ld;
   T* y = reinterpret_cast<T*>(p.y) + (long long)r * p.y_ld + (long long)h * p.vdim;
-  for (int e = warp; e < p.vdim; e += 8) {
-    float a = 0.f;
-    for (int c = lane; c < p.rank; c += 32) a = fmaf(so[c], Cvt<T>::to(uv[(long long)e * p.w_ld + c]), a);
-    a = warp_sum(a);
-    if (lane == 0) y[e] = Cvt<T>::from(a);
+  constexpr int N = Pack<T>::N, R = 4;                   // R rows of W_uv per warp and pass, 16-byte pieces
+  const int nv = p.coff / N;
+  for (int e0 = warp * R; e0 < p.vdim; e0 += 8 * R) {
+    float a[R];
+#pragma unroll
+    for (int r = 0; r < R; r++) a[r] = 0.f;
+    for (int c = lane; c < nv; c += 32) {
+      Pack<T> w[R];
+#pragma unroll
+      for (int r = 0; r < R; r++) w[r] = ld16(uv + (long long)min(e0 + r, p.vdim - 1) * p.w_ld + c * N);
+#pragma unroll
+      for (int q = 0; q < N; q++) {
+        const float x = so[c * N + q];
+#pragma unroll
+        for (int r = 0; r < R; r++) a[r] = fmaf(x, Cvt<T>::to(w[r].v[q]), a[r]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < R; r++) {
+      a[r] = warp_sum(a[r]);
+      if (lane == 0 && e0 + r < p.vdim) y[e0 + r] = Cvt<T>::from(a[r]);
+    }
   }
 }
 
@@ -384,20 +569,43 @@ static cudaError_t launch_ld(cudaStream_t s, const LaParams& p, dim3 grid, size_
   }
   return launch_pdl(latent_decode_attend_kernel<T, NR>, grid, dim3(256), smem, s, p);
 }
+template <typename T, int NW>
+static cudaError_t launch_lm(cudaStream_t s, const LaParams& p, dim3 grid, size_t smem) {
+  static bool attr = false;
+  if (!attr) {
+    cudaError_t e = cudaFuncSetAttribute(latent_decode_attend_mma_kernel<T, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+    if (e != cudaSuccess) return e;
+    attr = true;
+  }
+  return launch_pdl(latent_decode_attend_mma_kernel<T, NW>, grid, dim3(256), smem, s, p);
+}
 template <typename T>
 static cudaError_t latent_decode_t(cudaStream_t s, const LaParams& p) {
   const int rows = p.n_seq * p.T;
-  cudaError_t e = launch_pdl(latent_decode_prepare_kernel<T>, dim3((unsigned)(p.heads + 1), (unsigned)rows), dim3(256), (size_t)p.dim * sizeof(float), s, p);
+  const size_t psmem = ((size_t)p.dim + 256 * Pack<T>::N) * sizeof(float);
+  cudaError_t e = launch_pdl(latent_decode_prepare_kernel<T>, dim3((unsigned)(p.heads + 1), (unsigned)rows), dim3(256), psmem, s, p);
   if (e != cudaSuccess) return e;
-  const size_t smem = (size_t)kLdHeads * p.cld * sizeof(float) + (size_t)kLdKeys * (p.cld + 2) * sizeof(T);
-  const dim3 grid((unsigned)p.splits, (unsigned)((p.heads + kLdHeads - 1) / kLdHeads), (unsigned)rows);
-  if (p.rank <= 64) e = launch_ld<T, 2>(s, p, grid, smem);
-  else if (p.rank <= 128) e = launch_ld<T, 4>(s, p, grid, smem);
-  else if (p.rank <= 256) e = launch_ld<T, 8>(s, p, grid, smem);
-  else if (p.rank <= 512) e = launch_ld<T, 16>(s, p, grid, smem);
-  else e = launch_ld<T, 32>(s, p, grid, smem);
+  bool done = false;
+  if constexpr (sizeof(T) == 2) {
+    const size_t smem = lm_smem(p.cld);
+    if (smem <= 220 * 1024) {
+      const dim3 grid((unsigned)p.splits, (unsigned)((p.heads + kLmHeads - 1) / kLmHeads), (unsigned)rows);
+      e = p.rank <= 128 ? launch_lm<T, 2>(s, p, grid, smem) : p.rank <= 256 ? launch_lm<T, 4>(s, p, grid, smem) : p.rank <= 512 ? launch_lm<T, 8>(s, p, grid, smem)
+                                                                                                                                : launch_lm<T, 16>(s, p, grid, smem);
+      done = true;
+    }
+  }
+  if (!done) {
+    const size_t smem = (size_t)kLdHeads * p.cld * sizeof(float) + (size_t)kLdKeys * (p.cld + 2) * sizeof(T);
+    const dim3 grid((unsigned)p.splits, (unsigned)((p.heads + kLdHeads - 1) / kLdHeads), (unsigned)rows);
+    if (p.rank <= 64) e = launch_ld<T, 2>(s, p, grid, smem);
+    else if (p.rank <= 128) e = launch_ld<T, 4>(s, p, grid, smem);
+    else if (p.rank <= 256) e = launch_ld<T, 8>(s, p, grid, smem);
+    else if (p.rank <= 512) e = launch_ld<T, 16>(s, p, grid, smem);
+    else e = launch_ld<T, 32>(s, p, grid, smem);
+  }
   if (e != cudaSuccess) return e;
-  return launch_pdl(latent_decode_merge_kernel<T>, dim3((unsigned)p.heads, (unsigned)rows), dim3(256), (size_t)p.rank * sizeof(float), s, p);
+  return launch_pdl(latent_decode_merge_kernel<T>, dim3((unsigned)p.heads, (unsigned)rows), dim3(256), (size_t)p.coff * sizeof(float), s, p);
 }
 
 Status latent_decode(cudaStream_t s, const LatentDesc& d, void* work) {

@@ -130,36 +130,72 @@ __global__ void __launch_bounds__(256) ml_chunk_kernel(const MlParams p) {
 }
 
 // ── carry: the chunks' own states become the states in front of them ────────
-template <typename T>      // storage type of the planes the tensor-core output kernel reads; float: none, the states stay float32
-__global__ void __launch_bounds__(256) ml_carry_kernel(const MlParams p) {
+// A thread owns VEC neighbouring elements of a head's S (or one of n, by the blocks past S).
+template <typename T, int VEC>      // T: storage type of the planes the tensor-core output kernel reads; float: none, the states stay float32
+__global__ void __launch_bounds__(256) ml_carry_kernel(const MlParams p, int s_blocks) {
+  __shared__ float s_decay[256];
   pdl_wait();
   pdl_trigger();
   const int sh = blockIdx.y, s = sh / p.heads, h = sh % p.heads;
-  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
   const long long n_state = (long long)p.dim * p.vdim;
-  if (i >= n_state + p.dim) return;
-  const bool is_n = i >= n_state;
-  float* home = is_n ? p.n_of(s) + (long long)h * p.dim + (i - n_state) : p.S_of(s) + h * n_state + i;
-  float* own = is_n ? p.w.n + (long long)sh * p.w.chunks * p.dim + (i - n_state) : p.w.S + (long long)sh * p.w.chunks * n_state + i;
-  const long long step = is_n ? p.dim : n_state;
   const double* F = p.w.F + (long long)sh * p.T;
   const float* ms = p.w.m_start + (long long)sh * (p.w.chunks + 1);
-  float v = *home;
-#pragma unroll 4
-  for (int c = 0; c < p.w.chunks; c++) {
-    const int t1 = min(p.T, (c + 1) * kMlChunk);
-    const double Fc = F[t1 - 1] - (c ? F[c * kMlChunk - 1] : 0.0);
-    const float u = own[c * step];
-    if (sizeof(T) == 4 || is_n) own[c * step] = v;
-    else {
-      T* plane = reinterpret_cast<T*>(p.w.planes) + ((long long)sh * p.w.chunks + c) * 2 * n_state + i;
-      const T hi = Cvt<T>::from(v);
-      plane[0] = hi;
-      plane[n_state] = Cvt<T>::from(v - Cvt<T>::to(hi));
+  const bool is_n = (int)blockIdx.x >= s_blocks;
+  const long long i = is_n ? ((long long)(blockIdx.x - s_blocks) * 256 + threadIdx.x) : ((long long)blockIdx.x * 256 + threadIdx.x) * VEC;
+  const bool live = i < (is_n ? p.dim : n_state);
+  float* home = is_n ? p.n_of(s) + (long long)h * p.dim + i : p.S_of(s) + h * n_state + i;
+  float* own = is_n ? p.w.n + (long long)sh * p.w.chunks * p.dim + i : p.w.S + (long long)sh * p.w.chunks * n_state + i;
+  const long long step = is_n ? p.dim : n_state;
+  float v[VEC];
+  auto load = [&](const float* q, float (&o)[VEC]) {
+    if constexpr (VEC == 4) {
+      if (!is_n) { const float4 f = *reinterpret_cast<const float4*>(q); o[0] = f.x; o[1] = f.y; o[2] = f.z; o[3] = f.w; return; }
     }
-    v = fmaf(v, expf((float)Fc + ms[c] - ms[c + 1]), u);
+    o[0] = q[0];
+  };
+  auto store = [&](float* q, const float (&o)[VEC]) {
+    if constexpr (VEC == 4) {
+      if (!is_n) { *reinterpret_cast<float4*>(q) = make_float4(o[0], o[1], o[2], o[3]); return; }
+    }
+    q[0] = o[0];
+  };
+#pragma unroll
+  for (int e = 0; e < VEC; e++) v[e] = 0.f;
+  if (live) load(home, v);
+  for (int c0 = 0; c0 < p.w.chunks; c0 += 256) {
+    const int nc = min(256, p.w.chunks - c0);
+    __syncthreads();
+    if ((int)threadIdx.x < nc) {
+      const int c = c0 + threadIdx.x, t1 = min(p.T, (c + 1) * kMlChunk);
+      const double Fc = F[t1 - 1] - (c ? F[c * kMlChunk - 1] : 0.0);
+      s_decay[threadIdx.x] = expf((float)Fc + ms[c] - ms[c + 1]);
+    }
+    __syncthreads();
+    if (!live) continue;
+#pragma unroll 4
+    for (int k = 0; k < nc; k++) {
+      const int c = c0 + k;
+      float u[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; e++) u[e] = 0.f;
+      load(own + c * step, u);
+      if (sizeof(T) == 4 || is_n) store(own + c * step, v);
+      else {
+        T* plane = reinterpret_cast<T*>(p.w.planes) + ((long long)sh * p.w.chunks + c) * 2 * n_state + i;
+        alignas(8) T hi[VEC], lo[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; e++) { hi[e] = Cvt<T>::from(v[e]); lo[e] = Cvt<T>::from(v[e] - Cvt<T>::to(hi[e])); }
+        if constexpr (VEC * sizeof(T) == 8) { *reinterpret_cast<uint2*>(plane) = *reinterpret_cast<const uint2*>(hi); *reinterpret_cast<uint2*>(plane + n_state) = *reinterpret_cast<const uint2*>(lo); }
+        else {
+#pragma unroll
+          for (int e = 0; e < VEC; e++) { plane[e] = hi[e]; plane[n_state + e] = lo[e]; }
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; e++) v[e] = fmaf(v[e], s_decay[k], u[e]);
+    }
   }
-  *home = v;
+  if (live) store(home, v);
 }
 
 // ── output ──────────────────────────────────────────────────────────────────
@@ -299,10 +335,14 @@ Status mlstm_prefill(cudaStream_t s, const MlstmDesc& d) {
     AG_DISPATCH_FLOAT(d.dtype, T, (e = launch_pdl(ml_chunk_kernel<T>, dim3((unsigned)tiles, (unsigned)p.w.chunks, (unsigned)sh), dim3(256), 0, s, p)));
     if (e != cudaSuccess) return cuda_status(e, "mlstm chunk states");
   }
-  const long long per = (long long)d.dim * d.vdim + d.dim;
-  const dim3 cgrid((unsigned)((per + 255) / 256), (unsigned)sh);
-  if (tc) e = d.dtype == DType::BF16 ? launch_pdl(ml_carry_kernel<__nv_bfloat16>, cgrid, dim3(256), 0, s, p) : launch_pdl(ml_carry_kernel<__half>, cgrid, dim3(256), 0, s, p);
-  else e = launch_pdl(ml_carry_kernel<float>, cgrid, dim3(256), 0, s, p);
+  const bool vec = d.vdim % 4 == 0 && d.state_stride % 4 == 0 && aligned16(d.state);
+  const int s_blocks = (int)(((long long)d.dim * d.vdim + 256 * (vec ? 4 : 1) - 1) / (256 * (vec ? 4 : 1)));
+  const dim3 cgrid((unsigned)(s_blocks + (d.dim + 255) / 256), (unsigned)sh);
+  auto carry = [&](auto tag) {
+    using T = decltype(tag);
+    return vec ? launch_pdl(ml_carry_kernel<T, 4>, cgrid, dim3(256), 0, s, p, s_blocks) : launch_pdl(ml_carry_kernel<T, 1>, cgrid, dim3(256), 0, s, p, s_blocks);
+  };
+  e = !tc ? carry(0.f) : d.dtype == DType::BF16 ? carry(__nv_bfloat16()) : carry(__half());
   if (e != cudaSuccess) return cuda_status(e, "mlstm carry");
   if (tc) return mlstm_output_tc(s, d.dtype, p);
   const size_t lim = 220 * 1024;

@@ -25,9 +25,9 @@ __device__ __forceinline__ float ml_pow(float4 row, float4 key, float m2) { retu
 // ── chunk: U = sum_j w_j k_j v_j^T and n = sum_j w_j k_j over the chunk's tokens ────────────────────────────────
 // D[dim, vdim] = A[dim, tokens] B[tokens, vdim], both operands as they lie (tokens are rows, so A is M-major and B N-major).
 // Four converter warps scale the key rows by their decay in shared memory and split them; they also hold the sum for n and
-// write the result. grid: (chunks x tiles of 128 key dimensions, n_seq * heads).
+// write the result. grid: (chunks x tiles of 128 key dimensions x tiles of 256 value columns, n_seq * heads).
 constexpr int kMcStages = 3;
-struct MlChunkTc { MlParams p; int m_tiles, pv, n; int* status; };
+struct MlChunkTc { MlParams p; int m_tiles, n_tiles, pv; int* status; };
 template <typename T>
 __global__ void __launch_bounds__(192, 1) ml_chunk_tc_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv, const MlChunkTc a) {
   extern __shared__ uint8_t smem_raw[];
@@ -52,7 +52,8 @@ __global__ void __launch_bounds__(192, 1) ml_chunk_tc_kernel(const __grid_consta
   const uint32_t tmem = tmem_base_slot;
   pdl_wait();
   pdl_trigger();
-  const int c = (int)blockIdx.x / a.m_tiles, d0 = (int)blockIdx.x % a.m_tiles * 128;
+  const int e0 = (int)blockIdx.x % a.n_tiles * 256, d0 = (int)blockIdx.x / a.n_tiles % a.m_tiles * 128, c = (int)blockIdx.x / (a.n_tiles * a.m_tiles);
+  const int ne = min(256, p.vdim - e0);
   const int sh = blockIdx.y, s = sh / p.heads, h = sh % p.heads;
   const int t0 = c * kMlChunk, t1 = min(p.T, t0 + kMlChunk), blocks = (t1 - t0 + kMtTok - 1) / kMtTok;
   if (warp == 0) {
@@ -64,13 +65,13 @@ __global__ void __launch_bounds__(192, 1) ml_chunk_tc_kernel(const __grid_consta
         mbar_expect_tx(&k_full[st], 2 * kMtPanelBytes);
         for (int q = 0; q < 2; q++) tma_load_4d(base + q * kMtPanelBytes, &mk, &k_full[st], d0 + q * kMtPanel, t0 + j * kMtTok, h, s);
         mbar_expect_tx(&v_full[st], (uint32_t)(a.pv * kMtPanelBytes));
-        for (int q = 0; q < a.pv; q++) tma_load_4d(base + (4 + q) * kMtPanelBytes, &mv, &v_full[st], q * kMtPanel, t0 + j * kMtTok, h, s);
+        for (int q = 0; q < a.pv; q++) tma_load_4d(base + (4 + q) * kMtPanelBytes, &mv, &v_full[st], e0 + q * kMtPanel, t0 + j * kMtTok, h, s);
       }
     }
   } else if (warp == 1) {
     if (lane == 0) {
       constexpr int fmt = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
-      const uint32_t idesc = make_idesc_f16(fmt, 1, 1, 128, a.n);
+      const uint32_t idesc = make_idesc_f16(fmt, 1, 1, 128, (ne + 15) / 16 * 16);
       bool ok = true;
       for (int j = 0; j < blocks && ok; j++) {
         const int st = j % kMcStages;
@@ -134,7 +135,7 @@ __global__ void __launch_bounds__(192, 1) ml_chunk_tc_kernel(const __grid_consta
     for (int e = 0; e < 8; e++) s_n[r0][ch * 8 + e] = nacc[e];
     asm volatile("bar.sync 1, 128;" ::: "memory");
     const long long ci = (long long)sh * p.w.chunks + c;
-    if (d0 + tid < p.dim) {
+    if (e0 == 0 && d0 + tid < p.dim) {
       float v = 0.f;
 #pragma unroll
       for (int r = 0; r < 8; r++) v += s_n[r][tid];
@@ -143,15 +144,15 @@ __global__ void __launch_bounds__(192, 1) ml_chunk_tc_kernel(const __grid_consta
     if (ok && __all_sync(0xffffffffu, mbar_wait(&acc_full, 0, a.status, 48))) {
       tc_fence_after_sync();
       const int quarter = warp & 3, row = d0 + quarter * 32 + lane;
-      float* dst = p.w.S + (ci * p.dim + row) * p.vdim;
-      for (int g = 0; g * 32 < p.vdim; g++) {
+      float* dst = p.w.S + (ci * p.dim + row) * p.vdim + e0;
+      for (int g = 0; g * 32 < ne; g++) {
         uint32_t o[32];
         tmem_ld_32x32(tmem + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(g * 32), o);
         tmem_ld_wait();
         if (row >= p.dim) continue;
 #pragma unroll
         for (int q = 0; q < 8; q++)
-          if (g * 32 + q * 4 < p.vdim) *reinterpret_cast<uint4*>(dst + g * 32 + q * 4) = make_uint4(o[q * 4], o[q * 4 + 1], o[q * 4 + 2], o[q * 4 + 3]);
+          if (g * 32 + q * 4 < ne) *reinterpret_cast<uint4*>(dst + g * 32 + q * 4) = make_uint4(o[q * 4], o[q * 4 + 1], o[q * 4 + 2], o[q * 4 + 3]);
       }
       tc_fence_before_sync();
     }
@@ -163,19 +164,22 @@ __global__ void __launch_bounds__(192, 1) ml_chunk_tc_kernel(const __grid_consta
 }
 
 // ── output ──────────────────────────────────────────────────────────────────
-// A CTA: 128 rows of one head. O = (q S) r first (the state's planes stream through the value ring), then the chunk's key
+// A cluster: 128 rows of one head, each CTA 128 value columns (the scores are computed by every one; the head norm's sums meet
+// over distributed shared memory), small enough for two CTAs per SM. O = (q S) r first (the state's planes stream through the value ring), then the chunk's key
 // blocks: scores by tcgen05, times their decay by the row's thread, split, O += P V from tensor memory. The row's thread
 // also holds n . q, so it ends with the division, the head norm, the norm weight and the output gate.
-struct MlOutTc { MlParams p; int pd, pv, n, ks, vs, tmem_cols, y_vec; int* status; };
+constexpr int kMoCols = 128;
+struct MlOutTc { MlParams p; int pd, pv, ks, vs, ranks, y_vec; int* status; };
 constexpr int kMoMaxStages = 4;
 template <typename T>
-__global__ void __launch_bounds__(192) ml_output_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv,
+__global__ void __launch_bounds__(192, 2) ml_output_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv,
                                                            const __grid_constant__ CUtensorMap ms, const MlOutTc a) {
   extern __shared__ uint8_t smem_raw[];
   __shared__ uint64_t q_full, k_full[kMoMaxStages], k_empty[kMoMaxStages], v_full[kMoMaxStages], v_empty[kMoMaxStages], s_full[2], p_full[2], st_full, st_done, o_full;
   __shared__ uint32_t tmem_base_slot;
   __shared__ __align__(16) float2 s_b[kMlChunk];
   __shared__ float s_n[256];
+  __shared__ float s_sq[128];
   const MlParams& p = a.p;
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   uint8_t* sQ = smem;                                          // pd panels of 128 rows
@@ -189,14 +193,15 @@ __global__ void __launch_bounds__(192) ml_output_tc_kernel(const __grid_constant
     mbar_fence_init();
     prefetch_tmap(&mq); prefetch_tmap(&mk); prefetch_tmap(&mv); prefetch_tmap(&ms);
   }
-  if (warp == 1) { tmem_alloc(&tmem_base_slot, (uint32_t)a.tmem_cols); tmem_relinquish(); }
+  if (warp == 1) { tmem_alloc(&tmem_base_slot, 256); tmem_relinquish(); }
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
   const uint32_t tmem_s = tmem_base_slot, tmem_o = tmem_base_slot + 2 * kMtTok;
   pdl_wait();
   pdl_trigger();
-  const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * 128, sh = blockIdx.y, s = sh / p.heads, h = sh % p.heads;
+  const int rank = (int)blockIdx.x % a.ranks, e0 = rank * kMoCols, ne = min(kMoCols, p.vdim - e0);
+  const int q0 = (int)((gridDim.x - 1 - blockIdx.x) / a.ranks) * 128, sh = blockIdx.y, s = sh / p.heads, h = sh % p.heads;
   const int c = q0 / kMlChunk, t0 = c * kMlChunk;
   const int blocks = (min(p.T, q0 + 128) - t0 + kMtTok - 1) / kMtTok;
   const int dblocks = (p.dim + kMtTok - 1) / kMtTok, vblocks = 2 * dblocks;       // state planes in blocks of 64 rows, ahead of the values
@@ -219,8 +224,8 @@ __global__ void __launch_bounds__(192) ml_output_tc_kernel(const __grid_constant
         mbar_expect_tx(&v_full[st], (uint32_t)(a.pv * kMtPanelBytes));
         uint8_t* dst = sV + st * a.pv * kMtPanelBytes;
         for (int q = 0; q < a.pv; q++) {
-          if (jv < vblocks) tma_load_4d(dst + q * kMtPanelBytes, &ms, &v_full[st], q * kMtPanel, (jv >> 1) * kMtTok, c * 2 + (jv & 1), sh);
-          else tma_load_4d(dst + q * kMtPanelBytes, &mv, &v_full[st], q * kMtPanel, t0 + (jv - vblocks) * kMtTok, h, s);
+          if (jv < vblocks) tma_load_4d(dst + q * kMtPanelBytes, &ms, &v_full[st], e0 + q * kMtPanel, (jv >> 1) * kMtTok, c * 2 + (jv & 1), sh);
+          else tma_load_4d(dst + q * kMtPanelBytes, &mv, &v_full[st], e0 + q * kMtPanel, t0 + (jv - vblocks) * kMtTok, h, s);
         }
         jv++;
       };
@@ -235,7 +240,7 @@ __global__ void __launch_bounds__(192) ml_output_tc_kernel(const __grid_constant
   } else if (warp == 1) {
     if (lane == 0) {
       constexpr int fmt = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
-      const uint32_t idesc_s = make_idesc_f16(fmt, 0, 0, 128, kMtTok), idesc_o = make_idesc_f16(fmt, 0, 1, 128, a.n);
+      const uint32_t idesc_s = make_idesc_f16(fmt, 0, 0, 128, kMtTok), idesc_o = make_idesc_f16(fmt, 0, 1, 128, (ne + 15) / 16 * 16);
       auto steps = [&](int q) { const int left = p.dim - q * kMtPanel; return left >= kMtPanel ? 4 : (left + 15) / 16; };
       auto issue_s = [&](int j) -> bool {
         if (j >= blocks) return true;
@@ -282,10 +287,17 @@ __global__ void __launch_bounds__(192) ml_output_tc_kernel(const __grid_constant
       }
       if (ok) mma_commit(&o_full);
     }
-  } else {
-    const int tid = threadIdx.x - 64, quarter = warp & 3;
-    const int row = q0 + quarter * 32 + lane, rr = min(row, p.T - 1);
-    const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
+  }
+  // the row's thread (warps 2 .. 5)
+  const int tid = threadIdx.x - 64, quarter = warp & 3, lr = quarter * 32 + lane;
+  const int row = q0 + lr, rr = min(row, p.T - 1);
+  const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
+  const T* grow = reinterpret_cast<const T*>(p.proj) + ((long long)s * p.T + rr) * p.ld;
+  const int o_groups = (ne + 31) / 32;
+  float den = 0.f;
+  bool ok = warp >= 2;
+  uint4 z[kMoCols / 8];
+  if (warp >= 2) {
     const float4* ab = p.w.ab + (long long)sh * p.T;
     const float4 mine = ab[rr];
     const float m2 = p.w.m2[(long long)sh * p.T + rr];
@@ -300,19 +312,18 @@ __global__ void __launch_bounds__(192) ml_output_tc_kernel(const __grid_constant
     // what lies in front of the chunk reaches this row by r
     const float m_c = p.w.m_start[(long long)sh * (p.w.chunks + 1) + c] * 1.4426950408889634f;
     const float r = ex2_approx((mine.x + m_c) + (mine.y - m2)) * p.q_scale;
-    const T* grow = reinterpret_cast<const T*>(p.proj) + ((long long)s * p.T + rr) * p.ld;
     float nq = 0.f;
-    {
-      const T* q = grow + h * p.dim;
+    ok = __all_sync(0xffffffffu, mbar_wait(&q_full, 0, a.status, 49));
+    if (ok) {
       for (int i = 0; i < p.dim; i += 8) {
-        const Pack<T> v = ld16(q + i);
+        const uint4 raw = *reinterpret_cast<const uint4*>(sQ + (i >> 6) * 2 * kMtPanelBytes + lr * 128 + ((((i & 63) >> 3) ^ (lr & 7)) << 4));
+        const T* v = reinterpret_cast<const T*>(&raw);
 #pragma unroll
-        for (int e = 0; e < 8; e++) nq = fmaf(Cvt<T>::to(v.v[e]), s_n[i + e], nq);
+        for (int e = 0; e < 8; e++) nq = fmaf(Cvt<T>::to(v[e]), s_n[i + e], nq);
       }
       nq *= r;
     }
-    const int o_groups = (p.vdim + 31) / 32;
-    bool ok = __all_sync(0xffffffffu, mbar_wait(&st_full, 0, a.status, 58));
+    ok = ok && __all_sync(0xffffffffu, mbar_wait(&st_full, 0, a.status, 58));
     if (ok) {
       tc_fence_after_sync();
       for (int g = 0; g < o_groups; g++) {
@@ -362,9 +373,14 @@ __global__ void __launch_bounds__(192) ml_output_tc_kernel(const __grid_constant
       __syncwarp();
       if (lane == 0) mbar_arrive(&p_full[sb]);
     }
-    if (ok && __all_sync(0xffffffffu, mbar_wait(&o_full, 0, a.status, 60))) {
+    // the output gate's values are on their way while the last product finishes
+    const T* gp = grow + 2 * p.heads * p.dim + p.heads * p.vdim + h * p.vdim + e0;
+#pragma unroll
+    for (int q = 0; q < kMoCols / 8; q++) z[q] = q * 8 < ne ? *reinterpret_cast<const uint4*>(gp + q * 8) : make_uint4(0u, 0u, 0u, 0u);
+    ok = ok && __all_sync(0xffffffffu, mbar_wait(&o_full, 0, a.status, 60));
+    if (ok) {
       tc_fence_after_sync();
-      const float den = 1.0f / (fmaxf(fabsf(nq), ex2_approx(-m2)) + 1e-6f);
+      den = 1.0f / (fmaxf(fabsf(nq), ex2_approx(-m2)) + 1e-6f);
       float sq = 0.f;
       for (int g = 0; g < o_groups; g++) {
         uint32_t o[32];
@@ -372,65 +388,79 @@ __global__ void __launch_bounds__(192) ml_output_tc_kernel(const __grid_constant
         tmem_ld_wait();
 #pragma unroll
         for (int e = 0; e < 32; e++) {
-          const float v = g * 32 + e < p.vdim ? __uint_as_float(o[e]) * den : 0.f;
+          const float v = g * 32 + e < ne ? __uint_as_float(o[e]) * den : 0.f;
           sq = fmaf(v, v, sq);
         }
       }
-      const float rs = den / sqrtf(sq / (float)p.vdim + p.eps);
-      const T* gp = grow + 2 * p.heads * p.dim + p.heads * p.vdim + h * p.vdim;
-      T* y = reinterpret_cast<T*>(p.y) + ((long long)s * p.T + rr) * p.y_ld + h * p.vdim;
-      const float* nw = p.norm + h * p.vdim;
-      for (int g = 0; g < o_groups; g++) {
-        uint32_t o[32];
-        tmem_ld_32x32(tmem_o + lane_addr + (uint32_t)(g * 32), o);
-        tmem_ld_wait();
-        if (row >= p.T) continue;
-#pragma unroll
-        for (int q = 0; q < 4; q++) {
-          const int e0 = g * 32 + q * 8;
-          if (e0 >= p.vdim) break;
-          const Pack<T> z = ld16(gp + e0);
-          float v[8];
-#pragma unroll
-          for (int e = 0; e < 8; e++) v[e] = __uint_as_float(o[q * 8 + e]) * rs * __ldg(nw + e0 + e) * __fdividef(1.0f, 1.0f + __expf(-Cvt<T>::to(z.v[e])));
-          Pack<T> w;
-          pack_from_floats<T>(w, v);
-          if (a.y_vec) st16(y + e0, w);
-          else {
-#pragma unroll
-            for (int e = 0; e < 8; e++) y[e0 + e] = w.v[e];
-          }
-        }
-      }
-      tc_fence_before_sync();
+      s_sq[lr] = sq;
     }
   }
+  __syncwarp();
+  if (a.ranks > 1) cluster_sync_all();
+  if (ok) {
+    float sq = 0.f;
+    for (int q = 0; q < a.ranks; q++) {
+      float v = s_sq[lr];
+      if (a.ranks > 1) asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(mapa_u32(smem_u32(&s_sq[lr]), (uint32_t)q)));
+      sq += v;
+    }
+    const float rs = den / sqrtf(sq / (float)p.vdim + p.eps);
+    T* y = reinterpret_cast<T*>(p.y) + ((long long)s * p.T + rr) * p.y_ld + h * p.vdim + e0;
+    const float* nw = p.norm + h * p.vdim + e0;
+#pragma unroll
+    for (int g = 0; g < kMoCols / 32; g++) {
+      if (g >= o_groups) break;
+      uint32_t o[32];
+      tmem_ld_32x32(tmem_o + lane_addr + (uint32_t)(g * 32), o);
+      tmem_ld_wait();
+      if (row >= p.T) continue;
+#pragma unroll
+      for (int q = 0; q < 4; q++) {
+        const int c0 = g * 32 + q * 8;
+        if (c0 >= ne) break;
+        const T* zv = reinterpret_cast<const T*>(&z[g * 4 + q]);
+        float v[8];
+#pragma unroll
+        for (int e = 0; e < 8; e++) v[e] = __uint_as_float(o[q * 8 + e]) * rs * __ldg(nw + c0 + e) * __fdividef(1.0f, 1.0f + __expf(-Cvt<T>::to(zv[e])));
+        Pack<T> w;
+        pack_from_floats<T>(w, v);
+        if (a.y_vec) st16(y + c0, w);
+        else {
+#pragma unroll
+          for (int e = 0; e < 8; e++) y[c0 + e] = w.v[e];
+        }
+      }
+    }
+    tc_fence_before_sync();
+  }
   tc_fence_before_sync();
-  __syncthreads();
+  __syncwarp();
+  if (a.ranks > 1) cluster_sync_all(); else __syncthreads();      // also: no CTA leaves while its sums are being read
   tc_fence_after_sync();
-  if (warp == 1) tmem_dealloc(tmem_base_slot, (uint32_t)a.tmem_cols);
+  if (warp == 1) tmem_dealloc(tmem_base_slot, 256);
 }
 
 // ── host ────────────────────────────────────────────────────────────────────
 static int mt_panels(int n) { return (n + kMtPanel - 1) / kMtPanel; }
-// stages of the key and value rings: as much as fits half an SM when the accumulators take half the tensor memory
+// stages of the key and value rings: as much as fits half an SM where two value stages do
 static bool mo_stages(int pd, int pv, int* ks, int* vs, int* smem) {
-  const int q = pd * 2 * kMtPanelBytes;
-  const int most = kMtSmemMax - 4 * 1024, limit = pv <= 2 ? 108 * 1024 : most;
+  const int q = pd * 2 * kMtPanelBytes, most = kMtSmemMax - 6 * 1024;
   *ks = 2;
-  int left = limit - 1024 - q - *ks * pd * kMtPanelBytes;
-  *vs = left / (pv * kMtPanelBytes);
-  if (*vs < 2 && limit < most) { left = most - 1024 - q - *ks * pd * kMtPanelBytes; *vs = left / (pv * kMtPanelBytes); }
+  for (int limit : {107 * 1024, most}) {
+    *vs = (limit - 1024 - q - *ks * pd * kMtPanelBytes) / (pv * kMtPanelBytes);
+    if (*vs >= 2) break;
+  }
   if (*vs > kMoMaxStages) *vs = kMoMaxStages;
   *smem = q + (*ks * pd + *vs * pv) * kMtPanelBytes + 1024;
   return *vs >= 2;
 }
+static int mo_panels(int vdim) { return vdim >= kMoCols ? 2 : mt_panels(vdim); }
 
 bool mlstm_tc_eligible(const MlstmDesc& d) {
   if (!(d.dtype == DType::BF16 || d.dtype == DType::F16)) return false;
-  if (d.dim % 8 || d.vdim % 8 || d.dim > 256 || d.vdim > 256 || d.ld % 8 || !aligned16(d.proj)) return false;
+  if (d.dim % 8 || d.vdim % 8 || d.dim > 256 || d.vdim > 8 * kMoCols || d.ld % 8 || !aligned16(d.proj)) return false;
   int ks, vs, smem;
-  return mo_stages(mt_panels(d.dim), mt_panels(d.vdim), &ks, &vs, &smem) && matmul_status_word() != nullptr;
+  return mo_stages(mt_panels(d.dim), mo_panels(d.vdim), &ks, &vs, &smem) && matmul_status_word() != nullptr;
 }
 
 static Status token_map(CUtensorMap* m, DType dt, const MlParams& p, int64_t col, int width, int box_rows) {
@@ -453,9 +483,9 @@ Status mlstm_chunk_tc(cudaStream_t s, DType dt, const MlParams& p) {
   AG_RETURN_IF_ERROR(token_map(&mk, dt, p, (int64_t)p.heads * p.dim, p.dim, kMtTok));
   AG_RETURN_IF_ERROR(token_map(&mv, dt, p, 2 * (int64_t)p.heads * p.dim, p.vdim, kMtTok));
   MlChunkTc a;
-  a.p = p; a.m_tiles = (p.dim + 127) / 128; a.pv = mt_panels(p.vdim); a.n = (p.vdim + 15) / 16 * 16; a.status = matmul_status_word();
+  a.p = p; a.m_tiles = (p.dim + 127) / 128; a.n_tiles = (p.vdim + 255) / 256; a.pv = p.vdim > 256 ? 4 : mt_panels(p.vdim); a.status = matmul_status_word();
   const size_t smem = (size_t)kMcStages * (4 + a.pv) * kMtPanelBytes + 1024;
-  const dim3 grid((unsigned)(p.w.chunks * a.m_tiles), (unsigned)(p.n_seq * p.heads));
+  const dim3 grid((unsigned)(p.w.chunks * a.m_tiles * a.n_tiles), (unsigned)(p.n_seq * p.heads));
   const cudaError_t e = dt == DType::BF16 ? launch_mc<__nv_bfloat16>(s, mk, mv, a, grid, smem) : launch_mc<__half>(s, mk, mv, a, grid, smem);
   return cuda_status(e, "mlstm chunk states (tcgen05)");
 }
@@ -464,11 +494,17 @@ template <typename T>
 static cudaError_t launch_mo(cudaStream_t s, const CUtensorMap* m, const MlOutTc& a, dim3 grid, size_t smem) {
   static bool attr = false;
   if (!attr) {
-    cudaError_t e = cudaFuncSetAttribute(ml_output_tc_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMtSmemMax - 4 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(ml_output_tc_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMtSmemMax - 6 * 1024);
     if (e != cudaSuccess) return e;
     attr = true;
   }
-  return launch_pdl(ml_output_tc_kernel<T>, grid, dim3(192), smem, s, m[0], m[1], m[2], m[3], a);
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid; cfg.blockDim = dim3(192); cfg.dynamicSmemBytes = smem; cfg.stream = s;
+  cudaLaunchAttribute at[2];
+  at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization; at[0].val.programmaticStreamSerializationAllowed = pdl_enabled() ? 1 : 0;
+  at[1].id = cudaLaunchAttributeClusterDimension; at[1].val.clusterDim.x = (unsigned)a.ranks; at[1].val.clusterDim.y = 1; at[1].val.clusterDim.z = 1;
+  cfg.attrs = at; cfg.numAttrs = a.ranks > 1 ? 2 : 1;
+  return cudaLaunchKernelEx(&cfg, ml_output_tc_kernel<T>, m[0], m[1], m[2], m[3], a);
 }
 Status mlstm_output_tc(cudaStream_t s, DType dt, const MlParams& p) {
   CUtensorMap m[4];
@@ -479,11 +515,11 @@ Status mlstm_output_tc(cudaStream_t s, DType dt, const MlParams& p) {
   AG_RETURN_IF_ERROR(make_map(&m[3], dt, p.w.planes, (uint64_t)p.vdim, (uint64_t)p.dim, (uint64_t)p.w.chunks * 2, (uint64_t)p.n_seq * p.heads, (uint64_t)p.vdim, plane,
                               plane * p.w.chunks * 2, kMtPanel, kMtTok));
   MlOutTc a;
-  a.p = p; a.pd = mt_panels(p.dim); a.pv = mt_panels(p.vdim); a.n = (p.vdim + 15) / 16 * 16; a.tmem_cols = a.pv <= 2 ? 256 : 512; a.status = matmul_status_word();
+  a.p = p; a.pd = mt_panels(p.dim); a.pv = mo_panels(p.vdim); a.ranks = (p.vdim + kMoCols - 1) / kMoCols; a.status = matmul_status_word();
   a.y_vec = aligned16(p.y) && p.y_ld % 8 == 0 ? 1 : 0;
   int smem = 0;
   if (!mo_stages(a.pd, a.pv, &a.ks, &a.vs, &smem)) return Status::unsupported("mlstm output: head too large");
-  const dim3 grid((unsigned)((p.T + 127) / 128), (unsigned)(p.n_seq * p.heads));
+  const dim3 grid((unsigned)((p.T + 127) / 128 * a.ranks), (unsigned)(p.n_seq * p.heads));
   const cudaError_t e = dt == DType::BF16 ? launch_mo<__nv_bfloat16>(s, m, a, grid, (size_t)smem) : launch_mo<__half>(s, m, a, grid, (size_t)smem);
   return cuda_status(e, "mlstm output (tcgen05)");
 }

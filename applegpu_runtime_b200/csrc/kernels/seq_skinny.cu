@@ -8,6 +8,8 @@
 // float32 residual is updated in the epilogue of the output product.
 #include "common.cuh"
 #include "seq_kernels.h"
+#include "mma_sync.cuh"
+#include "sm100.cuh"
 
 namespace ag { namespace k {
 
@@ -141,31 +143,24 @@ __global__ void __launch_bounds__(kSsThreads) seq_skinny_kernel(const SsParams p
 // warps take every eighth 32-column block of K, and mma.m16n8k16 multiplies them with the input rows as the 8-wide
 // operand. The order of K inside a block is free as long as both operands agree on it, so a lane feeds two MMAs from one
 // 16-byte piece of each of its two weight rows and of its input row: no shared memory and no shuffles in the loop. The
-// first pieces of the weights are requested before the programmatic dependency wait. The warps' sums meet in shared memory.
+// first pieces of the weights are requested before the programmatic dependency wait. The warps' sums meet in shared memory;
+// a product with few result columns and long rows spreads K over a cluster, whose sums meet over distributed shared memory.
 struct SmSeg { const void* w; const void* a; void* out; long long ld, a_ld, out_ld; int n, mode, block0; float limit; };
-struct SmParams { SmSeg seg[kSeqSegs]; int n_seg, rows, kp; };
-
-template <typename T> __device__ __forceinline__ void mma_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1);
-template <> __device__ __forceinline__ void mma_16816<__nv_bfloat16>(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-template <> __device__ __forceinline__ void mma_16816<__half>(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
+struct SmParams { SmSeg seg[kSeqSegs]; int n_seg, rows, kp, ranks; };       // ranks: CTAs of a cluster along K
 
 template <typename T, int NT>        // NT groups of 8 input rows
 __global__ void __launch_bounds__(kSsThreads) seq_skinny_mma_kernel(const SmParams p) {
   constexpr int U = 4;               // 32-column blocks in flight per warp
   __shared__ float red[kSsWarps][NT * 8][17];
+  __shared__ float part[NT * 8][16];
+  const int rank = p.ranks > 1 ? (int)sm100::cluster_ctarank() : 0, stride = kSsWarps * p.ranks;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
   int si = 0;
 #pragma unroll
-  for (int i = 1; i < kSeqSegs; i++) if (i < p.n_seg && (int)blockIdx.x >= p.seg[i].block0) si = i;
+  for (int i = 1; i < kSeqSegs; i++) if (i < p.n_seg && (int)(blockIdx.x / p.ranks) >= p.seg[i].block0) si = i;
   const SmSeg sg = p.seg[si];
   const bool glu = sg.mode == (int)SeqOut::Glu;
-  const int group = (int)blockIdx.x - sg.block0;
+  const int group = (int)(blockIdx.x / p.ranks) - sg.block0;
   const int c0 = group * (glu ? 8 : 16);                        // first result column
   long long r0, r1;                                             // this lane's two weight rows
   if (glu) { r0 = c0 / kGluBlock * 2 * kGluBlock + c0 % kGluBlock + g; r1 = r0 + kGluBlock; }
@@ -184,19 +179,19 @@ __global__ void __launch_bounds__(kSsThreads) seq_skinny_mma_kernel(const SmPara
   auto fetch = [&](int kb) {
 #pragma unroll
     for (int u = 0; u < U; u++) {
-      const int kk = (kb + u * kSsWarps) * 32 + q * 8;
+      const int kk = (kb + u * stride) * 32 + q * 8;
       a0[u] = live0 && kk < p.kp ? __ldcs(reinterpret_cast<const uint4*>(w0 + kk)) : zero;
       a1[u] = live1 && kk < p.kp ? __ldcs(reinterpret_cast<const uint4*>(w1 + kk)) : zero;
     }
   };
-  fetch(warp);
+  fetch(rank * kSsWarps + warp);
   pdl_wait();
   pdl_trigger();
-  for (int kb = warp; kb * 32 < p.kp;) {
+  for (int kb = rank * kSsWarps + warp; kb * 32 < p.kp;) {
     uint4 b[U][NT];
 #pragma unroll
     for (int u = 0; u < U; u++) {
-      const int kk = (kb + u * kSsWarps) * 32 + q * 8;
+      const int kk = (kb + u * stride) * 32 + q * 8;
 #pragma unroll
       for (int t = 0; t < NT; t++) b[u][t] = x[t] && kk < p.kp ? *reinterpret_cast<const uint4*>(x[t] + kk) : zero;
     }
@@ -207,7 +202,7 @@ __global__ void __launch_bounds__(kSsThreads) seq_skinny_mma_kernel(const SmPara
         mma_16816<T>(acc[t], a0[u].x, a1[u].x, a0[u].y, a1[u].y, b[u][t].x, b[u][t].y);
         mma_16816<T>(acc[t], a0[u].z, a1[u].z, a0[u].w, a1[u].w, b[u][t].z, b[u][t].w);
       }
-    kb += U * kSsWarps;
+    kb += U * stride;
     if (kb * 32 < p.kp) fetch(kb);
   }
 #pragma unroll
@@ -216,19 +211,47 @@ __global__ void __launch_bounds__(kSsThreads) seq_skinny_mma_kernel(const SmPara
     red[warp][t * 8 + 2 * q][g + 8] = acc[t][2]; red[warp][t * 8 + 2 * q + 1][g + 8] = acc[t][3];
   }
   __syncthreads();
-  const int width = glu ? 8 : 16;
-  for (int i = threadIdx.x; i < NT * 8 * width; i += kSsThreads) {
-    const int m = i / width, n = i % width;
-    if (m >= p.rows || c0 + n >= sg.n) continue;
-    float v = 0.f, up = 0.f;
+  for (int i = threadIdx.x; i < NT * 8 * 16; i += kSsThreads) {
+    float v = 0.f;
 #pragma unroll
-    for (int w = 0; w < kSsWarps; w++) { v += red[w][m][n]; if (glu) up += red[w][m][n + 8]; }
-    const long long o = (long long)m * sg.out_ld + c0 + n;
-    if (glu) reinterpret_cast<T*>(sg.out)[o] = Cvt<T>::from(clamped_glu_f(v, up, sg.limit));
-    else if (sg.mode == (int)SeqOut::Store) reinterpret_cast<T*>(sg.out)[o] = Cvt<T>::from(v);
-    else if (sg.mode == (int)SeqOut::StoreF32) reinterpret_cast<float*>(sg.out)[o] = v;
-    else reinterpret_cast<float*>(sg.out)[o] += v;
+    for (int w = 0; w < kSsWarps; w++) v += red[w][i / 16][i % 16];
+    part[i / 16][i % 16] = v;
   }
+  if (p.ranks > 1) sm100::cluster_sync_all(); else __syncthreads();
+  if (rank == 0) {
+    auto total = [&](int m, int n) {
+      float v = part[m][n];
+      for (int r = 1; r < p.ranks; r++) {
+        float u;
+        asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(u) : "r"(sm100::mapa_u32(sm100::smem_u32(&part[m][n]), (uint32_t)r)));
+        v += u;
+      }
+      return v;
+    };
+    const int width = glu ? 8 : 16;
+    for (int i = threadIdx.x; i < NT * 8 * width; i += kSsThreads) {
+      const int m = i / width, n = i % width;
+      if (m >= p.rows || c0 + n >= sg.n) continue;
+      const float v = total(m, n);
+      const long long o = (long long)m * sg.out_ld + c0 + n;
+      if (glu) reinterpret_cast<T*>(sg.out)[o] = Cvt<T>::from(clamped_glu_f(v, total(m, n + 8), sg.limit));
+      else if (sg.mode == (int)SeqOut::Store) reinterpret_cast<T*>(sg.out)[o] = Cvt<T>::from(v);
+      else if (sg.mode == (int)SeqOut::StoreF32) reinterpret_cast<float*>(sg.out)[o] = v;
+      else reinterpret_cast<float*>(sg.out)[o] += v;
+    }
+  }
+  if (p.ranks > 1) sm100::cluster_sync_all();      // no CTA leaves while its sums are being read
+}
+
+template <typename T, int NT>
+static cudaError_t launch_sm(cudaStream_t s, const SmParams& p, int blocks) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3((unsigned)(blocks * p.ranks)); cfg.blockDim = dim3(kSsThreads); cfg.stream = s;
+  cudaLaunchAttribute at[2];
+  at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization; at[0].val.programmaticStreamSerializationAllowed = pdl_enabled() ? 1 : 0;
+  at[1].id = cudaLaunchAttributeClusterDimension; at[1].val.clusterDim.x = (unsigned)p.ranks; at[1].val.clusterDim.y = 1; at[1].val.clusterDim.z = 1;
+  cfg.attrs = at; cfg.numAttrs = p.ranks > 1 ? 2 : 1;
+  return cudaLaunchKernelEx(&cfg, seq_skinny_mma_kernel<T, NT>, p);
 }
 
 static Status seq_skinny_mma(cudaStream_t s, const SeqSkinnyDesc& d) {
@@ -243,13 +266,11 @@ static Status seq_skinny_mma(cudaStream_t s, const SeqSkinnyDesc& d) {
     const int per = g.mode == SeqOut::Glu ? 8 : 16;
     blocks += (g.n + per - 1) / per;
   }
+  p.ranks = 1;                                     // few blocks: more CTAs along K, as long as each warp keeps a full round of it
+  while (p.ranks < 4 && blocks * p.ranks < 2 * sm_count() && p.kp / 32 >= kSsWarps * p.ranks * 4) p.ranks *= 2;
   cudaError_t e;
-  if (d.dtype == DType::BF16)
-    e = d.rows <= 8 ? launch_pdl(seq_skinny_mma_kernel<__nv_bfloat16, 1>, dim3((unsigned)blocks), dim3(kSsThreads), 0, s, p)
-                    : launch_pdl(seq_skinny_mma_kernel<__nv_bfloat16, 2>, dim3((unsigned)blocks), dim3(kSsThreads), 0, s, p);
-  else
-    e = d.rows <= 8 ? launch_pdl(seq_skinny_mma_kernel<__half, 1>, dim3((unsigned)blocks), dim3(kSsThreads), 0, s, p)
-                    : launch_pdl(seq_skinny_mma_kernel<__half, 2>, dim3((unsigned)blocks), dim3(kSsThreads), 0, s, p);
+  if (d.dtype == DType::BF16) e = d.rows <= 8 ? launch_sm<__nv_bfloat16, 1>(s, p, blocks) : launch_sm<__nv_bfloat16, 2>(s, p, blocks);
+  else e = d.rows <= 8 ? launch_sm<__half, 1>(s, p, blocks) : launch_sm<__half, 2>(s, p, blocks);
   return cuda_status(e, "seq_skinny (tensor cores)");
 }
 

@@ -86,7 +86,7 @@ def state_parts(s, H, d, e):
     return s[:H * d * e].reshape(H, d, e), s[H * d * e:H * d * e + H * d].reshape(H, d), s[H * d * e + H * d:H * d * e + H * d + H]
 
 
-MLSTM_SIZES = [(1, 16, 16), (3, 20, 28), (2, 64, 128), (2, 8, 37), (1, 128, 256), (2, 72, 96), (2, 200, 40), (1, 24, 264)]
+MLSTM_SIZES = [(1, 16, 16), (3, 20, 28), (2, 64, 128), (2, 8, 37), (1, 128, 256), (2, 72, 96), (2, 200, 40), (1, 24, 264), (1, 136, 520)]
 
 
 @pytest.mark.parametrize("H,d,e", MLSTM_SIZES)
