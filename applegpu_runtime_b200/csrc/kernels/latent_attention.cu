@@ -39,18 +39,25 @@ static Status la_params(const LatentDesc& d, LaParams* out) {
 template <typename T>
 __device__ __forceinline__ void la_cache_row(const LaParams& p, const T* row, T* crow, int position, float* red) {
   const T* c = row + (long long)p.heads * (p.dim + p.rot_dim);
-  float sq = 0.f;
-  for (int i = threadIdx.x; i < p.rank; i += blockDim.x) { const float v = Cvt<T>::to(c[i]); sq = fmaf(v, v, sq); }
-  const float rs = 1.0f / sqrtf(block_sum(sq, red) / (float)p.rank + p.eps);
-  for (int i = threadIdx.x; i < p.rank; i += blockDim.x) crow[i] = Cvt<T>::from(Cvt<T>::to(c[i]) * rs * p.c_norm[i]);
   const T* kr = c + p.rank;
   T* dst = crow + p.coff;
+  constexpr int KEEP = 8;                                // values of the latent a thread keeps (the rest is read again)
+  float keep[KEEP], sq = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; k++) { const int i = threadIdx.x + k * blockDim.x; keep[k] = i < p.rank ? Cvt<T>::to(c[i]) : 0.f; }
   for (int i = threadIdx.x; i < p.pairs; i += blockDim.x) {
     const float2 cs = p.rot[(long long)position * p.pairs + i];
     const float u = Cvt<T>::to(kr[2 * i]), v = Cvt<T>::to(kr[2 * i + 1]);
     dst[2 * i] = Cvt<T>::from(u * cs.x - v * cs.y);
     dst[2 * i + 1] = Cvt<T>::from(v * cs.x + u * cs.y);
   }
+#pragma unroll
+  for (int k = 0; k < KEEP; k++) sq = fmaf(keep[k], keep[k], sq);
+  for (int i = threadIdx.x + KEEP * blockDim.x; i < p.rank; i += blockDim.x) { const float v = Cvt<T>::to(c[i]); sq = fmaf(v, v, sq); }
+  const float rs = 1.0f / sqrtf(block_sum(sq, red) / (float)p.rank + p.eps);
+#pragma unroll
+  for (int k = 0; k < KEEP; k++) { const int i = threadIdx.x + k * blockDim.x; if (i < p.rank) crow[i] = Cvt<T>::from(keep[k] * rs * p.c_norm[i]); }
+  for (int i = threadIdx.x + KEEP * blockDim.x; i < p.rank; i += blockDim.x) crow[i] = Cvt<T>::from(Cvt<T>::to(c[i]) * rs * p.c_norm[i]);
   for (int i = 2 * p.pairs + threadIdx.x; i < p.rot_dim; i += blockDim.x) dst[i] = kr[i];
 }
 
@@ -65,22 +72,35 @@ __global__ void __launch_bounds__(kLaThreads) latent_append_kernel(const LaParam
   if (position < 0 || position >= p.max_len) return;
   T* row = reinterpret_cast<T*>(p.proj) + (long long)r * p.ld;
   T* crow = reinterpret_cast<T*>(p.cache) + (long long)s * p.seq_stride + (long long)position * p.cld;
-  la_cache_row<T>(p, row, crow, position, red);
-  // a warp per head, a lane per pair (read and written as one word when pairs lie on words)
+  // a warp per head, a lane per pair (read and written as one word when pairs lie on words), four heads in flight
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, hd = p.dim + p.rot_dim;
-  const bool words = sizeof(T) == 2 && p.dim % 2 == 0 && hd % 2 == 0;
+  constexpr int HF = 4, HW = kLaThreads / 32;
+  const bool words = sizeof(T) == 2 && p.dim % 2 == 0 && hd % 2 == 0 && (reinterpret_cast<uintptr_t>(row) & 3u) == 0;
   for (int j = lane; j < p.pairs; j += 32) {
     const float2 cs = p.rot[(long long)position * p.pairs + j];
-    for (int h = warp; h < p.heads; h += kLaThreads / 32) {
-      T* q = row + (long long)h * hd + p.dim + 2 * j;
-      alignas(8) T t[2];
-      if (words) *reinterpret_cast<uint32_t*>(t) = *reinterpret_cast<const uint32_t*>(q); else { t[0] = q[0]; t[1] = q[1]; }
-      const float u = Cvt<T>::to(t[0]), v = Cvt<T>::to(t[1]);
-      t[0] = Cvt<T>::from(u * cs.x - v * cs.y);
-      t[1] = Cvt<T>::from(v * cs.x + u * cs.y);
-      if (words) *reinterpret_cast<uint32_t*>(q) = *reinterpret_cast<const uint32_t*>(t); else { q[0] = t[0]; q[1] = t[1]; }
+    T* q0 = row + p.dim + 2 * j;
+    for (int h0 = warp; h0 < p.heads; h0 += HW * HF) {
+      alignas(8) T t[HF][2];
+#pragma unroll
+      for (int k = 0; k < HF; k++) {
+        const int h = h0 + HW * k;
+        if (h >= p.heads) continue;
+        const T* q = q0 + (long long)h * hd;
+        if (words) *reinterpret_cast<uint32_t*>(t[k]) = *reinterpret_cast<const uint32_t*>(q); else { t[k][0] = q[0]; t[k][1] = q[1]; }
+      }
+#pragma unroll
+      for (int k = 0; k < HF; k++) {
+        const int h = h0 + HW * k;
+        if (h >= p.heads) continue;
+        T* q = q0 + (long long)h * hd;
+        const float u = Cvt<T>::to(t[k][0]), v = Cvt<T>::to(t[k][1]);
+        t[k][0] = Cvt<T>::from(u * cs.x - v * cs.y);
+        t[k][1] = Cvt<T>::from(v * cs.x + u * cs.y);
+        if (words) *reinterpret_cast<uint32_t*>(q) = *reinterpret_cast<const uint32_t*>(t[k]); else { q[0] = t[k][0]; q[1] = t[k][1]; }
+      }
     }
   }
+  la_cache_row<T>(p, row, crow, position, red);
 }
 
 Status latent_append(cudaStream_t s, const LatentDesc& d) {

@@ -80,6 +80,8 @@ def bench_gedenex(width, peaks, iters=10, batch=8, prompt=1024, steps=48):
         eng.decode(4, 0, n, use_graph=False)
         gpu.profile(False)
         row[f"decode_b{n}_kernels"] = _kernel_rows(peaks, 4)
+        bytes_ = sum(r["work"] for r in gpu.profile_report().values()) / 4      # weights, states and caches a step has to read
+        row[f"decode_b{n}_frac"] = round(bytes_ / (row[f"decode_b{n}_ms"] * 1e-3) / peaks["hbm_gbs"] / 1e9, 3)
     eng.close()
     return row
 
@@ -106,7 +108,8 @@ def bench_gpt2(width, peaks, iters=10, batch=8, prompt=1024, steps=48, vocab=327
     kern = {}
     for name, r in gpu.profile_report().items():
         if name.startswith(("fused_attention", "fused_linear", "matmul")):
-            rate = r["work"] / (r["ms"] * 1e-3)
+            work = r["launches"] * 2.0 * batch * width * prompt * (prompt + 1) if name.startswith("fused_attention") else r["work"]      # the unmasked half
+            rate = work / (r["ms"] * 1e-3)
             kern[name] = {"launches": r["launches"], "us": round(r["ms"] / r["launches"] * 1e3, 2), "rate": f"{rate / 1e12:.0f} TFLOP/s", "frac": round(rate / peaks["bf16_tflops"] / 1e12, 3)}
     row["prefill_kernels"] = kern
     for n in (1, batch):
