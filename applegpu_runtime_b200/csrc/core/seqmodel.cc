@@ -322,7 +322,7 @@ struct SeqEngine {
           AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h1.ptr(), wl, R, cfg.width, W[kWIn].data(), wl, mx.proj_cols(), proj.ptr(), pl, false, nullptr))));
         }
         if (mx.gate_cols()) {
-          Span span("linear_gates", product(R, mx.gate_cols(), cfg.width));
+          Span span("linear_gates", (double)R * (esz() * cfg.width + 4.0 * mx.gate_cols()));      // bound by reading its input
           AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h1.ptr(), wl, R, cfg.width, W[kWAux0].data(), wl, mx.gate_cols(), gates.ptr(), mx.gate_cols(), true, nullptr))));
         }
         if (c.ff) {

@@ -7,7 +7,7 @@
 import json
 import os
 
-from .bert import load_bert_state_dict
+from .bert import BERT_BASE, load_bert_state_dict
 from .checkpoint import read_safetensors
 from .gedenex import ARCHITECTURE as _GEDENEX, load_gedenex
 from .gpt2 import load_gpt2_state_dict
@@ -42,8 +42,13 @@ def _gpt2(config, weights, dtype):
     return load_gpt2_state_dict(state, {k: config[k] for k in ("n_layer", "n_head", "n_embd", "vocab_size", "n_positions")}, dtype=dtype)
 
 
+_BERT_KEYS = {"n_layer": "num_hidden_layers", "n_head": "num_attention_heads", "n_embd": "hidden_size", "d_ff": "intermediate_size", "vocab_size": "vocab_size",
+              "n_positions": "max_position_embeddings"}
+
+
 def _bert(config, weights, dtype):
-    return load_bert_state_dict(weights, config, dtype=dtype)
+    cfg = {k: config[hf] if hf in config else config[k] for k, hf in _BERT_KEYS.items()}
+    return load_bert_state_dict(weights, {**BERT_BASE, **cfg}, dtype=dtype)
 
 
 for _n in ("gpt2", "GPT2LMHeadModel"):

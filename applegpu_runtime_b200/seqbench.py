@@ -17,7 +17,7 @@ from .generate import Gpt2Decoder
 from .gpt2 import gpt2_forward, init_gpt2_weights
 
 SIZES = {1024: dict(heads=4, latent_heads=8, kv_rank=256, ff=2816), 2048: dict(heads=8, latent_heads=16, kv_rank=512, ff=5632)}
-BYTES = ("rms_rows", "clamped_glu", "mlstm_prefill", "mlstm_step", "latent_append", "latent_decode", "skinny_in", "skinny_out", "skinny_head")
+BYTES = ("rms_rows", "linear_gates", "clamped_glu", "mlstm_prefill", "mlstm_step", "latent_append", "latent_decode", "skinny_in", "skinny_out", "skinny_head")
 
 
 def config_of(width, vocab=32768):

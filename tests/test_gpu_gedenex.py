@@ -364,6 +364,46 @@ def test_batch_against_alone(gpu_dev):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_portions_longer_than_a_step(gpu_dev, dtype):
+    """A prompt, and a batch of prompts, with more rows than one step takes: the engine cuts them itself."""
+    cfg = config(32, [("mlstm", ml(1, 16, 16), None), ("latent_attention", la(1, 16, 8, 16, 24, base=1e5), (32, 2.0))], vocab=60)
+    w = weights(cfg, 21)
+    rng = np.random.default_rng(3)
+    model = gpu_dev.load_gedenex(cfg, w, dtype)
+    toks = rng.integers(0, 60, 8300).tolist()
+    eng = model.engine(1, 8300)
+    rows = [0, 17, 5000, 8191, 8192, 8193, 8299]
+    once = eng.forward(toks, want=rows)[0]
+    eng.reset(0)
+    parts, lo = [], 0
+    for n in (3001, 1, 4100, 1198):
+        here = [r - lo for r in rows if lo <= r < lo + n]
+        parts.append(eng.forward(toks[lo:lo + n], want=here)[0])
+        lo += n
+    assert rel(once, np.concatenate(parts)) < TOL[dtype]
+    batch = rng.integers(0, 60, (3, 3000)).astype(np.int32)
+    eng3 = model.engine(3, 3000)
+    both = eng3.forward(batch, want=[0, 2999, 3000 + 2730, 2 * 3000 + 2729, 2 * 3000 + 2999])[0]
+    alone = []
+    for i, r in ((0, [0, 2999]), (1, [2730]), (2, [2729, 2999])):
+        eng.reset(0)
+        alone.append(eng.forward(batch[i], want=r)[0])
+    assert rel(both, np.concatenate(alone)) < TOL[dtype]
+    assert gpu_dev.pipeline_status() == 0
+
+
+def test_more_sequences_than_step_rows(gpu_dev):
+    """Eighteen sequences: the linears of a step go to the GEMM, the mixers stay token by token."""
+    from applegpu_runtime_b200.generate import greedy_generate
+    cfg = CONFIGS["looped"]
+    model = gpu_dev.load_gedenex(cfg, weights(cfg, 9), "float32")
+    prompts = [np.random.default_rng(i).integers(0, cfg["vocab"], 3 + i).tolist() for i in range(18)]
+    out = greedy_generate(model, prompts, 6)
+    for i in (0, 7, 17):
+        assert greedy_generate(model, [prompts[i]], 6)[0].tolist() == out[i]
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_greedy_generation(gpu_dev, dtype):
     from applegpu_runtime_b200.generate import generate, greedy_generate
     cfg, g = CONFIGS["looped"], gpu_dev
