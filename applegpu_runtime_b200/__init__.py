@@ -25,4 +25,5 @@ from .bert import bert_forward, bert_forward_overlapped, init_bert_weights, load
 from .generate import generate, greedy_generate  # noqa: E402,F401
 from .seqmodel import SequenceModel, SequenceEngine  # noqa: E402,F401
 from .gedenex import load_gedenex, init_gedenex_weights  # noqa: E402,F401
+from .rurunex import load_rurunex, init_rurunex_weights  # noqa: E402,F401
 from .models import load_model, build_model, register as register_model  # noqa: E402,F401

@@ -1,12 +1,14 @@
 // Engine of the sequence models: weights, per-sequence memory, prompt portions and generated tokens.
 //
-// A model is a list of layers x <- x + mixer(rms(x) w1) + ff(rms(x) w2) over a float32 residual stream; a range of layers
-// may run several times with the same weights, every run with its own memory. What distinguishes the mixers (columns of
-// their input product, memory, kernels) sits behind the Mixer interface below, so another design adds a mixer kind and
-// keeps the rest.
+// A model is a list of layers over a float32 residual stream, in one of two forms:
+//     parallel    x <- x + mixer(rms(x) w1) + ff(rms(x) w2)
+//     sequential  x <- x + rms(mixer(rms(x) w1)) p1, then x <- x + rms(ff(rms(x) w2)) p2
+// A range of layers may run several times with the same weights, every run with its own memory. What distinguishes the mixers
+// (columns of their input product, memory, kernels) sits behind the Mixer interface below, so another design adds a mixer
+// kind and keeps the rest.
 //
 // Memory: the engine owns `slots` sequences of at most `max_len` tokens. A layer run keeps, for every slot, a fixed block
-// (recurrent state) or a row per token (cache); the number of tokens a slot holds lives in device memory (kernels read it
+// (recurrent state) or a row per token (cache); a layer may also use the cache of an earlier one. The number of tokens a slot holds lives in device memory (kernels read it
 // there, so that a captured step serves every length) with a mirror on the host.
 //
 // A step brings the next T tokens of n consecutive slots (R = n T rows) and picks its kernels by size: up to 16 rows the
@@ -182,14 +184,14 @@ struct LatentMixer : Mixer {
         g.batch = n; g.a_batch = d.seq_stride; g.c_batch = keys * kv_cols();
         AG_RETURN_IF_ERROR(k::matmul(x.s, g));
       }
-      k::LatentPrefillDesc p;
+      k::PromptAttnDesc p;
       p.dtype = dtype; p.n_seq = n; p.T = x.T; p.past = past; p.heads = c.heads; p.dim = c.dim; p.rot_dim = c.rot_dim; p.vdim = c.vdim; p.scale = c.score_scale;
       p.q = static_cast<uint8_t*>(proj) + (size_t)i * x.T * ld * esz; p.q_ld = ld; p.q_b = x.T * ld;
-      p.kv = kv; p.kv_ld = kv_cols(); p.v_off = v_off; p.kv_b = keys * kv_cols();
+      p.k = kv; p.k_ld = kv_cols(); p.v = static_cast<uint8_t*>(kv) + (size_t)v_off * esz; p.v_ld = kv_cols(); p.k_b = p.v_b = keys * kv_cols();
       p.k_rot = cache + (size_t)pad8(c.kv_rank) * esz; p.k_rot_ld = cld(); p.k_rot_b = d.seq_stride;
       p.y = static_cast<uint8_t*>(y) + (size_t)i * x.T * y_ld * esz; p.y_ld = y_ld; p.y_b = x.T * y_ld;
       Span span("latent_prefill", 2.0 * n * c.heads * (c.dim + c.rot_dim + c.vdim) * (past * (double)x.T + 0.5 * x.T * (x.T + 1.0)));
-      AG_RETURN_IF_ERROR(k::latent_prefill(x.s, p));
+      AG_RETURN_IF_ERROR(k::prompt_attention(x.s, p));
       *launches += 2;
       i += n;
     }
@@ -197,7 +199,125 @@ struct LatentMixer : Mixer {
   }
 };
 
-struct LayerRun { int layer; int pass; bool first; };   // pass -1 outside the loop
+// Matrix states with one decay per key channel: gated linear attention, the channel-wise gated delta rule.
+struct KeyDecayMixer : Mixer {
+  using Mixer::Mixer;
+  bool delta() const { return c.flags & kKdDelta; }
+  int qk_cols() const { return (int)pad8((int64_t)c.kv_heads * c.dim); }
+  int v_cols() const { return (int)pad8((int64_t)c.heads * c.vdim); }
+  int proj_cols() const override { return 2 * qk_cols() + v_cols() + (int)pad8(c.a_rank) + (c.g_rank ? (int)pad8(c.g_rank) : v_cols()); }
+  int gate_cols() const override { return delta() ? c.heads : 0; }
+  size_t slot_bytes(int) const override { return k::key_decay_mem_bytes(dtype, c.heads, c.kv_heads, c.dim, c.vdim, c.taps); }
+  bool clear_on_reset() const override { return true; }
+  Status check(const SeqModelCfg& m, int) const override {
+    if (c.kv_heads < 1 || c.heads % c.kv_heads || c.a_rank < 1 || c.g_rank < 0 || c.taps < 0 || !(c.tau > 0.f)) return Status::invalid("key decay sizes");
+    if (delta() && !is_matrix(w[kWAux0], dtype, c.heads, pad8(m.width))) return Status::invalid("write strengths");
+    if (!is_matrix(w[kWAux1], dtype, (int64_t)c.heads * c.dim, pad8(c.a_rank)) || !is_vector(w[kWAux2], (int64_t)c.heads * c.dim) || !is_vector(w[kWAux3], c.vdim))
+      return Status::invalid("decay weights, decay bias or head norm");
+    if (c.g_rank && !is_matrix(w[kWAux4], dtype, (int64_t)c.heads * c.vdim, pad8(c.g_rank))) return Status::invalid("gate weights");
+    if ((c.flags & kKdSoftplus) && !is_vector(w[kWAux5], c.heads)) return Status::invalid("decay rates");
+    if (c.taps && !is_vector(w[kWAux6], (int64_t)k::key_decay_channels(c.heads, c.kv_heads, c.dim, c.vdim) * c.taps)) return Status::invalid("convolution taps");
+    return Status::OK();
+  }
+  k::KeyDecayDesc desc(int n_seq, int T) const {
+    k::KeyDecayDesc d;
+    d.dtype = dtype; d.n_seq = n_seq; d.T = T; d.heads = c.heads; d.qk_heads = c.kv_heads; d.dim = c.dim; d.vdim = c.vdim;
+    d.delta = delta(); d.unit = c.flags & kKdUnit; d.softplus = c.flags & kKdSoftplus; d.gate_silu = c.flags & kKdGateSilu;
+    d.taps = c.taps; d.tau = c.tau; d.q_scale = (float)(1.0 / std::sqrt((double)c.dim));
+    d.q_off = 0; d.k_off = qk_cols(); d.v_off = 2 * qk_cols(); d.a_off = d.v_off + v_cols(); d.a_rank = c.a_rank; d.g_off = d.a_off + (int)pad8(c.a_rank); d.g_rank = c.g_rank;
+    return d;
+  }
+  size_t work_bytes(int n_seq, int T, int) const override { return k::key_decay_work_bytes(desc(n_seq, T)); }
+  Status run(const StepCtx& x, void* proj, int64_t ld, const float* gates, void* mem, int max_len, const int* pos, void* y, int64_t y_ld, void* work, void*, float eps,
+             int* launches) const override {
+    k::KeyDecayDesc d = desc(x.n_seq, x.T);
+    d.eps = eps; d.proj = proj; d.ld = ld; d.a2 = w[kWAux1].data(); d.bias = f32(w[kWAux2]); d.norm = f32(w[kWAux3]);
+    if (c.g_rank) d.g2 = w[kWAux4].data();
+    if (d.softplus) d.rate = f32(w[kWAux5]);
+    if (c.taps) d.conv = f32(w[kWAux6]);
+    d.beta = gates; d.beta_ld = gate_cols();
+    d.mem_stride = (int64_t)slot_bytes(max_len);
+    d.mem = static_cast<uint8_t*>(mem) + x.slot0 * d.mem_stride;
+    d.pos = pos; d.y = y; d.y_ld = y_ld; d.work = work;
+    const double esz = dtype_size(dtype), mem_rw = 8.0 * c.heads * c.dim * c.vdim;       // the state read and written once
+    const double row = esz * (2.0 * c.kv_heads * c.dim + c.heads * c.vdim * (c.g_rank ? 2.0 : 3.0) + c.a_rank + c.g_rank), wts = esz * c.heads * ((double)c.dim * c.a_rank + (double)c.vdim * c.g_rank);
+    const bool step = x.T <= k::kKeyDecayStepTokens;
+    Span span(step ? (delta() ? "delta_step" : "gla_step") : delta() ? "delta_prefill" : "gla_prefill", row * x.rows() + mem_rw * x.n_seq + wts);
+    return k::key_decay(x.s, d, launches);
+  }
+};
+
+// Query heads in groups over shared keys and values, all of them or a window, with per-head norms and rotation.
+struct GroupedMixer : Mixer {
+  using Mixer::Mixer;
+  bool shared() const { return c.kv_from >= 0; }
+  int q_cols() const { return (int)pad8((int64_t)c.heads * c.dim); }
+  int k_cols() const { return (int)pad8((int64_t)c.kv_heads * c.dim); }
+  int proj_cols() const override { return q_cols() + (shared() ? 0 : k_cols() + (int)pad8((int64_t)c.kv_heads * c.vdim)); }
+  int64_t cld() const { return k::grouped_cache_ld(c.kv_heads, c.dim, c.vdim); }
+  size_t cache_bytes(int max_len) const { return (size_t)max_len * cld() * dtype_size(dtype); }
+  size_t slot_bytes(int max_len) const override { return shared() ? 0 : cache_bytes(max_len); }
+  bool clear_on_reset() const override { return false; }
+  Status check(const SeqModelCfg& m, int max_len) const override {
+    if (c.kv_heads < 1 || c.heads % c.kv_heads || c.window < 0 || 2 * c.rot_pairs > c.dim) return Status::invalid("grouped attention sizes");
+    if (!is_vector(w[kWAux0], c.dim) || (!shared() && !is_vector(w[kWAux1], c.dim))) return Status::invalid("query or key norm");
+    if (c.rot_pairs && !(w[kWAux2].buf && w[kWAux2].contiguous() && w[kWAux2].dtype == DType::F32 && numel_of(w[kWAux2].shape) >= (int64_t)max_len * c.rot_pairs * 2))
+      return Status::invalid("rotation table");
+    if (shared()) {
+      if (c.kv_from >= (int)m.layers.size()) return Status::invalid("no such layer to take keys from");
+      const SeqLayerCfg& o = m.layers[c.kv_from];
+      if (o.mixer != MixerKind::GroupedAttention || o.kv_from >= 0 || o.kv_heads != c.kv_heads || o.dim != c.dim || o.vdim != c.vdim) return Status::invalid("the layer to take keys from has none of this kind");
+    }
+    return Status::OK();
+  }
+  size_t work_bytes(int, int, int) const override { return 0; }
+  double pairs_seen(int past, int T) const {            // (query, key) pairs of a portion
+    double n = 0;
+    for (int t = 0; t < T; t++) n += c.window ? std::min(c.window, past + t + 1) : past + t + 1;
+    return n;
+  }
+  Status run(const StepCtx& x, void* proj, int64_t ld, const float*, void* mem, int max_len, const int* pos, void* y, int64_t y_ld, void*, void*, float eps, int* launches) const override {
+    const size_t esz = dtype_size(dtype);
+    k::GroupedAttnDesc d;
+    d.dtype = dtype; d.n_seq = x.n_seq; d.T = x.T; d.heads = c.heads; d.kv_heads = c.kv_heads; d.dim = c.dim; d.vdim = c.vdim; d.rot_pairs = c.rot_pairs; d.window = c.window;
+    d.shared = shared(); d.scale = c.score_scale; d.softcap = c.softcap; d.eps = eps; d.proj = proj; d.ld = ld; d.k_off = q_cols(); d.v_off = q_cols() + k_cols();
+    d.q_norm = f32(w[kWAux0]); d.k_norm = shared() ? nullptr : f32(w[kWAux1]); d.rot_table = reinterpret_cast<const float2*>(w[kWAux2].data());
+    d.seq_stride = (int64_t)max_len * cld();
+    d.cache = static_cast<uint8_t*>(mem) + (size_t)x.slot0 * cache_bytes(max_len);
+    d.pos = pos; d.max_len = max_len; d.y = y; d.y_ld = y_ld;
+    {
+      Span span("grouped_append", esz * (double)x.rows() * 2.0 * (c.heads * c.dim + (shared() ? 0 : c.kv_heads * (c.dim + c.vdim))));
+      AG_RETURN_IF_ERROR(k::grouped_append(x.s, d));
+    }
+    *launches += 1;
+    if (x.T <= kShortT) {
+      double keys = 0;
+      for (int i = 0; i < x.n_seq; i++) keys += c.window ? std::min(c.window + x.T - 1, x.host_len[i] + x.T) : x.host_len[i] + x.T;
+      Span span("grouped_decode", esz * (keys * c.kv_heads + (double)x.rows() * c.heads) * (c.dim + c.vdim));
+      *launches += 1;
+      return k::grouped_decode(x.s, d);
+    }
+    // sequences that hold equally many tokens share a launch
+    for (int i = 0; i < x.n_seq;) {
+      int n = 1;
+      while (i + n < x.n_seq && x.host_len[i + n] == x.host_len[i]) n++;
+      const uint8_t* cache = static_cast<const uint8_t*>(d.cache) + (size_t)i * cache_bytes(max_len);
+      k::PromptAttnDesc p;
+      p.dtype = dtype; p.n_seq = n; p.T = x.T; p.past = x.host_len[i]; p.heads = c.heads; p.group = c.heads / c.kv_heads; p.dim = c.dim; p.vdim = c.vdim; p.window = c.window;
+      p.scale = c.score_scale; p.softcap = c.softcap;
+      p.q = static_cast<const uint8_t*>(proj) + (size_t)i * x.T * ld * esz; p.q_ld = ld; p.q_b = x.T * ld;
+      p.k = cache; p.v = cache + (size_t)k::grouped_v_col(c.kv_heads, c.dim) * esz; p.k_ld = p.v_ld = cld(); p.k_b = p.v_b = d.seq_stride;
+      p.y = static_cast<uint8_t*>(y) + (size_t)i * x.T * y_ld * esz; p.y_ld = y_ld; p.y_b = x.T * y_ld;
+      Span span("grouped_prefill", 2.0 * n * c.heads * (c.dim + c.vdim) * pairs_seen(p.past, x.T));
+      AG_RETURN_IF_ERROR(k::prompt_attention(x.s, p));
+      *launches += 1;
+      i += n;
+    }
+    return Status::OK();
+  }
+};
+
+struct LayerRun { int layer; int pass; bool first; int memory; };   // pass -1 outside the loop; memory: the run whose memory it uses
 
 struct SeqEngine {
   SeqModelCfg cfg;
@@ -205,10 +325,10 @@ struct SeqEngine {
   std::vector<TensorRec> w;
   std::vector<std::unique_ptr<Mixer>> mixers;
   std::vector<LayerRun> runs;
-  std::vector<std::shared_ptr<Buffer>> memory;     // per layer run, all slots
+  std::vector<std::shared_ptr<Buffer>> memory;     // per layer run, all slots (none where a run uses another one's)
   int slots = 0, max_len = 0;
   std::vector<int> len;                            // host mirror of pos
-  Scratch pos, tok, history, step, rowmap, x, h1, h2, proj, gates, gu, cat, work, kv, logits, picked;
+  Scratch pos, tok, history, step, rowmap, x, h1, h2, proj, gates, gu, cat, sub, work, kv, logits, picked;
   std::map<std::pair<int, int>, cudaGraphExec_t> graphs;
   int launches = 0, step_launches = 0;
   bool last_graph = false;
@@ -219,7 +339,8 @@ struct SeqEngine {
   size_t esz() const { return dtype_size(dtype); }
   const TensorRec* lw(int l) const { return &w[4 + (size_t)l * kSeqLayerWeights]; }
   int64_t y_cols(const SeqLayerCfg& c) const { return pad8((int64_t)c.heads * c.vdim); }       // where the feed-forward's columns start
-  int64_t cat_k(const SeqLayerCfg& c) const { return c.ff ? y_cols(c) + c.ff : (int64_t)c.heads * c.vdim; }
+  bool sequential() const { return cfg.form == LayerForm::Sequential; }
+  int64_t cat_k(const SeqLayerCfg& c) const { return c.ff && !sequential() ? y_cols(c) + c.ff : (int64_t)c.heads * c.vdim; }
   int64_t cat_ld(const SeqLayerCfg& c) const { return pad8(cat_k(c)); }
 
   // Grows a buffer (by half at least); graphs hold the old addresses of the buffers their step uses, so they are dropped and
@@ -242,7 +363,7 @@ struct SeqEngine {
     for (size_t l = 0; l < cfg.layers.size(); l++) {
       const SeqLayerCfg& c = cfg.layers[l];
       pc = std::max(pc, pad8(mixers[l]->proj_cols())); gc = std::max<int64_t>(gc, mixers[l]->gate_cols());
-      fc = std::max(fc, k::glu_rows(c.ff)); cc = std::max(cc, cat_ld(c));
+      fc = std::max(fc, k::glu_rows(c.ff)); cc = std::max({cc, cat_ld(c), pad8(c.ff)});
       wb = std::max(wb, mixers[l]->work_bytes(n_seq, T, max_len));
       if (T > kShortT) kb = std::max(kb, mixers[l]->kv_bytes(len.data() + slot0, n_seq, T));
     }
@@ -250,6 +371,7 @@ struct SeqEngine {
     AG_RETURN_IF_ERROR(ensure(&proj, R * pc * esz()));
     AG_RETURN_IF_ERROR(ensure(&gates, R * gc * sizeof(float)));
     AG_RETURN_IF_ERROR(ensure(&cat, R * cc * esz(), true));
+    if (sequential()) AG_RETURN_IF_ERROR(ensure(&sub, R * cfg.width * sizeof(float)));
     AG_RETURN_IF_ERROR(ensure(&work, wb));
     AG_RETURN_IF_ERROR(ensure(&kv, kb, false, false));
     const size_t hrows = std::max<size_t>(R, (size_t)n_want);
@@ -263,107 +385,202 @@ struct SeqEngine {
   }
   bool skinny_ok() const {
     int64_t kmax = cfg.width;
-    for (const SeqLayerCfg& c : cfg.layers) kmax = std::max(kmax, cat_k(c));
+    for (const SeqLayerCfg& c : cfg.layers) kmax = std::max({kmax, cat_k(c), (int64_t)c.ff});
     return k::seq_skinny_fits(kmax);
   }
 
   Status count(Status st) { launches++; return st; }
 
-  // All layers over the R rows whose tokens are in `tok`; x holds the residual stream afterwards.
-  Status enqueue_layers(const StepCtx& st, float* layers_out) {
+  void* mem_of(const LayerRun& run) const { return memory[run.memory]->ptr; }
+  // One product of a sequential layer: rows of `a` against wt, by the kernel the number of rows calls for.
+  Status enqueue_product(const StepCtx& st, const char* name, const void* a, int64_t a_ld, int64_t kdim, const TensorRec& wt, int64_t n, void* out, int64_t out_ld, bool out_f32,
+                         bool bytes = false) {
+    const int R = st.rows();
+    Span span(name, R <= k::kSeqSkinnyRows ? esz() * (double)n * pad8(kdim) : bytes ? R * (esz() * kdim + 4.0 * n) : product(R, n, kdim));
+    if (R <= k::kSeqSkinnyRows && skinny_ok()) {
+      k::SeqSkinnyDesc d;
+      d.dtype = dtype; d.rows = R; d.k = (int)kdim; d.a = a; d.a_ld = a_ld; d.n_seg = 1;
+      k::SeqSeg& g = d.seg[0];
+      g.a = a; g.a_ld = a_ld; g.w = wt.data(); g.ld = pad8(kdim); g.n = (int)n; g.mode = out_f32 ? k::SeqOut::StoreF32 : k::SeqOut::Store; g.out = out; g.out_ld = out_ld;
+      return count(k::seq_skinny(st.s, d));
+    }
+    return count(k::matmul(st.s, linear_desc(dtype, a, a_ld, R, kdim, wt.data(), pad8(kdim), n, out, out_ld, out_f32, nullptr)));
+  }
+  // The gated half of a feed-forward: out [R, ff] from the normed rows in h.
+  Status enqueue_glu(const StepCtx& st, const SeqLayerCfg& c, const void* h, const TensorRec& wt, void* out, int64_t out_ld) {
+    const int R = st.rows();
+    const int64_t wl = pad8(cfg.width), fn = k::glu_rows(c.ff);
+    if (R <= k::kSeqSkinnyRows && skinny_ok()) {
+      k::SeqSkinnyDesc d;
+      d.dtype = dtype; d.rows = R; d.k = cfg.width; d.a = h; d.a_ld = wl; d.n_seg = 1;
+      k::SeqSeg& g = d.seg[0];
+      g.a = h; g.a_ld = wl; g.w = wt.data(); g.ld = wl; g.n = c.ff; g.mode = k::SeqOut::Glu; g.glu = (k::Glu)c.glu; g.limit = c.ff_limit; g.out = out; g.out_ld = out_ld;
+      Span span("skinny_ff", esz() * 2.0 * c.ff * wl);
+      return count(k::seq_skinny(st.s, d));
+    }
+    k::GemmDesc g = linear_desc(dtype, h, wl, R, cfg.width, wt.data(), wl, fn, gu.ptr(), fn, false, nullptr);
+    Span span("linear_ff", product(R, 2.0 * c.ff, cfg.width));
+    if (k::matmul_tc_ready(g)) {                          // the gate rides in the product's epilogue
+      g.c = out; g.c_row = out_ld; g.ep.glu_n = c.ff; g.ep.glu = (k::Glu)c.glu; g.ep.glu_limit = c.ff_limit;
+      return count(k::matmul(st.s, g));
+    }
+    AG_RETURN_IF_ERROR(count(k::matmul(st.s, g)));
+    return count(k::glu(st.s, dtype, gu.ptr(), fn, out, out_ld, R, c.ff, k::kGluBlock, (k::Glu)c.glu, c.ff_limit));
+  }
+  // A sequential layer leaves its last sublayer's output in `sub`; *post is the weight of the norm through which the next norm
+  // kernel adds it to the stream.
+  Status enqueue_sequential(const StepCtx& st, const LayerRun& run, bool start, const float** post) {
+    const int R = st.rows();
+    float* X = static_cast<float*>(x.ptr());
+    const SeqLayerCfg& c = cfg.layers[run.layer];
+    const Mixer& mx = *mixers[run.layer];
+    const TensorRec* W = lw(run.layer);
+    const int64_t pl = pad8(mx.proj_cols()), cl = cat_ld(c), wl = pad8(cfg.width);
+    auto norm = [&](const TensorRec& w1, bool first) {
+      k::RmsRowsDesc n;
+      n.dtype = dtype; n.x = X; n.rows = R; n.width = cfg.width; n.eps = cfg.eps; n.w1 = f32(w1); n.out1 = h1.ptr(); n.ld1 = wl;
+      if (first && (start || (run.first && run.pass > 0))) {
+        n.tok = static_cast<const int32_t*>(tok.ptr()); n.embed = w[0].data(); n.embed_ld = w[0].shape[1]; n.vocab = cfg.vocab; n.embed_scale = cfg.embed_scale;
+        n.load_x = !start;
+      }
+      if (first && run.first) n.step = f32(w[3]) + (size_t)run.pass * cfg.width;
+      if (*post) { n.post = static_cast<const float*>(sub.ptr()); n.post_w = *post; }
+      *post = nullptr;
+      Span span("rms_rows", (double)R * cfg.width * ((n.post ? 12.0 : 4.0) + esz()));
+      return count(k::rms_rows(st.s, n));
+    };
+    AG_RETURN_IF_ERROR(norm(W[kWNorm1], true));
+    if (mx.gate_cols() && R <= k::kSeqSkinnyRows && skinny_ok()) {          // both input products in one launch
+      k::SeqSkinnyDesc d;
+      d.dtype = dtype; d.rows = R; d.k = cfg.width; d.a = h1.ptr(); d.a_ld = wl; d.n_seg = 2;
+      for (int i = 0; i < 2; i++) { d.seg[i].a = h1.ptr(); d.seg[i].a_ld = wl; d.seg[i].ld = wl; }
+      d.seg[0].w = W[kWIn].data(); d.seg[0].n = mx.proj_cols(); d.seg[0].mode = k::SeqOut::Store; d.seg[0].out = proj.ptr(); d.seg[0].out_ld = pl;
+      d.seg[1].w = W[kWAux0].data(); d.seg[1].n = mx.gate_cols(); d.seg[1].mode = k::SeqOut::StoreF32; d.seg[1].out = gates.ptr(); d.seg[1].out_ld = mx.gate_cols();
+      Span span("skinny_in", esz() * (double)wl * (mx.proj_cols() + mx.gate_cols()));
+      AG_RETURN_IF_ERROR(count(k::seq_skinny(st.s, d)));
+    } else {
+      AG_RETURN_IF_ERROR(enqueue_product(st, R <= k::kSeqSkinnyRows ? "skinny_in" : "linear_in", h1.ptr(), wl, cfg.width, W[kWIn], mx.proj_cols(), proj.ptr(), pl, false));
+      if (mx.gate_cols()) AG_RETURN_IF_ERROR(enqueue_product(st, "linear_gates", h1.ptr(), wl, cfg.width, W[kWAux0], mx.gate_cols(), gates.ptr(), mx.gate_cols(), true, true));
+    }
+    AG_RETURN_IF_ERROR(mx.run(st, proj.ptr(), pl, static_cast<const float*>(gates.ptr()), mem_of(run), max_len, static_cast<const int*>(pos.ptr()) + st.slot0, cat.ptr(), cl, work.ptr(),
+                              kv.ptr(), cfg.eps, &launches));
+    AG_RETURN_IF_ERROR(enqueue_product(st, R <= k::kSeqSkinnyRows ? "skinny_out" : "linear_out", cat.ptr(), cl, cat_k(c), W[kWOut], cfg.width, sub.ptr(), cfg.width, true));
+    *post = f32(W[kWPost1]);
+    if (!c.ff) return Status::OK();
+    AG_RETURN_IF_ERROR(norm(W[kWNorm2], false));
+    AG_RETURN_IF_ERROR(enqueue_glu(st, c, h1.ptr(), W[kWFf], cat.ptr(), pad8(c.ff)));
+    AG_RETURN_IF_ERROR(enqueue_product(st, R <= k::kSeqSkinnyRows ? "skinny_out" : "linear_out", cat.ptr(), pad8(c.ff), c.ff, W[kWDown], cfg.width, sub.ptr(), cfg.width, true));
+    *post = f32(W[kWPost2]);
+    return Status::OK();
+  }
+  Status enqueue_parallel(const StepCtx& st, const LayerRun& run, bool start) {
     const int R = st.rows();
     const bool skinny = R <= k::kSeqSkinnyRows && skinny_ok();
     float* X = static_cast<float*>(x.ptr());
     const int* p = static_cast<const int*>(pos.ptr()) + st.slot0;
-    for (size_t r = 0; r < runs.size(); r++) {
-      const LayerRun& run = runs[r];
-      const SeqLayerCfg& c = cfg.layers[run.layer];
-      const Mixer& mx = *mixers[run.layer];
-      const TensorRec* W = lw(run.layer);
-      const int64_t pl = pad8(mx.proj_cols()), cl = cat_ld(c), wl = pad8(cfg.width);
-      uint8_t* ff_out = static_cast<uint8_t*>(cat.ptr()) + (size_t)y_cols(c) * esz();
-      // what happens to the stream ahead of this run rides in the norm: the embedding, a pass's additions
-      k::RmsRowsDesc n;
-      n.dtype = dtype; n.x = X; n.rows = R; n.width = cfg.width; n.eps = cfg.eps;
-      const bool start = r == 0, again = run.first && run.pass > 0;
-      if (start || again) { n.tok = static_cast<const int32_t*>(tok.ptr()); n.embed = w[0].data(); n.embed_ld = w[0].shape[1]; n.vocab = cfg.vocab; }
-      n.load_x = !start;
-      if (run.first) n.step = f32(w[3]) + (size_t)run.pass * cfg.width;
-      if (skinny) {
-        // 16-bit: the norms are stored once and every product reads them; float32: the products take them in their prologue
-        const bool stored = dtype != DType::F32;
-        if (stored) {
-          n.w1 = f32(W[kWNorm1]); n.out1 = h1.ptr(); n.ld1 = wl;
-          if (c.ff) { n.w2 = f32(W[kWNorm2]); n.out2 = h2.ptr(); n.ld2 = wl; }
-        }
-        if (stored || start || n.step) AG_RETURN_IF_ERROR(count(k::rms_rows(st.s, n)));
-        k::SeqSkinnyDesc d;
-        d.dtype = dtype; d.rows = R; d.k = cfg.width; d.eps = cfg.eps;
-        if (!stored) d.x = X;
-        auto seg = [&](const TensorRec& wt, int64_t cols, const TensorRec& nw, const Scratch& h, k::SeqOut mode, void* out, int64_t ld) {
-          k::SeqSeg& g = d.seg[d.n_seg++];
-          g.w = wt.data(); g.ld = wl; g.n = (int)cols; g.mode = mode; g.limit = c.ff_limit; g.out = out; g.out_ld = ld;
-          if (stored) { g.a = h.ptr(); g.a_ld = wl; } else g.norm_w = f32(nw);
-        };
-        seg(W[kWIn], mx.proj_cols(), W[kWNorm1], h1, k::SeqOut::Store, proj.ptr(), pl);
-        if (mx.gate_cols()) seg(W[kWAux0], mx.gate_cols(), W[kWNorm1], h1, k::SeqOut::StoreF32, gates.ptr(), mx.gate_cols());
-        if (c.ff) seg(W[kWFf], c.ff, W[kWNorm2], h2, k::SeqOut::Glu, ff_out, cl);
-        Span span("skinny_in", esz() * (double)wl * (mx.proj_cols() + mx.gate_cols() + 2.0 * c.ff));
-        AG_RETURN_IF_ERROR(count(k::seq_skinny(st.s, d)));
-      } else {
+    const SeqLayerCfg& c = cfg.layers[run.layer];
+    const Mixer& mx = *mixers[run.layer];
+    const TensorRec* W = lw(run.layer);
+    const int64_t pl = pad8(mx.proj_cols()), cl = cat_ld(c), wl = pad8(cfg.width);
+    uint8_t* ff_out = static_cast<uint8_t*>(cat.ptr()) + (size_t)y_cols(c) * esz();
+    // what happens to the stream ahead of this run rides in the norm: the embedding, a pass's additions
+    k::RmsRowsDesc n;
+    n.dtype = dtype; n.x = X; n.rows = R; n.width = cfg.width; n.eps = cfg.eps;
+    const bool again = run.first && run.pass > 0;
+    if (start || again) { n.tok = static_cast<const int32_t*>(tok.ptr()); n.embed = w[0].data(); n.embed_ld = w[0].shape[1]; n.vocab = cfg.vocab; n.embed_scale = cfg.embed_scale; }
+    n.load_x = !start;
+    if (run.first) n.step = f32(w[3]) + (size_t)run.pass * cfg.width;
+    if (skinny) {
+      // 16-bit: the norms are stored once and every product reads them; float32: the products take them in their prologue
+      const bool stored = dtype != DType::F32;
+      if (stored) {
         n.w1 = f32(W[kWNorm1]); n.out1 = h1.ptr(); n.ld1 = wl;
         if (c.ff) { n.w2 = f32(W[kWNorm2]); n.out2 = h2.ptr(); n.ld2 = wl; }
-        {
-          Span span("rms_rows", (4.0 + (c.ff ? 2.0 : 1.0) * esz()) * R * cfg.width);
-          AG_RETURN_IF_ERROR(count(k::rms_rows(st.s, n)));
-        }
-        {
-          Span span("linear_in", product(R, mx.proj_cols(), cfg.width));
-          AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h1.ptr(), wl, R, cfg.width, W[kWIn].data(), wl, mx.proj_cols(), proj.ptr(), pl, false, nullptr))));
-        }
-        if (mx.gate_cols()) {
-          Span span("linear_gates", (double)R * (esz() * cfg.width + 4.0 * mx.gate_cols()));      // bound by reading its input
-          AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h1.ptr(), wl, R, cfg.width, W[kWAux0].data(), wl, mx.gate_cols(), gates.ptr(), mx.gate_cols(), true, nullptr))));
-        }
-        if (c.ff) {
-          const int64_t fn = k::glu_rows(c.ff);
-          k::GemmDesc g = linear_desc(dtype, h2.ptr(), wl, R, cfg.width, W[kWFf].data(), wl, fn, gu.ptr(), fn, false, nullptr);
-          if (k::matmul_tc_ready(g)) {                  // the gate rides in the product's epilogue
-            g.c = ff_out; g.c_row = cl; g.ep.glu_n = c.ff; g.ep.glu_limit = c.ff_limit;
+      }
+      if (stored || start || n.step) AG_RETURN_IF_ERROR(count(k::rms_rows(st.s, n)));
+      k::SeqSkinnyDesc d;
+      d.dtype = dtype; d.rows = R; d.k = cfg.width; d.eps = cfg.eps;
+      if (!stored) d.x = X;
+      auto seg = [&](const TensorRec& wt, int64_t cols, const TensorRec& nw, const Scratch& h, k::SeqOut mode, void* out, int64_t ld) {
+        k::SeqSeg& g = d.seg[d.n_seg++];
+        g.w = wt.data(); g.ld = wl; g.n = (int)cols; g.mode = mode; g.glu = (k::Glu)c.glu; g.limit = c.ff_limit; g.out = out; g.out_ld = ld;
+        if (stored) { g.a = h.ptr(); g.a_ld = wl; } else g.norm_w = f32(nw);
+      };
+      seg(W[kWIn], mx.proj_cols(), W[kWNorm1], h1, k::SeqOut::Store, proj.ptr(), pl);
+      if (mx.gate_cols()) seg(W[kWAux0], mx.gate_cols(), W[kWNorm1], h1, k::SeqOut::StoreF32, gates.ptr(), mx.gate_cols());
+      if (c.ff) seg(W[kWFf], c.ff, W[kWNorm2], h2, k::SeqOut::Glu, ff_out, cl);
+      Span span("skinny_in", esz() * (double)wl * (mx.proj_cols() + mx.gate_cols() + 2.0 * c.ff));
+      AG_RETURN_IF_ERROR(count(k::seq_skinny(st.s, d)));
+    } else {
+      n.w1 = f32(W[kWNorm1]); n.out1 = h1.ptr(); n.ld1 = wl;
+      if (c.ff) { n.w2 = f32(W[kWNorm2]); n.out2 = h2.ptr(); n.ld2 = wl; }
+      {
+        Span span("rms_rows", (4.0 + (c.ff ? 2.0 : 1.0) * esz()) * R * cfg.width);
+        AG_RETURN_IF_ERROR(count(k::rms_rows(st.s, n)));
+      }
+      {
+        Span span("linear_in", product(R, mx.proj_cols(), cfg.width));
+        AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h1.ptr(), wl, R, cfg.width, W[kWIn].data(), wl, mx.proj_cols(), proj.ptr(), pl, false, nullptr))));
+      }
+      if (mx.gate_cols()) {
+        Span span("linear_gates", (double)R * (esz() * cfg.width + 4.0 * mx.gate_cols()));      // bound by reading its input
+        AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, h1.ptr(), wl, R, cfg.width, W[kWAux0].data(), wl, mx.gate_cols(), gates.ptr(), mx.gate_cols(), true, nullptr))));
+      }
+      if (c.ff) {
+        const int64_t fn = k::glu_rows(c.ff);
+        k::GemmDesc g = linear_desc(dtype, h2.ptr(), wl, R, cfg.width, W[kWFf].data(), wl, fn, gu.ptr(), fn, false, nullptr);
+        if (k::matmul_tc_ready(g)) {                  // the gate rides in the product's epilogue
+          g.c = ff_out; g.c_row = cl; g.ep.glu_n = c.ff; g.ep.glu = (k::Glu)c.glu; g.ep.glu_limit = c.ff_limit;
+          Span span("linear_ff", product(R, 2.0 * c.ff, cfg.width));
+          AG_RETURN_IF_ERROR(count(k::matmul(st.s, g)));
+        } else {
+          {
             Span span("linear_ff", product(R, 2.0 * c.ff, cfg.width));
             AG_RETURN_IF_ERROR(count(k::matmul(st.s, g)));
-          } else {
-            {
-              Span span("linear_ff", product(R, 2.0 * c.ff, cfg.width));
-              AG_RETURN_IF_ERROR(count(k::matmul(st.s, g)));
-            }
-            Span span("clamped_glu", 3.0 * esz() * R * c.ff);
-            AG_RETURN_IF_ERROR(count(k::clamped_glu(st.s, dtype, gu.ptr(), fn, ff_out, cl, R, c.ff, k::kGluBlock, c.ff_limit)));
           }
+          Span span("clamped_glu", 3.0 * esz() * R * c.ff);
+          AG_RETURN_IF_ERROR(count(k::glu(st.s, dtype, gu.ptr(), fn, ff_out, cl, R, c.ff, k::kGluBlock, (k::Glu)c.glu, c.ff_limit)));
         }
       }
-      AG_RETURN_IF_ERROR(mx.run(st, proj.ptr(), pl, static_cast<const float*>(gates.ptr()), memory[r]->ptr, max_len, p, cat.ptr(), cl, work.ptr(), kv.ptr(), cfg.eps, &launches));
-      if (skinny) {
-        k::SeqSkinnyDesc d;
-        d.dtype = dtype; d.rows = R; d.k = (int)cat_k(c); d.a = cat.ptr(); d.a_ld = cl; d.n_seg = 1;
-        d.seg[0].a = cat.ptr(); d.seg[0].a_ld = cl;
-        d.seg[0].w = W[kWOut].data(); d.seg[0].ld = cl; d.seg[0].n = cfg.width; d.seg[0].mode = k::SeqOut::AddF32; d.seg[0].out = X; d.seg[0].out_ld = cfg.width;
-        Span span("skinny_out", esz() * (double)cl * cfg.width);
-        AG_RETURN_IF_ERROR(count(k::seq_skinny(st.s, d)));
-      } else {
-        Span span("linear_out", product(R, cfg.width, cat_k(c)));
-        AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, cat.ptr(), cl, R, cat_k(c), W[kWOut].data(), cl, cfg.width, X, cfg.width, true, X))));
-      }
+    }
+    AG_RETURN_IF_ERROR(mx.run(st, proj.ptr(), pl, static_cast<const float*>(gates.ptr()), mem_of(run), max_len, p, cat.ptr(), cl, work.ptr(), kv.ptr(), cfg.eps, &launches));
+    if (skinny) {
+      k::SeqSkinnyDesc d;
+      d.dtype = dtype; d.rows = R; d.k = (int)cat_k(c); d.a = cat.ptr(); d.a_ld = cl; d.n_seg = 1;
+      d.seg[0].a = cat.ptr(); d.seg[0].a_ld = cl;
+      d.seg[0].w = W[kWOut].data(); d.seg[0].ld = cl; d.seg[0].n = cfg.width; d.seg[0].mode = k::SeqOut::AddF32; d.seg[0].out = X; d.seg[0].out_ld = cfg.width;
+      Span span("skinny_out", esz() * (double)cl * cfg.width);
+      AG_RETURN_IF_ERROR(count(k::seq_skinny(st.s, d)));
+    } else {
+      Span span("linear_out", product(R, cfg.width, cat_k(c)));
+      AG_RETURN_IF_ERROR(count(k::matmul(st.s, linear_desc(dtype, cat.ptr(), cl, R, cat_k(c), W[kWOut].data(), cl, cfg.width, X, cfg.width, true, X))));
+    }
+    return Status::OK();
+  }
+
+  // All layers over the R rows whose tokens are in `tok`; x holds the residual stream afterwards, but for what *post (see
+  // enqueue_sequential) says is still to be added.
+  Status enqueue_layers(const StepCtx& st, float* layers_out, const float** post) {
+    const size_t R = (size_t)st.rows();
+    *post = nullptr;
+    for (size_t r = 0; r < runs.size(); r++) {
+      AG_RETURN_IF_ERROR(sequential() ? enqueue_sequential(st, runs[r], r == 0, post) : enqueue_parallel(st, runs[r], r == 0));
       if (layers_out) {
-        cudaError_t e = cudaMemcpyAsync(layers_out + r * (size_t)R * cfg.width, X, (size_t)R * cfg.width * sizeof(float), cudaMemcpyDeviceToHost, st.s);
+        if (*post) {
+          k::RmsRowsDesc n;
+          n.dtype = dtype; n.x = static_cast<float*>(x.ptr()); n.rows = R; n.width = cfg.width; n.eps = cfg.eps; n.post = static_cast<const float*>(sub.ptr()); n.post_w = *post;
+          *post = nullptr;
+          AG_RETURN_IF_ERROR(count(k::rms_rows(st.s, n)));
+        }
+        cudaError_t e = cudaMemcpyAsync(layers_out + r * R * cfg.width, x.ptr(), R * cfg.width * sizeof(float), cudaMemcpyDeviceToHost, st.s);
         if (e != cudaSuccess) return Status::compute("sequence engine: layer copy");
       }
     }
     return Status::OK();
   }
 
-  // Logits of n rows of x: all of them in order (map null), or the ones listed in the device array `map`.
-  Status enqueue_head(cudaStream_t s, int n, const int32_t* map) {
+  // Logits of n rows of x: all of them in order (map null), or the ones listed in the device array `map`; post: as enqueue_layers left it.
+  Status enqueue_head(cudaStream_t s, int n, const int32_t* map, const float* post) {
     const int64_t wl = pad8(cfg.width);
     Span span(n <= k::kSeqSkinnyRows ? "skinny_head" : "linear_head", n <= k::kSeqSkinnyRows ? esz() * (double)wl * cfg.vocab : product(n, cfg.vocab, cfg.width));
     const bool skinny = n <= k::kSeqSkinnyRows && k::seq_skinny_fits(cfg.width);
@@ -371,9 +588,10 @@ struct SeqEngine {
     d.dtype = dtype; d.rows = n; d.k = cfg.width; d.eps = cfg.eps; d.n_seg = 1;
     d.seg[0].w = w[1].data(); d.seg[0].ld = wl; d.seg[0].n = cfg.vocab; d.seg[0].norm_w = f32(w[2]); d.seg[0].mode = k::SeqOut::StoreF32; d.seg[0].out = logits.ptr();
     d.seg[0].out_ld = cfg.vocab;
-    if (skinny && !map && dtype == DType::F32) { d.x = static_cast<const float*>(x.ptr()); return count(k::seq_skinny(s, d)); }
+    if (skinny && !map && !post && dtype == DType::F32) { d.x = static_cast<const float*>(x.ptr()); return count(k::seq_skinny(s, d)); }
     k::RmsRowsDesc r;
     r.dtype = dtype; r.x = static_cast<float*>(x.ptr()); r.rows = n; r.width = cfg.width; r.eps = cfg.eps; r.row_map = map; r.w1 = f32(w[2]); r.out1 = h1.ptr(); r.ld1 = wl;
+    if (post) { r.post = static_cast<const float*>(sub.ptr()); r.post_w = post; }
     AG_RETURN_IF_ERROR(count(k::rms_rows(s, r)));
     if (skinny) { d.a = d.seg[0].a = h1.ptr(); d.a_ld = d.seg[0].a_ld = wl; return count(k::seq_skinny(s, d)); }
     return count(k::matmul(s, linear_desc(dtype, h1.ptr(), wl, n, cfg.width, w[1].data(), wl, cfg.vocab, logits.ptr(), cfg.vocab, true, nullptr)));
@@ -386,8 +604,9 @@ struct SeqEngine {
   Status enqueue_step(cudaStream_t s, int slot0, int n) {
     launches = 0;
     StepCtx st{s, slot0, n, 1, len.data() + slot0};
-    AG_RETURN_IF_ERROR(enqueue_layers(st, nullptr));
-    AG_RETURN_IF_ERROR(enqueue_head(s, n, nullptr));
+    const float* post = nullptr;
+    AG_RETURN_IF_ERROR(enqueue_layers(st, nullptr, &post));
+    AG_RETURN_IF_ERROR(enqueue_head(s, n, nullptr, post));
     AG_RETURN_IF_ERROR(enqueue_pick(s, n, tok.ptr()));
     AG_RETURN_IF_ERROR(count(k::seq_advance(s, static_cast<int*>(pos.ptr()) + slot0, n, 1, static_cast<const int32_t*>(tok.ptr()), static_cast<int32_t*>(history.ptr()),
                                             static_cast<int*>(step.ptr()), max_len)));
@@ -471,21 +690,35 @@ Status seq_create(const SeqModelCfg& cfg, const std::vector<TensorRec>& weights,
     if (c.heads < 1 || c.dim < 1 || c.vdim < 1 || c.ff < 0) return Status::invalid(at + "bad sizes");
     if (c.mixer == MixerKind::Mlstm) e->mixers.emplace_back(new MlstmMixer(c, t, dt));
     else if (c.mixer == MixerKind::LatentAttention) e->mixers.emplace_back(new LatentMixer(c, t, dt));
+    else if (c.mixer == MixerKind::KeyDecay) e->mixers.emplace_back(new KeyDecayMixer(c, t, dt));
+    else if (c.mixer == MixerKind::GroupedAttention) e->mixers.emplace_back(new GroupedMixer(c, t, dt));
     else return Status::invalid(at + "unknown mixer");
     const Mixer& m = *e->mixers.back();
     if (!is_vector(t[kWNorm1], W) || !is_matrix(t[kWIn], dt, m.proj_cols(), wl) || !is_matrix(t[kWOut], dt, W, e->cat_ld(c))) return Status::invalid(at + "norm, input or output weights");
     if (c.ff && (!is_vector(t[kWNorm2], W) || !is_matrix(t[kWFf], dt, k::glu_rows(c.ff), wl))) return Status::invalid(at + "feed-forward weights");
+    if (e->sequential() && (!is_vector(t[kWPost1], W) || (c.ff && (!is_vector(t[kWPost2], W) || !is_matrix(t[kWDown], dt, W, pad8(c.ff))))))
+      return Status::invalid(at + "norms behind the sublayers or feed-forward output");
+    if (c.kv_from >= l) return Status::invalid(at + "keys come from an earlier layer");
     const Status st = m.check(cfg, max_len);
     if (!st.ok()) return Status{st.kind, at + st.msg};
   }
-  auto add = [&](int lo, int hi, int pass) { for (int l = lo; l < hi; l++) e->runs.push_back({l, pass, pass >= 0 && l == lo}); };
+  auto add = [&](int lo, int hi, int pass) { for (int l = lo; l < hi; l++) e->runs.push_back({l, pass, pass >= 0 && l == lo, (int)e->runs.size()}); };
   if (cfg.loop_times) {
     add(0, cfg.loop_start, -1);
     for (int t = 0; t < cfg.loop_times; t++) add(cfg.loop_start, cfg.loop_stop, t);
     add(cfg.loop_stop, n_layers, -1);
   } else add(0, n_layers, -1);
+  for (size_t i = 0; i < e->runs.size(); i++) {         // keys of another layer: its latest run
+    const int from = e->cfg.layers[e->runs[i].layer].kv_from;
+    if (from < 0) continue;
+    size_t j = i;
+    while (j > 0 && e->runs[j].layer != from) j--;
+    if (e->runs[j].layer != from) return Status::invalid("sequence model: keys come from a layer that has not run");
+    e->runs[i].memory = (int)j;
+  }
   for (const LayerRun& r : e->runs) {
     std::shared_ptr<Buffer> b;
+    if (e->mixers[r.layer]->slot_bytes(max_len) == 0) { e->memory.push_back(nullptr); continue; }
     AG_RETURN_IF_ERROR(Shared::get().pool.acquire((size_t)slots * e->mixers[r.layer]->slot_bytes(max_len), &b));
     // padding columns of caches take part in products with zeros: they must hold numbers
     if (cudaMemsetAsync(b->ptr, 0, b->capacity, ctx.stream) != cudaSuccess) return Status::compute("sequence engine: clear");
@@ -566,10 +799,11 @@ Status seq_forward(uint64_t handle, int slot0, int n_seq, const int32_t* tokens,
     } else {
       e->launches = 0;
       StepCtx st{s, slot0, n_seq, Ts, e->len.data() + slot0};
-      AG_RETURN_IF_ERROR(e->enqueue_layers(st, layers_out));
+      const float* post = nullptr;
+      AG_RETURN_IF_ERROR(e->enqueue_layers(st, layers_out, &post));
       if (nw) {
         if (!in_order) AG_RETURN_IF_ERROR(copy_ok(cudaMemcpyAsync(e->rowmap.ptr(), rows.data(), (size_t)nw * 4, cudaMemcpyHostToDevice, s)));
-        AG_RETURN_IF_ERROR(e->enqueue_head(s, nw, in_order ? nullptr : static_cast<const int32_t*>(e->rowmap.ptr())));
+        AG_RETURN_IF_ERROR(e->enqueue_head(s, nw, in_order ? nullptr : static_cast<const int32_t*>(e->rowmap.ptr()), post));
         if (picked) {
           AG_RETURN_IF_ERROR(e->enqueue_pick(s, nw, e->picked.ptr()));
           std::vector<int32_t> got(nw);

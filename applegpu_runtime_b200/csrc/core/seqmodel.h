@@ -5,26 +5,36 @@
 
 namespace ag {
 
-enum class MixerKind : int { Mlstm = 1, LatentAttention = 2 };
+enum class MixerKind : int { Mlstm = 1, LatentAttention = 2, KeyDecay = 3, GroupedAttention = 4 };
+enum class LayerForm : int { Parallel = 0, Sequential = 1 };     // see seqmodel.cc
+enum KeyDecayFlag : int { kKdDelta = 1, kKdUnit = 2, kKdSoftplus = 4, kKdGateSilu = 8 };
 
 struct SeqLayerCfg {
   MixerKind mixer = MixerKind::Mlstm;
   int heads = 0, dim = 0, vdim = 0;
   int rot_dim = 0, rot_pairs = 0, kv_rank = 0;      // latent attention
   float gate_cap = 0.f;                             // mLSTM
-  float score_scale = 0.f;                          // latent attention
+  float score_scale = 0.f;                          // attention
+  int kv_heads = 0;                                 // grouped attention, key decay (heads of q and k)
+  int window = 0, kv_from = -1;                     // grouped attention: keys a token sees (0: all), layer whose keys it uses (-1: its own)
+  float softcap = 0.f;                              // grouped attention
+  int taps = 0, a_rank = 0, g_rank = 0, flags = 0;  // key decay (KeyDecayFlag)
+  float tau = 1.f;                                  // key decay
   int ff = 0;                                       // 0: no feed-forward
+  int glu = 0;                                      // k::Glu
   float ff_limit = 0.f;
 };
 struct SeqModelCfg {
   int vocab = 0, width = 0;
   float eps = 1e-5f;
+  LayerForm form = LayerForm::Parallel;
+  float embed_scale = 1.f;
   int loop_start = 0, loop_stop = 0, loop_times = 0;  // loop_times 0: no layer is repeated
   std::vector<SeqLayerCfg> layers;
 };
 // Weight tensors: embed, head, final norm, step vectors (or an empty record without a loop), then kSeqLayerWeights per layer
 // in the order of SeqLayerWeight (empty records where a layer has none).
-enum SeqLayerWeight : int { kWNorm1 = 0, kWNorm2, kWIn, kWOut, kWFf, kWAux0, kWAux1, kWAux2, kSeqLayerWeights };
+enum SeqLayerWeight : int { kWNorm1 = 0, kWNorm2, kWIn, kWOut, kWFf, kWAux0, kWAux1, kWAux2, kWPost1, kWPost2, kWDown, kWAux3, kWAux4, kWAux5, kWAux6, kSeqLayerWeights };
 
 Status seq_create(const SeqModelCfg& cfg, const std::vector<TensorRec>& weights, int slots, int max_len, uint64_t* handle);
 // The next T tokens of the sequences in slots slot0 .. slot0 + n_seq, all of them of the same portion length. `want`: rows

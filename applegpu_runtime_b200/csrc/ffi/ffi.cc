@@ -1361,11 +1361,14 @@ uint64_t applegpu_seq_create(const applegpu_seq_model* m, const applegpu_seq_lay
   std::lock_guard<std::mutex> g(st.mu);
   SeqModelCfg cfg;
   cfg.vocab = m->vocab; cfg.width = m->width; cfg.eps = m->eps; cfg.loop_start = m->loop_start; cfg.loop_stop = m->loop_stop; cfg.loop_times = m->loop_times;
+  cfg.form = (LayerForm)m->form; cfg.embed_scale = m->embed_scale;
   for (int32_t i = 0; i < m->n_layers; i++) {
     const applegpu_seq_layer& l = layers[i];
     SeqLayerCfg c;
     c.mixer = (MixerKind)l.mixer; c.heads = l.heads; c.dim = l.dim; c.vdim = l.vdim; c.rot_dim = l.rot_dim; c.rot_pairs = l.rot_pairs; c.kv_rank = l.kv_rank;
     c.gate_cap = l.gate_cap; c.score_scale = l.score_scale; c.ff = l.ff; c.ff_limit = l.ff_limit;
+    c.kv_heads = l.kv_heads; c.window = l.window; c.kv_from = l.kv_from; c.taps = l.taps; c.a_rank = l.a_rank; c.g_rank = l.g_rank; c.flags = l.flags; c.glu = l.glu;
+    c.softcap = l.softcap; c.tau = l.tau;
     cfg.layers.push_back(c);
   }
   std::vector<TensorRec> w(n_weights);
@@ -1455,7 +1458,7 @@ uint64_t applegpu_ffi_clamped_glu(uint64_t gate_up_id, float limit) {
     const int64_t c = o.back(), rows = numel_of(o) / (c ? c : 1);
     o.back() = c / 2;
     AG_RETURN_IF_ERROR(new_tensor(o, t.dtype, &out));
-    return k::clamped_glu(DeviceCtx::get().stream, t.dtype, t.data(), c, out.data(), c / 2, rows, (int)(c / 2), (int)(c / 2), limit);
+    return k::glu(DeviceCtx::get().stream, t.dtype, t.data(), c, out.data(), c / 2, rows, (int)(c / 2), (int)(c / 2), k::Glu::Clamped, limit);
   };
   const Status s = run();
   return immediate_result("clamped_glu", st.rt, s, out);
@@ -1526,13 +1529,13 @@ uint64_t applegpu_ffi_latent_attention(uint64_t proj_id, uint64_t norm_id, uint6
     m.dtype = dt; m.b_dtype = dt; m.a = d.cache; m.b = d.w_uk; m.c = work.data(); m.m = keys; m.n = cols; m.k = kv_rank; m.batch = B;
     m.a_row = cld; m.a_col = 1; m.a_batch = d.seq_stride; m.b_row = 1; m.b_col = w_ld; m.b_batch = 0; m.c_row = cols; m.c_batch = keys * cols;
     AG_RETURN_IF_ERROR(k::matmul(cs, m));
-    k::LatentPrefillDesc p;
+    k::PromptAttnDesc p;
     p.dtype = dt; p.n_seq = (int)B; p.T = (int)T; p.past = (int)past; p.heads = (int)heads; p.dim = (int)dim; p.rot_dim = (int)rot_dim; p.vdim = (int)vdim; p.scale = scale;
-    p.q = d.proj; p.q_ld = d.ld; p.q_b = T * d.ld; p.kv = work.data(); p.kv_ld = cols; p.v_off = v_off; p.kv_b = keys * cols;
+    p.q = d.proj; p.q_ld = d.ld; p.q_b = T * d.ld; p.k = work.data(); p.k_ld = cols; p.v = static_cast<uint8_t*>(work.data()) + (size_t)v_off * esz; p.v_ld = cols; p.k_b = p.v_b = keys * cols;
     p.k_rot = static_cast<uint8_t*>(d.cache) + (size_t)k::pad8(kv_rank) * esz; p.k_rot_ld = cld; p.k_rot_b = d.seq_stride;
     p.y = out.data(); p.y_ld = d.y_ld; p.y_b = T * d.y_ld;
-    if (form == 2) return k::latent_prefill_tc_eligible(p) ? k::latent_prefill_tc(cs, p) : Status::unsupported("these sizes do not take the tensor-core kernel");
-    AG_RETURN_IF_ERROR(k::latent_prefill(cs, p));
+    if (form == 2) return k::prompt_attention_tc_eligible(p) ? k::prompt_attention_tc(cs, p) : Status::unsupported("these sizes do not take the tensor-core kernel");
+    AG_RETURN_IF_ERROR(k::prompt_attention(cs, p));
     return Status::OK();
   };
   const Status s = run();

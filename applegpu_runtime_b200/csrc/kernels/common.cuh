@@ -162,6 +162,8 @@ __device__ __forceinline__ float clamped_glu_f(float gate, float up, float limit
   return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
 }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float glu_f(int kind, float gate, float up, float limit) { return kind == (int)Glu::Silu ? silu_f(gate) * up : clamped_glu_f(gate, up, limit); }
 
 inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
 

@@ -57,6 +57,7 @@ struct TcParams {
   long long* stats_out;              // folded layer_norm, producer side: row sums of what is stored (fixed point, integer atomics)
   long long* stats_zero;             // rows of the other statistics tensor to clear
   int glu_n, glu_vec;                // gated result: B rows come in blocks of 16 gate | 16 up, C has glu_n columns (16-byte rows: glu_vec)
+  int glu_kind;
   float glu_limit;
   int* status;
 #ifdef AG_GEMM_PROBE
@@ -251,8 +252,12 @@ __device__ __forceinline__ void glu_group(const TcParams& p, uint32_t taddr, lon
     float r[2];
 #pragma unroll
     for (int q = 0; q < 2; q++) {
-      const float g = fminf(__uint_as_float(acc[2 * w + q]), p.glu_limit), u = fminf(fmaxf(__uint_as_float(acc[16 + 2 * w + q]), -p.glu_limit), p.glu_limit);
-      r[q] = __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+      float g = __uint_as_float(acc[2 * w + q]), u = __uint_as_float(acc[16 + 2 * w + q]);
+      if (p.glu_kind == (int)Glu::Silu) r[q] = g * __frcp_rn(1.0f + __expf(-g)) * u;      // a quotient with so large a divisor that its reciprocal is subnormal is zero
+      else {
+        g = fminf(g, p.glu_limit); u = fminf(fmaxf(u, -p.glu_limit), p.glu_limit);
+        r[q] = __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+      }
     }
     o[w] = pack2<T>(r[0], r[1]);
   }
@@ -1969,7 +1974,7 @@ Status matmul_tc(cudaStream_t s, const GemmDesc& d, int* status_word) {
   p.c_f32 = d.c_f32 ? 1 : 0;
   p.ln_stats = d.ep.ln_stats; p.ln_colsum = d.ep.ln_colsum; p.ln_inv_k = d.k ? 1.0f / (float)d.k : 0.f; p.ln_eps = d.ep.ln_eps;
   p.stats_out = d.ep.stats_out; p.stats_zero = d.ep.stats_zero;
-  p.glu_n = d.ep.glu_n; p.glu_limit = d.ep.glu_limit;
+  p.glu_n = d.ep.glu_n; p.glu_kind = (int)d.ep.glu; p.glu_limit = d.ep.glu_limit;
   p.glu_vec = (reinterpret_cast<uintptr_t>(d.c) & 15u) == 0 && d.c_row % 8 == 0 ? 1 : 0;
 #ifdef AG_GEMM_PROBE
   p.probe = g_tc_probe;

@@ -13,6 +13,8 @@ enum class UnOp : int {
   Neg = 0, Relu, Exp, Log, Sqrt, Tanh, Sin, Cos, Gelu, GeluExact, Sigmoid, Abs, Sign, Copy
 };
 enum class Act : int { None = 0, GeluTanh = 1, GeluErf = 2, Relu = 3 };
+// Gated feed-forwards. Clamped: g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(value, -limit, limit). Silu: gate sigmoid(gate) value.
+enum class Glu : int { Clamped = 0, Silu = 1 };
 
 // Fused element-wise chain (reference: fusion.rs:167-238 emits MSL text; here the chain
 // is a register program interpreted per element). Registers 0..n_inputs-1 hold the loaded
@@ -84,8 +86,9 @@ struct GemmEpilogue {
   long long* stats_out = nullptr;
   long long* stats_zero = nullptr;
   // Gated result (tensor-core kernels, unbatched, 16-bit C): B's columns come in blocks of 16 gates | 16 values, n a multiple of
-  // 32, and C gets glu_n <= n / 2 columns g sigmoid(1.702 g) (u + 1), g = min(gate, glu_limit), u = clamp(value, +-glu_limit).
+  // 32, and C gets glu_n <= n / 2 columns.
   int glu_n = 0;
+  Glu glu = Glu::Clamped;
   float glu_limit = 0.f;
 };
 struct GemmDesc {

@@ -1,0 +1,52 @@
+// What the two files of key-decayed matrix states share: the parameters of their kernels, the raw inputs of the convolutions, the
+// decay.
+#pragma once
+#include "common.cuh"
+#include "seq_kernels.h"
+
+namespace ag { namespace k {
+
+constexpr int kKdChunk = 32;           // tokens per chunk
+
+struct KdParams {
+  const void* proj; const void* a2; const void* g2; const float* bias; const float* rate; const float* conv; const float* norm; const float* beta; const int* pos;
+  void* mem; void* y;
+  const float* z; const void* gate;      // decay inputs [rows, heads * dim] without bias and gates [rows, heads * vdim], where a product made them
+  long long ld, beta_ld, mem_stride, y_ld, gate_ld, ring_off;      // ring_off: bytes from a sequence's memory to its ring
+  int n_seq, T, heads, qk_heads, group, dim, vdim, taps, ring, channels;
+  int q_off, k_off, v_off, a_off, a_rank, a_ld, g_off, g_rank, g_ld;
+  int delta, unit, softplus, gate_silu;
+  float inv_tau, q_scale, eps;
+  uint8_t* ops; float* u; float* o;      // scratch of the chunk form
+  int chunks, dp;                        // dp: dim padded for the tensor cores
+  long long ops_bytes;                   // of one chunk of one head
+  __device__ float* state(int s) const { return reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(mem) + (long long)s * mem_stride); }
+  template <typename T> __device__ T* ring_of(int s) const { return reinterpret_cast<T*>(reinterpret_cast<uint8_t*>(mem) + (long long)s * mem_stride + ring_off); }
+};
+
+// Raw input of a channel: `col` its column in proj, `ch` its place among the q | k | v channels, t the token of the portion (negative:
+// before it; zero before the sequence's start).
+template <typename T>
+__device__ __forceinline__ float kd_raw(const KdParams& p, const T* base, const T* ring, int pos, int t, int col, int ch) {
+  if (t >= 0) return Cvt<T>::to(base[(long long)t * p.ld + col]);
+  const int at = pos + t;
+  return at < 0 ? 0.f : Cvt<T>::to(ring[(long long)(at % p.ring) * p.channels + ch]);
+}
+// One channel at token t behind its convolution and silu, or as it is.
+template <typename T>
+__device__ __forceinline__ float kd_input(const KdParams& p, const T* base, const T* ring, int pos, int t, int col, int ch) {
+  if (p.taps == 0) return Cvt<T>::to(base[(long long)t * p.ld + col]);
+  const float* w = p.conv + (long long)ch * p.taps;
+  float a = 0.f;
+  for (int i = 0; i < p.taps; i++) a = fmaf(__ldg(w + i), kd_raw(p, base, ring, pos, t - (p.taps - 1) + i, col, ch), a);
+  return silu_f(a);
+}
+__device__ __forceinline__ float kd_softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// decay of a key channel from its input z (bias included)
+__device__ __forceinline__ float kd_decay(const KdParams& p, int h, float z) { return p.softplus ? expf(-p.rate[h] * kd_softplus(z)) : expf(-kd_softplus(-z) * p.inv_tau); }
+__device__ __forceinline__ float kd_gate(const KdParams& p, float g) { return p.gate_silu ? silu_f(g) : sigmoid_f(g); }
+
+inline int kd_dp(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 96 ? 96 : dim <= 128 ? 128 : dim <= 192 ? 192 : 256; }
+Status key_decay_chunked(cudaStream_t s, DType dt, const KdParams& p, int* launches);
+
+}}  // namespace ag::k

@@ -2,8 +2,7 @@
 // key part shared by the heads; the cache holds only those two.
 //
 //   append    one row per CTA: rotates the query parts, norms the latent, rotates the key part, writes the cache row
-//   prefill   attention of a prompt portion over keys and values expanded from the cache (the GEMM that expands them is
-//             the caller's). The form here runs on CUDA cores in float32 arithmetic and takes any sizes.
+//   prefill   prompt_attention over keys and values expanded from the cache (the GEMM that expands them is the caller's)
 //   decode    short portions stay in the latent space: W_uk is applied to the query instead of to every key, W_uv to the
 //             attended latent instead of to every value, so that a step reads each cached row once for all heads.
 //             prepare -> attend over splits of the keys -> merge the splits and apply W_uv.
@@ -109,112 +108,6 @@ Status latent_append(cudaStream_t s, const LatentDesc& d) {
   cudaError_t e = cudaSuccess;
   AG_DISPATCH_FLOAT(d.dtype, T, (e = launch_pdl(latent_append_kernel<T>, dim3((unsigned)(d.n_seq * d.T)), dim3(kLaThreads), 0, s, p)));
   return cuda_status(e, "latent append");
-}
-
-// ── prefill, CUDA cores ─────────────────────────────────────────────────────
-struct LpParams {
-  const void* q; const void* kv; const void* kr; void* y;
-  long long q_ld, kv_ld, v_off, kr_ld, y_ld, q_b, kv_b, kr_b, y_b;
-  int T, past, heads, dim, rot, vdim;
-  float scale;
-};
-template <typename T, int TQ>
-__global__ void __launch_bounds__(256) latent_prefill_kernel(const LpParams p) {
-  extern __shared__ __align__(16) float sm[];
-  const int D = p.dim + p.rot, E = p.vdim;
-  float* sq = sm;                        // [TQ][D]
-  float* sk = sq + TQ * D;               // [TQ][D + 1]
-  float* sv = sk + TQ * (D + 1);         // [TQ][E]
-  float* so = sv + TQ * E;               // [TQ][E]
-  float* sp = so + TQ * E;               // [TQ][TQ + 1]
-  float* s_m = sp + TQ * (TQ + 1);       // [TQ] running maximum, sum, rescale factor
-  float* s_l = s_m + TQ;
-  float* s_a = s_l + TQ;
-  pdl_wait();
-  pdl_trigger();
-  const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * TQ, h = blockIdx.y;     // longest rows first
-  const int rows = min(TQ, p.T - q0);
-  const long long b = blockIdx.z;
-  const T* Q = reinterpret_cast<const T*>(p.q) + b * p.q_b + (long long)h * D;
-  const T* KV = reinterpret_cast<const T*>(p.kv) + b * p.kv_b;
-  const T* KR = reinterpret_cast<const T*>(p.kr) + b * p.kr_b;
-  for (int i = threadIdx.x; i < TQ * D; i += 256) {
-    const int t = i / D;
-    sq[i] = t < rows ? Cvt<T>::to(Q[(long long)(q0 + t) * p.q_ld + i % D]) * p.scale : 0.f;
-  }
-  for (int i = threadIdx.x; i < TQ * E; i += 256) so[i] = 0.f;
-  if (threadIdx.x < TQ) { s_m[threadIdx.x] = -INFINITY; s_l[threadIdx.x] = 0.f; }
-  const int n_keys = p.past + q0 + rows;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int k0 = 0; k0 < n_keys; k0 += TQ) {
-    const int nk = min(TQ, n_keys - k0);
-    __syncthreads();
-    for (int i = threadIdx.x; i < nk * D; i += 256) {
-      const int j = i / D, c = i % D;
-      sk[j * (D + 1) + c] = c < p.dim ? Cvt<T>::to(KV[(long long)(k0 + j) * p.kv_ld + h * p.dim + c]) : Cvt<T>::to(KR[(long long)(k0 + j) * p.kr_ld + c - p.dim]);
-    }
-    for (int i = threadIdx.x; i < nk * E; i += 256) sv[i] = Cvt<T>::to(KV[(long long)(k0 + i / E) * p.kv_ld + p.v_off + h * E + i % E]);
-    __syncthreads();
-    for (int i = threadIdx.x; i < TQ * TQ; i += 256) {
-      const int t = i / TQ, j = i % TQ;
-      float v = -INFINITY;
-      if (t < rows && j < nk && k0 + j <= p.past + q0 + t) {
-        v = 0.f;
-        for (int c = 0; c < D; c++) v = fmaf(sq[t * D + c], sk[j * (D + 1) + c], v);
-      }
-      sp[t * (TQ + 1) + j] = v;
-    }
-    __syncthreads();
-    for (int t = warp; t < rows; t += 8) {
-      const float v = lane < TQ ? sp[t * (TQ + 1) + lane] : -INFINITY;
-      const float m1 = fmaxf(s_m[t], warp_max(v));
-      const float e = v == -INFINITY ? 0.f : expf(v - m1);
-      const float sum = warp_sum(e);
-      if (lane < TQ) sp[t * (TQ + 1) + lane] = e;
-      __syncwarp();
-      if (lane == 0) {
-        const float a = m1 == -INFINITY ? 1.f : expf(s_m[t] - m1);
-        s_a[t] = a; s_l[t] = s_l[t] * a + sum; s_m[t] = m1;
-      }
-    }
-    __syncthreads();
-    for (int i = threadIdx.x; i < rows * E; i += 256) {
-      const int t = i / E, e = i % E;
-      float a = so[i] * s_a[t];
-      for (int j = 0; j < nk; j++) a = fmaf(sp[t * (TQ + 1) + j], sv[j * E + e], a);
-      so[i] = a;
-    }
-  }
-  __syncthreads();
-  T* Y = reinterpret_cast<T*>(p.y) + b * p.y_b + (long long)h * E;
-  for (int i = threadIdx.x; i < rows * E; i += 256) Y[(long long)(q0 + i / E) * p.y_ld + i % E] = Cvt<T>::from(so[i] / s_l[i / E]);
-}
-
-template <typename T, int TQ>
-static cudaError_t launch_lp(cudaStream_t s, const LpParams& p, int n_seq, size_t smem) {
-  static bool attr = false;
-  if (!attr) {
-    cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel<T, TQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
-    if (e != cudaSuccess) return e;
-    attr = true;
-  }
-  return launch_pdl(latent_prefill_kernel<T, TQ>, dim3((unsigned)((p.T + TQ - 1) / TQ), (unsigned)p.heads, (unsigned)n_seq), dim3(256), smem, s, p);
-}
-
-Status latent_prefill(cudaStream_t s, const LatentPrefillDesc& d) {
-  if (d.T < 1 || d.past < 0 || d.heads < 1 || d.heads > 65535 || d.dim < 1 || d.rot_dim < 0 || d.vdim < 1 || !d.q || !d.kv || !d.y || d.n_seq < 1 || d.n_seq > 65535)
-    return Status::invalid("latent prefill: bad description");
-  if (latent_prefill_tc_eligible(d)) return latent_prefill_tc(s, d);
-  LpParams p;
-  p.q = d.q; p.kv = d.kv; p.kr = d.k_rot; p.y = d.y; p.q_ld = d.q_ld; p.kv_ld = d.kv_ld; p.v_off = d.v_off; p.kr_ld = d.k_rot_ld; p.y_ld = d.y_ld;
-  p.q_b = d.q_b; p.kv_b = d.kv_b; p.kr_b = d.k_rot_b; p.y_b = d.y_b;
-  p.T = d.T; p.past = d.past; p.heads = d.heads; p.dim = d.dim; p.rot = d.rot_dim; p.vdim = d.vdim; p.scale = d.scale;
-  auto smem = [&](int tq) { return ((size_t)tq * (2 * (d.dim + d.rot_dim) + 1) + 2 * (size_t)tq * d.vdim + (size_t)tq * (tq + 1) + 3 * tq) * sizeof(float); };
-  const size_t lim = 220 * 1024;
-  if (smem(8) > lim) return Status::unsupported("latent prefill: head too large");
-  cudaError_t e = cudaSuccess;
-  AG_DISPATCH_FLOAT(d.dtype, T, (e = smem(32) <= lim ? launch_lp<T, 32>(s, p, d.n_seq, smem(32)) : smem(16) <= lim ? launch_lp<T, 16>(s, p, d.n_seq, smem(16)) : launch_lp<T, 8>(s, p, d.n_seq, smem(8))));
-  return cuda_status(e, "latent prefill");
 }
 
 // ── decode ──────────────────────────────────────────────────────────────────
@@ -364,13 +257,6 @@ constexpr int kLmKeys = 64, kLmHeads = 16;
 __host__ __device__ inline int lm_k(int cld) { return (cld + 31) / 32 * 32; }
 __host__ __device__ inline int lm_pitch(int cld) { const int p = lm_k(cld) / 8; return (p % 2 ? p : p + 1) * 8; }   // odd number of 16-byte pieces: no bank conflicts
 static size_t lm_smem(int cld) { return ((size_t)kLmKeys + 2 * kLmHeads) * lm_pitch(cld) * 2 + (size_t)kLmHeads * (kLmKeys + 1) * 4 + 2 * (size_t)kLmHeads * (kLmKeys + 8) * 2 + 4 * kLmHeads * 4; }
-__device__ __forceinline__ uint32_t lm_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
 template <typename T, int NW>          // NW: 8-column latent tiles per warp, rank <= 64 * NW
 __global__ void __launch_bounds__(256) latent_decode_attend_mma_kernel(const LaParams p) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -421,7 +307,7 @@ __global__ void __launch_bounds__(256) latent_decode_attend_mma_kernel(const LaP
     for (int i = threadIdx.x; i < kLmKeys * pieces; i += 256) {
       const int j = i / pieces, c = i % pieces * 8;
       T* dst = sk + j * P + c;
-      if (j < nk) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(lm_addr(dst)), "l"(cache + (long long)(k0 + j) * p.cld + c));
+      if (j < nk) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(dst)), "l"(cache + (long long)(k0 + j) * p.cld + c));
       else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -430,8 +316,8 @@ __global__ void __launch_bounds__(256) latent_decode_attend_mma_kernel(const LaP
     {
       // scores: 16 heads x 8 keys per warp
       float c4[4] = {0.f, 0.f, 0.f, 0.f};
-      const uint32_t qa = lm_addr(sqh + (lane & 15) * P + (lane >> 4) * 8), la = lm_addr(sql + (lane & 15) * P + (lane >> 4) * 8);
-      const uint32_t ka = lm_addr(sk + (warp * 8 + (lane & 7)) * P + (lane >> 3) * 8);
+      const uint32_t qa = smem_addr(sqh + (lane & 15) * P + (lane >> 4) * 8), la = smem_addr(sql + (lane & 15) * P + (lane >> 4) * 8);
+      const uint32_t ka = smem_addr(sk + (warp * 8 + (lane & 7)) * P + (lane >> 3) * 8);
       for (int kk = 0; kk < K; kk += 32) {
         uint32_t b[4], a0[4], a1[4];
         ldsm_x4(b, ka + kk * 2);
@@ -470,7 +356,7 @@ __global__ void __launch_bounds__(256) latent_decode_attend_mma_kernel(const LaP
       const float f0 = sm_a[g], f1 = sm_a[g + 8];
 #pragma unroll
       for (int j = 0; j < NW; j++) { o[j][0] *= f0; o[j][1] *= f0; o[j][2] *= f1; o[j][3] *= f1; }
-      const uint32_t pa = lm_addr(sph + (lane & 15) * (kLmKeys + 8) + (lane >> 4) * 8), pl = lm_addr(spl + (lane & 15) * (kLmKeys + 8) + (lane >> 4) * 8);
+      const uint32_t pa = smem_addr(sph + (lane & 15) * (kLmKeys + 8) + (lane >> 4) * 8), pl = smem_addr(spl + (lane & 15) * (kLmKeys + 8) + (lane >> 4) * 8);
 #pragma unroll
       for (int kk = 0; kk < kLmKeys; kk += 32) {
         uint32_t h0a[4], h1a[4], l0a[4], l1a[4];
@@ -481,7 +367,7 @@ __global__ void __launch_bounds__(256) latent_decode_attend_mma_kernel(const LaP
           const int c = (j * 8 + warp) * 8;
           if (c >= p.rank) break;
           uint32_t b[4];                               // keys kk .. kk + 31 of eight latent columns
-          ldsm_x4_t(b, lm_addr(sk + (kk + lane) * P + c));
+          ldsm_x4_t(b, smem_addr(sk + (kk + lane) * P + c));
           mma_16816<T>(o[j], h0a[0], h0a[1], h0a[2], h0a[3], b[0], b[1]);
           mma_16816<T>(o[j], h1a[0], h1a[1], h1a[2], h1a[3], b[2], b[3]);
           mma_16816<T>(o[j], l0a[0], l0a[1], l0a[2], l0a[3], b[0], b[1]);

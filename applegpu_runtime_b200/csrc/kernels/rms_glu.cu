@@ -1,4 +1,4 @@
-// RMS norms over a float32 residual stream and the clamped gated activation of a feed-forward.
+// RMS norms over a float32 residual stream and the gated activations of a feed-forward.
 //
 // rms_rows is the only kernel that touches the stream between two layers: it starts it from the embedding table, adds
 // what a repeated pass adds ahead of its first layer (the embedding output and a step vector), and writes the two
@@ -11,11 +11,11 @@ namespace ag { namespace k {
 constexpr int kRmsThreads = 128;      // small blocks: many rows in flight per SM
 
 struct RmsParams {
-  float* x; const int32_t* tok; const void* embed; const float* step; const float* w1; const float* w2; const int32_t* row_map;
+  float* x; const int32_t* tok; const void* embed; const float* step; const float* post; const float* wp; const float* w1; const float* w2; const int32_t* row_map;
   void* out1; void* out2;
   long long ld1, ld2, embed_ld;
   int width, vocab, load_x, write_x;
-  float eps;
+  float eps, embed_scale;
 };
 
 // VEC elements per thread and access (4 when width and pitches allow it), NREG accesses kept in registers (wider rows are read
@@ -37,6 +37,19 @@ __global__ void __launch_bounds__(kRmsThreads) rms_rows_kernel(const RmsParams p
   float v[NREG][VEC];
   float sq = 0.f;
   const int packs = p.width / VEC;
+  const float* y = p.post ? p.post + src * p.width : nullptr;
+  float rs_y = 0.f;
+  if (y) {                                               // the sublayer's output meets the stream through a norm of its own
+    float sy = 0.f;
+    for (int i = threadIdx.x; i < packs; i += kRmsThreads) {
+      const int c = i * VEC;
+      if constexpr (VEC == 4) {
+        const float4 q = *reinterpret_cast<const float4*>(y + c);
+        sy = fmaf(q.x, q.x, fmaf(q.y, q.y, fmaf(q.z, q.z, fmaf(q.w, q.w, sy))));
+      } else sy = fmaf(y[c], y[c], sy);
+    }
+    rs_y = 1.0f / sqrtf(block_sum(sy, red) / (float)p.width + p.eps);
+  }
   auto fetch = [&](int i, float (&o)[VEC]) {
     const int c = i * VEC;
     if (p.load_x) {
@@ -52,7 +65,14 @@ __global__ void __launch_bounds__(kRmsThreads) rms_rows_kernel(const RmsParams p
       else if constexpr (VEC == 4) *reinterpret_cast<uint4*>(t) = *reinterpret_cast<const uint4*>(e + c);
       else t[0] = e[c];
 #pragma unroll
-      for (int j = 0; j < VEC; j++) o[j] += Cvt<T>::to(t[j]);
+      for (int j = 0; j < VEC; j++) o[j] += Cvt<T>::to(t[j]) * p.embed_scale;
+    }
+    if (y) {
+      float yv[VEC];
+      if constexpr (VEC == 4) { const float4 q = *reinterpret_cast<const float4*>(y + c); yv[0] = q.x; yv[1] = q.y; yv[2] = q.z; yv[3] = q.w; }
+      else yv[0] = y[c];
+#pragma unroll
+      for (int j = 0; j < VEC; j++) o[j] += yv[j] * rs_y * __ldg(p.wp + c + j);
     }
     if (p.step) {
 #pragma unroll
@@ -115,13 +135,13 @@ __global__ void __launch_bounds__(kRmsThreads) rms_rows_kernel(const RmsParams p
 
 Status rms_rows(cudaStream_t s, const RmsRowsDesc& d) {
   if (d.rows <= 0) return Status::OK();
-  if (d.width < 1 || !d.x || (d.embed && !d.tok) || (d.out1 && !d.w1) || (d.out2 && !d.w2)) return Status::invalid("rms_rows: missing operand");
+  if (d.width < 1 || !d.x || (d.embed && !d.tok) || (d.out1 && !d.w1) || (d.out2 && !d.w2) || (d.post && !d.post_w)) return Status::invalid("rms_rows: missing operand");
   if (d.row_map && (d.embed || d.step || !d.load_x)) return Status::invalid("rms_rows: a gathered row is read only");
   RmsParams p;
-  p.x = d.x; p.tok = d.tok; p.embed = d.embed; p.step = d.step; p.w1 = d.w1; p.w2 = d.w2; p.row_map = d.row_map;
+  p.x = d.x; p.tok = d.tok; p.embed = d.embed; p.step = d.step; p.post = d.post; p.wp = d.post_w; p.embed_scale = d.embed_scale; p.w1 = d.w1; p.w2 = d.w2; p.row_map = d.row_map;
   p.out1 = d.out1; p.out2 = d.out2; p.ld1 = d.ld1; p.ld2 = d.ld2; p.embed_ld = d.embed_ld;
-  p.width = d.width; p.vocab = d.vocab; p.load_x = d.load_x ? 1 : 0; p.write_x = (!d.load_x || d.embed || d.step) ? 1 : 0; p.eps = d.eps;
-  const bool vec = d.width % 4 == 0 && d.ld1 % 4 == 0 && d.ld2 % 4 == 0 && aligned16(d.x) && (!d.embed || (d.embed_ld % 4 == 0 && aligned16(d.embed))) && (!d.out1 || aligned16(d.out1)) && (!d.out2 || aligned16(d.out2));
+  p.width = d.width; p.vocab = d.vocab; p.load_x = d.load_x ? 1 : 0; p.write_x = (!d.load_x || d.embed || d.step || (d.post && !d.row_map)) ? 1 : 0; p.eps = d.eps;
+  const bool vec = d.width % 4 == 0 && d.ld1 % 4 == 0 && d.ld2 % 4 == 0 && aligned16(d.x) && (!d.post || aligned16(d.post)) && (!d.embed || (d.embed_ld % 4 == 0 && aligned16(d.embed))) && (!d.out1 || aligned16(d.out1)) && (!d.out2 || aligned16(d.out2));
   cudaError_t e = cudaSuccess;
   AG_DISPATCH_FLOAT(d.dtype, T, {
     const dim3 grid((unsigned)d.rows), block(kRmsThreads);
@@ -134,10 +154,10 @@ Status rms_rows(cudaStream_t s, const RmsRowsDesc& d) {
   return cuda_status(e, "rms_rows");
 }
 
-// ── clamped gated activation ────────────────────────────────────────────────
+// ── gated activation ────────────────────────────────────────────────
 // gate of column c at (c / block) * 2 * block + c % block, the value it gates `block` columns later
 template <typename T, int VEC>
-__global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ gu, long long ld_in, T* __restrict__ out, long long ld_out, long long rows, int ff, int block, float limit) {
+__global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ gu, long long ld_in, T* __restrict__ out, long long ld_out, long long rows, int ff, int block, int kind, float limit) {
   pdl_wait();
   pdl_trigger();
   const int packs = ff / VEC;
@@ -151,27 +171,27 @@ __global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ 
       Pack<T> o;
       float t[VEC];
 #pragma unroll
-      for (int j = 0; j < VEC; j++) t[j] = clamped_glu_f(Cvt<T>::to(a.v[j]), Cvt<T>::to(b.v[j]), limit);
+      for (int j = 0; j < VEC; j++) t[j] = glu_f(kind, Cvt<T>::to(a.v[j]), Cvt<T>::to(b.v[j]), limit);
       pack_from_floats<T>(o, t);
       st16(out + r * ld_out + c, o);
     } else {
-      out[r * ld_out + c] = Cvt<T>::from(clamped_glu_f(Cvt<T>::to(g[0]), Cvt<T>::to(g[block]), limit));
+      out[r * ld_out + c] = Cvt<T>::from(glu_f(kind, Cvt<T>::to(g[0]), Cvt<T>::to(g[block]), limit));
     }
   }
 }
 
-Status clamped_glu(cudaStream_t s, DType dt, const void* gu, int64_t ld_in, void* out, int64_t ld_out, int64_t rows, int ff, int block, float limit) {
+Status glu(cudaStream_t s, DType dt, const void* gu, int64_t ld_in, void* out, int64_t ld_out, int64_t rows, int ff, int block, Glu kind, float limit) {
   if (rows <= 0 || ff <= 0) return Status::OK();
-  if (block < 1) return Status::invalid("clamped_glu: block");
+  if (block < 1) return Status::invalid("glu: block");
   cudaError_t e = cudaSuccess;
   AG_DISPATCH_FLOAT(dt, T, {
     constexpr int N = Pack<T>::N;
     const bool vec = ff % N == 0 && block % N == 0 && ld_in % N == 0 && ld_out % N == 0 && aligned16(gu) && aligned16(out);
     const int64_t work = rows * (ff / (vec ? N : 1));
-    if (vec) e = launch_pdl(clamped_glu_kernel<T, N>, dim3((unsigned)grid_for(work, 256)), dim3(256), 0, s, (const T*)gu, (long long)ld_in, (T*)out, (long long)ld_out, (long long)rows, ff, block, limit);
-    else e = launch_pdl(clamped_glu_kernel<T, 1>, dim3((unsigned)grid_for(work, 256)), dim3(256), 0, s, (const T*)gu, (long long)ld_in, (T*)out, (long long)ld_out, (long long)rows, ff, block, limit);
+    if (vec) e = launch_pdl(glu_kernel<T, N>, dim3((unsigned)grid_for(work, 256)), dim3(256), 0, s, (const T*)gu, (long long)ld_in, (T*)out, (long long)ld_out, (long long)rows, ff, block, (int)kind, limit);
+    else e = launch_pdl(glu_kernel<T, 1>, dim3((unsigned)grid_for(work, 256)), dim3(256), 0, s, (const T*)gu, (long long)ld_in, (T*)out, (long long)ld_out, (long long)rows, ff, block, (int)kind, limit);
   });
-  return cuda_status(e, "clamped_glu");
+  return cuda_status(e, "glu");
 }
 
 }}  // namespace ag::k

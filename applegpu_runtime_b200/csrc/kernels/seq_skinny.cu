@@ -20,7 +20,7 @@ constexpr size_t kSsMaxSmem = 200 * 1024;
 struct SsSeg {
   const void* w; void* out; const float* norm_w;
   long long ld, out_ld;
-  int n, mode, block0;               // block0: first block of this segment
+  int n, mode, glu, block0;          // block0: first block of this segment
   float limit;
 };
 struct SsParams {
@@ -122,7 +122,7 @@ __global__ void __launch_bounds__(kSsThreads) seq_skinny_kernel(const SsParams p
 #pragma unroll
         for (int r = 0; r < GW; r++) {
           if (((m * GW + r) & 31) != lane || n0 + r >= sg.n) continue;
-          reinterpret_cast<T*>(sg.out)[row * sg.out_ld + n0 + r] = Cvt<T>::from(clamped_glu_f(acc[m][r], acc[m][GW + r], sg.limit));
+          reinterpret_cast<T*>(sg.out)[row * sg.out_ld + n0 + r] = Cvt<T>::from(glu_f(sg.glu, acc[m][r], acc[m][GW + r], sg.limit));
         }
       }
       continue;
@@ -145,7 +145,7 @@ __global__ void __launch_bounds__(kSsThreads) seq_skinny_kernel(const SsParams p
 // 16-byte piece of each of its two weight rows and of its input row: no shared memory and no shuffles in the loop. The
 // first pieces of the weights are requested before the programmatic dependency wait. The warps' sums meet in shared memory;
 // a product with few result columns and long rows spreads K over a cluster, whose sums meet over distributed shared memory.
-struct SmSeg { const void* w; const void* a; void* out; long long ld, a_ld, out_ld; int n, mode, block0; float limit; };
+struct SmSeg { const void* w; const void* a; void* out; long long ld, a_ld, out_ld; int n, mode, glu, block0; float limit; };
 struct SmParams { SmSeg seg[kSeqSegs]; int n_seg, rows, kp, ranks; };       // ranks: CTAs of a cluster along K
 
 template <typename T, int NT>        // NT groups of 8 input rows
@@ -234,7 +234,7 @@ __global__ void __launch_bounds__(kSsThreads) seq_skinny_mma_kernel(const SmPara
       if (m >= p.rows || c0 + n >= sg.n) continue;
       const float v = total(m, n);
       const long long o = (long long)m * sg.out_ld + c0 + n;
-      if (glu) reinterpret_cast<T*>(sg.out)[o] = Cvt<T>::from(clamped_glu_f(v, total(m, n + 8), sg.limit));
+      if (glu) reinterpret_cast<T*>(sg.out)[o] = Cvt<T>::from(glu_f(sg.glu, v, total(m, n + 8), sg.limit));
       else if (sg.mode == (int)SeqOut::Store) reinterpret_cast<T*>(sg.out)[o] = Cvt<T>::from(v);
       else if (sg.mode == (int)SeqOut::StoreF32) reinterpret_cast<float*>(sg.out)[o] = v;
       else reinterpret_cast<float*>(sg.out)[o] += v;
@@ -262,7 +262,7 @@ static Status seq_skinny_mma(cudaStream_t s, const SeqSkinnyDesc& d) {
     const SeqSeg& g = d.seg[i];
     if (!g.w || !g.out || !g.a || g.n < 1 || g.ld % 8 != 0 || g.ld < d.k || g.a_ld % 8 != 0 || g.a_ld < p.kp || !aligned16(g.w) || !aligned16(g.a)) return Status::invalid("seq_skinny: bad segment");
     SmSeg& q = p.seg[i];
-    q.w = g.w; q.a = g.a; q.out = g.out; q.ld = g.ld; q.a_ld = g.a_ld; q.out_ld = g.out_ld; q.n = g.n; q.mode = (int)g.mode; q.block0 = blocks; q.limit = g.limit;
+    q.w = g.w; q.a = g.a; q.out = g.out; q.ld = g.ld; q.a_ld = g.a_ld; q.out_ld = g.out_ld; q.n = g.n; q.mode = (int)g.mode; q.glu = (int)g.glu; q.block0 = blocks; q.limit = g.limit;
     const int per = g.mode == SeqOut::Glu ? 8 : 16;
     blocks += (g.n + per - 1) / per;
   }
@@ -308,7 +308,7 @@ Status seq_skinny(cudaStream_t s, const SeqSkinnyDesc& d) {
     const SeqSeg& g = d.seg[i];
     if (!g.w || !g.out || g.n < 1 || g.ld % 8 != 0 || g.ld < d.k || !aligned16(g.w) || (d.x && !g.norm_w)) return Status::invalid("seq_skinny: bad segment");
     SsSeg& q = p.seg[i];
-    q.w = g.w; q.out = g.out; q.norm_w = g.norm_w; q.ld = g.ld; q.out_ld = g.out_ld; q.n = g.n; q.mode = (int)g.mode; q.limit = g.limit; q.block0 = blocks;
+    q.w = g.w; q.out = g.out; q.norm_w = g.norm_w; q.ld = g.ld; q.out_ld = g.out_ld; q.n = g.n; q.mode = (int)g.mode; q.glu = (int)g.glu; q.limit = g.limit; q.block0 = blocks;
     const int per = (g.mode == SeqOut::Glu ? rw / 2 : rw) * kSsWarps;
     blocks += (g.n + per - 1) / per;
   }

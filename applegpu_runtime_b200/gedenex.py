@@ -6,24 +6,9 @@ weights are [out, in].
 """
 import numpy as np
 
-from .seqmodel import Layer, Rotary, SequenceModel, interleaved, rows, side_by_side
+from .seqmodel import Layer, SequenceModel, Tensors, interleaved, rotary_of, rows, side_by_side
 
 ARCHITECTURE = "Gedenex"
-
-
-class _Tensors:
-    """Looks weights up by name and checks their shapes."""
-
-    def __init__(self, weights):
-        self._w = weights
-
-    def get(self, name, *shape):
-        if name not in self._w:
-            raise ValueError(f"missing tensor {name}")
-        a = np.asarray(self._w[name], np.float32)
-        if a.shape != tuple(shape):
-            raise ValueError(f"tensor {name} has shape {list(a.shape)}, the configuration asks for {list(shape)}")
-        return a
 
 
 def _mlstm(t, p, m, width):
@@ -37,12 +22,9 @@ def _mlstm(t, p, m, width):
 def _latent_attention(t, p, m, width):
     H, d, rd, e, r = int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"])
     layer = Layer("latent_attention", heads=H, dim=d, vdim=e, rot_dim=rd, kv_rank=r, score_scale=float(m["scale"]))
-    rot = m.get("rot")
-    if rot:
-        scaling = rot.get("scaling")
-        layer.rotary = Rotary(int(rot["dims"]), float(rot["base"]), None if not scaling else {k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")})
-        if layer.rotary.dims > rd or layer.rotary.dims % 2:
-            raise ValueError(f"{p}: {layer.rotary.dims} rotated dimensions of {rd}")
+    layer.rotary = rotary_of(m.get("rot"))
+    if layer.rotary and (layer.rotary.dims > rd or layer.rotary.dims % 2):
+        raise ValueError(f"{p}: {layer.rotary.dims} rotated dimensions of {rd}")
     layer.w_in = rows(t.get(p + "q", H * (d + rd), width), t.get(p + "dkv", r + rd, width))
     layer.own = [t.get(p + "dkv.norm", r), rows(t.get(p + "uk", H * d, r), t.get(p + "uv", H * e, r), pad_rows=True), None]
     return layer
@@ -53,7 +35,7 @@ _MIXERS = {"mlstm": _mlstm, "latent_attention": _latent_attention}
 
 def load_gedenex(config, weights, dtype="bfloat16"):
     """A SequenceModel from the parsed config.json and {tensor name: array}."""
-    width, vocab, t = int(config["width"]), int(config["vocab"]), _Tensors(weights)
+    width, vocab, t = int(config["width"]), int(config["vocab"]), Tensors(weights)
     layers = []
     for i, c in enumerate(config["layers"]):
         if c["type"] not in _MIXERS:

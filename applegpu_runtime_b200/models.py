@@ -11,6 +11,7 @@ from .bert import BERT_BASE, load_bert_state_dict
 from .checkpoint import read_safetensors
 from .gedenex import ARCHITECTURE as _GEDENEX, load_gedenex
 from .gpt2 import load_gpt2_state_dict
+from .rurunex import ARCHITECTURE as _RURUNEX, load_rurunex
 
 _LOADERS = {}
 
@@ -56,3 +57,4 @@ for _n in ("gpt2", "GPT2LMHeadModel"):
 for _n in ("bert", "BertModel"):
     register(_n, _bert)
 register(_GEDENEX, load_gedenex)
+register(_RURUNEX, load_rurunex)

@@ -2,7 +2,7 @@
 
 A `SequenceModel` holds uploaded weights and the list of layers; `engine(slots, max_len)` gives them memory for that many
 sequences and runs prompt portions and generated tokens (csrc/core/seqmodel.cc). A model family is a module that turns
-its configuration and tensor names into one (`gedenex.py`); it packs the weights with the helpers here and adds nothing
+its configuration and tensor names into one (`gedenex.py`, `rurunex.py`); it packs the weights with the helpers here and adds nothing
 to the run time.
 """
 import ctypes
@@ -14,7 +14,10 @@ from . import _lib
 from . import api as gpu
 from .rotary import rotary_table
 
-MIXERS = {"mlstm": 1, "latent_attention": 2}
+MIXERS = {"mlstm": 1, "latent_attention": 2, "key_decay": 3, "grouped_attention": 4}
+FORMS = {"parallel": 0, "sequential": 1}
+GLUS = {"clamped": 0, "silu": 1}
+DELTA, UNIT, SOFTPLUS, GATE_SILU = 1, 2, 4, 8          # key_decay options
 
 
 def pad8(n):
@@ -22,12 +25,13 @@ def pad8(n):
 
 
 class _ModelDesc(ctypes.Structure):
-    _fields_ = [(n, ctypes.c_int32) for n in ("vocab", "width", "n_layers", "loop_start", "loop_stop", "loop_times")] + [("eps", ctypes.c_float)]
+    _fields_ = [(n, ctypes.c_int32) for n in ("vocab", "width", "n_layers", "loop_start", "loop_stop", "loop_times", "form")] + [("eps", ctypes.c_float), ("embed_scale", ctypes.c_float)]
 
 
 class _LayerDesc(ctypes.Structure):
-    _fields_ = ([(n, ctypes.c_int32) for n in ("mixer", "heads", "dim", "vdim", "rot_dim", "rot_pairs", "kv_rank", "ff")]
-                + [(n, ctypes.c_float) for n in ("gate_cap", "score_scale", "ff_limit")])
+    _fields_ = ([(n, ctypes.c_int32) for n in ("mixer", "heads", "dim", "vdim", "rot_dim", "rot_pairs", "kv_rank", "ff", "kv_heads", "window", "kv_from", "taps",
+                                                 "a_rank", "g_rank", "flags", "glu")]
+                + [(n, ctypes.c_float) for n in ("gate_cap", "score_scale", "ff_limit", "softcap", "tau")])
 
 
 @dataclass
@@ -50,14 +54,63 @@ class Layer:
     gate_cap: float = 0.0
     score_scale: float = 0.0
     rotary: Rotary = None
+    kv_heads: int = 0          # grouped_attention, key_decay
+    window: int = 0            # keys a token sees, 0: all
+    kv_from: int = -1          # layer whose keys and values are used, -1: its own
+    softcap: float = 0.0
+    taps: int = 0
+    a_rank: int = 0
+    g_rank: int = 0
+    flags: int = 0
+    tau: float = 1.0
     ff: int = 0
+    glu: str = "clamped"
     ff_limit: float = 0.0
     norm1: np.ndarray = None
     norm2: np.ndarray = None
     w_in: np.ndarray = None
     w_out: np.ndarray = None
     w_ff: np.ndarray = None
-    own: list = field(default_factory=lambda: [None, None, None])
+    post1: np.ndarray = None   # sequential layers: norms behind the sublayers, feed-forward output
+    post2: np.ndarray = None
+    w_down: np.ndarray = None
+    own: list = field(default_factory=lambda: [None] * 7)
+
+    def weights(self):
+        own = self.own + [None] * (7 - len(self.own))
+        return [self.norm1, self.norm2, self.w_in, self.w_out, self.w_ff, *own[:3], self.post1, self.post2, self.w_down, *own[3:]]
+
+
+LAYER_WEIGHTS, ROTATION = 15, 7        # records per layer, place of the rotation table among them
+
+
+class Tensors:
+    """Looks weights up by name and checks their shapes."""
+
+    def __init__(self, weights):
+        self._w = weights
+
+    def get(self, name, *shape):
+        if name not in self._w:
+            raise ValueError(f"missing tensor {name}")
+        a = np.asarray(self._w[name], np.float32)
+        if a.shape != tuple(shape):
+            raise ValueError(f"tensor {name} has shape {list(a.shape)}, the configuration asks for {list(shape)}")
+        return a
+
+    def rank(self, name):
+        """Number of rows of a matrix whose size only its shape tells."""
+        if name not in self._w:
+            raise ValueError(f"missing tensor {name}")
+        return int(np.shape(self._w[name])[0])
+
+
+def rotary_of(rot):
+    """The `Rotary` of a configuration's "rot" entry (dims, base, optional scaling), None without one."""
+    if not rot or not int(rot["dims"]):
+        return None
+    scaling = rot.get("scaling")
+    return Rotary(int(rot["dims"]), float(rot["base"]), None if not scaling else {k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")})
 
 
 def rows(*parts, pad_rows=False):
@@ -97,18 +150,19 @@ def side_by_side(first, second):
 
 
 class SequenceModel:
-    def __init__(self, vocab, width, eps, layers, embed, head, final_norm, loop=None, dtype="bfloat16", config=None):
-        """`loop`: (start, stop, step vectors [times, width]) or None. Arrays are float32; matrices are stored as `dtype`."""
+    def __init__(self, vocab, width, eps, layers, embed, head, final_norm, loop=None, dtype="bfloat16", config=None, form="parallel", embed_scale=1.0):
+        """`loop`: (start, stop, step vectors [times, width]) or None; `form`: how a layer's sublayers meet the stream
+        (csrc/core/seqmodel.cc). Arrays are float32; matrices are stored as `dtype`."""
         if dtype not in ("float32", "bfloat16", "float16"):
             raise ValueError(f"sequence models run in float32, bfloat16 or float16, not {dtype}")
         self.vocab, self.width, self.eps, self.dtype, self.layers, self.config = int(vocab), int(width), float(eps), dtype, layers, config
+        self.form, self.embed_scale = form, float(embed_scale)
         self.loop = None if loop is None else (int(loop[0]), int(loop[1]), int(loop[2].shape[0]))
         self._weights = [self._matrix(np.asarray(embed, np.float32)), self._matrix(rows(head)), self._vector(final_norm), self._vector(loop[2]) if loop else None]
         for l in layers:
-            self._weights += [self._vector(l.norm1), self._vector(l.norm2), self._matrix(l.w_in), self._matrix(l.w_out), self._matrix(l.w_ff)]
-            self._weights += [a if a is None else (self._matrix(a) if a.ndim == 2 else self._vector(a)) for a in l.own]
-            l.norm1 = l.norm2 = l.w_in = l.w_out = l.w_ff = None      # uploaded
-            l.own = [None, None, None]
+            self._weights += [a if a is None else (self._matrix(a) if a.ndim == 2 else self._vector(a)) for a in l.weights()]
+            l.norm1 = l.norm2 = l.w_in = l.w_out = l.w_ff = l.post1 = l.post2 = l.w_down = None      # uploaded
+            l.own = []
 
     @staticmethod
     def _vector(a):
@@ -135,7 +189,7 @@ class SequenceEngine:
         self._lib = _lib.load()
         self.model, self.slots, self.max_len = model, int(slots), int(max_len)
         tables, w = {}, list(model._weights)
-        desc = _ModelDesc(model.vocab, model.width, len(model.layers), *(model.loop or (0, 0, 0)), model.eps)
+        desc = _ModelDesc(model.vocab, model.width, len(model.layers), *(model.loop or (0, 0, 0)), FORMS[model.form], model.eps, model.embed_scale)
         arr = (_LayerDesc * len(model.layers))()
         for i, l in enumerate(model.layers):
             pairs = 0
@@ -144,8 +198,9 @@ class SequenceEngine:
                 key = (l.rotary.dims, l.rotary.base, tuple(sorted((l.rotary.scaling or {}).items())))
                 if key not in tables:
                     tables[key] = gpu.from_numpy(rotary_table(self.max_len, l.rotary.dims, l.rotary.base, l.rotary.scaling))
-                w[4 + 8 * i + 7] = tables[key]
-            arr[i] = _LayerDesc(MIXERS[l.mixer], l.heads, l.dim, l.vdim, l.rot_dim, pairs, l.kv_rank, l.ff, l.gate_cap, l.score_scale, l.ff_limit)
+                w[4 + LAYER_WEIGHTS * i + ROTATION] = tables[key]
+            arr[i] = _LayerDesc(MIXERS[l.mixer], l.heads, l.dim, l.vdim, l.rot_dim, pairs, l.kv_rank, l.ff, l.kv_heads, l.window, l.kv_from, l.taps,
+                                l.a_rank, l.g_rank, l.flags, GLUS[l.glu], l.gate_cap, l.score_scale, l.ff_limit, l.softcap, l.tau)
         self._keep = w
         ids = (ctypes.c_uint64 * len(w))(*[0 if t is None else t.id for t in w])
         self.handle = int(self._lib.applegpu_seq_create(ctypes.byref(desc), arr, ids, len(w), self.slots, self.max_len))

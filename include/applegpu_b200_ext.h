@@ -312,10 +312,10 @@ APPLEGPU_API void applegpu_gpt2_decoder_destroy(uint64_t decoder);
  *            sequence; host_tokens [n_steps, n_seq]. use_graph replays one captured step per token.
  *   reset:   empties n slots. length: tokens a slot holds. info: 0 launches of the last one-token step, 1 whether it was
  *            replayed as a graph, 2 layer runs. */
-typedef struct { int32_t vocab, width, n_layers, loop_start, loop_stop, loop_times; float eps; } applegpu_seq_model;
+typedef struct { int32_t vocab, width, n_layers, loop_start, loop_stop, loop_times, form; float eps, embed_scale; } applegpu_seq_model;
 typedef struct {
-  int32_t mixer, heads, dim, vdim, rot_dim, rot_pairs, kv_rank, ff;
-  float gate_cap, score_scale, ff_limit;
+  int32_t mixer, heads, dim, vdim, rot_dim, rot_pairs, kv_rank, ff, kv_heads, window, kv_from, taps, a_rank, g_rank, flags, glu;
+  float gate_cap, score_scale, ff_limit, softcap, tau;
 } applegpu_seq_layer;
 APPLEGPU_API uint64_t applegpu_seq_create(const applegpu_seq_model* model, const applegpu_seq_layer* layers, const uint64_t* weight_ids, uint32_t n_weights, uint32_t slots, uint32_t max_len);
 APPLEGPU_API int32_t applegpu_seq_forward(uint64_t engine, uint32_t slot0, uint32_t n_seq, const int32_t* tokens, uint32_t n_tokens, const int32_t* want, uint32_t n_want,
