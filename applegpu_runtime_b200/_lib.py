@@ -206,6 +206,11 @@ EXT_SYMBOLS = {
     "applegpu_seq_destroy": (None, [u64]),
     "applegpu_ffi_rms_norm": (u64, [u64, u64, f32, i8]),
     "applegpu_ffi_clamped_glu": (u64, [u64, f32]),
+    "applegpu_ffi_silu_glu": (u64, [u64]),
+    "applegpu_ffi_rms_add": (u64, [u64, u64, u64, u64, f32, i8]),
+    "applegpu_key_decay_mem_bytes": (u64, [vp, i8]),
+    "applegpu_ffi_key_decay": (u64, [u64] * 10 + [vp, i32]),
+    "applegpu_ffi_grouped_attention": (u64, [u64] * 6 + [u32, vp, i32]),
     "applegpu_ffi_mlstm": (u64, [u64, u64, u64, u64, u64, u32, u32, u32, f32, f32, i32]),
     "applegpu_ffi_latent_attention": (u64, [u64, u64, u64, u64, u64, u64, u32, u32, u32, u32, u32, u32, f32, f32, i32]),
     "applegpu_test_wait_runs_out": (i32, [i32, u32]),

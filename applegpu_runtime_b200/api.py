@@ -446,6 +446,49 @@ def clamped_glu(gate_up, limit):
     return GpuTensor(_L().applegpu_ffi_clamped_glu(gate_up.id, float(limit)))
 
 
+def silu_glu(gate_up):
+    """[.., 2 n] (gate | up) -> gate sigmoid(gate) up."""
+    return GpuTensor(_L().applegpu_ffi_silu_glu(gate_up.id))
+
+
+def rms_add(x, y, post, weight, eps=1e-5, dtype="bfloat16"):
+    """x += y / rms(y) * post in place (float32); returns x / rms(x) * weight stored as `dtype`."""
+    return GpuTensor(_L().applegpu_ffi_rms_add(x.id, y.id, post.id, weight.id, float(eps), _DTYPE_CODES[_canon_dtype(dtype)]))
+
+
+class _KeyDecayDesc(ctypes.Structure):
+    _fields_ = [(n, ctypes.c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "taps", "a_rank", "g_rank", "flags")] + [(n, ctypes.c_float) for n in ("tau", "eps")]
+
+
+class _GroupedAttentionDesc(ctypes.Structure):
+    _fields_ = [(n, ctypes.c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "window", "shared")] + [(n, ctypes.c_float) for n in ("scale", "softcap", "eps")]
+
+
+def key_decay_memory(B, dtype, heads, kv_heads, dim, vdim, taps=0):
+    """Zeroed memory of B new sequences for `key_decay`: float32 [B, n], the state (heads * dim * vdim) first."""
+    d = _KeyDecayDesc(heads, kv_heads, dim, vdim, taps, 1, 0, 0, 1.0, 0.0)
+    return from_numpy(np.zeros((B, int(_L().applegpu_key_decay_mem_bytes(ctypes.byref(d), _DTYPE_CODES[_canon_dtype(dtype)])) // 4), np.float32))
+
+
+def key_decay(proj, a2, bias, norm, mem, pos, heads, kv_heads, dim, vdim, a_rank, g_rank=0, flags=0, taps=0, tau=1.0, eps=1e-5, beta=None, g2=None, rate=None, conv=None, form="auto"):
+    """Matrix states with one decay per key channel over proj [B, T, cols] (q | k | v | a1 | gate or g1, each part padded to a
+    multiple of 8 columns); flags: seqmodel.DELTA, UNIT, SOFTPLUS, GATE_SILU. `mem` is updated in place, `pos` (int32 [B]) says how
+    many tokens it holds. form: "auto" (chunks for longer 16-bit portions), "steps" (token by token). Returns [B, T, heads * vdim]."""
+    d = _KeyDecayDesc(heads, kv_heads, dim, vdim, taps, a_rank, g_rank, flags, float(tau), float(eps))
+    ids = [0 if t is None else t.id for t in (proj, beta, a2, bias, norm, g2, rate, conv, mem, pos)]
+    return GpuTensor(_L().applegpu_ffi_key_decay(*ids, ctypes.byref(d), {"auto": 0, "steps": 1}[form]))
+
+
+def grouped_attention(proj, q_norm, k_norm, rot_table, cache, pos, past, heads, kv_heads, dim, vdim, scale, softcap=0.0, window=0, shared=False, eps=1e-5, form="portion"):
+    """Causal attention of T new rows per sequence over a cache of normed, turned keys and plain values, query heads in groups. proj
+    [B, T, cols] holds q | k | v (q only when `shared`: the cache holds these tokens already), each part padded to a multiple of 8
+    columns; queries are normed and turned in place. form: "portion", "short" (splits of the keys), "tensor" (portion on the
+    tensor-core kernel or an error). Returns [B, T, heads * vdim]."""
+    d = _GroupedAttentionDesc(heads, kv_heads, dim, vdim, window, int(shared), float(scale), float(softcap), float(eps))
+    return GpuTensor(_L().applegpu_ffi_grouped_attention(proj.id, q_norm.id, 0 if k_norm is None else k_norm.id, 0 if rot_table is None else rot_table.id, cache.id, pos.id, int(past),
+                                                         ctypes.byref(d), {"portion": 0, "short": 1, "tensor": 2}[form]))
+
+
 def mlstm(proj, gates, gate_bias, norm, state, heads, dim, vdim, gate_cap, eps=1e-5, form="chunked"):
     """The mLSTM recurrence over proj [B, T, cols] (q | k | v | output gate) and float32 gates [B, T, 2 heads] (input | forget,
     without bias); `state` (float32 [B, n]) is updated in place. form: "chunked", "steps" (token by

@@ -1446,8 +1446,8 @@ uint64_t applegpu_ffi_rms_norm(uint64_t x_id, uint64_t weight_id, float eps, int
   const Status s = run();
   return immediate_result("rms_norm", st.rt, s, out);
 }
-uint64_t applegpu_ffi_clamped_glu(uint64_t gate_up_id, float limit) {
-  if (!ffi_ready("clamped_glu")) return 0;
+static uint64_t gated(const char* what, uint64_t gate_up_id, k::Glu kind, float limit) {
+  if (!ffi_ready(what)) return 0;
   LazyState& st = lazy_state();
   std::lock_guard<std::mutex> g(st.mu);
   TensorRec t, out;
@@ -1458,11 +1458,12 @@ uint64_t applegpu_ffi_clamped_glu(uint64_t gate_up_id, float limit) {
     const int64_t c = o.back(), rows = numel_of(o) / (c ? c : 1);
     o.back() = c / 2;
     AG_RETURN_IF_ERROR(new_tensor(o, t.dtype, &out));
-    return k::glu(DeviceCtx::get().stream, t.dtype, t.data(), c, out.data(), c / 2, rows, (int)(c / 2), (int)(c / 2), k::Glu::Clamped, limit);
+    return k::glu(DeviceCtx::get().stream, t.dtype, t.data(), c, out.data(), c / 2, rows, (int)(c / 2), (int)(c / 2), kind, limit);
   };
   const Status s = run();
-  return immediate_result("clamped_glu", st.rt, s, out);
+  return immediate_result(what, st.rt, s, out);
 }
+uint64_t applegpu_ffi_clamped_glu(uint64_t gate_up_id, float limit) { return gated("clamped_glu", gate_up_id, k::Glu::Clamped, limit); }
 uint64_t applegpu_ffi_mlstm(uint64_t proj_id, uint64_t gates_id, uint64_t gate_bias_id, uint64_t norm_id, uint64_t state_id, uint32_t heads, uint32_t dim, uint32_t vdim,
                             float gate_cap, float eps, int32_t form) {
   if (!ffi_ready("mlstm")) return 0;
@@ -1540,6 +1541,113 @@ uint64_t applegpu_ffi_latent_attention(uint64_t proj_id, uint64_t norm_id, uint6
   };
   const Status s = run();
   return immediate_result("latent_attention", st.rt, s, out);
+}
+
+uint64_t applegpu_ffi_silu_glu(uint64_t gate_up_id) { return gated("silu_glu", gate_up_id, k::Glu::Silu, 0.f); }
+uint64_t applegpu_ffi_rms_add(uint64_t x_id, uint64_t y_id, uint64_t post_id, uint64_t weight_id, float eps, int8_t out_dtype) {
+  if (!ffi_ready("rms_add")) return 0;
+  LazyState& st = lazy_state();
+  std::lock_guard<std::mutex> g(st.mu);
+  const uint64_t ids[4] = {x_id, y_id, post_id, weight_id};
+  TensorRec t[4], out;
+  DType dt = DType::Invalid;
+  auto run = [&]() -> Status {
+    AG_RETURN_IF_ERROR(immediate_operands(st.rt, ids, t, 4));
+    if (!dtype_from_wire(out_dtype, &dt)) return Status::invalid("unknown dtype");
+    if (t[0].shape.empty() || t[1].shape != t[0].shape || numel_of(t[2].shape) != t[0].shape.back() || numel_of(t[3].shape) != t[0].shape.back()) return Status::invalid("operand shapes");
+    for (const TensorRec& q : t) if (q.dtype != DType::F32) return Status::invalid("float32 operands");
+    const int64_t wd = t[0].shape.back();
+    AG_RETURN_IF_ERROR(new_tensor(t[0].shape, dt, &out));
+    k::RmsRowsDesc d;
+    d.dtype = dt; d.x = static_cast<float*>(t[0].data()); d.rows = numel_of(t[0].shape) / wd; d.width = (int)wd; d.eps = eps;
+    d.post = static_cast<const float*>(t[1].data()); d.post_w = static_cast<const float*>(t[2].data());
+    d.w1 = static_cast<const float*>(t[3].data()); d.out1 = out.data(); d.ld1 = wd;
+    return k::rms_rows(DeviceCtx::get().stream, d);
+  };
+  const Status s = run();
+  return immediate_result("rms_add", st.rt, s, out);
+}
+uint64_t applegpu_key_decay_mem_bytes(const applegpu_key_decay_desc* c, int8_t dtype) {
+  DType dt = DType::Invalid;
+  return c && dtype_from_wire(dtype, &dt) ? k::key_decay_mem_bytes(dt, c->heads, c->kv_heads, c->dim, c->vdim, c->taps) : 0;
+}
+uint64_t applegpu_ffi_key_decay(uint64_t proj_id, uint64_t beta_id, uint64_t a2_id, uint64_t bias_id, uint64_t norm_id, uint64_t g2_id, uint64_t rate_id, uint64_t conv_id,
+                                uint64_t mem_id, uint64_t pos_id, const applegpu_key_decay_desc* c, int32_t form) {
+  if (!ffi_ready("key_decay")) return 0;
+  if (!c) { set_ffi_error("key_decay failed: null argument"); return 0; }
+  LazyState& st = lazy_state();
+  std::lock_guard<std::mutex> g(st.mu);
+  const uint64_t ids[10] = {proj_id, beta_id, a2_id, bias_id, norm_id, g2_id, rate_id, conv_id, mem_id, pos_id};
+  TensorRec t[10], out, work;
+  auto run = [&]() -> Status {
+    AG_RETURN_IF_ERROR(immediate_operands(st.rt, ids, t, 10));
+    const int64_t H = c->heads, G = c->kv_heads, D = c->dim, E = c->vdim;
+    if (t[0].shape.size() != 3 || H < 1 || G < 1 || H % G || D < 1 || E < 1 || c->taps < 0 || c->a_rank < 1 || c->g_rank < 0) return Status::invalid("proj must be [sequences, tokens, columns]");
+    const int64_t B = t[0].shape[0], T = t[0].shape[1], qk = k::pad8(G * D), v = k::pad8(H * E), ar = k::pad8(c->a_rank);
+    const DType dt = t[0].dtype;
+    k::KeyDecayDesc d;
+    d.dtype = dt; d.n_seq = (int)B; d.T = (int)T; d.heads = (int)H; d.qk_heads = (int)G; d.dim = (int)D; d.vdim = (int)E;
+    d.delta = c->flags & kKdDelta; d.unit = c->flags & kKdUnit; d.softplus = c->flags & kKdSoftplus; d.gate_silu = c->flags & kKdGateSilu;
+    d.taps = c->taps; d.tau = c->tau; d.q_scale = (float)(1.0 / std::sqrt((double)D)); d.eps = c->eps;
+    d.q_off = 0; d.k_off = (int)qk; d.v_off = (int)(2 * qk); d.a_off = (int)(2 * qk + v); d.a_rank = c->a_rank; d.g_off = (int)(2 * qk + v + ar); d.g_rank = c->g_rank;
+    const int64_t mem = (int64_t)k::key_decay_mem_bytes(dt, (int)H, (int)G, (int)D, (int)E, c->taps), channels = k::key_decay_channels((int)H, (int)G, (int)D, (int)E);
+    auto vec = [&](const TensorRec& x, int64_t n) { return x.buf && x.dtype == DType::F32 && numel_of(x.shape) == n; };
+    if (t[0].shape[2] < 2 * qk + v + ar + (c->g_rank ? c->g_rank : H * E) || t[0].shape[2] % 8 || (d.delta && !vec(t[1], B * T * H)) || t[2].dtype != dt || t[2].shape != Dims{H * D, ar} ||
+        !vec(t[3], H * D) || !vec(t[4], E) || (c->g_rank && (t[5].dtype != dt || t[5].shape != Dims{H * E, k::pad8(c->g_rank)})) || (d.softplus && !vec(t[6], H)) ||
+        (c->taps && !vec(t[7], channels * c->taps)) || !vec(t[8], B * mem / 4) || t[9].dtype != DType::I32 || numel_of(t[9].shape) != B)
+      return Status::invalid("operand shapes or dtypes");
+    AG_RETURN_IF_ERROR(new_tensor({B, T, H * E}, dt, &out));
+    auto f = [](const TensorRec& x) { return static_cast<const float*>(x.data()); };
+    d.proj = t[0].data(); d.ld = t[0].shape[2]; d.beta = d.delta ? f(t[1]) : nullptr; d.beta_ld = H; d.a2 = t[2].data(); d.bias = f(t[3]); d.norm = f(t[4]);
+    d.g2 = c->g_rank ? t[5].data() : nullptr; d.rate = d.softplus ? f(t[6]) : nullptr; d.conv = c->taps ? f(t[7]) : nullptr;
+    d.mem = t[8].data(); d.mem_stride = mem; d.pos = static_cast<const int*>(t[9].data()); d.y = out.data(); d.y_ld = H * E; d.simple = form == 1;
+    const size_t wb = k::key_decay_work_bytes(d);
+    if (wb) { AG_RETURN_IF_ERROR(new_tensor({(int64_t)wb}, DType::U8, &work)); d.work = work.data(); }
+    int launches = 0;
+    return k::key_decay(DeviceCtx::get().stream, d, &launches);
+  };
+  const Status s = run();
+  return immediate_result("key_decay", st.rt, s, out);
+}
+uint64_t applegpu_ffi_grouped_attention(uint64_t proj_id, uint64_t q_norm_id, uint64_t k_norm_id, uint64_t rot_id, uint64_t cache_id, uint64_t pos_id, uint32_t past,
+                                        const applegpu_grouped_attention_desc* c, int32_t form) {
+  if (!ffi_ready("grouped_attention")) return 0;
+  if (!c) { set_ffi_error("grouped_attention failed: null argument"); return 0; }
+  LazyState& st = lazy_state();
+  std::lock_guard<std::mutex> g(st.mu);
+  const uint64_t ids[6] = {proj_id, q_norm_id, k_norm_id, rot_id, cache_id, pos_id};
+  TensorRec t[6], out;
+  auto run = [&]() -> Status {
+    AG_RETURN_IF_ERROR(immediate_operands(st.rt, ids, t, 6));
+    const int64_t H = c->heads, G = c->kv_heads, D = c->dim, E = c->vdim;
+    if (t[0].shape.size() != 3 || t[4].shape.size() != 3 || H < 1 || G < 1 || H % G || D < 1 || E < 1) return Status::invalid("proj [sequences, tokens, columns], cache [sequences, positions, columns]");
+    const int64_t B = t[0].shape[0], T = t[0].shape[1], q = k::pad8(H * D), kk = k::pad8(G * D), cld = k::grouped_cache_ld((int)G, (int)D, (int)E);
+    const DType dt = t[0].dtype;
+    if (t[0].shape[2] < q + (c->shared ? 0 : kk + G * E) || t[4].shape[0] != B || t[4].shape[2] != cld || (int64_t)past + T > t[4].shape[1] || numel_of(t[1].shape) != D ||
+        (!c->shared && numel_of(t[2].shape) != D) || numel_of(t[5].shape) != B)
+      return Status::invalid("operand shapes");
+    if (t[1].dtype != DType::F32 || (!c->shared && t[2].dtype != DType::F32) || t[4].dtype != dt || t[5].dtype != DType::I32) return Status::invalid("operand dtypes");
+    if (t[3].buf && (t[3].dtype != DType::F32 || t[3].shape.size() != 3 || t[3].shape[0] < t[4].shape[1] || t[3].shape[2] != 2)) return Status::invalid("rotation table");
+    AG_RETURN_IF_ERROR(new_tensor({B, T, H * E}, dt, &out));
+    const size_t esz = dtype_size(dt);
+    cudaStream_t cs = DeviceCtx::get().stream;
+    k::GroupedAttnDesc d;
+    d.dtype = dt; d.n_seq = (int)B; d.T = (int)T; d.heads = (int)H; d.kv_heads = (int)G; d.dim = (int)D; d.vdim = (int)E; d.rot_pairs = t[3].buf ? (int)t[3].shape[1] : 0; d.window = c->window;
+    d.shared = c->shared != 0; d.scale = c->scale; d.softcap = c->softcap; d.eps = c->eps; d.proj = t[0].data(); d.ld = t[0].shape[2]; d.k_off = (int)q; d.v_off = (int)(q + kk);
+    d.q_norm = static_cast<const float*>(t[1].data()); d.k_norm = c->shared ? nullptr : static_cast<const float*>(t[2].data());
+    d.rot_table = static_cast<const float2*>(t[3].data()); d.cache = t[4].data(); d.seq_stride = t[4].shape[1] * cld; d.pos = static_cast<const int*>(t[5].data());
+    d.max_len = (int)t[4].shape[1]; d.y = out.data(); d.y_ld = H * E;
+    AG_RETURN_IF_ERROR(k::grouped_append(cs, d));
+    if (form == 1) return k::grouped_decode(cs, d);
+    k::PromptAttnDesc p;
+    p.dtype = dt; p.n_seq = (int)B; p.T = (int)T; p.past = (int)past; p.heads = (int)H; p.group = (int)(H / G); p.dim = (int)D; p.vdim = (int)E; p.window = c->window; p.scale = c->scale;
+    p.softcap = c->softcap; p.q = d.proj; p.q_ld = d.ld; p.q_b = T * d.ld; p.k = d.cache; p.v = static_cast<uint8_t*>(d.cache) + (size_t)k::grouped_v_col((int)G, (int)D) * esz;
+    p.k_ld = p.v_ld = cld; p.k_b = p.v_b = d.seq_stride; p.y = out.data(); p.y_ld = d.y_ld; p.y_b = T * d.y_ld;
+    if (form == 2) return k::prompt_attention_tc_eligible(p) ? k::prompt_attention_tc(cs, p) : Status::unsupported("these sizes do not take the tensor-core kernel");
+    return k::prompt_attention(cs, p);
+  };
+  const Status s = run();
+  return immediate_result("grouped_attention", st.rt, s, out);
 }
 
 int32_t applegpu_test_wait_runs_out(int32_t code, uint32_t limit_us) {

@@ -274,7 +274,8 @@ Status key_decay(cudaStream_t s, const KeyDecayDesc& d, int* launches) {
   }
   if (w.ops) {
     p.chunks = (d.T + kKdChunk - 1) / kKdChunk; p.dp = kd_dp(d.dim); p.ops = w.ops; p.ops_bytes = kd_ops_bytes(p.dp, d.delta); p.u = w.u; p.o = w.o;
-    AG_RETURN_IF_ERROR(key_decay_chunked(s, d.dtype, p, launches));
+    *launches += 3;
+    AG_RETURN_IF_ERROR(d.dtype == DType::BF16 ? key_decay_chunked_bf16(s, p) : key_decay_chunked_f16(s, p));
   } else {
     *launches += 1;
     AG_RETURN_IF_ERROR(key_decay_step(s, d.dtype, p));

@@ -1,4 +1,4 @@
-// What the two files of key-decayed matrix states share: the parameters of their kernels, the raw inputs of the convolutions, the
+// What the files of key-decayed matrix states share: the parameters of their kernels, the raw inputs of the convolutions, the
 // decay.
 #pragma once
 #include "common.cuh"
@@ -47,6 +47,7 @@ __device__ __forceinline__ float kd_decay(const KdParams& p, int h, float z) { r
 __device__ __forceinline__ float kd_gate(const KdParams& p, float g) { return p.gate_silu ? silu_f(g) : sigmoid_f(g); }
 
 inline int kd_dp(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 96 ? 96 : dim <= 128 ? 128 : dim <= 192 ? 192 : 256; }
-Status key_decay_chunked(cudaStream_t s, DType dt, const KdParams& p, int* launches);
+Status key_decay_chunked_bf16(cudaStream_t s, const KdParams& p);
+Status key_decay_chunked_f16(cudaStream_t s, const KdParams& p);
 
 }}  // namespace ag::k

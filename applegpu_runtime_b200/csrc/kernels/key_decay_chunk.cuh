@@ -13,6 +13,7 @@
 // multiplied up term by term in float32; between blocks they split at block borders into factors of at most one, and the sums
 // over channels become small products. Values that the recurrence wants in float32 enter products as the sum of two 16-bit
 // numbers, high part and remainder (three products of four), which leaves an error near 2^-17.
+#pragma once
 #include "key_decay.cuh"
 #include "mma_sync.cuh"
 #include "sm100.cuh"
@@ -332,7 +333,7 @@ __global__ void __launch_bounds__(256) key_decay_scan_kernel(const KdParams p, i
 #pragma unroll
     for (int ks = 0; ks < NT / 2; ks++) {
       uint32_t uh[4], ul[4];
-      kd_frag<T>(u[2 * ks], u[2 * ks + 1], uh, ul);
+      kd_frag<T>(u[2 * ks], u[2 * ks + 1], uh, ul);      // without the delta rule and convolutions u is the stored v, without a remainder
 #pragma unroll
       for (int n = 0; n < NT; n += 2) {
         if (n + 1 < 2 * ks) continue;                    // tokens before these keys
@@ -343,7 +344,7 @@ __global__ void __launch_bounds__(256) key_decay_scan_kernel(const KdParams p, i
 #pragma unroll
         for (int x = 0; x < 2; x++) {
           mma_16816<T>(o[n + x], uh[0], uh[1], uh[2], uh[3], bh[2 * x], bh[2 * x + 1]);
-          if constexpr (DELTA) mma_16816<T>(o[n + x], ul[0], ul[1], ul[2], ul[3], bh[2 * x], bh[2 * x + 1]);
+          if (DELTA || p.taps) mma_16816<T>(o[n + x], ul[0], ul[1], ul[2], ul[3], bh[2 * x], bh[2 * x + 1]);
           mma_16816<T>(o[n + x], uh[0], uh[1], uh[2], uh[3], bl[2 * x], bl[2 * x + 1]);
         }
       }
@@ -356,7 +357,7 @@ __global__ void __launch_bounds__(256) key_decay_scan_kernel(const KdParams p, i
 #pragma unroll
         for (int x = 0; x < 2; x++) {
           mma_16816<T>(st[n + x], uh[0], uh[1], uh[2], uh[3], bh[2 * x], bh[2 * x + 1]);
-          if constexpr (DELTA) mma_16816<T>(st[n + x], ul[0], ul[1], ul[2], ul[3], bh[2 * x], bh[2 * x + 1]);
+          if (DELTA || p.taps) mma_16816<T>(st[n + x], ul[0], ul[1], ul[2], ul[3], bh[2 * x], bh[2 * x + 1]);
           mma_16816<T>(st[n + x], uh[0], uh[1], uh[2], uh[3], bl[2 * x], bl[2 * x + 1]);
         }
       }
@@ -440,20 +441,15 @@ static cudaError_t launch_kd_dp(cudaStream_t s, const KdParams& p, int warps) {
   }
 }
 template <typename T>
-static cudaError_t launch_chunked(cudaStream_t s, const KdParams& p) {
+static Status launch_chunked(cudaStream_t s, const KdParams& p) {
   // value columns per CTA: up to 128, fewer where that leaves SMs without work
   int warps = std::min(8, (p.vdim + 15) / 16);
   while (warps > 2 && (long long)p.n_seq * p.heads * ((p.vdim + 16 * warps - 1) / (16 * warps)) < sm_count()) warps = (warps + 1) / 2;
   cudaError_t e = p.delta ? launch_kd_dp<T, true>(s, p, warps) : launch_kd_dp<T, false>(s, p, warps);
-  if (e != cudaSuccess) return e;
+  if (e != cudaSuccess) return cuda_status(e, "key decay (chunked)");
   const unsigned blocks = (unsigned)(((long long)p.n_seq * p.T * p.heads + 7) / 8);
   const bool vec = p.vdim % 4 == 0 && p.y_ld % 4 == 0 && aligned16(p.y) && aligned16(p.norm) && (p.gate ? p.gate_ld % 4 == 0 : p.ld % 4 == 0 && p.g_off % 4 == 0 && aligned16(p.proj));
-  return vec ? launch_pdl(key_decay_finish_kernel<T, 4>, dim3(blocks), dim3(256), 0, s, p) : launch_pdl(key_decay_finish_kernel<T, 1>, dim3(blocks), dim3(256), 0, s, p);
-}
-
-Status key_decay_chunked(cudaStream_t s, DType dt, const KdParams& p, int* launches) {
-  *launches += 3;
-  const cudaError_t e = dt == DType::BF16 ? launch_chunked<__nv_bfloat16>(s, p) : launch_chunked<__half>(s, p);
+  e = vec ? launch_pdl(key_decay_finish_kernel<T, 4>, dim3(blocks), dim3(256), 0, s, p) : launch_pdl(key_decay_finish_kernel<T, 1>, dim3(blocks), dim3(256), 0, s, p);
   return cuda_status(e, "key decay (chunked)");
 }
 

@@ -109,7 +109,7 @@ Status latent_append(cudaStream_t s, const LatentDesc& d);
 size_t latent_decode_work_bytes(int rows, int heads, int kv_rank, int rot_dim, int max_len);
 Status latent_decode(cudaStream_t s, const LatentDesc& d, void* work);
 
-// ── matrix states with one decay per key channel (key_decay.cu, key_decay_chunk.cu) ──
+// ── matrix states with one decay per key channel (key_decay.cu, key_decay_chunk.cuh) ──
 // Per head S [dim, vdim], row d of which fades by a_d in every token:
 //     S <- diag(a) S,   u = v, or with the delta rule beta (v - S^T k),   S <- S + k u^T,   o = S^T q.
 // y rows receive o / rms(o) * norm * act(gate). Options, each on its own:

@@ -80,10 +80,11 @@ def load_rurunex(config, weights, dtype="bfloat16"):
                          form="sequential", embed_scale=config["embedding"]["scale"])
 
 
-def init_rurunex_weights(config, seed=0, std=0.02, ranks=(16, 16)):
+def init_rurunex_weights(config, seed=0, std=0.02, ranks=None):
     """Random weights for a configuration, {tensor name: float32 array}: N(0, std) matrices, unit norms, decays that keep most of a
-    state; `ranks`: inner sizes of the decay's and the gate's two-step projections."""
+    state; `ranks`: inner size of the two-step projections per mixer type."""
     rng = np.random.default_rng(seed)
+    ranks = {"gla": 16, "channel_delta": 16, **(ranks or {})}
     W, V, w = int(config["width"]), int(config["vocab"]), {}
 
     def mat(name, *shape):
@@ -104,10 +105,10 @@ def init_rurunex_weights(config, seed=0, std=0.02, ranks=(16, 16)):
                 mat(x + "v", m["kv_heads"] * e, W)
                 w[x + "k.norm"] = np.ones(d, np.float32)
         else:
-            G = m.get("kv_heads", H)
-            for n, k in (("q", G * d), ("k", G * d), ("v", H * e), ("a1", ranks[0])):
+            G, r = m.get("kv_heads", H), ranks[c["type"]]
+            for n, k in (("q", G * d), ("k", G * d), ("v", H * e), ("a1", r)):
                 mat(x + n, k, W)
-            mat(x + "a2", H * d, ranks[0])
+            mat(x + "a2", H * d, r)
             w[x + "norm"] = np.ones(e, np.float32)
             if c["type"] == "gla":
                 mat(x + "g", H * e, W)
@@ -116,8 +117,8 @@ def init_rurunex_weights(config, seed=0, std=0.02, ranks=(16, 16)):
                 for n, k in (("q", G * d), ("k", G * d), ("v", H * e)):
                     w[x + n + ".conv"] = (rng.standard_normal((k, m["conv"])) * 0.5).astype(np.float32)
                 mat(x + "b", H, W)
-                mat(x + "g1", ranks[1], W)
-                mat(x + "g2", H * e, ranks[1])
+                mat(x + "g1", r, W)
+                mat(x + "g2", H * e, r)
                 w[x + "A_log"] = np.log(rng.uniform(0.5, 4.0, H)).astype(np.float32)
                 w[x + "dt_bias"] = rng.uniform(-5.0, -2.0, H * d).astype(np.float32)
         mat(x + "o", W, H * e)

@@ -1,4 +1,4 @@
-"""Throughput of the Gedenex design beside GPT-2 at equal size, and what its kernels reach of the roofline.
+"""Throughput of the sequence-model designs at equal size, and what their kernels reach of the roofline.
 
 A size is a width; the mixers and feed-forwards take sizes a trained model of that width would have, weights are random
 (N(0, 0.02)), token ids uniform. The GPT-2 of equal size has the same width, one layer per layer run, heads of 64 and a
@@ -15,9 +15,12 @@ from . import api as gpu
 from .gedenex import init_gedenex_weights, load_gedenex
 from .generate import Gpt2Decoder
 from .gpt2 import gpt2_forward, init_gpt2_weights
+from .rurunex import init_rurunex_weights, load_rurunex
 
 SIZES = {1024: dict(heads=4, latent_heads=8, kv_rank=256, ff=2816), 2048: dict(heads=8, latent_heads=16, kv_rank=512, ff=5632)}
-BYTES = ("rms_rows", "linear_gates", "clamped_glu", "mlstm_prefill", "mlstm_step", "latent_append", "latent_decode", "skinny_in", "skinny_out", "skinny_head")
+RURUNEX_SIZES = {1024: dict(gla=4, delta=8, heads=8, kv_heads=2, ff=2816), 2048: dict(gla=8, delta=16, heads=16, kv_heads=4, ff=5632)}
+BYTES = ("rms_rows", "linear_gates", "clamped_glu", "mlstm_prefill", "mlstm_step", "latent_append", "latent_decode", "gla_prefill", "delta_prefill", "gla_step", "delta_step",
+         "grouped_append", "grouped_decode", "skinny_in", "skinny_ff", "skinny_out", "skinny_head")
 
 
 def config_of(width, vocab=32768):
@@ -28,6 +31,19 @@ def config_of(width, vocab=32768):
           "mixer": {"heads": s["latent_heads"], "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": s["kv_rank"], "scale": 192 ** -0.5,
                     "rot": {"dims": 64, "base": 10000.0, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
     return {"architecture": "Gedenex", "layers": [ml, ml, la, ml, ml, la], "loop": {"start": 0, "stop": 3, "times": 2}, "norm": {"eps": 1e-5}, "vocab": vocab, "width": width}
+
+
+def rurunex_config_of(width, vocab=32768):
+    """Nine layers like the nine layer runs above: matrix states of the same sizes, attention behind a window of 512 tokens."""
+    s = RURUNEX_SIZES[width]
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    gla = {"type": "gla", "mixer": {"heads": s["gla"], "dim": 128, "vdim": width // s["gla"], "tau": 16.0}, "mlp": mlp}
+    delta = {"type": "channel_delta", "mixer": {"heads": s["delta"], "kv_heads": s["delta"], "dim": 128, "vdim": 128, "conv": 4}, "mlp": mlp}
+    att = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": 128, "vdim": 128, "mask": {"size": 512}, "scale": 128 ** -0.5, "softcap": 30.0,
+           "rot": {"dims": 128, "base": 10000.0, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    att0, att1 = {"type": "attention", "mixer": att, "mlp": mlp}, {"type": "attention", "mixer": {**att, "kv_from": 2}, "mlp": mlp}
+    return {"architecture": "Rurunex", "embedding": {"scale": width ** 0.5}, "layers": [gla, delta, att0, gla, delta, att1, gla, delta, att1], "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "vocab": vocab, "width": width}
 
 
 def _timed(fn, iters, warmup=3):
@@ -51,12 +67,20 @@ def _kernel_rows(peaks, calls):
     return out
 
 
-def bench_gedenex(width, peaks, iters=10, batch=8, prompt=1024, steps=48):
+def bench_gedenex(width, peaks, iters=10):
     cfg = config_of(width)
-    model = load_gedenex(cfg, init_gedenex_weights(cfg, seed=0), "bfloat16")
+    return bench_sequence(load_gedenex(cfg, init_gedenex_weights(cfg, seed=0), "bfloat16"), width, peaks, iters)
+
+
+def bench_rurunex(width, peaks, iters=10):
+    cfg = rurunex_config_of(width)
+    return bench_sequence(load_rurunex(cfg, init_rurunex_weights(cfg, seed=0, ranks={"channel_delta": 128}), "bfloat16"), width, peaks, iters)
+
+
+def bench_sequence(model, width, peaks, iters=10, batch=8, prompt=1024, steps=48):
     eng = model.engine(slots=batch, max_len=prompt + 2 * steps + 16)
     rng = np.random.default_rng(1)
-    ids = rng.integers(0, cfg["vocab"], (batch, prompt)).astype(np.int32)
+    ids = rng.integers(0, model.vocab, (batch, prompt)).astype(np.int32)
 
     def prefill(n=batch):
         eng.reset(0, n)
@@ -125,12 +149,16 @@ def bench_gpt2(width, peaks, iters=10, batch=8, prompt=1024, steps=48, vocab=327
     return row
 
 
-def run(peaks, widths=(1024, 2048), iters=10):
+def run(peaks, widths=(1024, 2048), iters=10, design="gedenex"):
+    """The design at each width beside the closest existing model of equal size: GPT-2 for Gedenex, Gedenex for Rurunex."""
     gpu.init_backend()
     out = []
     t0 = time.time()
     for w in widths:
-        out.append({"gedenex": bench_gedenex(w, peaks, iters), "gpt2_equal_size": bench_gpt2(w, peaks, iters)})
+        if design == "gedenex":
+            out.append({"gedenex": bench_gedenex(w, peaks, iters), "gpt2_equal_size": bench_gpt2(w, peaks, iters)})
+        else:
+            out.append({"rurunex": bench_rurunex(w, peaks, iters), "gedenex_equal_size": bench_gedenex(w, peaks, iters)})
     st = gpu.pipeline_status()
     if st:
         raise RuntimeError(f"pipeline status {st}")

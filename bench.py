@@ -4,6 +4,7 @@
   python bench.py --gpus N --steps K --warmup W              the B200 path (this library)
   python bench.py --impl reference --gpus N --steps K ...    the reference's CPU path (PyTorch CPU eager)
   python bench.py --workload gedenex                         the Gedenex design beside GPT-2 at equal size
+  python bench.py --workload rurunex                         the Rurunex design beside Gedenex at equal size
 
 Workload at every N (both arms): GPT-2-small architecture (12 layers, d 768, 12 heads, MLP 3072, vocab
 50257, ctx 1024), weights N(0, 0.02) seed 0, token ids uniform over the vocab, batch 8 x seq 1024 per
@@ -611,17 +612,17 @@ def tensor_parallel_leg(gpu, lib, group):
         return {"error": f"{type(e).__name__}: {e}"}
 
 
-def run_gedenex(args):
+def run_sequence(args):
     from applegpu_runtime_b200 import seqbench
     peaks = measured_peaks()
     sampler = ClockSampler(0)
     sampler.start()
     t0 = time.perf_counter()
-    res = seqbench.run(peaks, iters=max(3, min(args.steps, 10)))
+    res = seqbench.run(peaks, iters=max(3, min(args.steps, 10)), design=args.workload)
     clocks = sampler.window(t0, time.perf_counter())
     sampler.stop()
-    big = res["sizes"][-1]["gedenex"]
-    print(json.dumps({"metric": "gedenex prefill tokens/s", "value": big["prefill_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "ms_per_step": big["prefill_ms"],
+    big = res["sizes"][-1][args.workload]
+    print(json.dumps({"metric": f"{args.workload} prefill tokens/s", "value": big["prefill_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "ms_per_step": big["prefill_ms"],
                       "higher_is_better": True, "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "peaks": peaks, "clocks": clocks, **res}), flush=True)
 
 
@@ -634,10 +635,11 @@ def main():
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--quick", action="store_true", help="headline, e2e, sustained and roofline only (no per-op rows, fp32, decode, strong / tp legs)")
     ap.add_argument("--sustained-seconds", type=float, default=2.0, help="length of the sustained loop; 0 runs it for --steps steps only (launch lists under a profiler)")
-    ap.add_argument("--workload", default="gpt2", choices=["gpt2", "gedenex"], help="gedenex: prefill and decode of the Gedenex design at two sizes beside GPT-2 at equal size (one GPU)")
+    ap.add_argument("--workload", default="gpt2", choices=["gpt2", "gedenex", "rurunex"],
+                    help="gedenex, rurunex: prefill and decode of the design at two sizes beside the closest existing model at equal size (one GPU)")
     args = ap.parse_args()
-    if args.workload == "gedenex":
-        run_gedenex(args)
+    if args.workload != "gpt2":
+        run_sequence(args)
     elif args.impl == "reference":
         run_reference(args)
     else:

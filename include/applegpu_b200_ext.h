@@ -288,21 +288,38 @@ APPLEGPU_API int32_t applegpu_gpt2_decoder_set_engine(uint64_t decoder, int32_t 
 APPLEGPU_API void applegpu_gpt2_decoder_destroy(uint64_t decoder);
 
 /* ── sequence models: layers with per-sequence memory, prompt portions, generation ──
- * No counterpart in the reference. An engine owns the weights of a decoder-only model given as a list of layers
- *     x <- x + (mixer(rms(x) norm1) + ff(rms(x) norm2))
- * over a float32 stream x, and `slots` sequences of at most max_len tokens. Each run of a layer keeps its own memory per
- * slot: mixer 1 (mLSTM) a float32 state, mixer 2 (latent attention) one cached row per token. Layers loop_start ..
- * loop_stop - 1 run loop_times times (0: no loop): before each pass but the first the embedding output is added to x, before
- * every pass a step vector.
+ * No counterpart in the reference. An engine owns the weights of a decoder-only model given as a list of layers over a float32
+ * stream x, and `slots` sequences of at most max_len tokens. form 0 (parallel): x <- x + (mixer(rms(x) norm1) + ff(rms(x) norm2));
+ * form 1 (sequential): x <- x + rms(mixer(rms(x) norm1)) post1, then x <- x + rms(ff(rms(x) norm2)) post2. The stream starts as
+ * embed[token] * embed_scale. Each run of a layer keeps its own memory per slot: mixer 1 (mLSTM) and 3 (key decay) a float32
+ * state, 3 with taps also the last inputs of its convolutions; mixer 2 (latent attention) and 4 (grouped attention) one cached
+ * row per token, unless kv_from names an earlier layer of mixer 4 whose rows are used. Layers loop_start .. loop_stop - 1 run
+ * loop_times times (0: no loop): before each pass but the first the embedding output is added to x, before every pass a step
+ * vector.
  *   create:  weight_ids = embed [vocab, width], head [vocab, P(width)], final norm f32 [width], step vectors f32
- *            [loop_times, width] (0 without a loop), then eight per layer: norm1, norm2 (f32 [width]; 0 without a
- *            feed-forward), the mixer's input rows [cols, P(width)], the output rows [width, P(K)] with K = P(heads * vdim) + ff
- *            (mixer columns, then feed-forward columns) or heads * vdim without a feed-forward, feed-forward rows in
- *            blocks of 16 gates | the 16 they gate (ff rounded up to 16, zero rows) [.., P(width)] (or 0), and three of the mixer's own:
- *              mLSTM    input rows q | k | v | g; own: i rows | f rows [2 heads, P(width)], f32 bias [2 heads], f32 norm [heads * vdim]
- *              latent   input rows q (per head: dim, rot_dim) | latent | rotated key part; own: f32 latent norm [kv_rank],
- *                       uk rows, padded to P(heads * dim), | uv rows, padded to P(heads * vdim), [.., P(kv_rank)], and
- *                       f32 (cos, sin) [>= max_len, rot_pairs, 2]
+ *            [loop_times, width] (0 without a loop), then fifteen per layer (0 where a layer has none):
+ *              norm1, norm2 (f32 [width]), the mixer's input rows [cols, P(width)], the output rows, feed-forward rows in blocks of
+ *              16 gates | the 16 they gate (ff rounded up to 16, zero rows) [.., P(width)], own0, own1, own2, post1, post2
+ *              (f32 [width]), feed-forward output rows [width, P(ff)], own3, own4, own5, own6.
+ *            Output rows: [width, P(K)], K = heads * vdim, or in form 0 with a feed-forward P(heads * vdim) + ff (mixer columns, then
+ *            feed-forward columns). Feed-forwards (glu): 0 g sigmoid(1.702 g) (u + 1), g = min(gate, ff_limit), u = clamp(value,
+ *            +-ff_limit); 1 gate sigmoid(gate) value. Mixers:
+ *              mLSTM    input rows q | k | v | g; own0 i rows | f rows [2 heads, P(width)], own1 f32 bias [2 heads], own2 f32 norm
+ *                       [heads * vdim]
+ *              latent   input rows q (per head: dim, rot_dim) | latent | rotated key part; own0 f32 latent norm [kv_rank], own1 uk
+ *                       rows, padded to P(heads * dim), | uv rows, padded to P(heads * vdim), [.., P(kv_rank)], own2 f32 (cos, sin)
+ *                       [>= max_len, rot_pairs, 2]
+ *              key decay  S <- diag(a) S, u = v (flags & 1: beta (v - S^T k)), S <- S + k u^T, o = S^T q, with q and k of kv_heads heads,
+ *                       q scaled by dim^-1/2; flags & 2: q and k unit vectors; taps > 0: q, k and v behind causal convolutions and
+ *                       silu; a = sigmoid(z)^(1 / tau) or (flags & 4) exp(-rate softplus(z)), z = own1 a1 + own2; result
+ *                       o / rms(o) own3 times sigmoid (flags & 8: silu) of the gate. Input rows q | k | v | a1 | gate, each part
+ *                       padded to P(rows), gate = own4 g1 if g_rank > 0 (the last part is then g1). own0 beta rows
+ *                       [heads, P(width)], own1 [heads * dim, P(a_rank)], own2 f32 [heads * dim], own3 f32 [vdim], own4
+ *                       [heads * vdim, P(g_rank)], own5 f32 rate [heads], own6 f32 taps [q | k | v channels, taps]
+ *              grouped  input rows q | k | v (q only with kv_from >= 0), each part padded to P(rows); heads / kv_heads query heads share a
+ *                       key head; q and k are normed per head and their first 2 rot_pairs entries turned, i with i + rot_pairs; a
+ *                       token sees the last `window` keys (0: all); softcap c > 0: c tanh(score / c). own0 f32 query norm [dim],
+ *                       own1 f32 key norm [dim], own2 f32 (cos, sin) [>= max_len, rot_pairs, 2]
  *            P(n) rounds up to a multiple of 8; padding holds zeros. All matrices share one float dtype, which is the
  *            storage type of activations and caches. Returns a handle, 0 on failure (applegpu_ffi_last_error).
  *   forward: the next n_tokens tokens of the n_seq sequences in slots slot0 .. (row s * n_tokens + t is token t of sequence
@@ -328,6 +345,14 @@ APPLEGPU_API void applegpu_seq_destroy(uint64_t engine);
 /* The mechanisms one by one, evaluated at once (operands contiguous; 0 on failure).
  *   rms_norm     float32 x [.., n], float32 weight [n] -> x / sqrt(mean(x^2) + eps) * weight in out_dtype
  *   clamped_glu  [.., 2 n] (gate | up) -> g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)
+ *   silu_glu     [.., 2 n] (gate | up) -> gate sigmoid(gate) up
+ *   rms_add      x f32 [.., n] += rms(y) * post (y f32 like x, post f32 [n]), in place -> rms(x) * weight in out_dtype
+ *   key_decay    proj [B, T, cols] and own tensors as in seq_create (beta f32 [B, T, heads], without sigmoid; 0 where unused), mem f32
+ *                [B, bytes / 4] (state, then the convolutions' ring; zeros for a new sequence), updated in place, pos int32 [B] ->
+ *                [B, T, heads * vdim]; form 0: by length and type, 1: token by token. key_decay_mem_bytes: of one sequence
+ *   grouped_attention  proj [B, T, cols] (turned in place), cache [B, max_len, P(kv_heads * dim) + P(kv_heads * vdim)] appended at pos
+ *                (int32 [B], all equal to `past`) unless `shared` -> [B, T, heads * vdim]; form 0: whole portions, 1: short ones, over
+ *                splits of the keys, 2: as 0, on the tensor-core kernel or not at all
  *   mlstm        proj [B, T, cols] (q | k | v | g), gates f32 [B, T, 2 heads] (i | f without bias), state f32 [B, S floats: per
  *                head dim * vdim, then heads * dim, then heads; S rounded up to 4], updated in place -> [B, T, heads * vdim];
  *                form 0: chunk-parallel, 1: token by token, 2: chunk-parallel on CUDA cores
@@ -337,6 +362,15 @@ APPLEGPU_API void applegpu_seq_destroy(uint64_t engine);
  *                kernel or not at all */
 APPLEGPU_API uint64_t applegpu_ffi_rms_norm(uint64_t x_id, uint64_t weight_id, float eps, int8_t out_dtype);
 APPLEGPU_API uint64_t applegpu_ffi_clamped_glu(uint64_t gate_up_id, float limit);
+APPLEGPU_API uint64_t applegpu_ffi_silu_glu(uint64_t gate_up_id);
+APPLEGPU_API uint64_t applegpu_ffi_rms_add(uint64_t x_id, uint64_t y_id, uint64_t post_id, uint64_t weight_id, float eps, int8_t out_dtype);
+typedef struct { int32_t heads, kv_heads, dim, vdim, taps, a_rank, g_rank, flags; float tau, eps; } applegpu_key_decay_desc;
+APPLEGPU_API uint64_t applegpu_key_decay_mem_bytes(const applegpu_key_decay_desc* desc, int8_t dtype);
+APPLEGPU_API uint64_t applegpu_ffi_key_decay(uint64_t proj_id, uint64_t beta_id, uint64_t a2_id, uint64_t bias_id, uint64_t norm_id, uint64_t g2_id, uint64_t rate_id,
+                                             uint64_t conv_id, uint64_t mem_id, uint64_t pos_id, const applegpu_key_decay_desc* desc, int32_t form);
+typedef struct { int32_t heads, kv_heads, dim, vdim, window, shared; float scale, softcap, eps; } applegpu_grouped_attention_desc;
+APPLEGPU_API uint64_t applegpu_ffi_grouped_attention(uint64_t proj_id, uint64_t q_norm_id, uint64_t k_norm_id, uint64_t rot_id, uint64_t cache_id, uint64_t pos_id, uint32_t past,
+                                                     const applegpu_grouped_attention_desc* desc, int32_t form);
 APPLEGPU_API uint64_t applegpu_ffi_mlstm(uint64_t proj_id, uint64_t gates_id, uint64_t gate_bias_id, uint64_t norm_id, uint64_t state_id, uint32_t heads, uint32_t dim,
                                          uint32_t vdim, float gate_cap, float eps, int32_t form);
 APPLEGPU_API uint64_t applegpu_ffi_latent_attention(uint64_t proj_id, uint64_t norm_id, uint64_t up_id, uint64_t rot_id, uint64_t cache_id, uint64_t pos_id, uint32_t past,
