@@ -214,7 +214,6 @@ static Status key_decay_step(cudaStream_t s, DType dt, const KdParams& p) {
 
 // Scratch of a portion longer than kKeyDecayStepTokens: z, the gates, and for the chunk form what its kernels hand on.
 struct KdWork { float* z; void* gate; uint8_t* ops; float* u; float* o; size_t total; };
-static long long kd_ops_bytes(int dp, bool delta) { return ((delta ? 6LL : 4LL) * kKdChunk * (dp + 8) + 2LL * kKdChunk * (kKdChunk + 8)) * 2 + dp * 4LL; }
 static KdWork kd_layout(const KeyDecayDesc& d, void* base) {
   KdWork w = {};
   uint8_t* p = static_cast<uint8_t*>(base);
@@ -225,7 +224,7 @@ static KdWork kd_layout(const KeyDecayDesc& d, void* base) {
   w.gate = d.g_rank ? take(rows * pad8((int64_t)d.heads * d.vdim) * dtype_size(d.dtype)) : nullptr;
   if (key_decay_chunk_eligible(d)) {
     const size_t n = (size_t)d.n_seq * d.heads * ((d.T + kKdChunk - 1) / kKdChunk);
-    w.ops = take(n * kd_ops_bytes(kd_dp(d.dim), d.delta));
+    w.ops = take(n * kd_ops_layout(kd_dp(d.dim), d.delta).stride);
     w.u = reinterpret_cast<float*>(take(n * d.vdim * kKdChunk * sizeof(float)));
     w.o = reinterpret_cast<float*>(take(rows * d.heads * d.vdim * sizeof(float)));
   }
@@ -273,8 +272,8 @@ Status key_decay(cudaStream_t s, const KeyDecayDesc& d, int* launches) {
     p.gate = w.gate;
   }
   if (w.ops) {
-    p.chunks = (d.T + kKdChunk - 1) / kKdChunk; p.dp = kd_dp(d.dim); p.ops = w.ops; p.ops_bytes = kd_ops_bytes(p.dp, d.delta); p.u = w.u; p.o = w.o;
-    *launches += 3;
+    p.chunks = (d.T + kKdChunk - 1) / kKdChunk; p.dp = kd_dp(d.dim); p.ops = w.ops; p.u = w.u; p.o = w.o;
+    *launches += kd_fused(p) ? 2 : 3;
     AG_RETURN_IF_ERROR(d.dtype == DType::BF16 ? key_decay_chunked_bf16(s, p) : key_decay_chunked_f16(s, p));
   } else {
     *launches += 1;

@@ -6,9 +6,11 @@
 //     S   = A_32 S_0 + sum_j (A_32 / A_j k_j) u_j^T.
 // (I + beta K) u = beta v - beta (A k) S_0 is solved for both right-hand sides ahead of the state, u = U - W S_0:
 //   prepare  every chunk on its own: convolutions, unit norms, decays, Q and K, U and W by forward substitution
-//   scan     the chunks of a head one after the other; a warp owns 16 value columns of S as accumulator fragments, so that S,
-//            u and the state's update chain from one product to the next without leaving registers
-//   finish   the head's norm, its weight and the gate
+//   scan     the chunks of a head one after the other, the transposed problem on tcgen05: S^T [value columns, channels], u^T and
+//            o^T are accumulators in tensor memory, S^T and u^T (split) A operands there; up to 128 channels and 128 value columns per
+//            CTA. Where that is all of a head, its norm, norm weight and gate follow, one chunk behind, in warps of their own.
+//            Wider keys take a warp-level form: a warp owns 16 value columns, its accumulator fragments chain in registers
+//   finish   norm and gate of wider heads
 // No decay is ever inverted: quotients A_i / A_j are products of the decays between j and i. Inside a block of 8 tokens they are
 // multiplied up term by term in float32; between blocks they split at block borders into factors of at most one, and the sums
 // over channels become small products. Values that the recurrence wants in float32 enter products as the sum of two 16-bit
@@ -19,6 +21,7 @@
 #include "sm100.cuh"
 #include "tc_math.cuh"
 #include <algorithm>
+#include <type_traits>
 
 namespace ag { namespace k {
 
@@ -27,22 +30,6 @@ using sm100::mbar_expect_tx;
 using sm100::mbar_wait;
 
 constexpr int kKdThreads = 256, kKdBlock = 8, kKdBlocks = kKdChunk / kKdBlock;
-constexpr int kKdAPitch = kKdChunk + 8;
-
-// What prepare hands to scan for one chunk of one head: planes of [32][dp + 8] (high part, remainder) of A q, then (delta) -W, then
-// A_32 / A k, planes of [32][40] of Q, the chunk's decay [dp] in float32.
-template <typename T>
-struct KdOps {
-  T* qg; T* w; T* kg; T* a; float* decay; int plane;
-  __device__ KdOps(uint8_t* base, int dp, bool delta) {
-    plane = kKdChunk * (dp + 8);
-    qg = reinterpret_cast<T*>(base);
-    w = qg + 2 * plane;
-    kg = w + (delta ? 2 * plane : 0);
-    a = kg + 2 * plane;
-    decay = reinterpret_cast<float*>(a + 2 * kKdChunk * kKdAPitch);
-  }
-};
 
 template <typename T>
 __device__ __forceinline__ void kd_split(float x, T& hi, T& lo) { hi = Cvt<T>::from(x); lo = Cvt<T>::from(x - Cvt<T>::to(hi)); }
@@ -53,9 +40,40 @@ __device__ __forceinline__ void kd_split2(float x, float y, uint32_t& hi, uint32
   lo = pack2_t<T>(x - Cvt<T>::to(v[0]), y - Cvt<T>::to(v[1]));
 }
 
+// log(1 + e) for 0 <= e <= 1 as 2 artanh(e / (2 + e)), the series of which converges within 1e-7 of the value there
+__device__ __forceinline__ float kd_log1p_unit(float e) {
+  const float s = __fdividef(e, 2.0f + e), t = s * s;
+  float r = fmaf(t, 1.0f / 13.0f, 1.0f / 11.0f);
+  r = fmaf(t, r, 1.0f / 9.0f);
+  r = fmaf(t, r, 1.0f / 7.0f);
+  r = fmaf(t, r, 1.0f / 5.0f);
+  r = fmaf(t, r, 1.0f / 3.0f);
+  return 2.0f * fmaf(s * t, r, s);
+}
+__device__ __forceinline__ float kd_softplus_fast(float x) { return fmaxf(x, 0.f) + kd_log1p_unit(__expf(-fabsf(x))); }
+__device__ __forceinline__ float kd_decay_fast(const KdParams& p, float rate, float z) { return __expf(p.softplus ? -rate * kd_softplus_fast(z) : -kd_softplus_fast(-z) * p.inv_tau); }
+template <typename T>
+__device__ __forceinline__ float kd_gate_fast(const KdParams& p, T g) { const float x = Cvt<T>::to(g), s = __fdividef(1.0f, 1.0f + __expf(-x)); return p.gate_silu ? x * s : s; }
+__device__ __forceinline__ float kd_silu_fast(float x) { return x * __fdividef(1.0f, 1.0f + __expf(-x)); }
+
+// Convolutions of up to kKdTaps taps slide over their raw inputs; longer ones read them tap by tap.
+constexpr int kKdTaps = 4;
+// The taps of channel ch, zeros in front
+__device__ __forceinline__ void kd_taps(const KdParams& p, int ch, float (&w)[kKdTaps]) {
+#pragma unroll
+  for (int j = 0; j < kKdTaps; j++) { const int at = j - (kKdTaps - p.taps); w[j] = at >= 0 ? __ldg(p.conv + (long long)ch * p.taps + at) : 0.f; }
+}
+template <typename T>
+__device__ __forceinline__ float2 kd_pair(const T* at) {
+  const uint32_t raw = *reinterpret_cast<const uint32_t*>(at);
+  const T* v = reinterpret_cast<const T*>(&raw);
+  return make_float2(Cvt<T>::to(v[0]), Cvt<T>::to(v[1]));
+}
+
 template <typename T, int DP, bool DELTA>
-__global__ void __launch_bounds__(kKdThreads) key_decay_prepare_kernel(const KdParams p) {
-  constexpr int P = DP + 4, NC = DP / 32;
+__global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const KdParams p) {
+  constexpr int P = DP + 4, NC = DP / 32, DH = DP / 2;
+  constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
   extern __shared__ __align__(16) float sm[];
   float* sq = sm;                        // [32][P]: q, later q times the decays from its block's start
   float* sk = sq + kKdChunk * P;         // [32][P]: k, later likewise
@@ -64,6 +82,7 @@ __global__ void __launch_bounds__(kKdThreads) key_decay_prepare_kernel(const KdP
   float* sQ = sb + kKdBlocks * DP;       // [32][36]
   float* sK = sQ + kKdChunk * 36;        // [32][36], times beta
   float* s_beta = sK + kKdChunk * 36;    // [32]
+  float2* s_f = reinterpret_cast<float2*>(s_beta + kKdChunk);      // [32] what makes q and k unit vectors
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int c = blockIdx.x, h = blockIdx.y, s = blockIdx.z, qh = h / p.group, D = p.dim, E = p.vdim;
   const int t0 = c * kKdChunk, nt = min(kKdChunk, p.T - t0);
@@ -73,30 +92,135 @@ __global__ void __launch_bounds__(kKdThreads) key_decay_prepare_kernel(const KdP
   const int pos = p.pos[s];
   const T* base = reinterpret_cast<const T*>(p.proj) + (long long)s * p.T * p.ld;
   const T* ring = p.ring_of<T>(s);
-  KdOps<T> ops(p.ops + chunk * p.ops_bytes, DP, DELTA);
-  for (int i = tid; i < kKdChunk * DP; i += kKdThreads) {
-    const int t = i / DP, d = i % DP;
-    float q = 0.f, k = 0.f, a = 1.f;
-    if (t < nt && d < D) {
-      const int ch = qh * D + d;
-      q = kd_input<T>(p, base, ring, pos, t0 + t, p.q_off + ch, ch);
-      k = kd_input<T>(p, base, ring, pos, t0 + t, p.k_off + ch, p.qk_heads * D + ch);
-      a = kd_decay(p, h, p.z[((long long)s * p.T + t0 + t) * p.heads * D + h * D + d] + p.bias[h * D + d]);
-      if (!p.unit) q *= p.q_scale;
+  uint8_t* ops = p.ops + chunk * L.stride;
+  // one value column over the chunk, and its u
+  auto load_v = [&](int e, float (&w)[kKdChunk]) {
+    const int ch = h * E + e, rc = 2 * p.qk_heads * D + ch;
+    const T* src = base + (long long)t0 * p.ld + p.v_off + ch;
+    if (p.taps > kKdTaps) {
+#pragma unroll 1
+      for (int i = 0; i < kKdChunk; i++) {
+        const float v = i < nt ? kd_input<T>(p, base, ring, pos, t0 + i, p.v_off + ch, rc) : 0.f;
+#pragma unroll
+        for (int j = 0; j < kKdChunk; j++) if (j == i) w[j] = v;
+      }
+      return;
     }
-    sq[t * P + d] = q; sk[t * P + d] = k; sa[t * P + d] = a;
+    if (nt == kKdChunk) {
+#pragma unroll
+      for (int i = 0; i < kKdChunk; i++) w[i] = Cvt<T>::to(src[(long long)i * p.ld]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < kKdChunk; i++) w[i] = i < nt ? Cvt<T>::to(src[(long long)i * p.ld]) : 0.f;
+    }
+    if (p.taps == 0) return;
+    float f[kKdTaps], x[kKdTaps - 1];
+    kd_taps(p, rc, f);
+#pragma unroll
+    for (int j = 0; j < kKdTaps - 1; j++) { const int back = kKdTaps - 1 - j; x[j] = back < p.taps ? kd_raw<T>(p, base, ring, pos, t0 - back, p.v_off + ch, rc) : 0.f; }
+#pragma unroll
+    for (int i = kKdChunk - 1; i >= 0; i--) {            // from the end, so that raw inputs are still there
+      float y = f[3] * w[i];
+#pragma unroll
+      for (int n = 1; n < kKdTaps; n++) y = fmaf(f[3 - n], i >= n ? w[i >= n ? i - n : 0] : x[i >= n ? 0 : kKdTaps - 1 + i - n], y);
+      w[i] = i < nt ? kd_silu_fast(y) : 0.f;
+    }
+  };
+  auto store_u = [&](int e, const float (&w)[kKdChunk]) {
+    float4* u = reinterpret_cast<float4*>(p.u + (chunk * E + e) * kKdChunk);
+#pragma unroll
+    for (int i = 0; i < kKdChunk; i += 4) u[i / 4] = make_float4(w[i], w[i + 1], w[i + 2], w[i + 3]);
+  };
+  float w[kKdChunk];                     // a right-hand side: this thread's channel of A k, or (threads past the channels) a value column
+  const int e_own = tid - DP;
+  const float rate = p.softplus ? p.rate[h] : 0.f;
+  if (D % 2 == 0 && p.taps <= kKdTaps) {
+    // two channels at a time; everything is requested before anything is used
+    float2 z[DP / 16];
+#pragma unroll
+    for (int n = 0; n < DP / 16; n++) {
+      const int i = tid + n * kKdThreads, t = i / DH, d = i % DH * 2;
+      z[n] = make_float2(0.f, 0.f);
+      if (t < nt && d < D) z[n] = __ldcs(reinterpret_cast<const float2*>(p.z + ((long long)s * p.T + t0 + t) * p.heads * D + h * D + d));
+    }
+    if (DELTA && e_own >= 0 && e_own < E) load_v(e_own, w);
+    for (int i = tid; i < kKdBlocks * DH; i += kKdThreads) {
+      const int d = i % DH * 2, o = i / DH * kKdBlock, first = t0 + o - (kKdTaps - 1);
+      constexpr int N = kKdBlock + kKdTaps - 1;
+      float2 x[2][N];
+      const bool inside = first >= 0 && first + N <= p.T;
+#pragma unroll
+      for (int m = 0; m < 2; m++) {
+        const int col = (m ? p.k_off : p.q_off) + qh * D + d, ch = (m ? p.qk_heads * D : 0) + qh * D + d;
+        const T* src = base + (long long)first * p.ld + col;
+#pragma unroll
+        for (int j = 0; j < N; j++) {
+          x[m][j] = make_float2(0.f, 0.f);
+          if (d >= D || (j < kKdTaps - 1 && !p.taps)) continue;
+          if (inside) x[m][j] = kd_pair<T>(src + (long long)j * p.ld);
+          else {
+            const int t = first + j;
+            if (t >= 0) { if (t < p.T) x[m][j] = kd_pair<T>(src + (long long)j * p.ld); }
+            else if (-t < p.taps) x[m][j] = make_float2(kd_raw<T>(p, base, ring, pos, t, col, ch), kd_raw<T>(p, base, ring, pos, t, col + 1, ch + 1));
+          }
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < 2; m++) {
+        float* dst = (m ? sk : sq) + o * P + d;
+        if (p.taps) {
+          float w0[kKdTaps], w1[kKdTaps];
+          const int ch = (m ? p.qk_heads * D : 0) + qh * D + min(d, D - 2);
+          kd_taps(p, ch, w0);
+          kd_taps(p, ch + 1, w1);
+#pragma unroll
+          for (int j = 0; j < kKdBlock; j++) {
+            float2 y = make_float2(0.f, 0.f);
+#pragma unroll
+            for (int n = 0; n < kKdTaps; n++) { y.x = fmaf(w0[n], x[m][j + n].x, y.x); y.y = fmaf(w1[n], x[m][j + n].y, y.y); }
+            const bool live = o + j < nt;                // channels past D are zero already
+            *reinterpret_cast<float2*>(dst + j * P) = make_float2(live ? kd_silu_fast(y.x) : 0.f, live ? kd_silu_fast(y.y) : 0.f);
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < kKdBlock; j++) *reinterpret_cast<float2*>(dst + j * P) = x[m][j + kKdTaps - 1];
+        }
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < DP / 16; n++) {
+      const int i = tid + n * kKdThreads, t = i / DH, d = i % DH * 2;
+      float2 a = make_float2(1.f, 1.f);
+      if (t < nt && d < D) a = make_float2(kd_decay_fast(p, rate, z[n].x + __ldg(p.bias + h * D + d)), kd_decay_fast(p, rate, z[n].y + __ldg(p.bias + h * D + d + 1)));
+      *reinterpret_cast<float2*>(sa + t * P + d) = a;
+    }
+  } else {
+    for (int i = tid; i < kKdChunk * DP; i += kKdThreads) {
+      const int t = i / DP, d = i % DP;
+      float q = 0.f, k = 0.f, a = 1.f;
+      if (t < nt && d < D) {
+        const int ch = qh * D + d;
+        q = kd_input<T>(p, base, ring, pos, t0 + t, p.q_off + ch, ch);
+        k = kd_input<T>(p, base, ring, pos, t0 + t, p.k_off + ch, p.qk_heads * D + ch);
+        a = kd_decay_fast(p, rate, p.z[((long long)s * p.T + t0 + t) * p.heads * D + h * D + d] + p.bias[h * D + d]);
+      }
+      sq[t * P + d] = q; sk[t * P + d] = k; sa[t * P + d] = a;
+    }
+    if (DELTA && e_own >= 0 && e_own < E) load_v(e_own, w);
   }
+  if constexpr (!DELTA) for (int e = tid; e < E; e += kKdThreads) { load_v(e, w); store_u(e, w); }
   for (int i = tid; i < kKdChunk * 36; i += kKdThreads) { sQ[i] = 0.f; sK[i] = 0.f; }
   if (tid < kKdChunk) s_beta[tid] = DELTA && tid < nt ? sigmoid_f(p.beta[((long long)s * p.T + t0 + tid) * p.beta_ld + h]) : 0.f;
   __syncthreads();
-  if (p.unit) {
-    for (int t = warp; t < kKdChunk; t += kKdThreads / 32) {
+  for (int t = warp; t < kKdChunk; t += kKdThreads / 32) {
+    float2 f = make_float2(p.q_scale, 1.f);
+    if (p.unit) {
       float qq = 0.f, kk = 0.f;
+#pragma unroll
       for (int d = lane; d < DP; d += 32) { const float a = sq[t * P + d], b = sk[t * P + d]; qq = fmaf(a, a, qq); kk = fmaf(b, b, kk); }
-      const float fq = p.q_scale / sqrtf(warp_sum(qq) + 1e-6f), fk = 1.0f / sqrtf(warp_sum(kk) + 1e-6f);
-      for (int d = lane; d < DP; d += 32) { sq[t * P + d] *= fq; sk[t * P + d] *= fk; }
+      f = make_float2(p.q_scale / sqrtf(warp_sum(qq) + 1e-6f), 1.0f / sqrtf(warp_sum(kk) + 1e-6f));
     }
-    __syncthreads();
+    if (lane == 0) s_f[t] = f;
   }
   {
     // pairs inside a block: eight lanes per key token j, which carry its decayed key from one query token to the next
@@ -132,20 +256,33 @@ __global__ void __launch_bounds__(kKdThreads) key_decay_prepare_kernel(const KdP
     }
   }
   __syncthreads();
-  float w[kKdChunk];                     // this thread's channel of A k, the right-hand side of W
+  {                                      // those pairs with the factors of their rows
+    const int i = tid >> 3, j = i / kKdBlock * kKdBlock + (tid & 7);
+    const float2 fi = s_f[i];
+    const float fk = s_f[j].y;
+    sQ[i * 36 + j] *= fi.x * fk;
+    if constexpr (DELTA) sK[i * 36 + j] *= fi.y * fk;
+  }
+  // element (row, channel tid) of a plane of `rows` rows, high part and remainder
+  auto put = [&](int plane0, int plane_bytes, int rows, int row, float x) {
+    T hi, lo;
+    kd_split<T>(x, hi, lo);
+    uint8_t* at = kd_tc(DP) ? ops + plane0 + (tid >> 6) * rows * 128 + row * 128 + (((tid & 63) * 2) ^ ((row & 7) << 4)) : ops + plane0 + (row * (DP + 8) + tid) * 2;
+    *reinterpret_cast<T*>(at) = hi;
+    *reinterpret_cast<T*>(at + plane_bytes) = lo;
+  };
   if (tid < DP) {
     const int d = tid;
     float kk[kKdChunk], pre = 1.f, loc = 1.f;
 #pragma unroll
     for (int i = 0; i < kKdChunk; i++) {
-      const float a = sa[i * P + d], q = sq[i * P + d];
-      kk[i] = sk[i * P + d];
+      const float2 f = s_f[i];
+      const float a = sa[i * P + d], q = sq[i * P + d] * f.x;
+      kk[i] = sk[i * P + d] * f.y;
       if (i % kKdBlock == 0) loc = 1.f;
       pre *= a; loc *= a;
-      T hi, lo;
-      kd_split<T>(q * pre, hi, lo);
-      ops.qg[i * (DP + 8) + d] = hi; ops.qg[ops.plane + i * (DP + 8) + d] = lo;
-      w[i] = kk[i] * pre;
+      put(L.qg, L.plane1, L.rows1, (kd_tc(DP) && DELTA ? kKdChunk : 0) + i, q * pre);
+      if constexpr (DELTA) w[i] = kk[i] * pre;
       sq[i * P + d] = q * loc; sk[i * P + d] = kk[i] * loc;
       if (i % kKdBlock == kKdBlock - 1) sb[i / kKdBlock * DP + d] = loc;
     }
@@ -155,13 +292,11 @@ __global__ void __launch_bounds__(kKdThreads) key_decay_prepare_kernel(const KdP
     for (int i = kKdChunk - 1; i >= 0; i--) {
       if (i % kKdBlock == kKdBlock - 1) loc = 1.f;
       const float a = sa[i * P + d];
-      T hi, lo;
-      kd_split<T>(kk[i] * suf, hi, lo);
-      ops.kg[i * (DP + 8) + d] = hi; ops.kg[ops.plane + i * (DP + 8) + d] = lo;
+      put(L.kg, L.plane2, kKdChunk, i, kk[i] * suf);
       sa[i * P + d] = kk[i] * loc;
       suf *= a; loc *= a;
     }
-    ops.decay[d] = suf;
+    reinterpret_cast<float*>(ops + L.decay)[d] = suf;
   }
   __syncthreads();
   if (warp < 6) {
@@ -196,50 +331,51 @@ __global__ void __launch_bounds__(kKdThreads) key_decay_prepare_kernel(const KdP
     if constexpr (DELTA) { sK[i * 36 + j] = acc[2] * s_beta[i]; sK[i * 36 + j + 1] = acc[3] * s_beta[i]; }
   }
   __syncthreads();
-  for (int i = tid; i < kKdChunk * kKdAPitch; i += kKdThreads) {
-    const int r = i / kKdAPitch, j = i % kKdAPitch;
-    T hi, lo;
-    kd_split<T>(j < kKdChunk ? sQ[r * 36 + j] : 0.f, hi, lo);
-    ops.a[i] = hi; ops.a[kKdChunk * kKdAPitch + i] = lo;
+  {
+    const int i = tid >> 3, j = (tid & 7) * 4;
+    const float4 v = *reinterpret_cast<const float4*>(sQ + i * 36 + j);
+    uint2 hi, lo;
+    kd_split2<T>(v.x, v.y, hi.x, lo.x);
+    kd_split2<T>(v.z, v.w, hi.y, lo.y);
+    uint8_t* at = ops + L.q + (kd_tc(DP) ? i * 128 : i * kKdAPitch * 2);
+    if constexpr (kd_tc(DP)) {
+      *reinterpret_cast<uint2*>(at + ((j * 2) ^ ((i & 7) << 4))) = hi;
+      *reinterpret_cast<uint2*>(at + ((64 + j * 2) ^ ((i & 7) << 4))) = lo;
+    } else {
+      *reinterpret_cast<uint2*>(at + j * 2) = hi;
+      *reinterpret_cast<uint2*>(at + kKdChunk * kKdAPitch * 2 + j * 2) = lo;
+    }
   }
-  // forward substitution, a thread per column: W first, then the value columns
-  auto solve = [&](float (&x)[kKdChunk]) {
+  if constexpr (DELTA) {
+    // forward substitution, a thread per column
+    auto solve = [&](float (&x)[kKdChunk]) {
 #pragma unroll
-    for (int i = 0; i < kKdChunk; i++) {
-      float v = x[i] * s_beta[i];
+      for (int i = 0; i < kKdChunk; i++) {
+        float v = x[i] * s_beta[i];
 #pragma unroll
-      for (int j = 0; j < i; j += 4) {
-        const float4 f = *reinterpret_cast<const float4*>(sK + i * 36 + j);      // zero from the diagonal on
-        v = fmaf(-f.x, x[j], v);
-        if (j + 1 < i) v = fmaf(-f.y, x[j + 1], v);
-        if (j + 2 < i) v = fmaf(-f.z, x[j + 2], v);
-        if (j + 3 < i) v = fmaf(-f.w, x[j + 3], v);
+        for (int j = 0; j < i; j += 4) {
+          const float4 f = *reinterpret_cast<const float4*>(sK + i * 36 + j);      // zero from the diagonal on
+          v = fmaf(-f.x, x[j], v);
+          if (j + 1 < i) v = fmaf(-f.y, x[j + 1], v);
+          if (j + 2 < i) v = fmaf(-f.z, x[j + 2], v);
+          if (j + 3 < i) v = fmaf(-f.w, x[j + 3], v);
+        }
+        x[i] = v;
       }
-      x[i] = v;
+    };
+    if (tid < DP || e_own < E) {
+      solve(w);
+      if (tid < DP) {
+#pragma unroll
+        for (int i = 0; i < kKdChunk; i++) put(L.w, L.plane1, L.rows1, i, -w[i]);
+      } else store_u(e_own, w);
     }
-  };
-  if (DELTA && tid < DP) {
-    solve(w);
-#pragma unroll
-    for (int i = 0; i < kKdChunk; i++) {
-      T hi, lo;
-      kd_split<T>(-w[i], hi, lo);
-      ops.w[i * (DP + 8) + tid] = hi; ops.w[ops.plane + i * (DP + 8) + tid] = lo;
-    }
-  }
-  const int first = DELTA ? DP : 0;
-  for (int e = tid < first ? tid + kKdThreads - first : tid - first; e < E; e += kKdThreads) {
-    const int ch = h * E + e;
-#pragma unroll
-    for (int i = 0; i < kKdChunk; i++) w[i] = i < nt ? kd_input<T>(p, base, ring, pos, t0 + i, p.v_off + ch, 2 * p.qk_heads * D + ch) : 0.f;
-    if constexpr (DELTA) solve(w);
-    float4* u = reinterpret_cast<float4*>(p.u + (chunk * E + e) * kKdChunk);
-#pragma unroll
-    for (int i = 0; i < kKdChunk; i += 4) u[i / 4] = make_float4(w[i], w[i + 1], w[i + 2], w[i + 3]);
+#pragma unroll 1
+    for (int e = tid + kKdThreads - DP; e < E; e += kKdThreads) { load_v(e, w); solve(w); store_u(e, w); }
   }
 }
 
-// ── scan ────────────────────────────────────────────────────────────────────
+// ── scan, warp-level products (more than 128 channels) ──────────────────────
 // Fragments of the transposed problem: accumulators hold S^T [16 value columns, DP], u^T and o^T [16, 32 tokens]; a pair of
 // neighbouring accumulator tiles is one A operand of the next product. The chunks' operands arrive in two stages by bulk copies,
 // issued by one lane when every warp is done with the stage.
@@ -258,6 +394,7 @@ template <typename T, int DP, bool DELTA>
 __global__ void __launch_bounds__(256) key_decay_scan_kernel(const KdParams p, int* status) {
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ uint64_t full[2], empty[2];
+  constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
   constexpr int P = DP + 8, DT = DP / 8, NT = kKdChunk / 8, plane = kKdChunk * P, aplane = kKdChunk * kKdAPitch;
   const int warps = (int)blockDim.x / 32, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
   const int h = blockIdx.y, s = blockIdx.z, E = p.vdim, D = p.dim;
@@ -270,8 +407,8 @@ __global__ void __launch_bounds__(256) key_decay_scan_kernel(const KdParams p, i
   pdl_wait();
   pdl_trigger();
   auto fetch = [&](int c) {
-    mbar_expect_tx(&full[c & 1], (uint32_t)p.ops_bytes);
-    kd_bulk_load(smem + (c & 1) * p.ops_bytes, p.ops + (sh * p.chunks + c) * p.ops_bytes, (uint32_t)p.ops_bytes, &full[c & 1]);
+    mbar_expect_tx(&full[c & 1], (uint32_t)L.bytes);
+    kd_bulk_load(smem + (c & 1) * L.stride, p.ops + (sh * p.chunks + c) * L.stride, (uint32_t)L.bytes, &full[c & 1]);
   };
   if (threadIdx.x == 0) { fetch(0); if (p.chunks > 1) fetch(1); }
   const int e0 = ((int)blockIdx.x * warps + warp) * 16 + g, e1 = e0 + 8;
@@ -298,7 +435,7 @@ __global__ void __launch_bounds__(256) key_decay_scan_kernel(const KdParams p, i
     if (threadIdx.x == 0 && c > 0 && c + 1 < p.chunks && mbar_wait(&empty[sg ^ 1], (uint32_t)(((c - 1) >> 1) & 1), status, 61)) fetch(c + 1);
     __syncwarp();
     if (!__all_sync(0xffffffffu, mbar_wait(&full[sg], (uint32_t)((c >> 1) & 1), status, 62))) return;
-    const T* qg = reinterpret_cast<const T*>(smem + sg * p.ops_bytes);
+    const T* qg = reinterpret_cast<const T*>(smem + sg * L.stride);
     const T* w = qg + 2 * plane;
     const T* kg = w + (DELTA ? 2 * plane : 0);
     const T* am = kg + 2 * plane;
@@ -380,76 +517,336 @@ __global__ void __launch_bounds__(256) key_decay_scan_kernel(const KdParams p, i
     for (int x = 0; x < 4; x++) { const int d = n * 8 + 2 * q + (x & 1), e = x < 2 ? e0 : e1; if (d < D && e < E) S[(long long)d * E + e] = st[n][x]; }
 }
 
-// ── finish: norm and gate of one head's outputs, a warp each ────────────────
-template <typename T, int VEC>
+// ── scan on tcgen05 (up to 128 channels) ────────────────────────────────────
+// A CTA: 128 value columns (lanes of tensor memory) of one head. Tensor memory columns: S^T in float32 [DP]; its high parts and
+// remainders as A operand [DP]; two buffers of (u^T | o^T) [32 | 32]; u^T split [16 + 16]. Per chunk:
+//   warps 0 - 3   split S, fade it in place                         (wait: update of the chunk before)
+//   warp 8        (u | o) = S (-W | A q)                            delta rule; otherwise o alone
+//   warps 0 - 3   u += U, split
+//   warp 8        o += u Q, S += u (A_32 / A k)
+//   warps 4 - 7   o to memory, or through the head's norm and gate
+// Warp 9 loads the chunks' operands. All waits are bounded.
+template <typename T, int DP, bool DELTA>
+__global__ void __launch_bounds__(320, 1) key_decay_scan_tc_kernel(const KdParams p, int fuse, int* status) {
+  using namespace sm100;
+  constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
+  constexpr uint32_t cS = 0, cA = 128, cO = 256, cU = 384;
+  constexpr int kSteps = DP / 16;
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ uint64_t full[2], empty[2], s_ready, u_ready, u_full, s_full, o_full[2], o_free[2], sums;
+  __shared__ uint32_t tmem_slot;
+  __shared__ float s_sum[2][4][32];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quarter = warp & 3;
+  const int h = blockIdx.y, s = blockIdx.z, E = p.vdim, D = p.dim;
+  const long long sh = (long long)s * p.heads + h;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < 2; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], 5); mbar_init(&o_full[i], 1); mbar_init(&o_free[i], 4); }
+    mbar_init(&s_ready, 4); mbar_init(&u_ready, 4); mbar_init(&u_full, 1); mbar_init(&s_full, 1); mbar_init(&sums, 4);
+    mbar_fence_init();
+  }
+  if (warp == 8) { tmem_alloc(&tmem_slot, 512); tmem_relinquish(); }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tm = tmem_slot;
+  pdl_wait();
+  pdl_trigger();
+  const int e = (int)blockIdx.x * 128 + quarter * 32 + lane;         // value column of the threads that own one
+  const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
+  if (warp == 9) {
+    if (lane == 0)
+      for (int c = 0; c < p.chunks; c++) {
+        const int st = c & 1;
+        if (!mbar_wait(&empty[st], (uint32_t)((c >> 1) & 1) ^ 1, status, 61)) break;
+        mbar_expect_tx(&full[st], (uint32_t)L.bytes);
+        kd_bulk_load(smem + st * L.stride, p.ops + (sh * p.chunks + c) * L.stride, (uint32_t)L.bytes, &full[st]);
+      }
+  } else if (warp == 8) {
+    if (lane == 0) {
+      constexpr int fmt = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
+      const uint32_t id_1 = make_idesc_f16(fmt, 0, 0, 128, L.rows1), id_o = make_idesc_f16(fmt, 0, 0, 128, kKdChunk), id_s = make_idesc_f16(fmt, 0, 1, 128, DP);
+      const bool exact = !DELTA && p.taps == 0;                      // u is the stored v: no remainder
+      for (int c = 0; c < p.chunks; c++) {
+        const int st = c & 1;
+        const uint32_t ph = (uint32_t)(c & 1), ph2 = (uint32_t)((c >> 1) & 1), base = smem_u32(smem + st * L.stride);
+        const uint32_t acc0 = tm + cO + (uint32_t)(st * 64), acc_o = acc0 + (DELTA ? 32u : 0u);
+        if (!mbar_wait(&full[st], ph2, status, 62) || !mbar_wait(&o_free[st], ph2 ^ 1, status, 63) || !mbar_wait(&s_ready, ph, status, 64)) break;
+        tc_fence_after_sync();
+#pragma unroll
+        for (int part = 0; part < 3; part++)                         // high x high, remainder x high, high x remainder
+#pragma unroll
+          for (int k = 0; k < kSteps; k++)
+            mma_f16_ts(acc0, tm + cA + (uint32_t)((part == 1 ? DP / 2 : 0) + k * 8),
+                       make_smem_desc_sw128(base + (part == 2 ? L.plane1 : 0) + (k >> 2) * L.rows1 * 128 + (k & 3) * 32, 16, 1024), id_1, part > 0 || k > 0 ? 1u : 0u);
+        if constexpr (DELTA) {
+          mma_commit(&u_full);
+          if (!mbar_wait(&u_ready, ph, status, 65)) break;
+          tc_fence_after_sync();
+        }
+#pragma unroll
+        for (int part = 0; part < 3; part++) {
+          if (part == 1 && exact) continue;
+#pragma unroll
+          for (int k = 0; k < kKdChunk / 16; k++) {
+            const uint32_t a = tm + cU + (uint32_t)((part == 1 ? 16 : 0) + k * 8);
+            mma_f16_ts(acc_o, a, make_smem_desc_sw128(base + L.q + (part == 2 ? 64 : 0) + k * 32, 16, 1024), id_o, 1u);
+            mma_f16_ts(tm + cS, a, make_smem_desc_sw128(base + L.kg + (part == 2 ? L.plane2 : 0) + k * 2048, kKdChunk * 128, 1024), id_s, 1u);
+          }
+        }
+        mma_commit(&o_full[st]);
+        mma_commit(&s_full);
+        mma_commit(&empty[st]);
+      }
+    }
+  } else if (warp < 4) {
+    float* S = p.state(s) + (long long)h * D * E;
+    uint32_t x[32];
+#pragma unroll 1
+    for (int g = 0; g < DP / 32; g++) {
+      const float* row = S + (long long)g * 32 * E + e;
+#pragma unroll
+      for (int i = 0; i < 32; i++, row += E) x[i] = g * 32 + i < D && e < E ? __float_as_uint(*row) : 0u;
+      tmem_st_32x32(tm + cS + lanes + (uint32_t)(g * 32), x);
+    }
+    tmem_st_wait();
+    bool ok = true;
+    auto split = [&](const float (&v)[32], uint32_t at, uint32_t lo_off) {
+      uint32_t hi[16], lo[16];
+#pragma unroll
+      for (int i = 0; i < 16; i++) kd_split2<T>(v[2 * i], v[2 * i + 1], hi[i], lo[i]);
+      tmem_st_32x16(at, hi);
+      tmem_st_32x16(at + lo_off, lo);
+    };
+    for (int c = 0; c < p.chunks; c++) {
+      const int st = c & 1;
+      const uint32_t ph = (uint32_t)(c & 1);
+      float u[32];
+      const float4* U = reinterpret_cast<const float4*>(p.u + ((sh * p.chunks + c) * E + min(e, E - 1)) * kKdChunk);
+#pragma unroll
+      for (int i = 0; i < 8; i++) {
+        const float4 f = e < E ? __ldcs(U + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        u[4 * i] = f.x; u[4 * i + 1] = f.y; u[4 * i + 2] = f.z; u[4 * i + 3] = f.w;
+      }
+      ok = __all_sync(0xffffffffu, mbar_wait(&full[st], (uint32_t)((c >> 1) & 1), status, 66) && (c == 0 || mbar_wait(&s_full, ph ^ 1, status, 67)));
+      if (!ok) break;
+      tc_fence_after_sync();
+      const float4* decay = reinterpret_cast<const float4*>(smem + st * L.stride + L.decay);
+#pragma unroll
+      for (int g = 0; g < DP / 32; g++) {
+        tmem_ld_32x32(tm + cS + lanes + (uint32_t)(g * 32), x);
+        tmem_ld_wait();
+        float v[32];
+#pragma unroll
+        for (int i = 0; i < 32; i++) v[i] = __uint_as_float(x[i]);
+        split(v, tm + cA + lanes + (uint32_t)(g * 16), DP / 2);
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+          const float4 f = decay[g * 8 + i];
+          x[4 * i] = __float_as_uint(v[4 * i] * f.x); x[4 * i + 1] = __float_as_uint(v[4 * i + 1] * f.y);
+          x[4 * i + 2] = __float_as_uint(v[4 * i + 2] * f.z); x[4 * i + 3] = __float_as_uint(v[4 * i + 3] * f.w);
+        }
+        tmem_st_32x32(tm + cS + lanes + (uint32_t)(g * 32), x);
+      }
+      if constexpr (!DELTA) split(u, tm + cU + lanes, 16);
+      tmem_st_wait();
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) { mbar_arrive(&s_ready); mbar_arrive(&empty[st]); }
+      if constexpr (DELTA) {
+        ok = __all_sync(0xffffffffu, mbar_wait(&u_full, ph, status, 68));
+        if (!ok) break;
+        tc_fence_after_sync();
+        tmem_ld_32x32(tm + cO + lanes + (uint32_t)(st * 64), x);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; i++) u[i] += __uint_as_float(x[i]);
+        split(u, tm + cU + lanes, 16);
+        tmem_st_wait();
+        tc_fence_before_sync();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&u_ready);
+      }
+    }
+    ok = ok && __all_sync(0xffffffffu, mbar_wait(&s_full, (uint32_t)((p.chunks - 1) & 1), status, 69));
+    if (ok) {
+      tc_fence_after_sync();
+#pragma unroll 1
+      for (int g = 0; g < DP / 32; g++) {
+        tmem_ld_32x32(tm + cS + lanes + (uint32_t)(g * 32), x);
+        tmem_ld_wait();
+        float* row = S + (long long)g * 32 * E + e;
+#pragma unroll
+        for (int i = 0; i < 32; i++, row += E) if (g * 32 + i < D && e < E) *row = __uint_as_float(x[i]);
+      }
+      tc_fence_before_sync();
+    }
+  } else {
+    const float nw = e < E ? p.norm[e] : 0.f;
+    for (int c = 0; c < p.chunks; c++) {
+      const int st = c & 1, t0 = c * kKdChunk, nt = min(kKdChunk, p.T - t0);
+      const long long row0 = (long long)s * p.T + t0;
+      uint16_t gate[kKdChunk];
+      if (fuse) {
+        const T* g = p.gate ? reinterpret_cast<const T*>(p.gate) + row0 * p.gate_ld + (long long)h * E + e : reinterpret_cast<const T*>(p.proj) + row0 * p.ld + p.g_off + (long long)h * E + e;
+        const long long ld = p.gate ? p.gate_ld : p.ld;
+#pragma unroll
+        for (int i = 0; i < kKdChunk; i++) gate[i] = e < E && i < nt ? *reinterpret_cast<const uint16_t*>(g + i * ld) : (uint16_t)0;
+      }
+      if (!__all_sync(0xffffffffu, mbar_wait(&o_full[st], (uint32_t)((c >> 1) & 1), status, 70))) break;
+      tc_fence_after_sync();
+      uint32_t o[32];
+      tmem_ld_32x32(tm + cO + lanes + (uint32_t)(st * 64 + (DELTA ? 32 : 0)), o);
+      tmem_ld_wait();
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&o_free[st]);
+      if (!fuse) {
+        float* O = p.o + (row0 * p.heads + h) * E + e;
+#pragma unroll
+        for (int i = 0; i < kKdChunk; i++) if (i < nt && e < E) O[(long long)i * p.heads * E] = __uint_as_float(o[i]);
+        continue;
+      }
+      // sums of squares over the value columns: after five halvings lane t holds token t's
+      float v[32];
+#pragma unroll
+      for (int i = 0; i < 32; i++) { const float f = __uint_as_float(o[i]); v[i] = f * f; }
+#pragma unroll
+      for (int w = 16; w > 0; w >>= 1) {
+        const bool up = lane & w;
+#pragma unroll
+        for (int i = 0; i < w; i++) {
+          const float other = __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + w], w);
+          v[i] = (up ? v[i + w] : v[i]) + other;
+        }
+      }
+      s_sum[st][quarter][lane] = v[0];
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&sums);
+      if (!__all_sync(0xffffffffu, mbar_wait(&sums, (uint32_t)st, status, 71))) break;
+      const float rs = 1.0f / sqrtf((s_sum[st][0][lane] + s_sum[st][1][lane] + s_sum[st][2][lane] + s_sum[st][3][lane]) / (float)E + p.eps);
+      T* y = reinterpret_cast<T*>(p.y) + row0 * p.y_ld + (long long)h * E + e;
+#pragma unroll
+      for (int i = 0; i < kKdChunk; i++) {
+        const float f = __shfl_sync(0xffffffffu, rs, i);
+        T g;
+        *reinterpret_cast<uint16_t*>(&g) = gate[i];
+        if (e < E && i < nt) y[i * p.y_ld] = Cvt<T>::from(__uint_as_float(o[i]) * f * nw * kd_gate_fast<T>(p, g));
+      }
+    }
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  if (warp == 8) tmem_dealloc(tm, 512);
+}
+
+// ── finish: norm and gate of the heads' outputs, a warp each ────────────────
+// REG: float4 pieces of a head a lane keeps; 0: any width and alignment, read twice
+constexpr int kKdItems = 2;            // heads a warp works on
+template <typename T, int REG>
 __global__ void __launch_bounds__(256) key_decay_finish_kernel(const KdParams p) {
   pdl_wait();
   pdl_trigger();
   const int lane = threadIdx.x & 31, E = p.vdim;
-  const long long i = (long long)blockIdx.x * 8 + (threadIdx.x >> 5), rows = (long long)p.n_seq * p.T;
-  if (i >= rows * p.heads) return;
-  const long long r = i / p.heads;
-  const int h = (int)(i % p.heads);
-  const float* o = p.o + i * E;
-  const T* gate = p.gate ? reinterpret_cast<const T*>(p.gate) + r * p.gate_ld + (long long)h * E : reinterpret_cast<const T*>(p.proj) + r * p.ld + p.g_off + (long long)h * E;
-  T* y = reinterpret_cast<T*>(p.y) + r * p.y_ld + (long long)h * E;
-  float sq = 0.f;
-  for (int e = lane * VEC; e < E; e += 32 * VEC) {
-    if constexpr (VEC == 4) { const float4 v = *reinterpret_cast<const float4*>(o + e); sq = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sq)))); }
-    else sq = fmaf(o[e], o[e], sq);
-  }
-  const float rs = 1.0f / sqrtf(warp_sum(sq) / (float)E + p.eps);
-  for (int e = lane * VEC; e < E; e += 32 * VEC) {
-    if constexpr (VEC == 4) {
-      const float4 v = *reinterpret_cast<const float4*>(o + e), w = *reinterpret_cast<const float4*>(p.norm + e);
-      const uint2 graw = *reinterpret_cast<const uint2*>(gate + e);
-      const T* gv = reinterpret_cast<const T*>(&graw);
-      uint2 out;
-      out.x = pack2_t<T>(v.x * rs * w.x * kd_gate(p, Cvt<T>::to(gv[0])), v.y * rs * w.y * kd_gate(p, Cvt<T>::to(gv[1])));
-      out.y = pack2_t<T>(v.z * rs * w.z * kd_gate(p, Cvt<T>::to(gv[2])), v.w * rs * w.w * kd_gate(p, Cvt<T>::to(gv[3])));
-      *reinterpret_cast<uint2*>(y + e) = out;
-    } else y[e] = Cvt<T>::from(o[e] * rs * p.norm[e] * kd_gate(p, Cvt<T>::to(gate[e])));
+  const long long items = (long long)p.n_seq * p.T * p.heads, i0 = ((long long)blockIdx.x * 8 + (threadIdx.x >> 5)) * kKdItems;
+  auto gate_of = [&](long long i) {
+    const long long r = (uint32_t)i / (uint32_t)p.heads, c = (long long)((uint32_t)i % (uint32_t)p.heads) * E;
+    return p.gate ? reinterpret_cast<const T*>(p.gate) + r * p.gate_ld + c : reinterpret_cast<const T*>(p.proj) + r * p.ld + p.g_off + c;
+  };
+  auto out_of = [&](long long i) { return reinterpret_cast<T*>(p.y) + (long long)((uint32_t)i / (uint32_t)p.heads) * p.y_ld + (long long)((uint32_t)i % (uint32_t)p.heads) * E; };
+  if constexpr (REG > 0) {
+    float4 v[kKdItems][REG];
+    uint2 z[kKdItems][REG];
+#pragma unroll
+    for (int n = 0; n < kKdItems; n++)
+#pragma unroll
+      for (int q = 0; q < REG; q++) {
+        const int e = (lane + 32 * q) * 4;
+        v[n][q] = make_float4(0.f, 0.f, 0.f, 0.f);
+        z[n][q] = make_uint2(0u, 0u);
+        if (i0 + n < items && e < E) { v[n][q] = __ldcs(reinterpret_cast<const float4*>(p.o + (i0 + n) * E + e)); z[n][q] = *reinterpret_cast<const uint2*>(gate_of(i0 + n) + e); }
+      }
+#pragma unroll
+    for (int n = 0; n < kKdItems; n++) {
+      float sq = 0.f;
+#pragma unroll
+      for (int q = 0; q < REG; q++) sq = fmaf(v[n][q].x, v[n][q].x, fmaf(v[n][q].y, v[n][q].y, fmaf(v[n][q].z, v[n][q].z, fmaf(v[n][q].w, v[n][q].w, sq))));
+      const float rs = 1.0f / sqrtf(warp_sum(sq) / (float)E + p.eps);
+#pragma unroll
+      for (int q = 0; q < REG; q++) {
+        const int e = (lane + 32 * q) * 4;
+        if (i0 + n >= items || e >= E) continue;
+        const float4 x = v[n][q], w = __ldg(reinterpret_cast<const float4*>(p.norm + e));
+        const T* gv = reinterpret_cast<const T*>(&z[n][q]);
+        uint2 out;
+        out.x = pack2_t<T>(x.x * rs * w.x * kd_gate_fast<T>(p, gv[0]), x.y * rs * w.y * kd_gate_fast<T>(p, gv[1]));
+        out.y = pack2_t<T>(x.z * rs * w.z * kd_gate_fast<T>(p, gv[2]), x.w * rs * w.w * kd_gate_fast<T>(p, gv[3]));
+        *reinterpret_cast<uint2*>(out_of(i0 + n) + e) = out;
+      }
+    }
+  } else {
+    for (long long i = i0; i < i0 + kKdItems && i < items; i++) {
+      const float* o = p.o + i * E;
+      const T* g = gate_of(i);
+      T* y = out_of(i);
+      float sq = 0.f;
+      for (int e = lane; e < E; e += 32) sq = fmaf(o[e], o[e], sq);
+      const float rs = 1.0f / sqrtf(warp_sum(sq) / (float)E + p.eps);
+      for (int e = lane; e < E; e += 32) y[e] = Cvt<T>::from(o[e] * rs * p.norm[e] * kd_gate_fast<T>(p, g[e]));
+    }
   }
 }
 
 // ── host ────────────────────────────────────────────────────────────────────
 template <typename T, int DP, bool DELTA>
-static cudaError_t launch_kd(cudaStream_t s, const KdParams& p, int warps) {
-  constexpr size_t prep = ((size_t)3 * kKdChunk * (DP + 4) + kKdBlocks * DP + 2 * kKdChunk * 36 + kKdChunk) * sizeof(float);
-  const size_t scan = 2 * (size_t)p.ops_bytes;
+static cudaError_t launch_kd(cudaStream_t s, const KdParams& p) {
+  constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
+  constexpr size_t prep = ((size_t)3 * kKdChunk * (DP + 4) + kKdBlocks * DP + 2 * kKdChunk * 36 + 3 * kKdChunk) * sizeof(float);
+  constexpr size_t scan = 2 * (size_t)L.stride + (kd_tc(DP) ? 1024 : 0);
   static bool attr = false;
   if (!attr) {
     cudaError_t e = cudaFuncSetAttribute(key_decay_prepare_kernel<T, DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(key_decay_scan_kernel<T, DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)scan);
+    if (e == cudaSuccess) {
+      if constexpr (kd_tc(DP)) e = cudaFuncSetAttribute(key_decay_scan_tc_kernel<T, DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)scan);
+      else e = cudaFuncSetAttribute(key_decay_scan_kernel<T, DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)scan);
+    }
     if (e != cudaSuccess) return e;
     attr = true;
   }
   cudaError_t e = launch_pdl(key_decay_prepare_kernel<T, DP, DELTA>, dim3((unsigned)p.chunks, (unsigned)p.heads, (unsigned)p.n_seq), dim3(kKdThreads), prep, s, p);
   if (e != cudaSuccess) return e;
-  const unsigned slices = (unsigned)((p.vdim + 16 * warps - 1) / (16 * warps));
-  return launch_pdl(key_decay_scan_kernel<T, DP, DELTA>, dim3(slices, (unsigned)p.heads, (unsigned)p.n_seq), dim3((unsigned)warps * 32), scan, s, p, matmul_status_word());
+  if constexpr (kd_tc(DP)) {
+    return launch_pdl(key_decay_scan_tc_kernel<T, DP, DELTA>, dim3((unsigned)((p.vdim + 127) / 128), (unsigned)p.heads, (unsigned)p.n_seq), dim3(320), scan, s, p, kd_fused(p) ? 1 : 0,
+                      matmul_status_word());
+  } else {
+    // value columns per CTA: up to 128, fewer where that leaves SMs without work
+    int warps = std::min(8, (p.vdim + 15) / 16);
+    while (warps > 2 && (long long)p.n_seq * p.heads * ((p.vdim + 16 * warps - 1) / (16 * warps)) < sm_count()) warps = (warps + 1) / 2;
+    return launch_pdl(key_decay_scan_kernel<T, DP, DELTA>, dim3((unsigned)((p.vdim + 16 * warps - 1) / (16 * warps)), (unsigned)p.heads, (unsigned)p.n_seq), dim3((unsigned)warps * 32), scan, s, p,
+                      matmul_status_word());
+  }
 }
 template <typename T, bool DELTA>
-static cudaError_t launch_kd_dp(cudaStream_t s, const KdParams& p, int warps) {
+static cudaError_t launch_kd_dp(cudaStream_t s, const KdParams& p) {
   switch (p.dp) {
-    case 32: return launch_kd<T, 32, DELTA>(s, p, warps);
-    case 64: return launch_kd<T, 64, DELTA>(s, p, warps);
-    case 96: return launch_kd<T, 96, DELTA>(s, p, warps);
-    case 128: return launch_kd<T, 128, DELTA>(s, p, warps);
-    case 192: return launch_kd<T, 192, DELTA>(s, p, warps);
-    default: return launch_kd<T, 256, DELTA>(s, p, warps);
+    case 32: return launch_kd<T, 32, DELTA>(s, p);
+    case 64: return launch_kd<T, 64, DELTA>(s, p);
+    case 96: return launch_kd<T, 96, DELTA>(s, p);
+    case 128: return launch_kd<T, 128, DELTA>(s, p);
+    case 192: return launch_kd<T, 192, DELTA>(s, p);
+    default: return launch_kd<T, 256, DELTA>(s, p);
   }
 }
 template <typename T>
 static Status launch_chunked(cudaStream_t s, const KdParams& p) {
-  // value columns per CTA: up to 128, fewer where that leaves SMs without work
-  int warps = std::min(8, (p.vdim + 15) / 16);
-  while (warps > 2 && (long long)p.n_seq * p.heads * ((p.vdim + 16 * warps - 1) / (16 * warps)) < sm_count()) warps = (warps + 1) / 2;
-  cudaError_t e = p.delta ? launch_kd_dp<T, true>(s, p, warps) : launch_kd_dp<T, false>(s, p, warps);
-  if (e != cudaSuccess) return cuda_status(e, "key decay (chunked)");
-  const unsigned blocks = (unsigned)(((long long)p.n_seq * p.T * p.heads + 7) / 8);
+  cudaError_t e = p.delta ? launch_kd_dp<T, true>(s, p) : launch_kd_dp<T, false>(s, p);
+  if (e != cudaSuccess || kd_fused(p)) return cuda_status(e, "key decay (chunked)");
+  const unsigned blocks = (unsigned)(((long long)p.n_seq * p.T * p.heads + 8 * kKdItems - 1) / (8 * kKdItems));
   const bool vec = p.vdim % 4 == 0 && p.y_ld % 4 == 0 && aligned16(p.y) && aligned16(p.norm) && (p.gate ? p.gate_ld % 4 == 0 : p.ld % 4 == 0 && p.g_off % 4 == 0 && aligned16(p.proj));
-  e = vec ? launch_pdl(key_decay_finish_kernel<T, 4>, dim3(blocks), dim3(256), 0, s, p) : launch_pdl(key_decay_finish_kernel<T, 1>, dim3(blocks), dim3(256), 0, s, p);
+  if (vec && p.vdim <= 128) e = launch_pdl(key_decay_finish_kernel<T, 1>, dim3(blocks), dim3(256), 0, s, p);
+  else if (vec && p.vdim <= 256) e = launch_pdl(key_decay_finish_kernel<T, 2>, dim3(blocks), dim3(256), 0, s, p);
+  else e = launch_pdl(key_decay_finish_kernel<T, 0>, dim3(blocks), dim3(256), 0, s, p);
   return cuda_status(e, "key decay (chunked)");
 }
 

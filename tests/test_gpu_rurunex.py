@@ -100,7 +100,7 @@ def kd_want(c, b):
         q, k = R.unit(q), R.unit(k)
     q, k = np.repeat(q * d ** -0.5, H // G, axis=1), np.repeat(k, H // G, axis=1)
     zz = (c["a1"][b].astype(np.float64) @ c["a2"].T + c["bias"]).reshape(T, H, d)
-    a = np.exp(-c["rate"][:, None] * R.softplus(zz)) if c["softplus"] else R.sigmoid(zz) ** (1 / c["tau"])
+    a = np.exp(-c["rate"][:, None] * R.softplus(zz) if c["softplus"] else R.log_sigmoid(zz) / c["tau"])
     S = np.zeros((H, d, e))
     if c["delta"]:
         o, S = R.delta_recurrence(q, k, v, a, R.sigmoid(c["beta"][b].astype(np.float64)), S)
