@@ -573,12 +573,14 @@ __global__ void __launch_bounds__(320, 1) key_decay_scan_tc_kernel(const KdParam
         const uint32_t acc0 = tm + cO + (uint32_t)(st * 64), acc_o = acc0 + (DELTA ? 32u : 0u);
         if (!mbar_wait(&full[st], ph2, status, 62) || !mbar_wait(&o_free[st], ph2 ^ 1, status, 63) || !mbar_wait(&s_ready, ph, status, 64)) break;
         tc_fence_after_sync();
+        // a descriptor's address field counts 16-byte units: offsets are added to it
+        const uint64_t d1 = make_smem_desc_sw128(base, 16, 1024), dq = d1 + (L.q >> 4), ds = make_smem_desc_sw128(base + L.kg, kKdChunk * 128, 1024);
 #pragma unroll
         for (int part = 0; part < 3; part++)                         // high x high, remainder x high, high x remainder
 #pragma unroll
           for (int k = 0; k < kSteps; k++)
-            mma_f16_ts(acc0, tm + cA + (uint32_t)((part == 1 ? DP / 2 : 0) + k * 8),
-                       make_smem_desc_sw128(base + (part == 2 ? L.plane1 : 0) + (k >> 2) * L.rows1 * 128 + (k & 3) * 32, 16, 1024), id_1, part > 0 || k > 0 ? 1u : 0u);
+            mma_f16_ts(acc0, tm + cA + (uint32_t)((part == 1 ? DP / 2 : 0) + k * 8), d1 + (((part == 2 ? L.plane1 : 0) + (k >> 2) * L.rows1 * 128 + (k & 3) * 32) >> 4), id_1,
+                       part > 0 || k > 0 ? 1u : 0u);
         if constexpr (DELTA) {
           mma_commit(&u_full);
           if (!mbar_wait(&u_ready, ph, status, 65)) break;
@@ -588,14 +590,18 @@ __global__ void __launch_bounds__(320, 1) key_decay_scan_tc_kernel(const KdParam
         for (int part = 0; part < 3; part++) {
           if (part == 1 && exact) continue;
 #pragma unroll
-          for (int k = 0; k < kKdChunk / 16; k++) {
-            const uint32_t a = tm + cU + (uint32_t)((part == 1 ? 16 : 0) + k * 8);
-            mma_f16_ts(acc_o, a, make_smem_desc_sw128(base + L.q + (part == 2 ? 64 : 0) + k * 32, 16, 1024), id_o, 1u);
-            mma_f16_ts(tm + cS, a, make_smem_desc_sw128(base + L.kg + (part == 2 ? L.plane2 : 0) + k * 2048, kKdChunk * 128, 1024), id_s, 1u);
-          }
+          for (int k = 0; k < kKdChunk / 16; k++)
+            mma_f16_ts(tm + cS, tm + cU + (uint32_t)((part == 1 ? 16 : 0) + k * 8), ds + (((part == 2 ? L.plane2 : 0) + k * 2048) >> 4), id_s, 1u);
+        }
+        mma_commit(&s_full);
+#pragma unroll
+        for (int part = 0; part < 3; part++) {
+          if (part == 1 && exact) continue;
+#pragma unroll
+          for (int k = 0; k < kKdChunk / 16; k++)
+            mma_f16_ts(acc_o, tm + cU + (uint32_t)((part == 1 ? 16 : 0) + k * 8), dq + (((part == 2 ? 64 : 0) + k * 32) >> 4), id_o, 1u);
         }
         mma_commit(&o_full[st]);
-        mma_commit(&s_full);
         mma_commit(&empty[st]);
       }
     }
@@ -632,23 +638,29 @@ __global__ void __launch_bounds__(320, 1) key_decay_scan_tc_kernel(const KdParam
       if (!ok) break;
       tc_fence_after_sync();
       const float4* decay = reinterpret_cast<const float4*>(smem + st * L.stride + L.decay);
+      uint32_t y[2][32];                                  // the next columns are on their way while these are split
+      tmem_ld_32x32(tm + cS + lanes, y[0]);
 #pragma unroll
       for (int g = 0; g < DP / 32; g++) {
-        tmem_ld_32x32(tm + cS + lanes + (uint32_t)(g * 32), x);
         tmem_ld_wait();
+        if (g + 1 < DP / 32) tmem_ld_32x32(tm + cS + lanes + (uint32_t)((g + 1) * 32), y[(g + 1) & 1]);
         float v[32];
 #pragma unroll
-        for (int i = 0; i < 32; i++) v[i] = __uint_as_float(x[i]);
+        for (int i = 0; i < 32; i++) v[i] = __uint_as_float(y[g & 1][i]);
         split(v, tm + cA + lanes + (uint32_t)(g * 16), DP / 2);
 #pragma unroll
         for (int i = 0; i < 8; i++) {
           const float4 f = decay[g * 8 + i];
-          x[4 * i] = __float_as_uint(v[4 * i] * f.x); x[4 * i + 1] = __float_as_uint(v[4 * i + 1] * f.y);
-          x[4 * i + 2] = __float_as_uint(v[4 * i + 2] * f.z); x[4 * i + 3] = __float_as_uint(v[4 * i + 3] * f.w);
+          y[g & 1][4 * i] = __float_as_uint(v[4 * i] * f.x); y[g & 1][4 * i + 1] = __float_as_uint(v[4 * i + 1] * f.y);
+          y[g & 1][4 * i + 2] = __float_as_uint(v[4 * i + 2] * f.z); y[g & 1][4 * i + 3] = __float_as_uint(v[4 * i + 3] * f.w);
         }
-        tmem_st_32x32(tm + cS + lanes + (uint32_t)(g * 32), x);
+        tmem_st_32x32(tm + cS + lanes + (uint32_t)(g * 32), y[g & 1]);
       }
-      if constexpr (!DELTA) split(u, tm + cU + lanes, 16);
+      if constexpr (!DELTA) {                             // the last o still reads the u before
+        ok = c == 0 || __all_sync(0xffffffffu, mbar_wait(&o_full[st ^ 1], (uint32_t)(((c - 1) >> 1) & 1), status, 72));
+        if (!ok) break;
+        split(u, tm + cU + lanes, 16);
+      }
       tmem_st_wait();
       tc_fence_before_sync();
       __syncwarp();
@@ -686,12 +698,18 @@ __global__ void __launch_bounds__(320, 1) key_decay_scan_tc_kernel(const KdParam
     for (int c = 0; c < p.chunks; c++) {
       const int st = c & 1, t0 = c * kKdChunk, nt = min(kKdChunk, p.T - t0);
       const long long row0 = (long long)s * p.T + t0;
+      const bool whole = __all_sync(0xffffffffu, e < E) && nt == kKdChunk;
       uint16_t gate[kKdChunk];
       if (fuse) {
         const T* g = p.gate ? reinterpret_cast<const T*>(p.gate) + row0 * p.gate_ld + (long long)h * E + e : reinterpret_cast<const T*>(p.proj) + row0 * p.ld + p.g_off + (long long)h * E + e;
         const long long ld = p.gate ? p.gate_ld : p.ld;
+        if (whole) {
 #pragma unroll
-        for (int i = 0; i < kKdChunk; i++) gate[i] = e < E && i < nt ? *reinterpret_cast<const uint16_t*>(g + i * ld) : (uint16_t)0;
+          for (int i = 0; i < kKdChunk; i++, g += ld) gate[i] = *reinterpret_cast<const uint16_t*>(g);
+        } else {
+#pragma unroll
+          for (int i = 0; i < kKdChunk; i++, g += ld) gate[i] = e < E && i < nt ? *reinterpret_cast<const uint16_t*>(g) : (uint16_t)0;
+        }
       }
       if (!__all_sync(0xffffffffu, mbar_wait(&o_full[st], (uint32_t)((c >> 1) & 1), status, 70))) break;
       tc_fence_after_sync();
@@ -726,12 +744,19 @@ __global__ void __launch_bounds__(320, 1) key_decay_scan_tc_kernel(const KdParam
       if (!__all_sync(0xffffffffu, mbar_wait(&sums, (uint32_t)st, status, 71))) break;
       const float rs = 1.0f / sqrtf((s_sum[st][0][lane] + s_sum[st][1][lane] + s_sum[st][2][lane] + s_sum[st][3][lane]) / (float)E + p.eps);
       T* y = reinterpret_cast<T*>(p.y) + row0 * p.y_ld + (long long)h * E + e;
+      T out[kKdChunk];
 #pragma unroll
       for (int i = 0; i < kKdChunk; i++) {
-        const float f = __shfl_sync(0xffffffffu, rs, i);
         T g;
         *reinterpret_cast<uint16_t*>(&g) = gate[i];
-        if (e < E && i < nt) y[i * p.y_ld] = Cvt<T>::from(__uint_as_float(o[i]) * f * nw * kd_gate_fast<T>(p, g));
+        out[i] = Cvt<T>::from(__uint_as_float(o[i]) * (__shfl_sync(0xffffffffu, rs, i) * nw) * kd_gate_fast<T>(p, g));
+      }
+      if (whole) {
+#pragma unroll
+        for (int i = 0; i < kKdChunk; i++, y += p.y_ld) *y = out[i];
+      } else {
+#pragma unroll
+        for (int i = 0; i < kKdChunk; i++, y += p.y_ld) if (e < E && i < nt) *y = out[i];
       }
     }
   }
