@@ -225,8 +225,8 @@ static KdWork kd_layout(const KeyDecayDesc& d, void* base) {
   if (key_decay_chunk_eligible(d)) {
     const size_t n = (size_t)d.n_seq * d.heads * ((d.T + kKdChunk - 1) / kKdChunk);
     w.ops = take(n * kd_ops_layout(kd_dp(d.dim), d.delta).stride);
-    w.u = reinterpret_cast<float*>(take(n * d.vdim * kKdChunk * sizeof(float)));
-    w.o = reinterpret_cast<float*>(take(rows * d.heads * d.vdim * sizeof(float)));
+    if (!kd_tc(kd_dp(d.dim))) w.u = reinterpret_cast<float*>(take(n * d.vdim * kKdChunk * sizeof(float)));
+    if (!kd_fused(kd_dp(d.dim), d.vdim)) w.o = reinterpret_cast<float*>(take(rows * d.heads * d.vdim * sizeof(float)));
   }
   w.total = o;
   return w;
@@ -273,7 +273,7 @@ Status key_decay(cudaStream_t s, const KeyDecayDesc& d, int* launches) {
   }
   if (w.ops) {
     p.chunks = (d.T + kKdChunk - 1) / kKdChunk; p.dp = kd_dp(d.dim); p.ops = w.ops; p.u = w.u; p.o = w.o;
-    *launches += kd_fused(p) ? 2 : 3;
+    *launches += kd_fused(p.dp, p.vdim) ? 2 : 3;
     AG_RETURN_IF_ERROR(d.dtype == DType::BF16 ? key_decay_chunked_bf16(s, p) : key_decay_chunked_f16(s, p));
   } else {
     *launches += 1;

@@ -3,13 +3,14 @@
 // With A_i = a_1 .. a_i the decay of a channel from the chunk's start through token i and S_0 the state in front of the chunk,
 //     u_i = beta_i (v_i - (A_i k_i) S_0 - sum_{j<i} K_ij u_j),  K_ij = k_i (A_i / A_j) k_j      (delta rule; otherwise u = v)
 //     o_i = (A_i q_i) S_0 + sum_{j<=i} Q_ij u_j,                Q_ij = q_i (A_i / A_j) k_j
-//     S   = A_32 S_0 + sum_j (A_32 / A_j k_j) u_j^T.
-// (I + beta K) u = beta v - beta (A k) S_0 is solved for both right-hand sides ahead of the state, u = U - W S_0:
-//   prepare  every chunk on its own: convolutions, unit norms, decays, Q and K, U and W by forward substitution
+//     S   = A_32 S_0 + sum_j (A_32 / A_j k_j) u_j^T,
+// so that u = T (beta v - beta (A k) S_0) with T = (I + beta K)^-1, unit lower triangular.
+//   prepare  every chunk on its own: convolutions, unit norms, decays, Q and T (by forward substitution), the scaled rows of q and k
 //   scan     the chunks of a head one after the other, the transposed problem on tcgen05: S^T [value columns, channels], u^T and
 //            o^T are accumulators in tensor memory, S^T and u^T (split) A operands there; up to 128 channels and 128 value columns per
 //            CTA. Where that is all of a head, its norm, norm weight and gate follow, one chunk behind, in warps of their own.
-//            Wider keys take a warp-level form: a warp owns 16 value columns, its accumulator fragments chain in registers
+//            Wider keys take a warp-level form: a warp owns 16 value columns, its accumulator fragments chain in registers; the
+//            prepare kernel solves for both right-hand sides there, u = U - W S_0
 //   finish   norm and gate of wider heads
 // No decay is ever inverted: quotients A_i / A_j are products of the decays between j and i. Inside a block of 8 tokens they are
 // multiplied up term by term in float32; between blocks they split at block borders into factors of at most one, and the sums
@@ -40,9 +41,15 @@ __device__ __forceinline__ void kd_split2(float x, float y, uint32_t& hi, uint32
   lo = pack2_t<T>(x - Cvt<T>::to(v[0]), y - Cvt<T>::to(v[1]));
 }
 
+__device__ __forceinline__ float kd_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+constexpr float kKdLog2e = 1.4426950408889634f;
 // log(1 + e) for 0 <= e <= 1 as 2 artanh(e / (2 + e)), the series of which converges within 1e-7 of the value there
 __device__ __forceinline__ float kd_log1p_unit(float e) {
-  const float s = __fdividef(e, 2.0f + e), t = s * s;
+  const float s = e * kd_rcp(2.0f + e), t = s * s;
   float r = fmaf(t, 1.0f / 13.0f, 1.0f / 11.0f);
   r = fmaf(t, r, 1.0f / 9.0f);
   r = fmaf(t, r, 1.0f / 7.0f);
@@ -50,11 +57,13 @@ __device__ __forceinline__ float kd_log1p_unit(float e) {
   r = fmaf(t, r, 1.0f / 3.0f);
   return 2.0f * fmaf(s * t, r, s);
 }
-__device__ __forceinline__ float kd_softplus_fast(float x) { return fmaxf(x, 0.f) + kd_log1p_unit(__expf(-fabsf(x))); }
-__device__ __forceinline__ float kd_decay_fast(const KdParams& p, float rate, float z) { return __expf(p.softplus ? -rate * kd_softplus_fast(z) : -kd_softplus_fast(-z) * p.inv_tau); }
+__device__ __forceinline__ float kd_softplus_fast(float x) { return fmaxf(x, 0.f) + kd_log1p_unit(ex2_approx(-kKdLog2e * fabsf(x))); }
+// exp(f softplus(x)): a decay from its input z, x = z and f = -rate or x = -z and f = -1 / tau; f comes in log2 units
+__device__ __forceinline__ float kd_decay_fast(float f_log2, float x) { return ex2_approx(f_log2 * kd_softplus_fast(x)); }
+__device__ __forceinline__ float kd_sigmoid_fast(float x) { return kd_rcp(1.0f + ex2_approx(-kKdLog2e * x)); }
 template <typename T>
-__device__ __forceinline__ float kd_gate_fast(const KdParams& p, T g) { const float x = Cvt<T>::to(g), s = __fdividef(1.0f, 1.0f + __expf(-x)); return p.gate_silu ? x * s : s; }
-__device__ __forceinline__ float kd_silu_fast(float x) { return x * __fdividef(1.0f, 1.0f + __expf(-x)); }
+__device__ __forceinline__ float kd_gate_fast(const KdParams& p, T g) { const float x = Cvt<T>::to(g), s = kd_sigmoid_fast(x); return p.gate_silu ? x * s : s; }
+__device__ __forceinline__ float kd_silu_fast(float x) { return x * kd_sigmoid_fast(x); }
 
 // Convolutions of up to kKdTaps taps slide over their raw inputs; longer ones read them tap by tap.
 constexpr int kKdTaps = 4;
@@ -82,6 +91,7 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
   float* sQ = sb + kKdBlocks * DP;       // [32][36]
   float* sK = sQ + kKdChunk * 36;        // [32][36], times beta
   float* s_beta = sK + kKdChunk * 36;    // [32]
+  float* s_one = s_beta + 3 * kKdChunk;  // [DP] ones
   float2* s_f = reinterpret_cast<float2*>(s_beta + kKdChunk);      // [32] what makes q and k unit vectors
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int c = blockIdx.x, h = blockIdx.y, s = blockIdx.z, qh = h / p.group, D = p.dim, E = p.vdim;
@@ -93,7 +103,8 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
   const T* base = reinterpret_cast<const T*>(p.proj) + (long long)s * p.T * p.ld;
   const T* ring = p.ring_of<T>(s);
   uint8_t* ops = p.ops + chunk * L.stride;
-  // one value column over the chunk, and its u
+  // one value column over the chunk, and its u (warp-level scan)
+  constexpr bool kSolveValues = !kd_tc(DP);
   auto load_v = [&](int e, float (&w)[kKdChunk]) {
     const int ch = h * E + e, rc = 2 * p.qk_heads * D + ch;
     const T* src = base + (long long)t0 * p.ld + p.v_off + ch;
@@ -133,35 +144,38 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
   };
   float w[kKdChunk];                     // a right-hand side: this thread's channel of A k, or (threads past the channels) a value column
   const int e_own = tid - DP;
-  const float rate = p.softplus ? p.rate[h] : 0.f;
+  const float sign = p.softplus ? 1.f : -1.f, f_log2 = -kKdLog2e * (p.softplus ? p.rate[h] : p.inv_tau);
   if (D % 2 == 0 && p.taps <= kKdTaps) {
     // two channels at a time; everything is requested before anything is used
-    float2 z[DP / 16];
+    constexpr int R = kKdThreads / DH, NZ = (kKdChunk + R - 1) / R;      // tokens per pass, passes
+    const int zd = tid % DH * 2, zt = tid / DH;
+    const bool z_mine = tid < R * DH, z_live = z_mine && zd < D;
+    const float* zp = p.z + ((long long)s * p.T + t0 + zt) * p.heads * D + h * D + zd;
+    const long long z_step = (long long)R * p.heads * D;
+    float2 z[NZ];
 #pragma unroll
-    for (int n = 0; n < DP / 16; n++) {
-      const int i = tid + n * kKdThreads, t = i / DH, d = i % DH * 2;
-      z[n] = make_float2(0.f, 0.f);
-      if (t < nt && d < D) z[n] = __ldcs(reinterpret_cast<const float2*>(p.z + ((long long)s * p.T + t0 + t) * p.heads * D + h * D + d));
-    }
-    if (DELTA && e_own >= 0 && e_own < E) load_v(e_own, w);
+    for (int n = 0; n < NZ; n++, zp += z_step) z[n] = z_live && zt + n * R < nt ? __ldcs(reinterpret_cast<const float2*>(zp)) : make_float2(0.f, 0.f);
+    const float b0 = z_live ? __ldg(p.bias + h * D + zd) : 0.f, b1 = z_live ? __ldg(p.bias + h * D + zd + 1) : 0.f;
+    if (kSolveValues && DELTA && e_own >= 0 && e_own < E) load_v(e_own, w);
     for (int i = tid; i < kKdBlocks * DH; i += kKdThreads) {
       const int d = i % DH * 2, o = i / DH * kKdBlock, first = t0 + o - (kKdTaps - 1);
       constexpr int N = kKdBlock + kKdTaps - 1;
       float2 x[2][N];
-      const bool inside = first >= 0 && first + N <= p.T;
+      const bool inside = d < D && first >= 0 && first + N <= p.T;
 #pragma unroll
       for (int m = 0; m < 2; m++) {
         const int col = (m ? p.k_off : p.q_off) + qh * D + d, ch = (m ? p.qk_heads * D : 0) + qh * D + d;
         const T* src = base + (long long)first * p.ld + col;
+        if (inside) {
 #pragma unroll
-        for (int j = 0; j < N; j++) {
-          x[m][j] = make_float2(0.f, 0.f);
-          if (d >= D || (j < kKdTaps - 1 && !p.taps)) continue;
-          if (inside) x[m][j] = kd_pair<T>(src + (long long)j * p.ld);
-          else {
+          for (int j = 0; j < N; j++, src += p.ld) x[m][j] = kd_pair<T>(src);
+        } else {
+#pragma unroll
+          for (int j = 0; j < N; j++) {
             const int t = first + j;
-            if (t >= 0) { if (t < p.T) x[m][j] = kd_pair<T>(src + (long long)j * p.ld); }
-            else if (-t < p.taps) x[m][j] = make_float2(kd_raw<T>(p, base, ring, pos, t, col, ch), kd_raw<T>(p, base, ring, pos, t, col + 1, ch + 1));
+            x[m][j] = make_float2(0.f, 0.f);
+            if (d >= D || t >= p.T || (t < 0 && -t >= p.taps)) continue;
+            x[m][j] = t >= 0 ? kd_pair<T>(src + (long long)j * p.ld) : make_float2(kd_raw<T>(p, base, ring, pos, t, col, ch), kd_raw<T>(p, base, ring, pos, t, col + 1, ch + 1));
           }
         }
       }
@@ -187,12 +201,15 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
         }
       }
     }
+    if (z_mine) {
 #pragma unroll
-    for (int n = 0; n < DP / 16; n++) {
-      const int i = tid + n * kKdThreads, t = i / DH, d = i % DH * 2;
-      float2 a = make_float2(1.f, 1.f);
-      if (t < nt && d < D) a = make_float2(kd_decay_fast(p, rate, z[n].x + __ldg(p.bias + h * D + d)), kd_decay_fast(p, rate, z[n].y + __ldg(p.bias + h * D + d + 1)));
-      *reinterpret_cast<float2*>(sa + t * P + d) = a;
+      for (int n = 0; n < NZ; n++) {
+        const int t = zt + n * R;
+        if (NZ * R > kKdChunk && t >= kKdChunk) break;
+        const bool live = z_live && t < nt;
+        const float a0 = kd_decay_fast(f_log2, sign * (z[n].x + b0)), a1 = kd_decay_fast(f_log2, sign * (z[n].y + b1));
+        *reinterpret_cast<float2*>(sa + t * P + zd) = make_float2(live ? a0 : 1.f, live ? a1 : 1.f);
+      }
     }
   } else {
     for (int i = tid; i < kKdChunk * DP; i += kKdThreads) {
@@ -202,14 +219,15 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
         const int ch = qh * D + d;
         q = kd_input<T>(p, base, ring, pos, t0 + t, p.q_off + ch, ch);
         k = kd_input<T>(p, base, ring, pos, t0 + t, p.k_off + ch, p.qk_heads * D + ch);
-        a = kd_decay_fast(p, rate, p.z[((long long)s * p.T + t0 + t) * p.heads * D + h * D + d] + p.bias[h * D + d]);
+        a = kd_decay_fast(f_log2, sign * (p.z[((long long)s * p.T + t0 + t) * p.heads * D + h * D + d] + p.bias[h * D + d]));
       }
       sq[t * P + d] = q; sk[t * P + d] = k; sa[t * P + d] = a;
     }
-    if (DELTA && e_own >= 0 && e_own < E) load_v(e_own, w);
+    if (kSolveValues && DELTA && e_own >= 0 && e_own < E) load_v(e_own, w);
   }
-  if constexpr (!DELTA) for (int e = tid; e < E; e += kKdThreads) { load_v(e, w); store_u(e, w); }
-  for (int i = tid; i < kKdChunk * 36; i += kKdThreads) { sQ[i] = 0.f; sK[i] = 0.f; }
+  if constexpr (kSolveValues && !DELTA) for (int e = tid; e < E; e += kKdThreads) { load_v(e, w); store_u(e, w); }
+  for (int i = tid; i < kKdChunk * 36 / 2; i += kKdThreads) reinterpret_cast<float4*>(sQ)[i] = make_float4(0.f, 0.f, 0.f, 0.f);      // Q and K
+  if (tid < DP) s_one[tid] = 1.f;
   if (tid < kKdChunk) s_beta[tid] = DELTA && tid < nt ? sigmoid_f(p.beta[((long long)s * p.T + t0 + tid) * p.beta_ld + h]) : 0.f;
   __syncthreads();
   for (int t = warp; t < kKdChunk; t += kKdThreads / 32) {
@@ -230,13 +248,12 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
     for (int n = 0; n < NC; n++) kk[n] = *reinterpret_cast<const float4*>(sk + j * P + (sl + 8 * n) * 4);
     for (int i = j & ~3; i <= last; i++) {               // the four keys of a warp walk the same rows
       float s1 = 0.f, s2 = 0.f;
+      const float* fade = i > j ? sa + i * P : s_one;
 #pragma unroll
       for (int n = 0; n < NC; n++) {
         const int at = i * P + (sl + 8 * n) * 4;
-        if (i > j) {
-          const float4 a = *reinterpret_cast<const float4*>(sa + at);
-          kk[n].x *= a.x; kk[n].y *= a.y; kk[n].z *= a.z; kk[n].w *= a.w;
-        }
+        const float4 a = *reinterpret_cast<const float4*>(fade + (sl + 8 * n) * 4);
+        kk[n].x *= a.x; kk[n].y *= a.y; kk[n].z *= a.z; kk[n].w *= a.w;
         const float4 q = *reinterpret_cast<const float4*>(sq + at);
         s1 = fmaf(q.x, kk[n].x, fmaf(q.y, kk[n].y, fmaf(q.z, kk[n].z, fmaf(q.w, kk[n].w, s1))));
         if constexpr (DELTA) {
@@ -263,13 +280,14 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
     sQ[i * 36 + j] *= fi.x * fk;
     if constexpr (DELTA) sK[i * 36 + j] *= fi.y * fk;
   }
-  // element (row, channel tid) of a plane of `rows` rows, high part and remainder
-  auto put = [&](int plane0, int plane_bytes, int rows, int row, float x) {
+  // element (row, channel tid) of a plane and its remainder; panels: a row's 16-byte pieces are swapped by its number's low bits
+  const uintptr_t own = reinterpret_cast<uintptr_t>(ops) + (tid & 63) * 2;
+  auto put = [&](int plane0, int to_lo, int panel_bytes, int row, float x) {
     T hi, lo;
     kd_split<T>(x, hi, lo);
-    uint8_t* at = kd_tc(DP) ? ops + plane0 + (tid >> 6) * rows * 128 + row * 128 + (((tid & 63) * 2) ^ ((row & 7) << 4)) : ops + plane0 + (row * (DP + 8) + tid) * 2;
+    uint8_t* at = kd_tc(DP) ? reinterpret_cast<uint8_t*>((own + (tid >> 6) * panel_bytes) ^ (uintptr_t)((row & 7) << 4)) + plane0 + row * 128 : ops + plane0 + (row * (DP + 8) + tid) * 2;
     *reinterpret_cast<T*>(at) = hi;
-    *reinterpret_cast<T*>(at + plane_bytes) = lo;
+    *reinterpret_cast<T*>(at + to_lo) = lo;
   };
   if (tid < DP) {
     const int d = tid;
@@ -281,8 +299,9 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
       kk[i] = sk[i * P + d] * f.y;
       if (i % kKdBlock == 0) loc = 1.f;
       pre *= a; loc *= a;
-      put(L.qg, L.plane1, L.rows1, (kd_tc(DP) && DELTA ? kKdChunk : 0) + i, q * pre);
-      if constexpr (DELTA) w[i] = kk[i] * pre;
+      put(L.qg, L.plane1, 2 * L.plane1, i, q * pre);
+      if constexpr (DELTA && kSolveValues) w[i] = kk[i] * pre;
+      else if constexpr (DELTA) put(L.w, L.plane1, 2 * L.plane1, i, kk[i] * pre);
       sq[i * P + d] = q * loc; sk[i * P + d] = kk[i] * loc;
       if (i % kKdBlock == kKdBlock - 1) sb[i / kKdBlock * DP + d] = loc;
     }
@@ -292,7 +311,7 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
     for (int i = kKdChunk - 1; i >= 0; i--) {
       if (i % kKdBlock == kKdBlock - 1) loc = 1.f;
       const float a = sa[i * P + d];
-      put(L.kg, L.plane2, kKdChunk, i, kk[i] * suf);
+      put(L.kg, L.plane2, kKdChunk * 128, i, kk[i] * suf);
       sa[i * P + d] = kk[i] * loc;
       suf *= a; loc *= a;
     }
@@ -347,11 +366,11 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
     }
   }
   if constexpr (DELTA) {
-    // forward substitution, a thread per column
+    // forward substitution with I + beta K, a thread per column
     auto solve = [&](float (&x)[kKdChunk]) {
 #pragma unroll
       for (int i = 0; i < kKdChunk; i++) {
-        float v = x[i] * s_beta[i];
+        float v = kSolveValues ? x[i] * s_beta[i] : x[i];
 #pragma unroll
         for (int j = 0; j < i; j += 4) {
           const float4 f = *reinterpret_cast<const float4*>(sK + i * 36 + j);      // zero from the diagonal on
@@ -363,11 +382,28 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
         x[i] = v;
       }
     };
+    if constexpr (!kSolveValues) {
+      // T, column by column: a column of the identity as right-hand side
+      if (tid < kKdChunk) reinterpret_cast<float*>(ops + L.beta)[tid] = s_beta[tid];
+      if (warp != kKdThreads / 32 - 1) return;
+#pragma unroll
+      for (int i = 0; i < kKdChunk; i++) w[i] = i == lane ? 1.f : 0.f;
+      solve(w);
+#pragma unroll
+      for (int i = 0; i < kKdChunk; i++) {
+        T hi, lo;
+        kd_split<T>(w[i], hi, lo);
+        uint8_t* at = ops + L.t + i * 128 + ((lane * 2) ^ ((i & 7) << 4));
+        *reinterpret_cast<T*>(at) = hi;
+        *reinterpret_cast<T*>(at + kKdChunk * 128) = lo;
+      }
+      return;
+    }
     if (tid < DP || e_own < E) {
       solve(w);
       if (tid < DP) {
 #pragma unroll
-        for (int i = 0; i < kKdChunk; i++) put(L.w, L.plane1, L.rows1, i, -w[i]);
+        for (int i = 0; i < kKdChunk; i++) put(L.w, L.plane1, 0, i, -w[i]);
       } else store_u(e_own, w);
     }
 #pragma unroll 1
@@ -518,34 +554,40 @@ __global__ void __launch_bounds__(256) key_decay_scan_kernel(const KdParams p, i
 }
 
 // ── scan on tcgen05 (up to 128 channels) ────────────────────────────────────
-// A CTA: 128 value columns (lanes of tensor memory) of one head. Tensor memory columns: S^T in float32 [DP]; its high parts and
-// remainders as A operand [DP]; two buffers of (u^T | o^T) [32 | 32]; u^T split [16 + 16]. Per chunk:
-//   warps 0 - 3   split S, fade it in place                         (wait: update of the chunk before)
-//   warp 8        (u | o) = S (-W | A q)                            delta rule; otherwise o alone
-//   warps 0 - 3   u += U, split
-//   warp 8        o += u Q, S += u (A_32 / A k)
-//   warps 4 - 7   o to memory, or through the head's norm and gate
-// Warp 9 loads the chunks' operands. All waits are bounded.
+// A CTA: 128 value columns (lanes of tensor memory) of one head; two warps share a quarter of the lanes, each with half of the channels
+// or tokens. Tensor memory columns: S^T in float32 [DP]; its high parts and remainders as A operand [DP]; two buffers of 128 columns,
+// the products with high parts and remainders of the chunk's rows: (x | o | x' | o') with x = S (A k), otherwise (o | o').
+// Per chunk:
+//   warps 0 - 7    split S, fade it in place                        (after the update of the chunk before)
+//   warp 16        (x | o) = S (A k | A q); without the delta rule o alone, u = v
+//   warps 0 - 7    v behind its convolution, r = beta (v - x), split
+//   warp 16        u = T r
+//   warps 0 - 7    split u
+//   warp 16        S += u (A_32 / A k), o += u Q
+//   warps 8 - 15   o to memory, or through the head's norm and gate
+// Warp 17 loads the chunks' operands. All waits are bounded.
+constexpr int kKdStateWarps = 8, kKdScanThreads = 18 * 32, kKdHalf = kKdChunk / 2;
 template <typename T, int DP, bool DELTA>
-__global__ void __launch_bounds__(320, 1) key_decay_scan_tc_kernel(const KdParams p, int fuse, int* status) {
+__global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(const KdParams p, int fuse, int* status) {
   using namespace sm100;
   constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
-  constexpr uint32_t cS = 0, cA = 128, cO = 256, cU = 384;
+  constexpr uint32_t cS = 0, cA = 128, cO = 256, cR = cA + 64, cU = 64, kLo = L.rows1;      // cU: within a buffer; kLo: from a product to its remainder's
   constexpr int kSteps = DP / 16;
   extern __shared__ uint8_t smem_raw[];
-  __shared__ uint64_t full[2], empty[2], s_ready, u_ready, u_full, s_full, o_full[2], o_free[2], sums;
+  __shared__ uint64_t full[2], empty[2], s_ready, r_ready, u_ready, x_full, u_full, s_full, o_full[2], o_free[2], sums[2];
   __shared__ uint32_t tmem_slot;
-  __shared__ float s_sum[2][4][32];
+  __shared__ float s_sum[2][2][4][kKdHalf];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quarter = warp & 3;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quarter = warp & 3, half = (warp >> 2) & 1;
   const int h = blockIdx.y, s = blockIdx.z, E = p.vdim, D = p.dim;
   const long long sh = (long long)s * p.heads + h;
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 2; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], 5); mbar_init(&o_full[i], 1); mbar_init(&o_free[i], 4); }
-    mbar_init(&s_ready, 4); mbar_init(&u_ready, 4); mbar_init(&u_full, 1); mbar_init(&s_full, 1); mbar_init(&sums, 4);
+    for (int i = 0; i < 2; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], kKdStateWarps + 1); mbar_init(&o_full[i], 1); mbar_init(&o_free[i], 8); mbar_init(&sums[i], 4); }
+    mbar_init(&s_ready, kKdStateWarps); mbar_init(&r_ready, kKdStateWarps); mbar_init(&u_ready, kKdStateWarps);
+    mbar_init(&x_full, 1); mbar_init(&u_full, 1); mbar_init(&s_full, 1);
     mbar_fence_init();
   }
-  if (warp == 8) { tmem_alloc(&tmem_slot, 512); tmem_relinquish(); }
+  if (warp == 16) { tmem_alloc(&tmem_slot, 512); tmem_relinquish(); }
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
@@ -553,8 +595,8 @@ __global__ void __launch_bounds__(320, 1) key_decay_scan_tc_kernel(const KdParam
   pdl_wait();
   pdl_trigger();
   const int e = (int)blockIdx.x * 128 + quarter * 32 + lane;         // value column of the threads that own one
-  const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
-  if (warp == 9) {
+  const uint32_t lanes = tm + ((uint32_t)(quarter * 32) << 16);
+  if (warp == 17) {
     if (lane == 0)
       for (int c = 0; c < p.chunks; c++) {
         const int st = c & 1;
@@ -562,36 +604,44 @@ __global__ void __launch_bounds__(320, 1) key_decay_scan_tc_kernel(const KdParam
         mbar_expect_tx(&full[st], (uint32_t)L.bytes);
         kd_bulk_load(smem + st * L.stride, p.ops + (sh * p.chunks + c) * L.stride, (uint32_t)L.bytes, &full[st]);
       }
-  } else if (warp == 8) {
+  } else if (warp == 16) {
     if (lane == 0) {
       constexpr int fmt = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
-      const uint32_t id_1 = make_idesc_f16(fmt, 0, 0, 128, L.rows1), id_o = make_idesc_f16(fmt, 0, 0, 128, kKdChunk), id_s = make_idesc_f16(fmt, 0, 1, 128, DP);
+      const uint32_t id_1 = make_idesc_f16(fmt, 0, 0, 128, 2 * L.rows1), id_2 = make_idesc_f16(fmt, 0, 0, 128, L.rows1);
+      const uint32_t id_64 = make_idesc_f16(fmt, 0, 0, 128, 64), id_32 = make_idesc_f16(fmt, 0, 0, 128, 32), id_s = make_idesc_f16(fmt, 0, 1, 128, DP);
       const bool exact = !DELTA && p.taps == 0;                      // u is the stored v: no remainder
       for (int c = 0; c < p.chunks; c++) {
         const int st = c & 1;
         const uint32_t ph = (uint32_t)(c & 1), ph2 = (uint32_t)((c >> 1) & 1), base = smem_u32(smem + st * L.stride);
-        const uint32_t acc0 = tm + cO + (uint32_t)(st * 64), acc_o = acc0 + (DELTA ? 32u : 0u);
+        const uint32_t buf = tm + cO + (uint32_t)(st * 128), acc_o = buf + (DELTA ? 32u : 0u), cu = buf + cU;
         if (!mbar_wait(&full[st], ph2, status, 62) || !mbar_wait(&o_free[st], ph2 ^ 1, status, 63) || !mbar_wait(&s_ready, ph, status, 64)) break;
         tc_fence_after_sync();
         // a descriptor's address field counts 16-byte units: offsets are added to it
-        const uint64_t d1 = make_smem_desc_sw128(base, 16, 1024), dq = d1 + (L.q >> 4), ds = make_smem_desc_sw128(base + L.kg, kKdChunk * 128, 1024);
+        const uint64_t d1 = make_smem_desc_sw128(base, 16, 1024), dq = d1 + (L.q >> 4), dt = d1 + (L.t >> 4), ds = make_smem_desc_sw128(base + L.kg, kKdChunk * 128, 1024);
 #pragma unroll
-        for (int part = 0; part < 3; part++)                         // high x high, remainder x high, high x remainder
+        for (int k = 0; k < kSteps; k++)                             // high parts with rows and their remainders side by side
+          mma_f16_ts(buf, tm + cA + (uint32_t)(k * 8), d1 + (((k >> 2) * 2 * L.plane1 + (k & 3) * 32) >> 4), id_1, k > 0 ? 1u : 0u);
 #pragma unroll
-          for (int k = 0; k < kSteps; k++)
-            mma_f16_ts(acc0, tm + cA + (uint32_t)((part == 1 ? DP / 2 : 0) + k * 8), d1 + (((part == 2 ? L.plane1 : 0) + (k >> 2) * L.rows1 * 128 + (k & 3) * 32) >> 4), id_1,
-                       part > 0 || k > 0 ? 1u : 0u);
+        for (int k = 0; k < kSteps; k++)                             // remainders with the rows
+          mma_f16_ts(buf, tm + cA + (uint32_t)(DP / 2 + k * 8), d1 + (((k >> 2) * 2 * L.plane1 + (k & 3) * 32) >> 4), id_2, 1u);
         if constexpr (DELTA) {
+          mma_commit(&x_full);
+          if (!mbar_wait(&r_ready, ph, status, 65)) break;
+          tc_fence_after_sync();
+          mma_f16_ts(tm + cA, tm + cR, dt, id_64, 0u);               // the operand S is no longer needed: u and its remainder take its place
+          mma_f16_ts(tm + cA, tm + cR + 8, dt + 2, id_64, 1u);
+          mma_f16_ts(tm + cA, tm + cR + 16, dt, id_32, 1u);
+          mma_f16_ts(tm + cA, tm + cR + 24, dt + 2, id_32, 1u);
           mma_commit(&u_full);
-          if (!mbar_wait(&u_ready, ph, status, 65)) break;
+          if (!mbar_wait(&u_ready, ph, status, 73)) break;
           tc_fence_after_sync();
         }
 #pragma unroll
-        for (int part = 0; part < 3; part++) {
+        for (int part = 0; part < 3; part++) {                       // high x high, remainder x high, high x remainder
           if (part == 1 && exact) continue;
 #pragma unroll
           for (int k = 0; k < kKdChunk / 16; k++)
-            mma_f16_ts(tm + cS, tm + cU + (uint32_t)((part == 1 ? 16 : 0) + k * 8), ds + (((part == 2 ? L.plane2 : 0) + k * 2048) >> 4), id_s, 1u);
+            mma_f16_ts(tm + cS, cu + (uint32_t)((part == 1 ? 16 : 0) + k * 8), ds + (((part == 2 ? L.plane2 : 0) + k * 2048) >> 4), id_s, 1u);
         }
         mma_commit(&s_full);
 #pragma unroll
@@ -599,171 +649,237 @@ __global__ void __launch_bounds__(320, 1) key_decay_scan_tc_kernel(const KdParam
           if (part == 1 && exact) continue;
 #pragma unroll
           for (int k = 0; k < kKdChunk / 16; k++)
-            mma_f16_ts(acc_o, tm + cU + (uint32_t)((part == 1 ? 16 : 0) + k * 8), dq + (((part == 2 ? 64 : 0) + k * 32) >> 4), id_o, 1u);
+            mma_f16_ts(acc_o, cu + (uint32_t)((part == 1 ? 16 : 0) + k * 8), dq + (((part == 2 ? 64 : 0) + k * 32) >> 4), id_32, 1u);
         }
         mma_commit(&o_full[st]);
         mma_commit(&empty[st]);
       }
     }
-  } else if (warp < 4) {
-    float* S = p.state(s) + (long long)h * D * E;
-    uint32_t x[32];
-#pragma unroll 1
-    for (int g = 0; g < DP / 32; g++) {
-      const float* row = S + (long long)g * 32 * E + e;
+  } else if (warp < kKdStateWarps) {
+    constexpr int G = DP / 16;                                       // pieces of 16 channels, every other one is this warp's
+    const int ec = min(e, E - 1), vcol = p.v_off + h * E + ec, vch = 2 * p.qk_heads * D + h * E + ec, tb = half * kKdHalf;
+    const T* base = reinterpret_cast<const T*>(p.proj) + (long long)s * p.T * p.ld;
+    const T* ring = p.ring_of<T>(s);
+    const int pos = p.pos[s];
+    float taps[kKdTaps];
 #pragma unroll
-      for (int i = 0; i < 32; i++, row += E) x[i] = g * 32 + i < D && e < E ? __float_as_uint(*row) : 0u;
-      tmem_st_32x32(tm + cS + lanes + (uint32_t)(g * 32), x);
+    for (int i = 0; i < kKdTaps; i++) taps[i] = i == kKdTaps - 1 ? 1.f : 0.f;
+    if (p.taps && p.taps <= kKdTaps) kd_taps(p, vch, taps);
+    float* S = p.state(s) + (long long)h * D * E;
+    uint32_t x[16];
+#pragma unroll 1
+    for (int g = half; g < G; g += 2) {
+      const float* row = S + (long long)g * 16 * E + e;
+#pragma unroll
+      for (int i = 0; i < 16; i++, row += E) x[i] = g * 16 + i < D && e < E ? __float_as_uint(*row) : 0u;
+      tmem_st_32x16(lanes + cS + (uint32_t)(g * 16), x);
     }
     tmem_st_wait();
     bool ok = true;
-    auto split = [&](const float (&v)[32], uint32_t at, uint32_t lo_off) {
-      uint32_t hi[16], lo[16];
+    auto split = [&](const float (&v)[16], uint32_t at, uint32_t lo_off) {
+      uint32_t hi[8], lo[8];
 #pragma unroll
-      for (int i = 0; i < 16; i++) kd_split2<T>(v[2 * i], v[2 * i + 1], hi[i], lo[i]);
-      tmem_st_32x16(at, hi);
-      tmem_st_32x16(at + lo_off, lo);
+      for (int i = 0; i < 8; i++) kd_split2<T>(v[2 * i], v[2 * i + 1], hi[i], lo[i]);
+      tmem_st_32x8(at, hi);
+      tmem_st_32x8(at + lo_off, lo);
+    };
+    auto arrive = [&](uint64_t* bar) {
+      tmem_st_wait();
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar);
     };
     for (int c = 0; c < p.chunks; c++) {
-      const int st = c & 1;
-      const uint32_t ph = (uint32_t)(c & 1);
-      float u[32];
-      const float4* U = reinterpret_cast<const float4*>(p.u + ((sh * p.chunks + c) * E + min(e, E - 1)) * kKdChunk);
+      const int st = c & 1, t0 = c * kKdChunk + tb;
+      const uint32_t ph = (uint32_t)(c & 1), buf = lanes + cO + (uint32_t)(st * 128);
+      T raw[kKdHalf + kKdTaps - 1];                                  // this thread's values and the ones before them
+      {
+        const T* src = base + (long long)(t0 - (kKdTaps - 1)) * p.ld + vcol;
+        if (t0 >= kKdTaps - 1 && t0 + kKdHalf <= p.T) {
 #pragma unroll
-      for (int i = 0; i < 8; i++) {
-        const float4 f = e < E ? __ldcs(U + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-        u[4 * i] = f.x; u[4 * i + 1] = f.y; u[4 * i + 2] = f.z; u[4 * i + 3] = f.w;
+          for (int i = 0; i < kKdHalf + kKdTaps - 1; i++, src += p.ld) raw[i] = *src;
+        } else {
+#pragma unroll
+          for (int i = 0; i < kKdHalf + kKdTaps - 1; i++) {
+            const int t = t0 - (kKdTaps - 1) + i;
+            raw[i] = t >= p.T || (t < 0 && -t >= p.taps) ? Cvt<T>::from(0.f) : t >= 0 ? src[(long long)i * p.ld] : Cvt<T>::from(kd_raw<T>(p, base, ring, pos, t, vcol, vch));
+          }
+        }
       }
+      float v[kKdHalf];
+      auto values = [&]() {
+        if (p.taps == 0) {
+#pragma unroll
+          for (int i = 0; i < kKdHalf; i++) v[i] = Cvt<T>::to(raw[i + kKdTaps - 1]);
+        } else if (p.taps <= kKdTaps) {
+#pragma unroll
+          for (int i = 0; i < kKdHalf; i++) {
+            float y = 0.f;
+#pragma unroll
+            for (int n = 0; n < kKdTaps; n++) y = fmaf(taps[n], Cvt<T>::to(raw[i + n]), y);
+            v[i] = kd_silu_fast(y);
+          }
+        } else {
+#pragma unroll 1
+          for (int i = 0; i < kKdHalf; i++) {
+            const float y = t0 + i < p.T ? kd_input<T>(p, base, ring, pos, t0 + i, vcol, vch) : 0.f;
+#pragma unroll
+            for (int j = 0; j < kKdHalf; j++) if (j == i) v[j] = y;
+          }
+        }
+        if (t0 + kKdHalf > p.T || e >= E) {
+#pragma unroll
+          for (int i = 0; i < kKdHalf; i++) if (t0 + i >= p.T || e >= E) v[i] = 0.f;
+        }
+      };
       ok = __all_sync(0xffffffffu, mbar_wait(&full[st], (uint32_t)((c >> 1) & 1), status, 66) && (c == 0 || mbar_wait(&s_full, ph ^ 1, status, 67)));
       if (!ok) break;
       tc_fence_after_sync();
       const float4* decay = reinterpret_cast<const float4*>(smem + st * L.stride + L.decay);
-      uint32_t y[2][32];                                  // the next columns are on their way while these are split
-      tmem_ld_32x32(tm + cS + lanes, y[0]);
-#pragma unroll
-      for (int g = 0; g < DP / 32; g++) {
+#pragma unroll 2
+      for (int g = half; g < G; g += 2) {
+        tmem_ld_32x16(lanes + cS + (uint32_t)(g * 16), x);
         tmem_ld_wait();
-        if (g + 1 < DP / 32) tmem_ld_32x32(tm + cS + lanes + (uint32_t)((g + 1) * 32), y[(g + 1) & 1]);
-        float v[32];
+        float y[16];
 #pragma unroll
-        for (int i = 0; i < 32; i++) v[i] = __uint_as_float(y[g & 1][i]);
-        split(v, tm + cA + lanes + (uint32_t)(g * 16), DP / 2);
+        for (int i = 0; i < 16; i++) y[i] = __uint_as_float(x[i]);
+        split(y, lanes + cA + (uint32_t)(g * 8), DP / 2);
 #pragma unroll
-        for (int i = 0; i < 8; i++) {
-          const float4 f = decay[g * 8 + i];
-          y[g & 1][4 * i] = __float_as_uint(v[4 * i] * f.x); y[g & 1][4 * i + 1] = __float_as_uint(v[4 * i + 1] * f.y);
-          y[g & 1][4 * i + 2] = __float_as_uint(v[4 * i + 2] * f.z); y[g & 1][4 * i + 3] = __float_as_uint(v[4 * i + 3] * f.w);
+        for (int i = 0; i < 4; i++) {
+          const float4 f = decay[g * 4 + i];
+          x[4 * i] = __float_as_uint(y[4 * i] * f.x); x[4 * i + 1] = __float_as_uint(y[4 * i + 1] * f.y);
+          x[4 * i + 2] = __float_as_uint(y[4 * i + 2] * f.z); x[4 * i + 3] = __float_as_uint(y[4 * i + 3] * f.w);
         }
-        tmem_st_32x32(tm + cS + lanes + (uint32_t)(g * 32), y[g & 1]);
+        tmem_st_32x16(lanes + cS + (uint32_t)(g * 16), x);
       }
-      if constexpr (!DELTA) {                             // the last o still reads the u before
-        ok = c == 0 || __all_sync(0xffffffffu, mbar_wait(&o_full[st ^ 1], (uint32_t)(((c - 1) >> 1) & 1), status, 72));
-        if (!ok) break;
-        split(u, tm + cU + lanes, 16);
-      }
-      tmem_st_wait();
-      tc_fence_before_sync();
-      __syncwarp();
-      if (lane == 0) { mbar_arrive(&s_ready); mbar_arrive(&empty[st]); }
-      if constexpr (DELTA) {
-        ok = __all_sync(0xffffffffu, mbar_wait(&u_full, ph, status, 68));
+      if constexpr (!DELTA) {
+        values();
+        split(v, buf + cU + (uint32_t)(half * 8), 16);               // its last reader was this buffer's o, two chunks ago
+        arrive(&s_ready);
+        if (lane == 0) mbar_arrive(&empty[st]);
+      } else {
+        arrive(&s_ready);
+        values();
+        const float4* beta = reinterpret_cast<const float4*>(smem + st * L.stride + L.beta) + tb / 4;
+        float b[kKdHalf];
+#pragma unroll
+        for (int i = 0; i < kKdHalf / 4; i++) { const float4 f = beta[i]; b[4 * i] = f.x; b[4 * i + 1] = f.y; b[4 * i + 2] = f.z; b[4 * i + 3] = f.w; }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&empty[st]);
+        uint32_t y[16];
+        ok = __all_sync(0xffffffffu, mbar_wait(&x_full, ph, status, 68));
         if (!ok) break;
         tc_fence_after_sync();
-        tmem_ld_32x32(tm + cO + lanes + (uint32_t)(st * 64), x);
+        tmem_ld_32x16(buf + (uint32_t)tb, x);
+        tmem_ld_32x16(buf + kLo + (uint32_t)tb, y);
         tmem_ld_wait();
 #pragma unroll
-        for (int i = 0; i < 32; i++) u[i] += __uint_as_float(x[i]);
-        split(u, tm + cU + lanes, 16);
-        tmem_st_wait();
-        tc_fence_before_sync();
-        __syncwarp();
-        if (lane == 0) mbar_arrive(&u_ready);
+        for (int i = 0; i < kKdHalf; i++) v[i] = b[i] * (v[i] - (__uint_as_float(x[i]) + __uint_as_float(y[i])));
+        split(v, lanes + cR + (uint32_t)(half * 8), 16);
+        arrive(&r_ready);
+        ok = __all_sync(0xffffffffu, mbar_wait(&u_full, ph, status, 74));
+        if (!ok) break;
+        tc_fence_after_sync();
+        tmem_ld_32x16(lanes + cA + (uint32_t)tb, x);
+        tmem_ld_32x16(lanes + cA + 32u + (uint32_t)tb, y);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < kKdHalf; i++) v[i] = __uint_as_float(x[i]) + __uint_as_float(y[i]);
+        split(v, buf + cU + (uint32_t)(half * 8), 16);
+        arrive(&u_ready);
       }
     }
     ok = ok && __all_sync(0xffffffffu, mbar_wait(&s_full, (uint32_t)((p.chunks - 1) & 1), status, 69));
     if (ok) {
       tc_fence_after_sync();
 #pragma unroll 1
-      for (int g = 0; g < DP / 32; g++) {
-        tmem_ld_32x32(tm + cS + lanes + (uint32_t)(g * 32), x);
+      for (int g = half; g < G; g += 2) {
+        tmem_ld_32x16(lanes + cS + (uint32_t)(g * 16), x);
         tmem_ld_wait();
-        float* row = S + (long long)g * 32 * E + e;
+        float* row = S + (long long)g * 16 * E + e;
 #pragma unroll
-        for (int i = 0; i < 32; i++, row += E) if (g * 32 + i < D && e < E) *row = __uint_as_float(x[i]);
+        for (int i = 0; i < 16; i++, row += E) if (g * 16 + i < D && e < E) *row = __uint_as_float(x[i]);
       }
       tc_fence_before_sync();
     }
   } else {
     const float nw = e < E ? p.norm[e] : 0.f;
     for (int c = 0; c < p.chunks; c++) {
-      const int st = c & 1, t0 = c * kKdChunk, nt = min(kKdChunk, p.T - t0);
+      const int st = c & 1, t0 = c * kKdChunk + half * kKdHalf, nt = min(kKdHalf, p.T - t0);       // may be none
       const long long row0 = (long long)s * p.T + t0;
-      const bool whole = __all_sync(0xffffffffu, e < E) && nt == kKdChunk;
-      uint16_t gate[kKdChunk];
+      const bool whole = __all_sync(0xffffffffu, e < E) && nt == kKdHalf;
+      uint16_t gate[kKdHalf];
       if (fuse) {
         const T* g = p.gate ? reinterpret_cast<const T*>(p.gate) + row0 * p.gate_ld + (long long)h * E + e : reinterpret_cast<const T*>(p.proj) + row0 * p.ld + p.g_off + (long long)h * E + e;
         const long long ld = p.gate ? p.gate_ld : p.ld;
         if (whole) {
 #pragma unroll
-          for (int i = 0; i < kKdChunk; i++, g += ld) gate[i] = *reinterpret_cast<const uint16_t*>(g);
+          for (int i = 0; i < kKdHalf; i++, g += ld) gate[i] = *reinterpret_cast<const uint16_t*>(g);
         } else {
 #pragma unroll
-          for (int i = 0; i < kKdChunk; i++, g += ld) gate[i] = e < E && i < nt ? *reinterpret_cast<const uint16_t*>(g) : (uint16_t)0;
+          for (int i = 0; i < kKdHalf; i++, g += ld) gate[i] = e < E && i < nt ? *reinterpret_cast<const uint16_t*>(g) : (uint16_t)0;
         }
       }
       if (!__all_sync(0xffffffffu, mbar_wait(&o_full[st], (uint32_t)((c >> 1) & 1), status, 70))) break;
       tc_fence_after_sync();
-      uint32_t o[32];
-      tmem_ld_32x32(tm + cO + lanes + (uint32_t)(st * 64 + (DELTA ? 32 : 0)), o);
+      uint32_t x[16], y[16];
+      const uint32_t at = lanes + cO + (uint32_t)(st * 128 + (DELTA ? 32 : 0) + half * kKdHalf);
+      tmem_ld_32x16(at, x);
+      tmem_ld_32x16(at + kLo, y);
       tmem_ld_wait();
       tc_fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(&o_free[st]);
+      float o[kKdHalf];
+#pragma unroll
+      for (int i = 0; i < kKdHalf; i++) o[i] = __uint_as_float(x[i]) + __uint_as_float(y[i]);
       if (!fuse) {
         float* O = p.o + (row0 * p.heads + h) * E + e;
 #pragma unroll
-        for (int i = 0; i < kKdChunk; i++) if (i < nt && e < E) O[(long long)i * p.heads * E] = __uint_as_float(o[i]);
+        for (int i = 0; i < kKdHalf; i++) if (i < nt && e < E) O[(long long)i * p.heads * E] = o[i];
         continue;
       }
-      // sums of squares over the value columns: after five halvings lane t holds token t's
-      float v[32];
+      // sums of squares over the value columns: after four halvings and one sum over pairs lane l holds token l / 2's
+      float v[kKdHalf];
 #pragma unroll
-      for (int i = 0; i < 32; i++) { const float f = __uint_as_float(o[i]); v[i] = f * f; }
+      for (int i = 0; i < kKdHalf; i++) v[i] = o[i] * o[i];
 #pragma unroll
-      for (int w = 16; w > 0; w >>= 1) {
-        const bool up = lane & w;
+      for (int w = 8; w > 0; w >>= 1) {
+        const bool up = lane & (2 * w);
 #pragma unroll
         for (int i = 0; i < w; i++) {
-          const float other = __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + w], w);
+          const float other = __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + w], 2 * w);
           v[i] = (up ? v[i + w] : v[i]) + other;
         }
       }
-      s_sum[st][quarter][lane] = v[0];
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
+      if (!(lane & 1)) s_sum[st][half][quarter][lane >> 1] = v[0];
       __syncwarp();
-      if (lane == 0) mbar_arrive(&sums);
-      if (!__all_sync(0xffffffffu, mbar_wait(&sums, (uint32_t)st, status, 71))) break;
-      const float rs = 1.0f / sqrtf((s_sum[st][0][lane] + s_sum[st][1][lane] + s_sum[st][2][lane] + s_sum[st][3][lane]) / (float)E + p.eps);
-      T* y = reinterpret_cast<T*>(p.y) + row0 * p.y_ld + (long long)h * E + e;
-      T out[kKdChunk];
+      if (lane == 0) mbar_arrive(&sums[half]);
+      if (!__all_sync(0xffffffffu, mbar_wait(&sums[half], (uint32_t)st, status, 71))) break;
+      const float (&q)[4][kKdHalf] = s_sum[st][half];
+      const float rs = 1.0f / sqrtf((q[0][lane >> 1] + q[1][lane >> 1] + q[2][lane >> 1] + q[3][lane >> 1]) / (float)E + p.eps);
+      T* out = reinterpret_cast<T*>(p.y) + row0 * p.y_ld + (long long)h * E + e;
+      T res[kKdHalf];
 #pragma unroll
-      for (int i = 0; i < kKdChunk; i++) {
+      for (int i = 0; i < kKdHalf; i++) {
         T g;
         *reinterpret_cast<uint16_t*>(&g) = gate[i];
-        out[i] = Cvt<T>::from(__uint_as_float(o[i]) * (__shfl_sync(0xffffffffu, rs, i) * nw) * kd_gate_fast<T>(p, g));
+        res[i] = Cvt<T>::from(o[i] * (__shfl_sync(0xffffffffu, rs, 2 * i) * nw) * kd_gate_fast<T>(p, g));
       }
       if (whole) {
 #pragma unroll
-        for (int i = 0; i < kKdChunk; i++, y += p.y_ld) *y = out[i];
+        for (int i = 0; i < kKdHalf; i++, out += p.y_ld) *out = res[i];
       } else {
 #pragma unroll
-        for (int i = 0; i < kKdChunk; i++, y += p.y_ld) if (e < E && i < nt) *y = out[i];
+        for (int i = 0; i < kKdHalf; i++, out += p.y_ld) if (e < E && i < nt) *out = res[i];
       }
     }
   }
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
-  if (warp == 8) tmem_dealloc(tm, 512);
+  if (warp == 16) tmem_dealloc(tm, 512);
 }
 
 // ── finish: norm and gate of the heads' outputs, a warp each ────────────────
@@ -827,7 +943,7 @@ __global__ void __launch_bounds__(256) key_decay_finish_kernel(const KdParams p)
 template <typename T, int DP, bool DELTA>
 static cudaError_t launch_kd(cudaStream_t s, const KdParams& p) {
   constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
-  constexpr size_t prep = ((size_t)3 * kKdChunk * (DP + 4) + kKdBlocks * DP + 2 * kKdChunk * 36 + 3 * kKdChunk) * sizeof(float);
+  constexpr size_t prep = ((size_t)3 * kKdChunk * (DP + 4) + kKdBlocks * DP + 2 * kKdChunk * 36 + 3 * kKdChunk + DP) * sizeof(float);
   constexpr size_t scan = 2 * (size_t)L.stride + (kd_tc(DP) ? 1024 : 0);
   static bool attr = false;
   if (!attr) {
@@ -842,7 +958,7 @@ static cudaError_t launch_kd(cudaStream_t s, const KdParams& p) {
   cudaError_t e = launch_pdl(key_decay_prepare_kernel<T, DP, DELTA>, dim3((unsigned)p.chunks, (unsigned)p.heads, (unsigned)p.n_seq), dim3(kKdThreads), prep, s, p);
   if (e != cudaSuccess) return e;
   if constexpr (kd_tc(DP)) {
-    return launch_pdl(key_decay_scan_tc_kernel<T, DP, DELTA>, dim3((unsigned)((p.vdim + 127) / 128), (unsigned)p.heads, (unsigned)p.n_seq), dim3(320), scan, s, p, kd_fused(p) ? 1 : 0,
+    return launch_pdl(key_decay_scan_tc_kernel<T, DP, DELTA>, dim3((unsigned)((p.vdim + 127) / 128), (unsigned)p.heads, (unsigned)p.n_seq), dim3(kKdScanThreads), scan, s, p, kd_fused(p.dp, p.vdim) ? 1 : 0,
                       matmul_status_word());
   } else {
     // value columns per CTA: up to 128, fewer where that leaves SMs without work
@@ -866,7 +982,7 @@ static cudaError_t launch_kd_dp(cudaStream_t s, const KdParams& p) {
 template <typename T>
 static Status launch_chunked(cudaStream_t s, const KdParams& p) {
   cudaError_t e = p.delta ? launch_kd_dp<T, true>(s, p) : launch_kd_dp<T, false>(s, p);
-  if (e != cudaSuccess || kd_fused(p)) return cuda_status(e, "key decay (chunked)");
+  if (e != cudaSuccess || kd_fused(p.dp, p.vdim)) return cuda_status(e, "key decay (chunked)");
   const unsigned blocks = (unsigned)(((long long)p.n_seq * p.T * p.heads + 8 * kKdItems - 1) / (8 * kKdItems));
   const bool vec = p.vdim % 4 == 0 && p.y_ld % 4 == 0 && aligned16(p.y) && aligned16(p.norm) && (p.gate ? p.gate_ld % 4 == 0 : p.ld % 4 == 0 && p.g_off % 4 == 0 && aligned16(p.proj));
   if (vec && p.vdim <= 128) e = launch_pdl(key_decay_finish_kernel<T, 1>, dim3(blocks), dim3(256), 0, s, p);
