@@ -280,42 +280,26 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
     sQ[i * 36 + j] *= fi.x * fk;
     if constexpr (DELTA) sK[i * 36 + j] *= fi.y * fk;
   }
-  // element (row, channel tid) of a plane and its remainder; panels: a row's 16-byte pieces are swapped by its number's low bits
-  const uintptr_t own = reinterpret_cast<uintptr_t>(ops) + (tid & 63) * 2;
-  auto put = [&](int plane0, int to_lo, int panel_bytes, int row, float x) {
-    T hi, lo;
-    kd_split<T>(x, hi, lo);
-    uint8_t* at = kd_tc(DP) ? reinterpret_cast<uint8_t*>((own + (tid >> 6) * panel_bytes) ^ (uintptr_t)((row & 7) << 4)) + plane0 + row * 128 : ops + plane0 + (row * (DP + 8) + tid) * 2;
-    *reinterpret_cast<T*>(at) = hi;
-    *reinterpret_cast<T*>(at + to_lo) = lo;
-  };
-  if (tid < DP) {
-    const int d = tid;
-    float kk[kKdChunk], pre = 1.f, loc = 1.f;
+  // q, k and the keys of a block with the decays from the block's start or to its end
+  for (int i = tid; i < kKdBlocks * DP; i += kKdThreads) {
+    const int d = i % DP, b = i / DP;
+    float* q = sq + b * kKdBlock * P + d;
+    float* k = sk + b * kKdBlock * P + d;
+    float* a = sa + b * kKdBlock * P + d;
+    float kk[kKdBlock], aa[kKdBlock], f = 1.f;
 #pragma unroll
-    for (int i = 0; i < kKdChunk; i++) {
-      const float2 f = s_f[i];
-      const float a = sa[i * P + d], q = sq[i * P + d] * f.x;
-      kk[i] = sk[i * P + d] * f.y;
-      if (i % kKdBlock == 0) loc = 1.f;
-      pre *= a; loc *= a;
-      put(L.qg, L.plane1, 2 * L.plane1, i, q * pre);
-      if constexpr (DELTA && kSolveValues) w[i] = kk[i] * pre;
-      else if constexpr (DELTA) put(L.w, L.plane1, 2 * L.plane1, i, kk[i] * pre);
-      sq[i * P + d] = q * loc; sk[i * P + d] = kk[i] * loc;
-      if (i % kKdBlock == kKdBlock - 1) sb[i / kKdBlock * DP + d] = loc;
+    for (int j = 0; j < kKdBlock; j++) {
+      const float2 n = s_f[b * kKdBlock + j];
+      aa[j] = a[j * P];
+      kk[j] = k[j * P] * n.y;
+      f *= aa[j];
+      q[j * P] *= n.x * f;
+      k[j * P] = kk[j] * f;
     }
-    float suf = 1.f;
-    loc = 1.f;
+    sb[b * DP + d] = f;
+    f = 1.f;
 #pragma unroll
-    for (int i = kKdChunk - 1; i >= 0; i--) {
-      if (i % kKdBlock == kKdBlock - 1) loc = 1.f;
-      const float a = sa[i * P + d];
-      put(L.kg, L.plane2, kKdChunk * 128, i, kk[i] * suf);
-      sa[i * P + d] = kk[i] * loc;
-      suf *= a; loc *= a;
-    }
-    reinterpret_cast<float*>(ops + L.decay)[d] = suf;
+    for (int j = kKdBlock - 1; j >= 0; j--) { a[j * P] = kk[j] * f; f *= aa[j]; }
   }
   __syncthreads();
   if (warp < 6) {
@@ -350,27 +334,113 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
     if constexpr (DELTA) { sK[i * 36 + j] = acc[2] * s_beta[i]; sK[i * 36 + j + 1] = acc[3] * s_beta[i]; }
   }
   __syncthreads();
-  {
-    const int i = tid >> 3, j = (tid & 7) * 4;
+  const auto store_q = [&](int i, int j) {               // four entries of Q
     const float4 v = *reinterpret_cast<const float4*>(sQ + i * 36 + j);
     uint2 hi, lo;
     kd_split2<T>(v.x, v.y, hi.x, lo.x);
     kd_split2<T>(v.z, v.w, hi.y, lo.y);
     uint8_t* at = ops + L.q + (kd_tc(DP) ? i * 128 : i * kKdAPitch * 2);
-    if constexpr (kd_tc(DP)) {
-      *reinterpret_cast<uint2*>(at + ((j * 2) ^ ((i & 7) << 4))) = hi;
-      *reinterpret_cast<uint2*>(at + ((64 + j * 2) ^ ((i & 7) << 4))) = lo;
-    } else {
-      *reinterpret_cast<uint2*>(at + j * 2) = hi;
-      *reinterpret_cast<uint2*>(at + kKdChunk * kKdAPitch * 2 + j * 2) = lo;
+    *reinterpret_cast<uint2*>(at + (kd_tc(DP) ? (j * 2) ^ ((i & 7) << 4) : j * 2)) = hi;
+    *reinterpret_cast<uint2*>(at + (kd_tc(DP) ? (64 + j * 2) ^ ((i & 7) << 4) : kKdChunk * kKdAPitch * 2 + j * 2)) = lo;
+  };
+  // rows of A q, A k and A_32 / A k, two channels at a time, and the chunk's decay
+  const auto store_rows = [&](int first, int threads) {
+    for (int i = first; i < kKdBlocks * DH; i += threads) {
+      const int d = i % DH * 2, b = i / DH;
+      float2 pre = make_float2(1.f, 1.f), suf = make_float2(1.f, 1.f);
+#pragma unroll
+      for (int m = 0; m < kKdBlocks; m++) {
+        const float2 f = *reinterpret_cast<const float2*>(sb + m * DP + d);
+        if (m < b) { pre.x *= f.x; pre.y *= f.y; }
+        if (m > b) { suf.x *= f.x; suf.y *= f.y; }
+      }
+      if (b == 0) { float2* all = reinterpret_cast<float2*>(ops + L.decay + d * 4); const float2 f = *reinterpret_cast<const float2*>(sb + d); *all = make_float2(f.x * suf.x, f.y * suf.y); }
+      uint8_t* row0 = ops + (kd_tc(DP) ? (d & 63) * 2 + b * kKdBlock * 128 : b * kKdBlock * (DP + 8) * 2 + d * 2);
+      const int panel1 = kd_tc(DP) ? (d >> 6) * 2 * L.plane1 : 0, panel2 = kd_tc(DP) ? (d >> 6) * kKdChunk * 128 : 0;
+#pragma unroll
+      for (int j = 0; j < kKdBlock; j++) {
+        const int at = (b * kKdBlock + j) * P + d;
+        // panels: a row's 16-byte pieces are swapped by its number's low bits
+        uint8_t* row = kd_tc(DP) ? ops + (((d & 63) * 2) ^ (j << 4)) + b * kKdBlock * 128 + j * 128 : row0 + j * (DP + 8) * 2;
+        auto put = [&](uint8_t* to, int to_lo, float x, float y) {
+          uint32_t hi, lo;
+          kd_split2<T>(x, y, hi, lo);
+          *reinterpret_cast<uint32_t*>(to) = hi;
+          *reinterpret_cast<uint32_t*>(to + to_lo) = lo;
+        };
+        const float2 q = *reinterpret_cast<const float2*>(sq + at), v = *reinterpret_cast<const float2*>(sa + at);
+        put(row + L.qg + panel1, L.plane1, q.x * pre.x, q.y * pre.y);
+        put(row + L.kg + panel2, L.plane2, v.x * suf.x, v.y * suf.y);
+        if constexpr (DELTA && !kSolveValues) {
+          const float2 k = *reinterpret_cast<const float2*>(sk + at);
+          put(row + L.w + panel1, L.plane1, k.x * pre.x, k.y * pre.y);
+        }
+      }
     }
+  };
+  if constexpr (!DELTA || kSolveValues) {
+    store_q(tid >> 3, (tid & 7) * 4);
+    store_rows(tid, kKdThreads);
   }
-  if constexpr (DELTA) {
-    // forward substitution with I + beta K, a thread per column
+  if constexpr (DELTA && !kSolveValues) {
+    // T: the inverses of its two diagonal blocks of 16 by forward substitution, a lane per column, while the others store; then
+    // T_21 = -T_22 (beta K_21) T_11, a thread per entry
+    constexpr int N = 16;
+    float* sT = sQ;                                      // [32][36], once Q is stored
+    float x[N];
+    const int col = lane & (N - 1), blk = lane & N;
+    if (warp == kKdThreads / 32 - 1) {
+#pragma unroll
+      for (int i = 0; i < N; i++) {
+        float v = i == col ? 1.f : 0.f;
+#pragma unroll
+        for (int j = 0; j < i; j += 4) {
+          const float4 f = *reinterpret_cast<const float4*>(sK + (blk + i) * 36 + blk + j);      // zero from the diagonal on
+          v = fmaf(-f.x, x[j], v);
+          if (j + 1 < i) v = fmaf(-f.y, x[j + 1], v);
+          if (j + 2 < i) v = fmaf(-f.z, x[j + 2], v);
+          if (j + 3 < i) v = fmaf(-f.w, x[j + 3], v);
+        }
+        x[i] = v;
+      }
+      reinterpret_cast<float*>(ops + L.beta)[lane] = s_beta[lane];
+    } else {
+      for (int i = tid; i < kKdChunk * 8; i += kKdThreads - 32) store_q(i >> 3, (i & 7) * 4);
+      store_rows(tid, kKdThreads - 32);
+    }
+    __syncthreads();
+    if (warp == kKdThreads / 32 - 1) {
+#pragma unroll
+      for (int i = 0; i < N; i++) sT[(blk + i) * 36 + blk + col] = x[i];
+    }
+    __syncthreads();
+    const int i = tid >> 4, j = tid & 15;
+    float m = 0.f;
+#pragma unroll
+    for (int n = 0; n < N; n++) m = fmaf(sK[(N + i) * 36 + n], sT[n * 36 + j], m);
+    __syncthreads();
+    sK[i * 36 + j] = m;                                  // the first block of K is no longer needed
+    __syncthreads();
+    m = 0.f;
+#pragma unroll
+    for (int n = 0; n < N; n++) m = fmaf(-sT[(N + i) * 36 + N + n], sK[n * 36 + j], m);
+    auto put = [&](int r, int k, float v) {
+      T hi, lo;
+      kd_split<T>(v, hi, lo);
+      uint8_t* at = ops + L.t + r * 128 + ((k * 2) ^ ((r & 7) << 4));
+      *reinterpret_cast<T*>(at) = hi;
+      *reinterpret_cast<T*>(at + kKdChunk * 128) = lo;
+    };
+    put(i, j, sT[i * 36 + j]);
+    put(i, N + j, 0.f);
+    put(N + i, j, m);
+    put(N + i, N + j, sT[(N + i) * 36 + N + j]);
+  } else if constexpr (DELTA) {
+    // forward substitution with I + beta K, a thread per column: channels of A k, then value columns
     auto solve = [&](float (&x)[kKdChunk]) {
 #pragma unroll
       for (int i = 0; i < kKdChunk; i++) {
-        float v = kSolveValues ? x[i] * s_beta[i] : x[i];
+        float v = x[i] * s_beta[i];
 #pragma unroll
         for (int j = 0; j < i; j += 4) {
           const float4 f = *reinterpret_cast<const float4*>(sK + i * 36 + j);      // zero from the diagonal on
@@ -382,28 +452,25 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
         x[i] = v;
       }
     };
-    if constexpr (!kSolveValues) {
-      // T, column by column: a column of the identity as right-hand side
-      if (tid < kKdChunk) reinterpret_cast<float*>(ops + L.beta)[tid] = s_beta[tid];
-      if (warp != kKdThreads / 32 - 1) return;
-#pragma unroll
-      for (int i = 0; i < kKdChunk; i++) w[i] = i == lane ? 1.f : 0.f;
-      solve(w);
+    if (tid < DP) {
+      float f = 1.f;
 #pragma unroll
       for (int i = 0; i < kKdChunk; i++) {
-        T hi, lo;
-        kd_split<T>(w[i], hi, lo);
-        uint8_t* at = ops + L.t + i * 128 + ((lane * 2) ^ ((i & 7) << 4));
-        *reinterpret_cast<T*>(at) = hi;
-        *reinterpret_cast<T*>(at + kKdChunk * 128) = lo;
+        w[i] = sk[i * P + tid] * f;
+        if (i % kKdBlock == kKdBlock - 1) f *= sb[i / kKdBlock * DP + tid];
       }
-      return;
     }
     if (tid < DP || e_own < E) {
       solve(w);
       if (tid < DP) {
+        T* at = reinterpret_cast<T*>(ops + L.w) + tid;
 #pragma unroll
-        for (int i = 0; i < kKdChunk; i++) put(L.w, L.plane1, 0, i, -w[i]);
+        for (int i = 0; i < kKdChunk; i++) {
+          T hi, lo;
+          kd_split<T>(-w[i], hi, lo);
+          at[i * (DP + 8)] = hi;
+          at[i * (DP + 8) + L.plane1 / 2] = lo;
+        }
       } else store_u(e_own, w);
     }
 #pragma unroll 1
@@ -559,14 +626,14 @@ __global__ void __launch_bounds__(256) key_decay_scan_kernel(const KdParams p, i
 // the products with high parts and remainders of the chunk's rows: (x | o | x' | o') with x = S (A k), otherwise (o | o').
 // Per chunk:
 //   warps 0 - 7    split S, fade it in place                        (after the update of the chunk before)
-//   warp 16        (x | o) = S (A k | A q); without the delta rule o alone, u = v
+//   warp 12        (x | o) = S (A k | A q); without the delta rule o alone, u = v
 //   warps 0 - 7    v behind its convolution, r = beta (v - x), split
-//   warp 16        u = T r
+//   warp 12        u = T r
 //   warps 0 - 7    split u
-//   warp 16        S += u (A_32 / A k), o += u Q
-//   warps 8 - 15   o to memory, or through the head's norm and gate
-// Warp 17 loads the chunks' operands. All waits are bounded.
-constexpr int kKdStateWarps = 8, kKdScanThreads = 18 * 32, kKdHalf = kKdChunk / 2;
+//   warp 12        S += u (A_32 / A k), o += u Q
+//   warps 8 - 11   o to memory, or through the head's norm and gate
+// Warp 13 loads the chunks' operands. All waits are bounded.
+constexpr int kKdStateWarps = 8, kKdMmaWarp = 12, kKdLoadWarp = 13, kKdScanThreads = 14 * 32, kKdHalf = kKdChunk / 2;
 template <typename T, int DP, bool DELTA>
 __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(const KdParams p, int fuse, int* status) {
   using namespace sm100;
@@ -574,20 +641,21 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
   constexpr uint32_t cS = 0, cA = 128, cO = 256, cR = cA + 64, cU = 64, kLo = L.rows1;      // cU: within a buffer; kLo: from a product to its remainder's
   constexpr int kSteps = DP / 16;
   extern __shared__ uint8_t smem_raw[];
-  __shared__ uint64_t full[2], empty[2], s_ready, r_ready, u_ready, x_full, u_full, s_full, o_full[2], o_free[2], sums[2];
+  __shared__ uint64_t full[2], empty[2], s_ready, r_ready, u_ready, x_full, u_full, s_full, o_full[2], o_free[2], sums;
   __shared__ uint32_t tmem_slot;
-  __shared__ float s_sum[2][2][4][kKdHalf];
+  __shared__ float s_sum[2][4][kKdChunk];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quarter = warp & 3, half = (warp >> 2) & 1;
   const int h = blockIdx.y, s = blockIdx.z, E = p.vdim, D = p.dim;
   const long long sh = (long long)s * p.heads + h;
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 2; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], kKdStateWarps + 1); mbar_init(&o_full[i], 1); mbar_init(&o_free[i], 8); mbar_init(&sums[i], 4); }
+    for (int i = 0; i < 2; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], kKdStateWarps + 1); mbar_init(&o_full[i], 1); mbar_init(&o_free[i], 4); }
+    mbar_init(&sums, 4);
     mbar_init(&s_ready, kKdStateWarps); mbar_init(&r_ready, kKdStateWarps); mbar_init(&u_ready, kKdStateWarps);
     mbar_init(&x_full, 1); mbar_init(&u_full, 1); mbar_init(&s_full, 1);
     mbar_fence_init();
   }
-  if (warp == 16) { tmem_alloc(&tmem_slot, 512); tmem_relinquish(); }
+  if (warp == kKdMmaWarp) { tmem_alloc(&tmem_slot, 512); tmem_relinquish(); }
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
@@ -596,7 +664,7 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
   pdl_trigger();
   const int e = (int)blockIdx.x * 128 + quarter * 32 + lane;         // value column of the threads that own one
   const uint32_t lanes = tm + ((uint32_t)(quarter * 32) << 16);
-  if (warp == 17) {
+  if (warp == kKdLoadWarp) {
     if (lane == 0)
       for (int c = 0; c < p.chunks; c++) {
         const int st = c & 1;
@@ -604,7 +672,7 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
         mbar_expect_tx(&full[st], (uint32_t)L.bytes);
         kd_bulk_load(smem + st * L.stride, p.ops + (sh * p.chunks + c) * L.stride, (uint32_t)L.bytes, &full[st]);
       }
-  } else if (warp == 16) {
+  } else if (warp == kKdMmaWarp) {
     if (lane == 0) {
       constexpr int fmt = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
       const uint32_t id_1 = make_idesc_f16(fmt, 0, 0, 128, 2 * L.rows1), id_2 = make_idesc_f16(fmt, 0, 0, 128, L.rows1);
@@ -689,23 +757,25 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
       __syncwarp();
       if (lane == 0) mbar_arrive(bar);
     };
+    // this thread's raw values of a chunk and the ones before them, requested a chunk ahead
+    T raw[kKdHalf + kKdTaps - 1];
+    auto request = [&](int t0) {
+      const T* src = base + (long long)(t0 - (kKdTaps - 1)) * p.ld + vcol;
+      if (t0 >= kKdTaps - 1 && t0 + kKdHalf <= p.T) {
+#pragma unroll
+        for (int i = 0; i < kKdHalf + kKdTaps - 1; i++, src += p.ld) raw[i] = *src;
+      } else {
+#pragma unroll
+        for (int i = 0; i < kKdHalf + kKdTaps - 1; i++) {
+          const int t = t0 - (kKdTaps - 1) + i;
+          raw[i] = t >= p.T || (t < 0 && -t >= p.taps) ? Cvt<T>::from(0.f) : t >= 0 ? src[(long long)i * p.ld] : Cvt<T>::from(kd_raw<T>(p, base, ring, pos, t, vcol, vch));
+        }
+      }
+    };
+    request(tb);
     for (int c = 0; c < p.chunks; c++) {
       const int st = c & 1, t0 = c * kKdChunk + tb;
       const uint32_t ph = (uint32_t)(c & 1), buf = lanes + cO + (uint32_t)(st * 128);
-      T raw[kKdHalf + kKdTaps - 1];                                  // this thread's values and the ones before them
-      {
-        const T* src = base + (long long)(t0 - (kKdTaps - 1)) * p.ld + vcol;
-        if (t0 >= kKdTaps - 1 && t0 + kKdHalf <= p.T) {
-#pragma unroll
-          for (int i = 0; i < kKdHalf + kKdTaps - 1; i++, src += p.ld) raw[i] = *src;
-        } else {
-#pragma unroll
-          for (int i = 0; i < kKdHalf + kKdTaps - 1; i++) {
-            const int t = t0 - (kKdTaps - 1) + i;
-            raw[i] = t >= p.T || (t < 0 && -t >= p.taps) ? Cvt<T>::from(0.f) : t >= 0 ? src[(long long)i * p.ld] : Cvt<T>::from(kd_raw<T>(p, base, ring, pos, t, vcol, vch));
-          }
-        }
-      }
       float v[kKdHalf];
       auto values = [&]() {
         if (p.taps == 0) {
@@ -731,18 +801,23 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
 #pragma unroll
           for (int i = 0; i < kKdHalf; i++) if (t0 + i >= p.T || e >= E) v[i] = 0.f;
         }
+        if (c + 1 < p.chunks) request(t0 + kKdChunk);
       };
       ok = __all_sync(0xffffffffu, mbar_wait(&full[st], (uint32_t)((c >> 1) & 1), status, 66) && (c == 0 || mbar_wait(&s_full, ph ^ 1, status, 67)));
       if (!ok) break;
       tc_fence_after_sync();
       const float4* decay = reinterpret_cast<const float4*>(smem + st * L.stride + L.decay);
-#pragma unroll 2
-      for (int g = half; g < G; g += 2) {
-        tmem_ld_32x16(lanes + cS + (uint32_t)(g * 16), x);
+      uint32_t next[16];                                             // on its way while a piece is split
+      if (half < G) tmem_ld_32x16(lanes + cS + (uint32_t)(half * 16), next);
+#pragma unroll
+      for (int n = 0; n < (G + 1) / 2; n++) {
+        const int g = 2 * n + half;
+        if (G % 2 && g >= G) break;
         tmem_ld_wait();
         float y[16];
 #pragma unroll
-        for (int i = 0; i < 16; i++) y[i] = __uint_as_float(x[i]);
+        for (int i = 0; i < 16; i++) y[i] = __uint_as_float(next[i]);
+        if (g + 2 < G) tmem_ld_32x16(lanes + cS + (uint32_t)((g + 2) * 16), next);
         split(y, lanes + cA + (uint32_t)(g * 8), DP / 2);
 #pragma unroll
         for (int i = 0; i < 4; i++) {
@@ -805,81 +880,88 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
   } else {
     const float nw = e < E ? p.norm[e] : 0.f;
     for (int c = 0; c < p.chunks; c++) {
-      const int st = c & 1, t0 = c * kKdChunk + half * kKdHalf, nt = min(kKdHalf, p.T - t0);       // may be none
+      const int st = c & 1, t0 = c * kKdChunk, nt = min(kKdChunk, p.T - t0);
       const long long row0 = (long long)s * p.T + t0;
-      const bool whole = __all_sync(0xffffffffu, e < E) && nt == kKdHalf;
-      uint16_t gate[kKdHalf];
+      const bool whole = __all_sync(0xffffffffu, e < E) && nt == kKdChunk;
+      uint16_t gate[kKdChunk];
       if (fuse) {
         const T* g = p.gate ? reinterpret_cast<const T*>(p.gate) + row0 * p.gate_ld + (long long)h * E + e : reinterpret_cast<const T*>(p.proj) + row0 * p.ld + p.g_off + (long long)h * E + e;
         const long long ld = p.gate ? p.gate_ld : p.ld;
         if (whole) {
 #pragma unroll
-          for (int i = 0; i < kKdHalf; i++, g += ld) gate[i] = *reinterpret_cast<const uint16_t*>(g);
+          for (int i = 0; i < kKdChunk; i++, g += ld) gate[i] = *reinterpret_cast<const uint16_t*>(g);
         } else {
 #pragma unroll
-          for (int i = 0; i < kKdHalf; i++, g += ld) gate[i] = e < E && i < nt ? *reinterpret_cast<const uint16_t*>(g) : (uint16_t)0;
+          for (int i = 0; i < kKdChunk; i++, g += ld) gate[i] = e < E && i < nt ? *reinterpret_cast<const uint16_t*>(g) : (uint16_t)0;
         }
       }
       if (!__all_sync(0xffffffffu, mbar_wait(&o_full[st], (uint32_t)((c >> 1) & 1), status, 70))) break;
       tc_fence_after_sync();
-      uint32_t x[16], y[16];
-      const uint32_t at = lanes + cO + (uint32_t)(st * 128 + (DELTA ? 32 : 0) + half * kKdHalf);
-      tmem_ld_32x16(at, x);
-      tmem_ld_32x16(at + kLo, y);
-      tmem_ld_wait();
+      float o[kKdChunk];
+#pragma unroll
+      for (int n = 0; n < 2; n++) {
+        uint32_t x[16], y[16];
+        const uint32_t at = lanes + cO + (uint32_t)(st * 128 + (DELTA ? 32 : 0) + n * kKdHalf);
+        tmem_ld_32x16(at, x);
+        tmem_ld_32x16(at + kLo, y);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < kKdHalf; i++) o[n * kKdHalf + i] = __uint_as_float(x[i]) + __uint_as_float(y[i]);
+      }
       tc_fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(&o_free[st]);
-      float o[kKdHalf];
-#pragma unroll
-      for (int i = 0; i < kKdHalf; i++) o[i] = __uint_as_float(x[i]) + __uint_as_float(y[i]);
       if (!fuse) {
         float* O = p.o + (row0 * p.heads + h) * E + e;
 #pragma unroll
-        for (int i = 0; i < kKdHalf; i++) if (i < nt && e < E) O[(long long)i * p.heads * E] = o[i];
+        for (int i = 0; i < kKdChunk; i++) if (i < nt && e < E) O[(long long)i * p.heads * E] = o[i];
         continue;
       }
-      // sums of squares over the value columns: after four halvings and one sum over pairs lane l holds token l / 2's
+      // sums of squares over the value columns: after five halvings lane t holds token t's
       float v[kKdHalf];
+      {
+        const bool up = lane & 16;
 #pragma unroll
-      for (int i = 0; i < kKdHalf; i++) v[i] = o[i] * o[i];
+        for (int i = 0; i < kKdHalf; i++) {
+          const float a = o[i] * o[i], b = o[i + kKdHalf] * o[i + kKdHalf], other = __shfl_xor_sync(0xffffffffu, up ? a : b, 16);
+          v[i] = (up ? b : a) + other;
+        }
+      }
 #pragma unroll
       for (int w = 8; w > 0; w >>= 1) {
-        const bool up = lane & (2 * w);
+        const bool up = lane & w;
 #pragma unroll
         for (int i = 0; i < w; i++) {
-          const float other = __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + w], 2 * w);
+          const float other = __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + w], w);
           v[i] = (up ? v[i + w] : v[i]) + other;
         }
       }
-      v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
-      if (!(lane & 1)) s_sum[st][half][quarter][lane >> 1] = v[0];
+      s_sum[st][quarter][lane] = v[0];
       __syncwarp();
-      if (lane == 0) mbar_arrive(&sums[half]);
-      if (!__all_sync(0xffffffffu, mbar_wait(&sums[half], (uint32_t)st, status, 71))) break;
-      const float (&q)[4][kKdHalf] = s_sum[st][half];
-      const float rs = 1.0f / sqrtf((q[0][lane >> 1] + q[1][lane >> 1] + q[2][lane >> 1] + q[3][lane >> 1]) / (float)E + p.eps);
+      if (lane == 0) mbar_arrive(&sums);
+      if (!__all_sync(0xffffffffu, mbar_wait(&sums, (uint32_t)st, status, 71))) break;
+      const float rs = 1.0f / sqrtf((s_sum[st][0][lane] + s_sum[st][1][lane] + s_sum[st][2][lane] + s_sum[st][3][lane]) / (float)E + p.eps);
       T* out = reinterpret_cast<T*>(p.y) + row0 * p.y_ld + (long long)h * E + e;
-      T res[kKdHalf];
+      T res[kKdChunk];
 #pragma unroll
-      for (int i = 0; i < kKdHalf; i++) {
+      for (int i = 0; i < kKdChunk; i++) {
         T g;
         *reinterpret_cast<uint16_t*>(&g) = gate[i];
-        res[i] = Cvt<T>::from(o[i] * (__shfl_sync(0xffffffffu, rs, 2 * i) * nw) * kd_gate_fast<T>(p, g));
+        res[i] = Cvt<T>::from(o[i] * (__shfl_sync(0xffffffffu, rs, i) * nw) * kd_gate_fast<T>(p, g));
       }
       if (whole) {
 #pragma unroll
-        for (int i = 0; i < kKdHalf; i++, out += p.y_ld) *out = res[i];
+        for (int i = 0; i < kKdChunk; i++, out += p.y_ld) *out = res[i];
       } else {
 #pragma unroll
-        for (int i = 0; i < kKdHalf; i++, out += p.y_ld) if (e < E && i < nt) *out = res[i];
+        for (int i = 0; i < kKdChunk; i++, out += p.y_ld) if (e < E && i < nt) *out = res[i];
       }
     }
   }
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
-  if (warp == 16) tmem_dealloc(tm, 512);
+  if (warp == kKdMmaWarp) tmem_dealloc(tm, 512);
 }
 
 // ── finish: norm and gate of the heads' outputs, a warp each ────────────────
