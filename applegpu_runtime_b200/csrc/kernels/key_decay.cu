@@ -1,6 +1,7 @@
 // Matrix states with one decay per key channel: the token-by-token form and the choice between it and the chunked one.
 //
-// A cluster works on one head of one sequence, each CTA on a slice of the value columns of S. With r = (diag(a) S)^T k and
+// A cluster works on one head of one sequence, each CTA on a slice of the value columns of S. The channels of q, k and the decay are
+// computed once, a slice per CTA, and go to all CTAs over distributed shared memory. With r = (diag(a) S)^T k and
 // p = (diag(a) S)^T q taken in one pass over S, the rest of a token is u = beta (v - r) (or v), o = p + (k . q) u and the update
 // S <- diag(a) S + k u^T, which is the order of the recurrence: the read-out sees the current token's write. S stays in registers
 // from token to token where a CTA's columns fit one per thread.
@@ -50,14 +51,28 @@ __global__ void __launch_bounds__(kKsThreads) key_decay_step_kernel(const KdPara
   float* so = sg + slice;
   float* sx = so + slice;                // a1 and g1 of the token, padded with zeros to whole packs
   float* sy = sx + p.a_ld;
-  float* part = sy + p.g_ld;             // [ty][tx] twice
+  float* sz = sy + p.g_ld;               // [D] decay inputs of this CTA's channels
+  float* part = sz + D;                  // [ty][tx] twice
   const int ty_n = kKsThreads / tx_n, tx = threadIdx.x % tx_n, ty = threadIdx.x / tx_n, lane = threadIdx.x & 31;
+  const int cs = (D + n_rank - 1) / n_rank, c0 = min(D, rank * cs), nc = min(cs, D - c0);       // this CTA's channels
+  float* S = p.state(s) + (long long)h * D * E + e0;
+  // weights and state start towards the L2 before the previous kernel is waited for
+  {
+    constexpr int line = 128 / (int)sizeof(T);
+    const T* a2 = reinterpret_cast<const T*>(p.a2) + ((long long)h * D + c0) * p.a_ld;
+    if (!p.z) for (int i = threadIdx.x * line; i < nc * p.a_ld; i += kKsThreads * line) asm volatile("prefetch.global.L2 [%0];" ::"l"(a2 + i));
+    if (!p.gate && p.g_rank) {
+      const T* g2 = reinterpret_cast<const T*>(p.g2) + ((long long)h * E + e0) * p.g_ld;
+      for (int i = threadIdx.x * line; i < ne * p.g_ld; i += kKsThreads * line) asm volatile("prefetch.global.L2 [%0];" ::"l"(g2 + i));
+    }
+    if (ne > 0) for (int d = threadIdx.x; d < D; d += kKsThreads) asm volatile("prefetch.global.L2 [%0];" ::"l"(S + (long long)d * E));
+  }
+  if (n_rank > 1) sm100::cluster_sync_all();        // every CTA has started before another one writes into it
   pdl_wait();
   pdl_trigger();
   const int pos = p.pos[s];
   const T* base = reinterpret_cast<const T*>(p.proj) + (long long)s * p.T * p.ld;
   T* ring = p.ring_of<T>(s);
-  float* S = p.state(s) + (long long)h * D * E + e0;
   const bool resident = slice <= tx_n;
   float st[NR];
   auto load = [&](int c) {
@@ -73,13 +88,19 @@ __global__ void __launch_bounds__(kKsThreads) key_decay_step_kernel(const KdPara
     const T* row = base + (long long)t * p.ld;
     const long long r = (long long)s * p.T + t;
     __syncthreads();
-    for (int i = threadIdx.x; i < 2 * D; i += kKsThreads) {
-      const bool is_k = i >= D;
-      const int c = qh * D + (is_k ? i - D : i);
-      sq[i] = kd_input<T>(p, base, ring, pos, t, (is_k ? p.k_off : p.q_off) + c, (is_k ? p.qk_heads * D : 0) + c);
+    // own channels of q and k go to every CTA of the cluster
+    auto push = [&](float* at, float v) {
+      if (n_rank == 1) *at = v;
+      else
+        for (int r = 0; r < n_rank; r++) asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(sm100::mapa_u32(sm100::smem_u32(at), (uint32_t)r)), "f"(v) : "memory");
+    };
+    for (int i = threadIdx.x; i < 2 * nc; i += kKsThreads) {
+      const bool is_k = i >= nc;
+      const int d = c0 + (is_k ? i - nc : i), c = qh * D + d;
+      push((is_k ? sk : sq) + d, kd_input<T>(p, base, ring, pos, t, (is_k ? p.k_off : p.q_off) + c, (is_k ? p.qk_heads * D : 0) + c));
     }
     for (int i = threadIdx.x; i < ne; i += kKsThreads) { const int c = h * E + e0 + i; sv[i] = kd_input<T>(p, base, ring, pos, t, p.v_off + c, 2 * p.qk_heads * D + c); }
-    if (p.z) for (int i = threadIdx.x; i < D; i += kKsThreads) sa[i] = p.z[r * p.heads * D + h * D + i];
+    if (p.z) for (int i = threadIdx.x; i < nc; i += kKsThreads) sz[i] = p.z[r * p.heads * D + h * D + c0 + i];
     else for (int i = threadIdx.x; i < p.a_ld; i += kKsThreads) sx[i] = i < p.a_rank ? Cvt<T>::to(row[p.a_off + i]) : 0.f;
     if (p.gate || p.g_rank == 0)
       for (int i = threadIdx.x; i < ne; i += kKsThreads)
@@ -94,24 +115,20 @@ __global__ void __launch_bounds__(kKsThreads) key_decay_step_kernel(const KdPara
         for (int i = threadIdx.x; i < 2 * D; i += kKsThreads) { const int c = qh * D + i % D; dst[(i / D) * p.qk_heads * D + c] = row[(i < D ? p.q_off : p.k_off) + c]; }
     }
     __syncthreads();
-    if (!p.z) kd_rows<T>(reinterpret_cast<const T*>(p.a2) + (long long)h * D * p.a_ld, p.a_ld, p.a_rank, sx, D, sa);
+    if (!p.z) kd_rows<T>(reinterpret_cast<const T*>(p.a2) + ((long long)h * D + c0) * p.a_ld, p.a_ld, p.a_rank, sx, nc, sz);
     if (!p.gate && p.g_rank) kd_rows<T>(reinterpret_cast<const T*>(p.g2) + ((long long)h * E + e0) * p.g_ld, p.g_ld, p.g_rank, sy, ne, sg);
+    __syncthreads();
+    for (int i = threadIdx.x; i < nc; i += kKsThreads) push(sa + c0 + i, kd_decay(p, h, sz[i] + p.bias[h * D + c0 + i]));
+    if (n_rank > 1) sm100::cluster_sync_all(); else __syncthreads();
     // sums over the head, by every warp for itself
     float qq = 0.f, kk = 0.f, qk = 0.f;
     for (int i = lane; i < D; i += 32) { const float a = sq[i], b = sk[i]; qq = fmaf(a, a, qq); kk = fmaf(b, b, kk); qk = fmaf(a, b, qk); }
     qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
     const float fq = p.unit ? p.q_scale / sqrtf(qq + 1e-6f) : p.q_scale, fk = p.unit ? 1.0f / sqrtf(kk + 1e-6f) : 1.0f;
     qk *= fq * fk;
-    __syncthreads();
-    for (int i = threadIdx.x; i < D; i += kKsThreads) {
-      sa[i] = kd_decay(p, h, sa[i] + p.bias[h * D + i]);
-      sq[i] *= fq;
-      sk[i] *= fk;
-    }
     const float beta = p.delta ? sigmoid_f(p.beta[r * p.beta_ld + h]) : 1.f;
-    __syncthreads();
-    for (int c0 = 0; c0 < slice; c0 += tx_n) {
-      const int c = c0 + tx;
+    for (int col = 0; col < slice; col += tx_n) {
+      const int c = col + tx;
       if (!resident) load(c);
       float rk = 0.f, rq = 0.f;
 #pragma unroll
@@ -128,12 +145,13 @@ __global__ void __launch_bounds__(kKsThreads) key_decay_step_kernel(const KdPara
       __syncthreads();
       rk = 0.f; rq = 0.f;
       for (int y = 0; y < ty_n; y++) { rk += part[y * tx_n + tx]; rq += part[kKsThreads + y * tx_n + tx]; }
+      rk *= fk; rq *= fq;
       const float v = c < ne ? sv[c] : 0.f;
       const float u = p.delta ? beta * (v - rk) : v;
 #pragma unroll
       for (int n = 0; n < NR; n++) {
         const int d = n * ty_n + ty;
-        if (d < D) st[n] = fmaf(sk[d], u, st[n]);
+        if (d < D) st[n] = fmaf(sk[d], fk * u, st[n]);
       }
       if (ty == 0 && c < slice) so[c] = c < ne ? fmaf(qk, u, rq) : 0.f;
       if (!resident) { store(c); __syncthreads(); }
@@ -199,7 +217,7 @@ static Status key_decay_step(cudaStream_t s, DType dt, const KdParams& p) {
   int tx_n = 4;
   while (tx_n < 32 && tx_n < slice) tx_n *= 2;
   const int nr = (p.dim + kKsThreads / tx_n - 1) / (kKsThreads / tx_n);
-  const size_t smem = (3 * (size_t)p.dim + 3 * (size_t)slice + p.a_ld + p.g_ld + 2 * kKsThreads) * sizeof(float);
+  const size_t smem = (4 * (size_t)p.dim + 3 * (size_t)slice + p.a_ld + p.g_ld + 2 * kKsThreads) * sizeof(float);
   if (nr > 64 || smem > 100 * 1024) return Status::unsupported("key decay: head too large");
   cudaError_t e = cudaSuccess;
   AG_DISPATCH_FLOAT(dt, T, {

@@ -93,6 +93,9 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
   float* s_beta = sK + kKdChunk * 36;    // [32]
   float* s_one = s_beta + 3 * kKdChunk;  // [DP] ones
   float2* s_f = reinterpret_cast<float2*>(s_beta + kKdChunk);      // [32] what makes q and k unit vectors
+  float* s_pre = s_one + DP;             // [4][DP] decays of the blocks before one, and behind it
+  float* s_suf = s_pre + kKdBlocks * DP;
+  float* s_part = s_suf + kKdBlocks * DP;                          // [8][6][16][8] shares of the products between blocks
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int c = blockIdx.x, h = blockIdx.y, s = blockIdx.z, qh = h / p.group, D = p.dim, E = p.vdim;
   const int t0 = c * kKdChunk, nt = min(kKdChunk, p.T - t0);
@@ -192,9 +195,10 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
             float2 y = make_float2(0.f, 0.f);
 #pragma unroll
             for (int n = 0; n < kKdTaps; n++) { y.x = fmaf(w0[n], x[m][j + n].x, y.x); y.y = fmaf(w1[n], x[m][j + n].y, y.y); }
-            const bool live = o + j < nt;                // channels past D are zero already
-            *reinterpret_cast<float2*>(dst + j * P) = make_float2(live ? kd_silu_fast(y.x) : 0.f, live ? kd_silu_fast(y.y) : 0.f);
+            *reinterpret_cast<float2*>(dst + j * P) = make_float2(kd_silu_fast(y.x), kd_silu_fast(y.y));      // channels past D are zero already
           }
+          if (o + kKdBlock > nt)                         // tokens past the end are not
+            for (int j = max(0, nt - o); j < kKdBlock; j++) *reinterpret_cast<float2*>(dst + j * P) = make_float2(0.f, 0.f);
         } else {
 #pragma unroll
           for (int j = 0; j < kKdBlock; j++) *reinterpret_cast<float2*>(dst + j * P) = x[m][j + kKdTaps - 1];
@@ -230,42 +234,43 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
   if (tid < DP) s_one[tid] = 1.f;
   if (tid < kKdChunk) s_beta[tid] = DELTA && tid < nt ? sigmoid_f(p.beta[((long long)s * p.T + t0 + tid) * p.beta_ld + h]) : 0.f;
   __syncthreads();
-  for (int t = warp; t < kKdChunk; t += kKdThreads / 32) {
-    float2 f = make_float2(p.q_scale, 1.f);
-    if (p.unit) {
-      float qq = 0.f, kk = 0.f;
-#pragma unroll
-      for (int d = lane; d < DP; d += 32) { const float a = sq[t * P + d], b = sk[t * P + d]; qq = fmaf(a, a, qq); kk = fmaf(b, b, kk); }
-      f = make_float2(p.q_scale / sqrtf(warp_sum(qq) + 1e-6f), 1.0f / sqrtf(warp_sum(kk) + 1e-6f));
-    }
-    if (lane == 0) s_f[t] = f;
-  }
   {
-    // pairs inside a block: eight lanes per key token j, which carry its decayed key from one query token to the next
+    // pairs inside a block: eight lanes per key token j, which carry its decayed key from one query token to the next (two channels to
+    // an operation); before that the lengths of the token's own q and k
     const int j = tid >> 3, sl = tid & 7, last = j / kKdBlock * kKdBlock + kKdBlock - 1;
-    float4 kk[NC];
+    uint64_t kk[2 * NC];
+    auto row = [&](const float* x, int n) { return *reinterpret_cast<const ulonglong2*>(x + (sl + 8 * n) * 4); };
+    uint64_t a1 = 0ull, a2 = 0ull;
 #pragma unroll
-    for (int n = 0; n < NC; n++) kk[n] = *reinterpret_cast<const float4*>(sk + j * P + (sl + 8 * n) * 4);
+    for (int n = 0; n < NC; n++) {
+      const ulonglong2 k = row(sk + j * P, n), q = row(sq + j * P, n);
+      kk[2 * n] = k.x; kk[2 * n + 1] = k.y;
+      a1 = fma_f32x2(q.x, q.x, fma_f32x2(q.y, q.y, a1));
+      a2 = fma_f32x2(k.x, k.x, fma_f32x2(k.y, k.y, a2));
+    }
+    auto over_lanes = [&](float v) {
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+      return v;
+    };
+    {
+      const float qq = over_lanes(sum_f32x2(a1)), kq = over_lanes(sum_f32x2(a2));
+      if (sl == 0) s_f[j] = p.unit ? make_float2(p.q_scale / sqrtf(qq + 1e-6f), 1.0f / sqrtf(kq + 1e-6f)) : make_float2(p.q_scale, 1.f);
+    }
     for (int i = j & ~3; i <= last; i++) {               // the four keys of a warp walk the same rows
-      float s1 = 0.f, s2 = 0.f;
       const float* fade = i > j ? sa + i * P : s_one;
+      a1 = 0ull; a2 = 0ull;
 #pragma unroll
       for (int n = 0; n < NC; n++) {
-        const int at = i * P + (sl + 8 * n) * 4;
-        const float4 a = *reinterpret_cast<const float4*>(fade + (sl + 8 * n) * 4);
-        kk[n].x *= a.x; kk[n].y *= a.y; kk[n].z *= a.z; kk[n].w *= a.w;
-        const float4 q = *reinterpret_cast<const float4*>(sq + at);
-        s1 = fmaf(q.x, kk[n].x, fmaf(q.y, kk[n].y, fmaf(q.z, kk[n].z, fmaf(q.w, kk[n].w, s1))));
+        const ulonglong2 a = row(fade, n), q = row(sq + i * P, n);
+        kk[2 * n] = mul_f32x2(kk[2 * n], a.x); kk[2 * n + 1] = mul_f32x2(kk[2 * n + 1], a.y);
+        a1 = fma_f32x2(q.x, kk[2 * n], fma_f32x2(q.y, kk[2 * n + 1], a1));
         if constexpr (DELTA) {
-          const float4 k = *reinterpret_cast<const float4*>(sk + at);
-          s2 = fmaf(k.x, kk[n].x, fmaf(k.y, kk[n].y, fmaf(k.z, kk[n].z, fmaf(k.w, kk[n].w, s2))));
+          const ulonglong2 k = row(sk + i * P, n);
+          a2 = fma_f32x2(k.x, kk[2 * n], fma_f32x2(k.y, kk[2 * n + 1], a2));
         }
       }
-#pragma unroll
-      for (int o = 4; o > 0; o >>= 1) {
-        s1 += __shfl_xor_sync(0xffffffffu, s1, o);
-        if constexpr (DELTA) s2 += __shfl_xor_sync(0xffffffffu, s2, o);
-      }
+      const float s1 = over_lanes(sum_f32x2(a1)), s2 = DELTA ? over_lanes(sum_f32x2(a2)) : 0.f;
       if (sl == 0 && i >= j) {
         sQ[i * 36 + j] = s1;
         if (DELTA && i > j) sK[i * 36 + j] = s2 * s_beta[i];
@@ -302,36 +307,72 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
     for (int j = kKdBlock - 1; j >= 0; j--) { a[j * P] = kk[j] * f; f *= aa[j]; }
   }
   __syncthreads();
-  if (warp < 6) {
-    // pairs of different blocks, queries of block b with keys of block a: rows 0 .. 7 of the product are q, rows 8 .. 15 k
-    const int b = warp < 1 ? 1 : warp < 3 ? 2 : 3, a = warp - b * (b - 1) / 2, g = lane >> 2, q = lane & 3;
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    const float* rq = sq + (b * kKdBlock + g) * P + 2 * q;
-    const float* rk = sk + (b * kKdBlock + g) * P + 2 * q;
-    const float* rj = sa + (a * kKdBlock + g) * P + 2 * q;
-#pragma unroll 2
-    for (int k0 = 0; k0 < DP; k0 += 16) {
-      uint32_t ah[4], al[4], bh[2], bl[2];
+  if (tid < DP) {                        // a chunk's decays across blocks
+    const float f0 = sb[tid], f1 = sb[DP + tid], f2 = sb[2 * DP + tid], f3 = sb[3 * DP + tid];
+    s_pre[tid] = 1.f; s_pre[DP + tid] = f0; s_pre[2 * DP + tid] = f0 * f1; s_pre[3 * DP + tid] = f0 * f1 * f2;
+    s_suf[tid] = f1 * f2 * f3; s_suf[DP + tid] = f2 * f3; s_suf[2 * DP + tid] = f3; s_suf[3 * DP + tid] = 1.f;
+    reinterpret_cast<float*>(ops + L.decay)[tid] = f0 * f1 * f2 * f3;
+  }
+  // pairs of different blocks, queries of block b with keys of block a < b: rows 0 .. 7 of a product are q, rows 8 .. 15 k. A warp takes
+  // every eighth 16 channels of all six.
+  constexpr int kShares = DP / 16 < 8 ? DP / 16 : 8;
+  if (warp < kShares) {
+    const int g = lane >> 2, q = lane & 3;
+    float acc[6][4];
 #pragma unroll
-      for (int x = 0; x < 2; x++) {
-        const int at = k0 + 8 * x;
-        const float2 fq = *reinterpret_cast<const float2*>(rq + at);
-        kd_split2<T>(fq.x, fq.y, ah[2 * x], al[2 * x]);
-        if constexpr (DELTA) {
-          const float2 fk = *reinterpret_cast<const float2*>(rk + at);
-          kd_split2<T>(fk.x, fk.y, ah[2 * x + 1], al[2 * x + 1]);
-        } else { ah[2 * x + 1] = 0u; al[2 * x + 1] = 0u; }
-        float2 fj = *reinterpret_cast<const float2*>(rj + at);
-        for (int m = a + 1; m < b; m++) { const float2 fb = *reinterpret_cast<const float2*>(sb + m * DP + at + 2 * q); fj.x *= fb.x; fj.y *= fb.y; }
-        kd_split2<T>(fj.x, fj.y, bh[x], bl[x]);
+    for (int i = 0; i < 6; i++) { acc[i][0] = 0.f; acc[i][1] = 0.f; acc[i][2] = 0.f; acc[i][3] = 0.f; }
+#pragma unroll 1
+    for (int k0 = warp * 16; k0 < DP; k0 += kShares * 16) {
+      uint32_t ah[3][4], al[3][4];
+      const int c0 = k0 + 2 * q;
+      auto at = [&](const float* x, int r, int c) { return *reinterpret_cast<const float2*>(x + r * P + c); };
+#pragma unroll
+      for (int b = 1; b < kKdBlocks; b++)
+#pragma unroll
+        for (int x = 0; x < 2; x++) {
+          const float2 fq = at(sq, b * kKdBlock + g, c0 + 8 * x);
+          kd_split2<T>(fq.x, fq.y, ah[b - 1][2 * x], al[b - 1][2 * x]);
+          ah[b - 1][2 * x + 1] = 0u; al[b - 1][2 * x + 1] = 0u;
+          if constexpr (DELTA) {
+            const float2 fk = at(sk, b * kKdBlock + g, c0 + 8 * x);
+            kd_split2<T>(fk.x, fk.y, ah[b - 1][2 * x + 1], al[b - 1][2 * x + 1]);
+          }
+        }
+#pragma unroll
+      for (int a = 0; a < kKdBlocks - 1; a++) {
+        float2 f[2] = {at(sa, a * kKdBlock + g, c0), at(sa, a * kKdBlock + g, c0 + 8)};
+#pragma unroll
+        for (int b = a + 1; b < kKdBlocks; b++) {
+          uint32_t bh[2], bl[2];
+          float (&cc)[4] = acc[b * (b - 1) / 2 + a];
+#pragma unroll
+          for (int x = 0; x < 2; x++) {
+            if (b > a + 1) { const float2 m = *reinterpret_cast<const float2*>(sb + (b - 1) * DP + c0 + 8 * x); f[x].x *= m.x; f[x].y *= m.y; }
+            kd_split2<T>(f[x].x, f[x].y, bh[x], bl[x]);
+          }
+          mma_16816<T>(cc, ah[b - 1][0], ah[b - 1][1], ah[b - 1][2], ah[b - 1][3], bh[0], bh[1]);
+          mma_16816<T>(cc, al[b - 1][0], al[b - 1][1], al[b - 1][2], al[b - 1][3], bh[0], bh[1]);
+          mma_16816<T>(cc, ah[b - 1][0], ah[b - 1][1], ah[b - 1][2], ah[b - 1][3], bl[0], bl[1]);
+        }
       }
-      mma_16816<T>(acc, ah[0], ah[1], ah[2], ah[3], bh[0], bh[1]);
-      mma_16816<T>(acc, al[0], al[1], al[2], al[3], bh[0], bh[1]);
-      mma_16816<T>(acc, ah[0], ah[1], ah[2], ah[3], bl[0], bl[1]);
     }
-    const int i = b * kKdBlock + g, j = a * kKdBlock + 2 * q;
-    sQ[i * 36 + j] = acc[0]; sQ[i * 36 + j + 1] = acc[1];
-    if constexpr (DELTA) { sK[i * 36 + j] = acc[2] * s_beta[i]; sK[i * 36 + j + 1] = acc[3] * s_beta[i]; }
+#pragma unroll
+    for (int i = 0; i < 6; i++) {
+      float* to = s_part + warp * 768 + i * 128 + g * 8 + 2 * q;
+      *reinterpret_cast<float2*>(to) = make_float2(acc[i][0], acc[i][1]);
+      *reinterpret_cast<float2*>(to + 64) = make_float2(acc[i][2], acc[i][3]);
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int n = 0; n < 3; n++) {
+    const int i = tid + n * kKdThreads, pair = i >> 7, r = (i >> 3) & 15, j = i & 7;
+    float v = 0.f;
+#pragma unroll
+    for (int m = 0; m < kShares; m++) v += s_part[m * 768 + i];
+    const int b = pair < 1 ? 1 : pair < 3 ? 2 : 3, a = pair - b * (b - 1) / 2, row = b * kKdBlock + (r & 7), col = a * kKdBlock + j;
+    if (r < 8) sQ[row * 36 + col] = v;
+    else if constexpr (DELTA) sK[row * 36 + col] = v * s_beta[row];
   }
   __syncthreads();
   const auto store_q = [&](int i, int j) {               // four entries of Q
@@ -343,39 +384,27 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
     *reinterpret_cast<uint2*>(at + (kd_tc(DP) ? (j * 2) ^ ((i & 7) << 4) : j * 2)) = hi;
     *reinterpret_cast<uint2*>(at + (kd_tc(DP) ? (64 + j * 2) ^ ((i & 7) << 4) : kKdChunk * kKdAPitch * 2 + j * 2)) = lo;
   };
-  // rows of A q, A k and A_32 / A k, two channels at a time, and the chunk's decay
+  // rows of A q, A k and A_32 / A k, eight channels at a time
   const auto store_rows = [&](int first, int threads) {
-    for (int i = first; i < kKdBlocks * DH; i += threads) {
-      const int d = i % DH * 2, b = i / DH;
-      float2 pre = make_float2(1.f, 1.f), suf = make_float2(1.f, 1.f);
-#pragma unroll
-      for (int m = 0; m < kKdBlocks; m++) {
-        const float2 f = *reinterpret_cast<const float2*>(sb + m * DP + d);
-        if (m < b) { pre.x *= f.x; pre.y *= f.y; }
-        if (m > b) { suf.x *= f.x; suf.y *= f.y; }
-      }
-      if (b == 0) { float2* all = reinterpret_cast<float2*>(ops + L.decay + d * 4); const float2 f = *reinterpret_cast<const float2*>(sb + d); *all = make_float2(f.x * suf.x, f.y * suf.y); }
-      uint8_t* row0 = ops + (kd_tc(DP) ? (d & 63) * 2 + b * kKdBlock * 128 : b * kKdBlock * (DP + 8) * 2 + d * 2);
-      const int panel1 = kd_tc(DP) ? (d >> 6) * 2 * L.plane1 : 0, panel2 = kd_tc(DP) ? (d >> 6) * kKdChunk * 128 : 0;
-#pragma unroll
-      for (int j = 0; j < kKdBlock; j++) {
-        const int at = (b * kKdBlock + j) * P + d;
-        // panels: a row's 16-byte pieces are swapped by its number's low bits
-        uint8_t* row = kd_tc(DP) ? ops + (((d & 63) * 2) ^ (j << 4)) + b * kKdBlock * 128 + j * 128 : row0 + j * (DP + 8) * 2;
-        auto put = [&](uint8_t* to, int to_lo, float x, float y) {
-          uint32_t hi, lo;
-          kd_split2<T>(x, y, hi, lo);
-          *reinterpret_cast<uint32_t*>(to) = hi;
-          *reinterpret_cast<uint32_t*>(to + to_lo) = lo;
-        };
-        const float2 q = *reinterpret_cast<const float2*>(sq + at), v = *reinterpret_cast<const float2*>(sa + at);
-        put(row + L.qg + panel1, L.plane1, q.x * pre.x, q.y * pre.y);
-        put(row + L.kg + panel2, L.plane2, v.x * suf.x, v.y * suf.y);
-        if constexpr (DELTA && !kSolveValues) {
-          const float2 k = *reinterpret_cast<const float2*>(sk + at);
-          put(row + L.w + panel1, L.plane1, k.x * pre.x, k.y * pre.y);
-        }
-      }
+    for (int i = first; i < kKdChunk * DP / 8; i += threads) {
+      const int r = i / (DP / 8), unit = i % (DP / 8), b = r / kKdBlock, d = unit * 8;
+      // panels: a row's 16-byte pieces are swapped by its number's low bits
+      uint8_t* at = ops + (kd_tc(DP) ? r * 128 + (((unit & 7) ^ (r & 7)) << 4) : r * (DP + 8) * 2 + unit * 16);
+      const int panel1 = kd_tc(DP) ? (unit >> 3) * 2 * L.plane1 : 0, panel2 = kd_tc(DP) ? (unit >> 3) * kKdChunk * 128 : 0;
+      auto put = [&](uint8_t* to, int to_lo, const float* x, const float* f) {
+        uint4 hi, lo;
+        const float4 x0 = *reinterpret_cast<const float4*>(x + r * P + d), x1 = *reinterpret_cast<const float4*>(x + r * P + d + 4);
+        const float4 f0 = *reinterpret_cast<const float4*>(f + b * DP + d), f1 = *reinterpret_cast<const float4*>(f + b * DP + d + 4);
+        kd_split2<T>(x0.x * f0.x, x0.y * f0.y, hi.x, lo.x);
+        kd_split2<T>(x0.z * f0.z, x0.w * f0.w, hi.y, lo.y);
+        kd_split2<T>(x1.x * f1.x, x1.y * f1.y, hi.z, lo.z);
+        kd_split2<T>(x1.z * f1.z, x1.w * f1.w, hi.w, lo.w);
+        *reinterpret_cast<uint4*>(to) = hi;
+        *reinterpret_cast<uint4*>(to + to_lo) = lo;
+      };
+      put(at + L.qg + panel1, L.plane1, sq, s_pre);
+      put(at + L.kg + panel2, L.plane2, sa, s_suf);
+      if constexpr (DELTA && !kSolveValues) put(at + L.w + panel1, L.plane1, sk, s_pre);
     }
   };
   if constexpr (!DELTA || kSolveValues) {
@@ -1025,7 +1054,7 @@ __global__ void __launch_bounds__(256) key_decay_finish_kernel(const KdParams p)
 template <typename T, int DP, bool DELTA>
 static cudaError_t launch_kd(cudaStream_t s, const KdParams& p) {
   constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
-  constexpr size_t prep = ((size_t)3 * kKdChunk * (DP + 4) + kKdBlocks * DP + 2 * kKdChunk * 36 + 3 * kKdChunk + DP) * sizeof(float);
+  constexpr size_t prep = ((size_t)3 * kKdChunk * (DP + 4) + kKdBlocks * DP + 2 * kKdChunk * 36 + 3 * kKdChunk + DP + 2 * kKdBlocks * DP + 8 * 768) * sizeof(float);
   constexpr size_t scan = 2 * (size_t)L.stride + (kd_tc(DP) ? 1024 : 0);
   static bool attr = false;
   if (!attr) {
