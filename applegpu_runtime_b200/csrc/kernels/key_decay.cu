@@ -1,17 +1,16 @@
 // Matrix states with one decay per key channel: the token-by-token form and the choice between it and the chunked one.
 //
-// A cluster works on one head of one sequence, each CTA on a slice of the value columns of S. The channels of q, k and the decay are
-// computed once, a slice per CTA, and go to all CTAs over distributed shared memory. With r = (diag(a) S)^T k and
-// p = (diag(a) S)^T q taken in one pass over S, the rest of a token is u = beta (v - r) (or v), o = p + (k . q) u and the update
-// S <- diag(a) S + k u^T, which is the order of the recurrence: the read-out sees the current token's write. S stays in registers
-// from token to token where a CTA's columns fit one per thread.
+// A CTA works on up to 128 value columns of one head of one sequence (a cluster where a head has more: the head's norm adds their
+// sums of squares over distributed shared memory). With r = (diag(a) S)^T k and p = (diag(a) S)^T q taken in one pass over S, the
+// rest of a token is u = beta (v - r) (or v), o = p + (k . q) u and the update S <- diag(a) S + k u^T, which is the order of the
+// recurrence: the read-out sees the current token's write. S stays in registers from token to token where the CTA's columns fit.
 #include "key_decay.cuh"
 #include "sm100.cuh"
 #include <algorithm>
 
 namespace ag { namespace k {
 
-constexpr int kKsThreads = 256;
+constexpr int kKsThreads = 512;
 
 // out[i] = sum_r w[row0 + i][r] x[r] for n rows of a [.., ld] matrix: a few lanes per row, 16-byte pieces
 template <typename T>
@@ -19,31 +18,40 @@ __device__ __forceinline__ void kd_rows(const T* w, int ld, int rank, const floa
   constexpr int N = Pack<T>::N;
   const int pieces = (rank + N - 1) / N;
   int g = 1;
-  while (g < 8 && g * 2 <= pieces) g *= 2;
+  while (g < 4 && g * 2 <= pieces) g *= 2;
   const int lane = threadIdx.x % g;
   for (int i0 = 0; i0 < n; i0 += kKsThreads / g) {
     const int i = i0 + (int)threadIdx.x / g;
     float a = 0.f;
-    if (i < n)
+    if (i < n) {
+      const T* row = w + (long long)i * ld;
+#pragma unroll 4
       for (int q = lane; q < pieces; q += g) {
-        const Pack<T> v = ld16(w + (long long)i * ld + q * N);
+        const Pack<T> v = ld16(row + q * N);
 #pragma unroll
         for (int e = 0; e < N; e++) a = fmaf(Cvt<T>::to(v.v[e]), x[q * N + e], a);
       }
+    }
     for (int o = g >> 1; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
     if (i < n && lane == 0) out[i] = a;
   }
 }
+__device__ __forceinline__ void kd_prefetch(const void* at, int bytes) {
+  for (int i = threadIdx.x * 128; i < bytes; i += kKsThreads * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const uint8_t*>(at) + i));
+}
 
-template <typename T, int NR>          // NR rows of S per thread
-__global__ void __launch_bounds__(kKsThreads) key_decay_step_kernel(const KdParams p, int slice, int tx_n) {
+template <typename T, int VEC, int NR>          // NR rows of S per thread, VEC neighbouring columns of each
+__global__ void __launch_bounds__(kKsThreads, VEC * NR <= 32 ? 2 : 1) key_decay_step_kernel(const KdParams p, int slice, int tx_n) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float s_sq[2];
-  const int D = p.dim, E = p.vdim;
+  const int D = p.dim, E = p.vdim, cw = tx_n * VEC;       // cw: columns of a pass
   const int rank = (int)sm100::cluster_ctarank(), n_rank = (int)gridDim.x;
   const int h = blockIdx.y, s = blockIdx.z, qh = h / p.group;
   const int e0 = rank * slice, ne = max(0, min(slice, E - e0));
-  float* sq = sm;                        // [D] each
+  const int ty_n = kKsThreads / tx_n, tx = threadIdx.x % tx_n, ty = threadIdx.x / tx_n, lane = threadIdx.x & 31;
+  float* part = sm;                      // [2][ty][cw] shares of r and p
+  float* s_r = part + 2 * kKsThreads * VEC;      // [2][cw] their sums
+  float* sq = s_r + 2 * cw;              // [D] each
   float* sk = sq + D;
   float* sa = sk + D;
   float* sv = sa + D;                    // [slice] each
@@ -51,110 +59,141 @@ __global__ void __launch_bounds__(kKsThreads) key_decay_step_kernel(const KdPara
   float* so = sg + slice;
   float* sx = so + slice;                // a1 and g1 of the token, padded with zeros to whole packs
   float* sy = sx + p.a_ld;
-  float* sz = sy + p.g_ld;               // [D] decay inputs of this CTA's channels
-  float* part = sz + D;                  // [ty][tx] twice
-  const int ty_n = kKsThreads / tx_n, tx = threadIdx.x % tx_n, ty = threadIdx.x / tx_n, lane = threadIdx.x & 31;
-  const int cs = (D + n_rank - 1) / n_rank, c0 = min(D, rank * cs), nc = min(cs, D - c0);       // this CTA's channels
-  float* S = p.state(s) + (long long)h * D * E + e0;
-  // weights and state start towards the L2 before the previous kernel is waited for
-  {
-    constexpr int line = 128 / (int)sizeof(T);
-    const T* a2 = reinterpret_cast<const T*>(p.a2) + ((long long)h * D + c0) * p.a_ld;
-    if (!p.z) for (int i = threadIdx.x * line; i < nc * p.a_ld; i += kKsThreads * line) asm volatile("prefetch.global.L2 [%0];" ::"l"(a2 + i));
-    if (!p.gate && p.g_rank) {
-      const T* g2 = reinterpret_cast<const T*>(p.g2) + ((long long)h * E + e0) * p.g_ld;
-      for (int i = threadIdx.x * line; i < ne * p.g_ld; i += kKsThreads * line) asm volatile("prefetch.global.L2 [%0];" ::"l"(g2 + i));
-    }
-    if (ne > 0) for (int d = threadIdx.x; d < D; d += kKsThreads) asm volatile("prefetch.global.L2 [%0];" ::"l"(S + (long long)d * E));
+  // weights start towards the L2 before the previous kernel is waited for
+  kd_prefetch(p.bias + h * D, D * 4);
+  if (!p.z) kd_prefetch(reinterpret_cast<const T*>(p.a2) + (long long)h * D * p.a_ld, D * p.a_ld * (int)sizeof(T));
+  if (!p.gate && p.g_rank) kd_prefetch(reinterpret_cast<const T*>(p.g2) + ((long long)h * E + e0) * p.g_ld, ne * p.g_ld * (int)sizeof(T));
+  if (p.taps) {
+    const int qk = p.qk_heads * D;
+    kd_prefetch(p.conv + (long long)qh * D * p.taps, D * p.taps * 4);
+    kd_prefetch(p.conv + (long long)(qk + qh * D) * p.taps, D * p.taps * 4);
+    kd_prefetch(p.conv + (long long)(2 * qk + h * E + e0) * p.taps, ne * p.taps * 4);
   }
-  if (n_rank > 1) sm100::cluster_sync_all();        // every CTA has started before another one writes into it
   pdl_wait();
   pdl_trigger();
+  float* S = p.state(s) + (long long)h * D * E + e0;
+  const bool resident = slice <= cw;
+  float st[NR][VEC];
+  const int step = ty_n * E;
+  auto load = [&](int c) {
+    const float* at = S + ty * E + c;
+#pragma unroll
+    for (int n = 0; n < NR; n++, at += step) {
+      const bool in = n * ty_n + ty < D && c < ne;
+      if constexpr (VEC == 4) {
+        const float4 f = in ? *reinterpret_cast<const float4*>(at) : make_float4(0.f, 0.f, 0.f, 0.f);
+        st[n][0] = f.x; st[n][1] = f.y; st[n][2] = f.z; st[n][3] = f.w;
+      } else st[n][0] = in ? *at : 0.f;
+    }
+  };
+  auto store = [&](int c) {
+    float* at = S + ty * E + c;
+#pragma unroll
+    for (int n = 0; n < NR; n++, at += step) {
+      if (n * ty_n + ty >= D || c >= ne) continue;
+      if constexpr (VEC == 4) *reinterpret_cast<float4*>(at) = make_float4(st[n][0], st[n][1], st[n][2], st[n][3]);
+      else *at = st[n][0];
+    }
+  };
+  if (resident) load(tx * VEC);
   const int pos = p.pos[s];
   const T* base = reinterpret_cast<const T*>(p.proj) + (long long)s * p.T * p.ld;
   T* ring = p.ring_of<T>(s);
-  const bool resident = slice <= tx_n;
-  float st[NR];
-  auto load = [&](int c) {
-#pragma unroll
-    for (int n = 0; n < NR; n++) { const int d = n * ty_n + ty; st[n] = d < D && c < ne ? S[(long long)d * E + c] : 0.f; }
-  };
-  auto store = [&](int c) {
-#pragma unroll
-    for (int n = 0; n < NR; n++) { const int d = n * ty_n + ty; if (d < D && c < ne) S[(long long)d * E + c] = st[n]; }
-  };
-  if (resident) load(tx);
+  const float rate = p.softplus ? p.rate[h] : 0.f;
   for (int t = 0; t < p.T; t++) {
     const T* row = base + (long long)t * p.ld;
     const long long r = (long long)s * p.T + t;
+    const float beta_raw = p.delta ? p.beta[r * p.beta_ld + h] : 0.f;
+    const int place = p.ring ? (pos + t) % p.ring : 0;            // of this token's raw inputs among the ring's rows
+    const bool keep = p.ring && p.T <= kKeyDecayStepTokens;       // nothing of this launch reads the row they take
     __syncthreads();
-    // own channels of q and k go to every CTA of the cluster
-    auto push = [&](float* at, float v) {
-      if (n_rank == 1) *at = v;
-      else
-        for (int r = 0; r < n_rank; r++) asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(sm100::mapa_u32(sm100::smem_u32(at), (uint32_t)r)), "f"(v) : "memory");
-    };
-    for (int i = threadIdx.x; i < 2 * nc; i += kKsThreads) {
-      const bool is_k = i >= nc;
-      const int d = c0 + (is_k ? i - nc : i), c = qh * D + d;
-      push((is_k ? sk : sq) + d, kd_input<T>(p, base, ring, pos, t, (is_k ? p.k_off : p.q_off) + c, (is_k ? p.qk_heads * D : 0) + c));
+    for (int i = threadIdx.x; i < 2 * D + ne; i += kKsThreads) {
+      const int part_of = i < D ? 0 : i < 2 * D ? 1 : 2;
+      const int c = part_of < 2 ? qh * D + i - part_of * D : h * E + e0 + i - 2 * D;
+      const int col = (part_of == 0 ? p.q_off : part_of == 1 ? p.k_off : p.v_off) + c, ch = part_of * p.qk_heads * D + c;
+      const T raw = row[col];
+      float v = Cvt<T>::to(raw);
+      if (p.taps) {
+        const float* w = p.conv + (long long)ch * p.taps + p.taps - 1;
+        v *= __ldg(w);
+        for (int b = 1; b < p.taps; b++) {
+          float x = 0.f;
+          if (t >= b) x = Cvt<T>::to(row[col - (long long)b * p.ld]);
+          else if (pos + t >= b) { int q = place - b; if (q < 0) q += p.ring; x = Cvt<T>::to(ring[(long long)q * p.channels + ch]); }
+          v = fmaf(__ldg(w - b), x, v);
+        }
+        v = silu_f(v);
+      }
+      (part_of == 0 ? sq : part_of == 1 ? sk - D : sv - 2 * D)[i] = v;
+      if (keep && (part_of == 2 || (rank == 0 && h % p.group == 0))) ring[(long long)place * p.channels + ch] = raw;
     }
-    for (int i = threadIdx.x; i < ne; i += kKsThreads) { const int c = h * E + e0 + i; sv[i] = kd_input<T>(p, base, ring, pos, t, p.v_off + c, 2 * p.qk_heads * D + c); }
-    if (p.z) for (int i = threadIdx.x; i < nc; i += kKsThreads) sz[i] = p.z[r * p.heads * D + h * D + c0 + i];
+    if (p.z) for (int i = threadIdx.x; i < D; i += kKsThreads) sa[i] = p.z[r * p.heads * D + h * D + i];
     else for (int i = threadIdx.x; i < p.a_ld; i += kKsThreads) sx[i] = i < p.a_rank ? Cvt<T>::to(row[p.a_off + i]) : 0.f;
     if (p.gate || p.g_rank == 0)
       for (int i = threadIdx.x; i < ne; i += kKsThreads)
         sg[i] = p.gate ? Cvt<T>::to(reinterpret_cast<const T*>(p.gate)[r * p.gate_ld + h * E + e0 + i]) : Cvt<T>::to(row[p.g_off + h * E + e0 + i]);
     else for (int i = threadIdx.x; i < p.g_ld; i += kKsThreads) sy[i] = i < p.g_rank ? Cvt<T>::to(row[p.g_off + i]) : 0.f;
-    // this token's raw inputs for the convolutions of later portions; nothing of this launch reads the row they take
-    if (p.ring && p.T <= kKeyDecayStepTokens) {
-      T* dst = ring + (long long)((pos + t) % p.ring) * p.channels;
-      const int vc = 2 * p.qk_heads * D + h * E + e0;
-      for (int i = threadIdx.x; i < ne; i += kKsThreads) dst[vc + i] = row[p.v_off + h * E + e0 + i];
-      if (rank == 0 && h % p.group == 0)
-        for (int i = threadIdx.x; i < 2 * D; i += kKsThreads) { const int c = qh * D + i % D; dst[(i / D) * p.qk_heads * D + c] = row[(i < D ? p.q_off : p.k_off) + c]; }
-    }
     __syncthreads();
-    if (!p.z) kd_rows<T>(reinterpret_cast<const T*>(p.a2) + ((long long)h * D + c0) * p.a_ld, p.a_ld, p.a_rank, sx, nc, sz);
+    if (!p.z) kd_rows<T>(reinterpret_cast<const T*>(p.a2) + (long long)h * D * p.a_ld, p.a_ld, p.a_rank, sx, D, sa);
     if (!p.gate && p.g_rank) kd_rows<T>(reinterpret_cast<const T*>(p.g2) + ((long long)h * E + e0) * p.g_ld, p.g_ld, p.g_rank, sy, ne, sg);
-    __syncthreads();
-    for (int i = threadIdx.x; i < nc; i += kKsThreads) push(sa + c0 + i, kd_decay(p, h, sz[i] + p.bias[h * D + c0 + i]));
-    if (n_rank > 1) sm100::cluster_sync_all(); else __syncthreads();
     // sums over the head, by every warp for itself
     float qq = 0.f, kk = 0.f, qk = 0.f;
     for (int i = lane; i < D; i += 32) { const float a = sq[i], b = sk[i]; qq = fmaf(a, a, qq); kk = fmaf(b, b, kk); qk = fmaf(a, b, qk); }
     qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
     const float fq = p.unit ? p.q_scale / sqrtf(qq + 1e-6f) : p.q_scale, fk = p.unit ? 1.0f / sqrtf(kk + 1e-6f) : 1.0f;
     qk *= fq * fk;
-    const float beta = p.delta ? sigmoid_f(p.beta[r * p.beta_ld + h]) : 1.f;
-    for (int col = 0; col < slice; col += tx_n) {
-      const int c = col + tx;
+    const float beta = p.delta ? sigmoid_f(beta_raw) : 1.f;
+    __syncthreads();
+    for (int i = threadIdx.x; i < D; i += kKsThreads) {
+      const float z = sa[i] + p.bias[h * D + i];
+      sa[i] = p.softplus ? expf(-rate * kd_softplus(z)) : expf(-kd_softplus(-z) * p.inv_tau);
+    }
+    __syncthreads();
+    for (int c0 = 0; c0 < slice; c0 += cw) {
+      const int c = c0 + tx * VEC;
       if (!resident) load(c);
-      float rk = 0.f, rq = 0.f;
+      float rk[VEC], rq[VEC];
+#pragma unroll
+      for (int v = 0; v < VEC; v++) { rk[v] = 0.f; rq[v] = 0.f; }
 #pragma unroll
       for (int n = 0; n < NR; n++) {
         const int d = n * ty_n + ty;
-        if (d < D) {
-          st[n] *= sa[d];
-          rk = fmaf(st[n], sk[d], rk);
-          rq = fmaf(st[n], sq[d], rq);
-        }
+        if (d >= D) break;
+        const float a = sa[d], k = sk[d], q = sq[d];
+#pragma unroll
+        for (int v = 0; v < VEC; v++) { st[n][v] *= a; rk[v] = fmaf(st[n][v], k, rk[v]); rq[v] = fmaf(st[n][v], q, rq[v]); }
       }
-      part[threadIdx.x] = rk;
-      part[kKsThreads + threadIdx.x] = rq;
+      if constexpr (VEC == 4) {
+        *reinterpret_cast<float4*>(part + threadIdx.x * 4) = make_float4(rk[0], rk[1], rk[2], rk[3]);
+        *reinterpret_cast<float4*>(part + (kKsThreads + threadIdx.x) * 4) = make_float4(rq[0], rq[1], rq[2], rq[3]);
+      } else { part[threadIdx.x] = rk[0]; part[kKsThreads + threadIdx.x] = rq[0]; }
       __syncthreads();
-      rk = 0.f; rq = 0.f;
-      for (int y = 0; y < ty_n; y++) { rk += part[y * tx_n + tx]; rq += part[kKsThreads + y * tx_n + tx]; }
-      rk *= fk; rq *= fq;
-      const float v = c < ne ? sv[c] : 0.f;
-      const float u = p.delta ? beta * (v - rk) : v;
+      for (int i = threadIdx.x; i < 2 * cw; i += kKsThreads) {
+        const float* at = part + (i < cw ? i : kKsThreads * VEC + i - cw);
+        float a = 0.f;
+#pragma unroll 8
+        for (int y = 0; y < ty_n; y++) a += at[y * cw];
+        s_r[i] = a * (i < cw ? fk : fq);
+      }
+      __syncthreads();
+      float u[VEC];
+#pragma unroll
+      for (int v = 0; v < VEC; v++) {
+        const float x = c + v < ne ? sv[c + v] : 0.f;
+        u[v] = p.delta ? beta * (x - s_r[tx * VEC + v]) : x;
+        if (ty == 0 && c + v < ne) so[c + v] = fmaf(qk, u[v], s_r[cw + tx * VEC + v]);
+        u[v] *= fk;
+      }
 #pragma unroll
       for (int n = 0; n < NR; n++) {
         const int d = n * ty_n + ty;
-        if (d < D) st[n] = fmaf(sk[d], fk * u, st[n]);
+        if (d >= D) break;
+        const float k = sk[d];
+#pragma unroll
+        for (int v = 0; v < VEC; v++) st[n][v] = fmaf(k, u[v], st[n][v]);
       }
-      if (ty == 0 && c < slice) so[c] = c < ne ? fmaf(qk, u, rq) : 0.f;
       if (!resident) { store(c); __syncthreads(); }
+      else if (t + 1 == p.T) store(c);
     }
     __syncthreads();
     float ss = 0.f;
@@ -175,7 +214,6 @@ __global__ void __launch_bounds__(kKsThreads) key_decay_step_kernel(const KdPara
     T* y = reinterpret_cast<T*>(p.y) + r * p.y_ld + h * E + e0;
     for (int i = threadIdx.x; i < ne; i += kKsThreads) y[i] = Cvt<T>::from(so[i] * rs * p.norm[e0 + i] * kd_gate(p, sg[i]));
   }
-  if (resident) store(tx);
   if (n_rank > 1) sm100::cluster_sync_all();        // no CTA leaves while another may still read its sum
 }
 
@@ -193,11 +231,11 @@ __global__ void __launch_bounds__(256) key_decay_tail_kernel(const KdParams p) {
   }
 }
 
-template <typename T, int NR>
+template <typename T, int VEC, int NR>
 static cudaError_t launch_ks(cudaStream_t s, const KdParams& p, int ranks, int slice, int tx_n, size_t smem) {
   static bool attr = false;
   if (!attr) {
-    cudaError_t e = cudaFuncSetAttribute(key_decay_step_kernel<T, NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(key_decay_step_kernel<T, VEC, NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
     if (e != cudaSuccess) return e;
     attr = true;
   }
@@ -207,25 +245,29 @@ static cudaError_t launch_ks(cudaStream_t s, const KdParams& p, int ranks, int s
   at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization; at[0].val.programmaticStreamSerializationAllowed = pdl_enabled() ? 1 : 0;
   at[1].id = cudaLaunchAttributeClusterDimension; at[1].val.clusterDim.x = (unsigned)ranks; at[1].val.clusterDim.y = 1; at[1].val.clusterDim.z = 1;
   cfg.attrs = at; cfg.numAttrs = 2;
-  return cudaLaunchKernelEx(&cfg, key_decay_step_kernel<T, NR>, p, slice, tx_n);
+  return cudaLaunchKernelEx(&cfg, key_decay_step_kernel<T, VEC, NR>, p, slice, tx_n);
 }
 
 static Status key_decay_step(cudaStream_t s, DType dt, const KdParams& p) {
-  int ranks = 1;
-  while (ranks < 8 && p.vdim / (ranks * 2) >= 16) ranks *= 2;
-  const int slice = (p.vdim + ranks - 1) / ranks;
-  int tx_n = 4;
-  while (tx_n < 32 && tx_n < slice) tx_n *= 2;
-  const int nr = (p.dim + kKsThreads / tx_n - 1) / (kKsThreads / tx_n);
-  const size_t smem = (4 * (size_t)p.dim + 3 * (size_t)slice + p.a_ld + p.g_ld + 2 * kKsThreads) * sizeof(float);
-  if (nr > 64 || smem > 100 * 1024) return Status::unsupported("key decay: head too large");
+  // four columns a thread where rows of S lie on 16 bytes and a thread's share of them fits its registers
+  auto shape = [&](int vec, int* ranks, int* slice, int* tx_n) {
+    const int most = 32 * vec;
+    *ranks = 1;
+    while (*ranks < 8 && (p.vdim + *ranks - 1) / *ranks > most) *ranks *= 2;
+    *slice = ((p.vdim + *ranks - 1) / *ranks + vec - 1) / vec * vec;
+    *tx_n = 4;
+    while (*tx_n < 32 && *tx_n * vec < *slice) *tx_n *= 2;
+    return (p.dim + kKsThreads / *tx_n - 1) / (kKsThreads / *tx_n);
+  };
+  int ranks, slice, tx_n, vec = 4, nr = shape(4, &ranks, &slice, &tx_n);
+  if (p.vdim % 4 || nr > 16) { vec = 1; nr = shape(1, &ranks, &slice, &tx_n); }
+  const size_t smem = (2 * (size_t)kKsThreads * vec + 2 * (size_t)tx_n * vec + 3 * (size_t)p.dim + 3 * (size_t)slice + p.a_ld + p.g_ld) * sizeof(float);
+  if (nr > 32 || smem > 100 * 1024) return Status::unsupported("key decay: head too large");
   cudaError_t e = cudaSuccess;
   AG_DISPATCH_FLOAT(dt, T, {
-    if (nr <= 4) e = launch_ks<T, 4>(s, p, ranks, slice, tx_n, smem);
-    else if (nr <= 8) e = launch_ks<T, 8>(s, p, ranks, slice, tx_n, smem);
-    else if (nr <= 16) e = launch_ks<T, 16>(s, p, ranks, slice, tx_n, smem);
-    else if (nr <= 32) e = launch_ks<T, 32>(s, p, ranks, slice, tx_n, smem);
-    else e = launch_ks<T, 64>(s, p, ranks, slice, tx_n, smem);
+    if (vec == 4) e = nr <= 2 ? launch_ks<T, 4, 2>(s, p, ranks, slice, tx_n, smem) : nr <= 4 ? launch_ks<T, 4, 4>(s, p, ranks, slice, tx_n, smem)
+                    : nr <= 8 ? launch_ks<T, 4, 8>(s, p, ranks, slice, tx_n, smem) : launch_ks<T, 4, 16>(s, p, ranks, slice, tx_n, smem);
+    else e = nr <= 8 ? launch_ks<T, 1, 8>(s, p, ranks, slice, tx_n, smem) : launch_ks<T, 1, 32>(s, p, ranks, slice, tx_n, smem);
   });
   return cuda_status(e, "key decay step");
 }

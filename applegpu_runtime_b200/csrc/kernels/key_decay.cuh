@@ -41,8 +41,6 @@ __device__ __forceinline__ float kd_input(const KdParams& p, const T* base, cons
   return silu_f(a);
 }
 __device__ __forceinline__ float kd_softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
-// decay of a key channel from its input z (bias included)
-__device__ __forceinline__ float kd_decay(const KdParams& p, int h, float z) { return p.softplus ? expf(-p.rate[h] * kd_softplus(z)) : expf(-kd_softplus(-z) * p.inv_tau); }
 __device__ __forceinline__ float kd_gate(const KdParams& p, float g) { return p.gate_silu ? silu_f(g) : sigmoid_f(g); }
 
 // What the prepare kernel hands to the scan for one chunk of one head. Up to 128 channels (tcgen05 scan): 128-byte swizzled panels of 64
