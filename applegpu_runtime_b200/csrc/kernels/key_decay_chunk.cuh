@@ -61,8 +61,7 @@ __device__ __forceinline__ float kd_softplus_fast(float x) { return fmaxf(x, 0.f
 // exp(f softplus(x)): a decay from its input z, x = z and f = -rate or x = -z and f = -1 / tau; f comes in log2 units
 __device__ __forceinline__ float kd_decay_fast(float f_log2, float x) { return ex2_approx(f_log2 * kd_softplus_fast(x)); }
 __device__ __forceinline__ float kd_sigmoid_fast(float x) { return kd_rcp(1.0f + ex2_approx(-kKdLog2e * x)); }
-template <typename T>
-__device__ __forceinline__ float kd_gate_fast(const KdParams& p, T g) { const float x = Cvt<T>::to(g), s = kd_sigmoid_fast(x); return p.gate_silu ? x * s : s; }
+__device__ __forceinline__ float kd_gate_fast(const KdParams& p, float x) { const float s = kd_sigmoid_fast(x); return p.gate_silu ? x * s : s; }
 __device__ __forceinline__ float kd_silu_fast(float x) { return x * kd_sigmoid_fast(x); }
 
 // Convolutions of up to kKdTaps taps slide over their raw inputs; longer ones read them tap by tap.
@@ -72,6 +71,15 @@ __device__ __forceinline__ void kd_taps(const KdParams& p, int ch, float (&w)[kK
 #pragma unroll
   for (int j = 0; j < kKdTaps; j++) { const int at = j - (kKdTaps - p.taps); w[j] = at >= 0 ? __ldg(p.conv + (long long)ch * p.taps + at) : 0.f; }
 }
+// A 16-bit element in a register of its own: an array of these is not packed in pairs, which would wait for the loads
+template <typename T> __device__ __forceinline__ uint32_t kd_bits(const T* at) { return *reinterpret_cast<const uint16_t*>(at); }
+template <typename T> __device__ __forceinline__ float kd_value(uint32_t bits) {
+  const uint16_t b = (uint16_t)bits;
+  return Cvt<T>::to(*reinterpret_cast<const T*>(&b));
+}
+template <> __device__ __forceinline__ float kd_value<__nv_bfloat16>(uint32_t bits) { return __uint_as_float(bits << 16); }
+template <typename T>
+__device__ __forceinline__ uint32_t kd_round_bits(float x) { const T v = Cvt<T>::from(x); return kd_bits<T>(&v); }
 template <typename T>
 __device__ __forceinline__ float2 kd_pair(const T* at) {
   const uint32_t raw = *reinterpret_cast<const uint32_t*>(at);
@@ -668,9 +676,9 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
   using namespace sm100;
   constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
   constexpr uint32_t cS = 0, cA = 128, cO = 256, cR = cA + 64, cU = 64, kLo = L.rows1;      // cU: within a buffer; kLo: from a product to its remainder's
-  constexpr int kSteps = DP / 16;
+  constexpr int kSteps = DP / 16, kFirst = DELTA ? (kSteps + 1) / 4 * 2 : 0;      // steps of 16 channels; those whose products start ahead of the others
   extern __shared__ uint8_t smem_raw[];
-  __shared__ uint64_t full[2], empty[2], s_ready, r_ready, u_ready, x_full, u_full, s_full, o_full[2], o_free[2], sums;
+  __shared__ uint64_t full[2], empty[2], s_first, s_ready, r_ready, u_ready, x_full, u_full, s_full, o_full[2], o_free[2], sums;
   __shared__ uint32_t tmem_slot;
   __shared__ float s_sum[2][4][kKdChunk];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -680,7 +688,7 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
   if (threadIdx.x == 0) {
     for (int i = 0; i < 2; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], kKdStateWarps + 1); mbar_init(&o_full[i], 1); mbar_init(&o_free[i], 4); }
     mbar_init(&sums, 4);
-    mbar_init(&s_ready, kKdStateWarps); mbar_init(&r_ready, kKdStateWarps); mbar_init(&u_ready, kKdStateWarps);
+    mbar_init(&s_first, kKdStateWarps); mbar_init(&s_ready, kKdStateWarps); mbar_init(&r_ready, kKdStateWarps); mbar_init(&u_ready, kKdStateWarps);
     mbar_init(&x_full, 1); mbar_init(&u_full, 1); mbar_init(&s_full, 1);
     mbar_fence_init();
   }
@@ -711,17 +719,35 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
         const int st = c & 1;
         const uint32_t ph = (uint32_t)(c & 1), ph2 = (uint32_t)((c >> 1) & 1), base = smem_u32(smem + st * L.stride);
         const uint32_t buf = tm + cO + (uint32_t)(st * 128), acc_o = buf + (DELTA ? 32u : 0u), cu = buf + cU;
-        if (!mbar_wait(&full[st], ph2, status, 62) || !mbar_wait(&o_free[st], ph2 ^ 1, status, 63) || !mbar_wait(&s_ready, ph, status, 64)) break;
-        tc_fence_after_sync();
+        if (!mbar_wait(&full[st], ph2, status, 62) || !mbar_wait(&o_free[st], ph2 ^ 1, status, 63)) break;
         // a descriptor's address field counts 16-byte units: offsets are added to it
         const uint64_t d1 = make_smem_desc_sw128(base, 16, 1024), dq = d1 + (L.q >> 4), dt = d1 + (L.t >> 4), ds = make_smem_desc_sw128(base + L.kg, kKdChunk * 128, 1024);
+        auto rows_product = [&](int k) {                             // high parts with the rows and their remainders side by side, remainders with the rows
+          const uint64_t d = d1 + (((k >> 2) * 2 * L.plane1 + (k & 3) * 32) >> 4);
+          mma_f16_ts(buf, tm + cA + (uint32_t)(k * 8), d, id_1, k > 0 ? 1u : 0u);
+          mma_f16_ts(buf, tm + cA + (uint32_t)(DP / 2 + k * 8), d, id_2, 1u);
+        };
+        auto state_product = [&]() {                                 // high x high, remainder x high, high x remainder
 #pragma unroll
-        for (int k = 0; k < kSteps; k++)                             // high parts with rows and their remainders side by side
-          mma_f16_ts(buf, tm + cA + (uint32_t)(k * 8), d1 + (((k >> 2) * 2 * L.plane1 + (k & 3) * 32) >> 4), id_1, k > 0 ? 1u : 0u);
+          for (int part = 0; part < 3; part++) {
+            if (part == 1 && exact) continue;
 #pragma unroll
-        for (int k = 0; k < kSteps; k++)                             // remainders with the rows
-          mma_f16_ts(buf, tm + cA + (uint32_t)(DP / 2 + k * 8), d1 + (((k >> 2) * 2 * L.plane1 + (k & 3) * 32) >> 4), id_2, 1u);
+            for (int k = 0; k < kKdChunk / 16; k++)
+              mma_f16_ts(tm + cS, cu + (uint32_t)((part == 1 ? 16 : 0) + k * 8), ds + (((part == 2 ? L.plane2 : 0) + k * 2048) >> 4), id_s, 1u);
+          }
+          mma_commit(&s_full);
+        };
         if constexpr (DELTA) {
+          if constexpr (kFirst > 0) {
+            if (!mbar_wait(&s_first, ph, status, 64)) break;
+            tc_fence_after_sync();
+#pragma unroll
+            for (int k = 0; k < kFirst; k++) rows_product(k);
+          }
+          if (!mbar_wait(&s_ready, ph, status, 64)) break;
+          tc_fence_after_sync();
+#pragma unroll
+          for (int k = kFirst; k < kSteps; k++) rows_product(k);
           mma_commit(&x_full);
           if (!mbar_wait(&r_ready, ph, status, 65)) break;
           tc_fence_after_sync();
@@ -732,15 +758,15 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
           mma_commit(&u_full);
           if (!mbar_wait(&u_ready, ph, status, 73)) break;
           tc_fence_after_sync();
-        }
+          state_product();
+        } else {
+          if (!mbar_wait(&s_ready, ph, status, 64)) break;
+          tc_fence_after_sync();
+          state_product();                                           // needs no more than u: ahead of the rows, which read the split copy of S
 #pragma unroll
-        for (int part = 0; part < 3; part++) {                       // high x high, remainder x high, high x remainder
-          if (part == 1 && exact) continue;
-#pragma unroll
-          for (int k = 0; k < kKdChunk / 16; k++)
-            mma_f16_ts(tm + cS, cu + (uint32_t)((part == 1 ? 16 : 0) + k * 8), ds + (((part == 2 ? L.plane2 : 0) + k * 2048) >> 4), id_s, 1u);
+          for (int k = 0; k < kSteps; k++) rows_product(k);
+          mma_commit(&x_full);
         }
-        mma_commit(&s_full);
 #pragma unroll
         for (int part = 0; part < 3; part++) {
           if (part == 1 && exact) continue;
@@ -787,17 +813,17 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
       if (lane == 0) mbar_arrive(bar);
     };
     // this thread's raw values of a chunk and the ones before them, requested a chunk ahead
-    T raw[kKdHalf + kKdTaps - 1];
+    uint32_t raw[kKdHalf + kKdTaps - 1];
     auto request = [&](int t0) {
       const T* src = base + (long long)(t0 - (kKdTaps - 1)) * p.ld + vcol;
       if (t0 >= kKdTaps - 1 && t0 + kKdHalf <= p.T) {
 #pragma unroll
-        for (int i = 0; i < kKdHalf + kKdTaps - 1; i++, src += p.ld) raw[i] = *src;
+        for (int i = 0; i < kKdHalf + kKdTaps - 1; i++, src += p.ld) raw[i] = kd_bits<T>(src);
       } else {
 #pragma unroll
         for (int i = 0; i < kKdHalf + kKdTaps - 1; i++) {
           const int t = t0 - (kKdTaps - 1) + i;
-          raw[i] = t >= p.T || (t < 0 && -t >= p.taps) ? Cvt<T>::from(0.f) : t >= 0 ? src[(long long)i * p.ld] : Cvt<T>::from(kd_raw<T>(p, base, ring, pos, t, vcol, vch));
+          raw[i] = t >= p.T || (t < 0 && -t >= p.taps) ? 0u : t >= 0 ? kd_bits<T>(src + (long long)i * p.ld) : kd_round_bits<T>(kd_raw<T>(p, base, ring, pos, t, vcol, vch));
         }
       }
     };
@@ -809,13 +835,13 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
       auto values = [&]() {
         if (p.taps == 0) {
 #pragma unroll
-          for (int i = 0; i < kKdHalf; i++) v[i] = Cvt<T>::to(raw[i + kKdTaps - 1]);
+          for (int i = 0; i < kKdHalf; i++) v[i] = kd_value<T>(raw[i + kKdTaps - 1]);
         } else if (p.taps <= kKdTaps) {
 #pragma unroll
           for (int i = 0; i < kKdHalf; i++) {
             float y = 0.f;
 #pragma unroll
-            for (int n = 0; n < kKdTaps; n++) y = fmaf(taps[n], Cvt<T>::to(raw[i + n]), y);
+            for (int n = 0; n < kKdTaps; n++) y = fmaf(taps[n], kd_value<T>(raw[i + n]), y);
             v[i] = kd_silu_fast(y);
           }
         } else {
@@ -837,7 +863,12 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
       tc_fence_after_sync();
       const float4* decay = reinterpret_cast<const float4*>(smem + st * L.stride + L.decay);
       uint32_t next[16];                                             // on its way while a piece is split
-      if (half < G) tmem_ld_32x16(lanes + cS + (uint32_t)(half * 16), next);
+      tmem_ld_32x16(lanes + cS + (uint32_t)(half * 16), next);
+      if (!DELTA && c > 0) {                                         // the copy of S is still an operand of the last rows
+        ok = __all_sync(0xffffffffu, mbar_wait(&x_full, ph ^ 1, status, 72));
+        if (!ok) break;
+        tc_fence_after_sync();
+      }
 #pragma unroll
       for (int n = 0; n < (G + 1) / 2; n++) {
         const int g = 2 * n + half;
@@ -855,6 +886,7 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
           x[4 * i + 2] = __float_as_uint(y[4 * i + 2] * f.z); x[4 * i + 3] = __float_as_uint(y[4 * i + 3] * f.w);
         }
         tmem_st_32x16(lanes + cS + (uint32_t)(g * 16), x);
+        if (kFirst > 0 && 2 * n + 2 == kFirst) arrive(&s_first);
       }
       if constexpr (!DELTA) {
         values();
@@ -912,16 +944,16 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
       const int st = c & 1, t0 = c * kKdChunk, nt = min(kKdChunk, p.T - t0);
       const long long row0 = (long long)s * p.T + t0;
       const bool whole = __all_sync(0xffffffffu, e < E) && nt == kKdChunk;
-      uint16_t gate[kKdChunk];
+      uint32_t gate[kKdChunk];
       if (fuse) {
         const T* g = p.gate ? reinterpret_cast<const T*>(p.gate) + row0 * p.gate_ld + (long long)h * E + e : reinterpret_cast<const T*>(p.proj) + row0 * p.ld + p.g_off + (long long)h * E + e;
         const long long ld = p.gate ? p.gate_ld : p.ld;
         if (whole) {
 #pragma unroll
-          for (int i = 0; i < kKdChunk; i++, g += ld) gate[i] = *reinterpret_cast<const uint16_t*>(g);
+          for (int i = 0; i < kKdChunk; i++, g += ld) gate[i] = kd_bits<T>(g);
         } else {
 #pragma unroll
-          for (int i = 0; i < kKdChunk; i++, g += ld) gate[i] = e < E && i < nt ? *reinterpret_cast<const uint16_t*>(g) : (uint16_t)0;
+          for (int i = 0; i < kKdChunk; i++, g += ld) gate[i] = e < E && i < nt ? kd_bits<T>(g) : 0u;
         }
       }
       if (!__all_sync(0xffffffffu, mbar_wait(&o_full[st], (uint32_t)((c >> 1) & 1), status, 70))) break;
@@ -974,9 +1006,7 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
       T res[kKdChunk];
 #pragma unroll
       for (int i = 0; i < kKdChunk; i++) {
-        T g;
-        *reinterpret_cast<uint16_t*>(&g) = gate[i];
-        res[i] = Cvt<T>::from(o[i] * (__shfl_sync(0xffffffffu, rs, i) * nw) * kd_gate_fast<T>(p, g));
+        res[i] = Cvt<T>::from(o[i] * (__shfl_sync(0xffffffffu, rs, i) * nw) * kd_gate_fast(p, kd_value<T>(gate[i])));
       }
       if (whole) {
 #pragma unroll
@@ -1032,8 +1062,8 @@ __global__ void __launch_bounds__(256) key_decay_finish_kernel(const KdParams p)
         const float4 x = v[n][q], w = __ldg(reinterpret_cast<const float4*>(p.norm + e));
         const T* gv = reinterpret_cast<const T*>(&z[n][q]);
         uint2 out;
-        out.x = pack2_t<T>(x.x * rs * w.x * kd_gate_fast<T>(p, gv[0]), x.y * rs * w.y * kd_gate_fast<T>(p, gv[1]));
-        out.y = pack2_t<T>(x.z * rs * w.z * kd_gate_fast<T>(p, gv[2]), x.w * rs * w.w * kd_gate_fast<T>(p, gv[3]));
+        out.x = pack2_t<T>(x.x * rs * w.x * kd_gate_fast(p, Cvt<T>::to(gv[0])), x.y * rs * w.y * kd_gate_fast(p, Cvt<T>::to(gv[1])));
+        out.y = pack2_t<T>(x.z * rs * w.z * kd_gate_fast(p, Cvt<T>::to(gv[2])), x.w * rs * w.w * kd_gate_fast(p, Cvt<T>::to(gv[3])));
         *reinterpret_cast<uint2*>(out_of(i0 + n) + e) = out;
       }
     }
@@ -1045,7 +1075,7 @@ __global__ void __launch_bounds__(256) key_decay_finish_kernel(const KdParams p)
       float sq = 0.f;
       for (int e = lane; e < E; e += 32) sq = fmaf(o[e], o[e], sq);
       const float rs = 1.0f / sqrtf(warp_sum(sq) / (float)E + p.eps);
-      for (int e = lane; e < E; e += 32) y[e] = Cvt<T>::from(o[e] * rs * p.norm[e] * kd_gate_fast<T>(p, g[e]));
+      for (int e = lane; e < E; e += 32) y[e] = Cvt<T>::from(o[e] * rs * p.norm[e] * kd_gate_fast(p, Cvt<T>::to(g[e])));
     }
   }
 }
