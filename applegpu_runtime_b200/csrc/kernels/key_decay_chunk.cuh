@@ -38,7 +38,9 @@ template <typename T>
 __device__ __forceinline__ void kd_split2(float x, float y, uint32_t& hi, uint32_t& lo) {
   hi = pack2_t<T>(x, y);
   const T* v = reinterpret_cast<const T*>(&hi);
-  lo = pack2_t<T>(x - Cvt<T>::to(v[0]), y - Cvt<T>::to(v[1]));
+  float a, b;
+  unpack_f32x2(fma_f32x2(pack_f32x2(Cvt<T>::to(v[0]), Cvt<T>::to(v[1])), pack_f32x2(-1.0f, -1.0f), pack_f32x2(x, y)), a, b);
+  lo = pack2_t<T>(a, b);
 }
 
 __device__ __forceinline__ float kd_rcp(float x) {
@@ -670,6 +672,7 @@ __global__ void __launch_bounds__(256) key_decay_scan_kernel(const KdParams p, i
 //   warp 12        S += u (A_32 / A k), o += u Q
 //   warps 8 - 11   o to memory, or through the head's norm and gate
 // Warp 13 loads the chunks' operands. All waits are bounded.
+constexpr int kd_stages(bool delta) { return delta ? 2 : 3; }      // chunks on their way; more shared memory would cost the delta rule's other loads their L1
 constexpr int kKdStateWarps = 8, kKdMmaWarp = 12, kKdLoadWarp = 13, kKdScanThreads = 14 * 32, kKdHalf = kKdChunk / 2;
 template <typename T, int DP, bool DELTA>
 __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(const KdParams p, int fuse, int* status) {
@@ -678,7 +681,8 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
   constexpr uint32_t cS = 0, cA = 128, cO = 256, cR = cA + 64, cU = 64, kLo = L.rows1;      // cU: within a buffer; kLo: from a product to its remainder's
   constexpr int kSteps = DP / 16, kFirst = DELTA ? (kSteps + 1) / 4 * 2 : 0;      // steps of 16 channels; those whose products start ahead of the others
   extern __shared__ uint8_t smem_raw[];
-  __shared__ uint64_t full[2], empty[2], s_first, s_ready, r_ready, u_ready, x_full, u_full, s_full, o_full[2], o_free[2], sums;
+  constexpr int kStages = kd_stages(DELTA);
+  __shared__ uint64_t full[kStages], empty[kStages], s_first, s_ready, r_ready, u_ready, x_full, u_full, s_full, o_full[2], o_free[2], sums;
   __shared__ uint32_t tmem_slot;
   __shared__ float s_sum[2][4][kKdChunk];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -686,7 +690,8 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
   const int h = blockIdx.y, s = blockIdx.z, E = p.vdim, D = p.dim;
   const long long sh = (long long)s * p.heads + h;
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 2; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], kKdStateWarps + 1); mbar_init(&o_full[i], 1); mbar_init(&o_free[i], 4); }
+    for (int i = 0; i < kStages; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], kKdStateWarps + 1); }
+    for (int i = 0; i < 2; i++) { mbar_init(&o_full[i], 1); mbar_init(&o_free[i], 4); }
     mbar_init(&sums, 4);
     mbar_init(&s_first, kKdStateWarps); mbar_init(&s_ready, kKdStateWarps); mbar_init(&r_ready, kKdStateWarps); mbar_init(&u_ready, kKdStateWarps);
     mbar_init(&x_full, 1); mbar_init(&u_full, 1); mbar_init(&s_full, 1);
@@ -704,8 +709,8 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
   if (warp == kKdLoadWarp) {
     if (lane == 0)
       for (int c = 0; c < p.chunks; c++) {
-        const int st = c & 1;
-        if (!mbar_wait(&empty[st], (uint32_t)((c >> 1) & 1) ^ 1, status, 61)) break;
+        const int st = c % kStages;
+        if (!mbar_wait(&empty[st], (uint32_t)((c / kStages) & 1) ^ 1, status, 61)) break;
         mbar_expect_tx(&full[st], (uint32_t)L.bytes);
         kd_bulk_load(smem + st * L.stride, p.ops + (sh * p.chunks + c) * L.stride, (uint32_t)L.bytes, &full[st]);
       }
@@ -716,10 +721,10 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
       const uint32_t id_64 = make_idesc_f16(fmt, 0, 0, 128, 64), id_32 = make_idesc_f16(fmt, 0, 0, 128, 32), id_s = make_idesc_f16(fmt, 0, 1, 128, DP);
       const bool exact = !DELTA && p.taps == 0;                      // u is the stored v: no remainder
       for (int c = 0; c < p.chunks; c++) {
-        const int st = c & 1;
-        const uint32_t ph = (uint32_t)(c & 1), ph2 = (uint32_t)((c >> 1) & 1), base = smem_u32(smem + st * L.stride);
+        const int st = c & 1, sg = c % kStages;
+        const uint32_t ph = (uint32_t)(c & 1), ph2 = (uint32_t)((c >> 1) & 1), base = smem_u32(smem + sg * L.stride);
         const uint32_t buf = tm + cO + (uint32_t)(st * 128), acc_o = buf + (DELTA ? 32u : 0u), cu = buf + cU;
-        if (!mbar_wait(&full[st], ph2, status, 62) || !mbar_wait(&o_free[st], ph2 ^ 1, status, 63)) break;
+        if (!mbar_wait(&full[sg], (uint32_t)((c / kStages) & 1), status, 62) || !mbar_wait(&o_free[st], ph2 ^ 1, status, 63)) break;
         // a descriptor's address field counts 16-byte units: offsets are added to it
         const uint64_t d1 = make_smem_desc_sw128(base, 16, 1024), dq = d1 + (L.q >> 4), dt = d1 + (L.t >> 4), ds = make_smem_desc_sw128(base + L.kg, kKdChunk * 128, 1024);
         auto rows_product = [&](int k) {                             // high parts with the rows and their remainders side by side, remainders with the rows
@@ -775,7 +780,7 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
             mma_f16_ts(acc_o, cu + (uint32_t)((part == 1 ? 16 : 0) + k * 8), dq + (((part == 2 ? 64 : 0) + k * 32) >> 4), id_32, 1u);
         }
         mma_commit(&o_full[st]);
-        mma_commit(&empty[st]);
+        mma_commit(&empty[sg]);
       }
     }
   } else if (warp < kKdStateWarps) {
@@ -829,7 +834,7 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
     };
     request(tb);
     for (int c = 0; c < p.chunks; c++) {
-      const int st = c & 1, t0 = c * kKdChunk + tb;
+      const int st = c & 1, sg = c % kStages, t0 = c * kKdChunk + tb;
       const uint32_t ph = (uint32_t)(c & 1), buf = lanes + cO + (uint32_t)(st * 128);
       float v[kKdHalf];
       auto values = [&]() {
@@ -858,10 +863,10 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
         }
         if (c + 1 < p.chunks) request(t0 + kKdChunk);
       };
-      ok = __all_sync(0xffffffffu, mbar_wait(&full[st], (uint32_t)((c >> 1) & 1), status, 66) && (c == 0 || mbar_wait(&s_full, ph ^ 1, status, 67)));
+      ok = __all_sync(0xffffffffu, mbar_wait(&full[sg], (uint32_t)((c / kStages) & 1), status, 66) && (c == 0 || mbar_wait(&s_full, ph ^ 1, status, 67)));
       if (!ok) break;
       tc_fence_after_sync();
-      const float4* decay = reinterpret_cast<const float4*>(smem + st * L.stride + L.decay);
+      const float4* decay = reinterpret_cast<const float4*>(smem + sg * L.stride + L.decay);
       uint32_t next[16];                                             // on its way while a piece is split
       tmem_ld_32x16(lanes + cS + (uint32_t)(half * 16), next);
       if (!DELTA && c > 0) {                                         // the copy of S is still an operand of the last rows
@@ -882,8 +887,8 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
 #pragma unroll
         for (int i = 0; i < 4; i++) {
           const float4 f = decay[g * 4 + i];
-          x[4 * i] = __float_as_uint(y[4 * i] * f.x); x[4 * i + 1] = __float_as_uint(y[4 * i + 1] * f.y);
-          x[4 * i + 2] = __float_as_uint(y[4 * i + 2] * f.z); x[4 * i + 3] = __float_as_uint(y[4 * i + 3] * f.w);
+          const uint64_t a = mul_f32x2(pack_f32x2(y[4 * i], y[4 * i + 1]), pack_f32x2(f.x, f.y)), b = mul_f32x2(pack_f32x2(y[4 * i + 2], y[4 * i + 3]), pack_f32x2(f.z, f.w));
+          x[4 * i] = (uint32_t)a; x[4 * i + 1] = (uint32_t)(a >> 32); x[4 * i + 2] = (uint32_t)b; x[4 * i + 3] = (uint32_t)(b >> 32);
         }
         tmem_st_32x16(lanes + cS + (uint32_t)(g * 16), x);
         if (kFirst > 0 && 2 * n + 2 == kFirst) arrive(&s_first);
@@ -892,16 +897,16 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
         values();
         split(v, buf + cU + (uint32_t)(half * 8), 16);               // its last reader was this buffer's o, two chunks ago
         arrive(&s_ready);
-        if (lane == 0) mbar_arrive(&empty[st]);
+        if (lane == 0) mbar_arrive(&empty[sg]);
       } else {
         arrive(&s_ready);
         values();
-        const float4* beta = reinterpret_cast<const float4*>(smem + st * L.stride + L.beta) + tb / 4;
+        const float4* beta = reinterpret_cast<const float4*>(smem + sg * L.stride + L.beta) + tb / 4;
         float b[kKdHalf];
 #pragma unroll
         for (int i = 0; i < kKdHalf / 4; i++) { const float4 f = beta[i]; b[4 * i] = f.x; b[4 * i + 1] = f.y; b[4 * i + 2] = f.z; b[4 * i + 3] = f.w; }
         __syncwarp();
-        if (lane == 0) mbar_arrive(&empty[st]);
+        if (lane == 0) mbar_arrive(&empty[sg]);
         uint32_t y[16];
         ok = __all_sync(0xffffffffu, mbar_wait(&x_full, ph, status, 68));
         if (!ok) break;
@@ -1085,7 +1090,7 @@ template <typename T, int DP, bool DELTA>
 static cudaError_t launch_kd(cudaStream_t s, const KdParams& p) {
   constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
   constexpr size_t prep = ((size_t)3 * kKdChunk * (DP + 4) + kKdBlocks * DP + 2 * kKdChunk * 36 + 3 * kKdChunk + DP + 2 * kKdBlocks * DP + 8 * 768) * sizeof(float);
-  constexpr size_t scan = 2 * (size_t)L.stride + (kd_tc(DP) ? 1024 : 0);
+  constexpr size_t scan = kd_tc(DP) ? kd_stages(DELTA) * (size_t)L.stride + 1024 : 2 * (size_t)L.stride;
   static bool attr = false;
   if (!attr) {
     cudaError_t e = cudaFuncSetAttribute(key_decay_prepare_kernel<T, DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep);

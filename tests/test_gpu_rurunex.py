@@ -64,7 +64,7 @@ KD_CASES = {
     "gla_192": dict(GLA, H=1, G=1, d=160, e=40, ar=8),
     "delta": dict(DELTA, H=2, G=2, d=32, e=32, ar=12), "delta_groups": dict(DELTA, H=6, G=2, d=24, e=40, ar=24, gr=9), "delta_odd": dict(DELTA, H=3, G=1, d=11, e=19, ar=3, gr=7, taps=2),
     "delta_128": dict(DELTA, H=1, G=1, d=128, e=128, ar=64, gr=64), "delta_96": dict(DELTA, H=2, G=1, d=72, e=80, ar=8), "delta_256": dict(DELTA, H=1, G=1, d=256, e=24, ar=8, taps=5),
-    "six_taps": dict(DELTA, H=2, G=1, d=40, e=24, ar=8, taps=6), "one_tap": dict(DELTA, H=2, G=1, d=16, e=16, ar=8, taps=1), "plain_delta": dict(DELTA, H=2, G=2, d=16, e=24, ar=8, unit=True, taps=0, gr=0, softplus=False),
+    "delta_values_200": dict(DELTA, H=1, G=1, d=64, e=200, ar=8), "six_taps": dict(DELTA, H=2, G=1, d=40, e=24, ar=8, taps=6), "one_tap": dict(DELTA, H=2, G=1, d=16, e=16, ar=8, taps=1), "plain_delta": dict(DELTA, H=2, G=2, d=16, e=24, ar=8, unit=True, taps=0, gr=0, softplus=False),
     "conv_without_delta": dict(GLA, H=2, G=1, d=24, e=16, ar=8, taps=3, softplus=True, gr=6), "beyond_chunks": dict(DELTA, H=1, G=1, d=300, e=20, ar=8),
 }
 
