@@ -90,7 +90,7 @@ __device__ __forceinline__ float2 kd_pair(const T* at) {
 }
 
 template <typename T, int DP, bool DELTA>
-__global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const KdParams p) {
+__global__ void __launch_bounds__(kKdThreads, kd_tc(DP) ? 3 : DP <= 192 ? 2 : 1) key_decay_prepare_kernel(const KdParams p) {
   constexpr int P = DP + 4, NC = DP / 32, DH = DP / 2;
   constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
   extern __shared__ __align__(16) float sm[];
@@ -103,9 +103,9 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
   float* s_beta = sK + kKdChunk * 36;    // [32]
   float* s_one = s_beta + 3 * kKdChunk;  // [DP] ones
   float2* s_f = reinterpret_cast<float2*>(s_beta + kKdChunk);      // [32] what makes q and k unit vectors
-  float* s_pre = s_one + DP;             // [4][DP] decays of the blocks before one, and behind it
+  float* s_part = s_one + DP;            // [4][6][16][8] shares of the products between blocks
+  float* s_pre = s_part;                 // [4][DP] then the decays of the blocks before one, and behind it
   float* s_suf = s_pre + kKdBlocks * DP;
-  float* s_part = s_suf + kKdBlocks * DP;                          // [8][6][16][8] shares of the products between blocks
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int c = blockIdx.x, h = blockIdx.y, s = blockIdx.z, qh = h / p.group, D = p.dim, E = p.vdim;
   const int t0 = c * kKdChunk, nt = min(kKdChunk, p.T - t0);
@@ -173,45 +173,44 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
     for (int i = tid; i < kKdBlocks * DH; i += kKdThreads) {
       const int d = i % DH * 2, o = i / DH * kKdBlock, first = t0 + o - (kKdTaps - 1);
       constexpr int N = kKdBlock + kKdTaps - 1;
-      float2 x[2][N];
       const bool inside = d < D && first >= 0 && first + N <= p.T;
-#pragma unroll
+#pragma unroll 1
       for (int m = 0; m < 2; m++) {
+        float2 x[N];
         const int col = (m ? p.k_off : p.q_off) + qh * D + d, ch = (m ? p.qk_heads * D : 0) + qh * D + d;
         const T* src = base + (long long)first * p.ld + col;
         if (inside) {
 #pragma unroll
-          for (int j = 0; j < N; j++, src += p.ld) x[m][j] = kd_pair<T>(src);
+          for (int j = 0; j < N; j++, src += p.ld) x[j] = kd_pair<T>(src);
         } else {
 #pragma unroll
           for (int j = 0; j < N; j++) {
             const int t = first + j;
-            x[m][j] = make_float2(0.f, 0.f);
+            x[j] = make_float2(0.f, 0.f);
             if (d >= D || t >= p.T || (t < 0 && -t >= p.taps)) continue;
-            x[m][j] = t >= 0 ? kd_pair<T>(src + (long long)j * p.ld) : make_float2(kd_raw<T>(p, base, ring, pos, t, col, ch), kd_raw<T>(p, base, ring, pos, t, col + 1, ch + 1));
+            x[j] = t >= 0 ? kd_pair<T>(src + (long long)j * p.ld) : make_float2(kd_raw<T>(p, base, ring, pos, t, col, ch), kd_raw<T>(p, base, ring, pos, t, col + 1, ch + 1));
           }
         }
-      }
-#pragma unroll
-      for (int m = 0; m < 2; m++) {
         float* dst = (m ? sk : sq) + o * P + d;
         if (p.taps) {
           float w0[kKdTaps], w1[kKdTaps];
-          const int ch = (m ? p.qk_heads * D : 0) + qh * D + min(d, D - 2);
-          kd_taps(p, ch, w0);
-          kd_taps(p, ch + 1, w1);
+          const int wch = ch - d + min(d, D - 2);
+          kd_taps(p, wch, w0);
+          kd_taps(p, wch + 1, w1);
 #pragma unroll
           for (int j = 0; j < kKdBlock; j++) {
-            float2 y = make_float2(0.f, 0.f);
+            uint64_t sum = 0ull;
 #pragma unroll
-            for (int n = 0; n < kKdTaps; n++) { y.x = fmaf(w0[n], x[m][j + n].x, y.x); y.y = fmaf(w1[n], x[m][j + n].y, y.y); }
+            for (int n = 0; n < kKdTaps; n++) sum = fma_f32x2(pack_f32x2(w0[n], w1[n]), pack_f32x2(x[j + n].x, x[j + n].y), sum);
+            float2 y;
+            unpack_f32x2(sum, y.x, y.y);
             *reinterpret_cast<float2*>(dst + j * P) = make_float2(kd_silu_fast(y.x), kd_silu_fast(y.y));      // channels past D are zero already
           }
           if (o + kKdBlock > nt)                         // tokens past the end are not
             for (int j = max(0, nt - o); j < kKdBlock; j++) *reinterpret_cast<float2*>(dst + j * P) = make_float2(0.f, 0.f);
         } else {
 #pragma unroll
-          for (int j = 0; j < kKdBlock; j++) *reinterpret_cast<float2*>(dst + j * P) = x[m][j + kKdTaps - 1];
+          for (int j = 0; j < kKdBlock; j++) *reinterpret_cast<float2*>(dst + j * P) = x[j + kKdTaps - 1];
         }
       }
     }
@@ -317,15 +316,9 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
     for (int j = kKdBlock - 1; j >= 0; j--) { a[j * P] = kk[j] * f; f *= aa[j]; }
   }
   __syncthreads();
-  if (tid < DP) {                        // a chunk's decays across blocks
-    const float f0 = sb[tid], f1 = sb[DP + tid], f2 = sb[2 * DP + tid], f3 = sb[3 * DP + tid];
-    s_pre[tid] = 1.f; s_pre[DP + tid] = f0; s_pre[2 * DP + tid] = f0 * f1; s_pre[3 * DP + tid] = f0 * f1 * f2;
-    s_suf[tid] = f1 * f2 * f3; s_suf[DP + tid] = f2 * f3; s_suf[2 * DP + tid] = f3; s_suf[3 * DP + tid] = 1.f;
-    reinterpret_cast<float*>(ops + L.decay)[tid] = f0 * f1 * f2 * f3;
-  }
-  // pairs of different blocks, queries of block b with keys of block a < b: rows 0 .. 7 of a product are q, rows 8 .. 15 k. A warp takes
-  // every eighth 16 channels of all six.
-  constexpr int kShares = DP / 16 < 8 ? DP / 16 : 8;
+  // pairs of different blocks, queries of block b with keys of block a < b: rows 0 .. 7 of a product are q, rows 8 .. 15 k. Four warps
+  // take every fourth 16 channels of all six.
+  constexpr int kShares = DP / 16 < 4 ? DP / 16 : 4;
   if (warp < kShares) {
     const int g = lane >> 2, q = lane & 3;
     float acc[6][4];
@@ -383,6 +376,13 @@ __global__ void __launch_bounds__(kKdThreads, 2) key_decay_prepare_kernel(const 
     const int b = pair < 1 ? 1 : pair < 3 ? 2 : 3, a = pair - b * (b - 1) / 2, row = b * kKdBlock + (r & 7), col = a * kKdBlock + j;
     if (r < 8) sQ[row * 36 + col] = v;
     else if constexpr (DELTA) sK[row * 36 + col] = v * s_beta[row];
+  }
+  __syncthreads();
+  if (tid < DP) {                        // a chunk's decays across blocks
+    const float f0 = sb[tid], f1 = sb[DP + tid], f2 = sb[2 * DP + tid], f3 = sb[3 * DP + tid];
+    s_pre[tid] = 1.f; s_pre[DP + tid] = f0; s_pre[2 * DP + tid] = f0 * f1; s_pre[3 * DP + tid] = f0 * f1 * f2;
+    s_suf[tid] = f1 * f2 * f3; s_suf[DP + tid] = f2 * f3; s_suf[2 * DP + tid] = f3; s_suf[3 * DP + tid] = 1.f;
+    reinterpret_cast<float*>(ops + L.decay)[tid] = f0 * f1 * f2 * f3;
   }
   __syncthreads();
   const auto store_q = [&](int i, int j) {               // four entries of Q
@@ -1089,7 +1089,7 @@ __global__ void __launch_bounds__(256) key_decay_finish_kernel(const KdParams p)
 template <typename T, int DP, bool DELTA>
 static cudaError_t launch_kd(cudaStream_t s, const KdParams& p) {
   constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
-  constexpr size_t prep = ((size_t)3 * kKdChunk * (DP + 4) + kKdBlocks * DP + 2 * kKdChunk * 36 + 3 * kKdChunk + DP + 2 * kKdBlocks * DP + 8 * 768) * sizeof(float);
+  constexpr size_t prep = ((size_t)3 * kKdChunk * (DP + 4) + kKdBlocks * DP + 2 * kKdChunk * 36 + 3 * kKdChunk + DP + (2 * kKdBlocks * DP > 4 * 768 ? 2 * kKdBlocks * DP : 4 * 768)) * sizeof(float);
   constexpr size_t scan = kd_tc(DP) ? kd_stages(DELTA) * (size_t)L.stride + 1024 : 2 * (size_t)L.stride;
   static bool attr = false;
   if (!attr) {
