@@ -34,12 +34,13 @@ constexpr int kKdThreads = 256, kKdBlock = 8, kKdBlocks = kKdChunk / kKdBlock;
 
 template <typename T>
 __device__ __forceinline__ void kd_split(float x, T& hi, T& lo) { hi = Cvt<T>::from(x); lo = Cvt<T>::from(x - Cvt<T>::to(hi)); }
-template <typename T>
+// PACKED: the remainders of the pair in one operation (which form the register allocation favours differs by kernel)
+template <typename T, bool PACKED = false>
 __device__ __forceinline__ void kd_split2(float x, float y, uint32_t& hi, uint32_t& lo) {
   hi = pack2_t<T>(x, y);
   const T* v = reinterpret_cast<const T*>(&hi);
-  float a, b;
-  unpack_f32x2(fma_f32x2(pack_f32x2(Cvt<T>::to(v[0]), Cvt<T>::to(v[1])), pack_f32x2(-1.0f, -1.0f), pack_f32x2(x, y)), a, b);
+  float a = x - Cvt<T>::to(v[0]), b = y - Cvt<T>::to(v[1]);
+  if constexpr (PACKED) unpack_f32x2(fma_f32x2(pack_f32x2(Cvt<T>::to(v[0]), Cvt<T>::to(v[1])), pack_f32x2(-1.0f, -1.0f), pack_f32x2(x, y)), a, b);
   lo = pack2_t<T>(a, b);
 }
 
@@ -679,10 +680,10 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
   using namespace sm100;
   constexpr KdOpsLayout L = kd_ops_layout(DP, DELTA);
   constexpr uint32_t cS = 0, cA = 128, cO = 256, cR = cA + 64, cU = 64, kLo = L.rows1;      // cU: within a buffer; kLo: from a product to its remainder's
-  constexpr int kSteps = DP / 16, kFirst = DELTA ? (kSteps + 1) / 4 * 2 : 0;      // steps of 16 channels; those whose products start ahead of the others
+  constexpr int kSteps = DP / 16;
   extern __shared__ uint8_t smem_raw[];
   constexpr int kStages = kd_stages(DELTA);
-  __shared__ uint64_t full[kStages], empty[kStages], s_first, s_ready, r_ready, u_ready, x_full, u_full, s_full, o_full[2], o_free[2], sums;
+  __shared__ uint64_t full[kStages], empty[kStages], s_ready, r_ready, u_ready, x_full, u_full, s_full, o_full[2], o_free[2], sums;
   __shared__ uint32_t tmem_slot;
   __shared__ float s_sum[2][4][kKdChunk];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -693,7 +694,7 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
     for (int i = 0; i < kStages; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], kKdStateWarps + 1); }
     for (int i = 0; i < 2; i++) { mbar_init(&o_full[i], 1); mbar_init(&o_free[i], 4); }
     mbar_init(&sums, 4);
-    mbar_init(&s_first, kKdStateWarps); mbar_init(&s_ready, kKdStateWarps); mbar_init(&r_ready, kKdStateWarps); mbar_init(&u_ready, kKdStateWarps);
+    mbar_init(&s_ready, kKdStateWarps); mbar_init(&r_ready, kKdStateWarps); mbar_init(&u_ready, kKdStateWarps);
     mbar_init(&x_full, 1); mbar_init(&u_full, 1); mbar_init(&s_full, 1);
     mbar_fence_init();
   }
@@ -743,16 +744,10 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
           mma_commit(&s_full);
         };
         if constexpr (DELTA) {
-          if constexpr (kFirst > 0) {
-            if (!mbar_wait(&s_first, ph, status, 64)) break;
-            tc_fence_after_sync();
-#pragma unroll
-            for (int k = 0; k < kFirst; k++) rows_product(k);
-          }
           if (!mbar_wait(&s_ready, ph, status, 64)) break;
           tc_fence_after_sync();
 #pragma unroll
-          for (int k = kFirst; k < kSteps; k++) rows_product(k);
+          for (int k = 0; k < kSteps; k++) rows_product(k);
           mma_commit(&x_full);
           if (!mbar_wait(&r_ready, ph, status, 65)) break;
           tc_fence_after_sync();
@@ -807,7 +802,7 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
     auto split = [&](const float (&v)[16], uint32_t at, uint32_t lo_off) {
       uint32_t hi[8], lo[8];
 #pragma unroll
-      for (int i = 0; i < 8; i++) kd_split2<T>(v[2 * i], v[2 * i + 1], hi[i], lo[i]);
+      for (int i = 0; i < 8; i++) kd_split2<T, !DELTA>(v[2 * i], v[2 * i + 1], hi[i], lo[i]);
       tmem_st_32x8(at, hi);
       tmem_st_32x8(at + lo_off, lo);
     };
@@ -874,7 +869,7 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
         if (!ok) break;
         tc_fence_after_sync();
       }
-#pragma unroll
+#pragma unroll(DELTA ? 1 : 8)
       for (int n = 0; n < (G + 1) / 2; n++) {
         const int g = 2 * n + half;
         if (G % 2 && g >= G) break;
@@ -887,11 +882,15 @@ __global__ void __launch_bounds__(kKdScanThreads, 1) key_decay_scan_tc_kernel(co
 #pragma unroll
         for (int i = 0; i < 4; i++) {
           const float4 f = decay[g * 4 + i];
-          const uint64_t a = mul_f32x2(pack_f32x2(y[4 * i], y[4 * i + 1]), pack_f32x2(f.x, f.y)), b = mul_f32x2(pack_f32x2(y[4 * i + 2], y[4 * i + 3]), pack_f32x2(f.z, f.w));
-          x[4 * i] = (uint32_t)a; x[4 * i + 1] = (uint32_t)(a >> 32); x[4 * i + 2] = (uint32_t)b; x[4 * i + 3] = (uint32_t)(b >> 32);
+          if constexpr (DELTA) {
+            x[4 * i] = __float_as_uint(y[4 * i] * f.x); x[4 * i + 1] = __float_as_uint(y[4 * i + 1] * f.y);
+            x[4 * i + 2] = __float_as_uint(y[4 * i + 2] * f.z); x[4 * i + 3] = __float_as_uint(y[4 * i + 3] * f.w);
+          } else {
+            const uint64_t a = mul_f32x2(pack_f32x2(y[4 * i], y[4 * i + 1]), pack_f32x2(f.x, f.y)), b = mul_f32x2(pack_f32x2(y[4 * i + 2], y[4 * i + 3]), pack_f32x2(f.z, f.w));
+            x[4 * i] = (uint32_t)a; x[4 * i + 1] = (uint32_t)(a >> 32); x[4 * i + 2] = (uint32_t)b; x[4 * i + 3] = (uint32_t)(b >> 32);
+          }
         }
         tmem_st_32x16(lanes + cS + (uint32_t)(g * 16), x);
-        if (kFirst > 0 && 2 * n + 2 == kFirst) arrive(&s_first);
       }
       if constexpr (!DELTA) {
         values();
