@@ -3,7 +3,7 @@
 // A CTA works on up to 128 value columns of one head of one sequence (a cluster where a head has more: the head's norm adds their
 // sums of squares over distributed shared memory). With r = (diag(a) S)^T k and p = (diag(a) S)^T q taken in one pass over S, the
 // rest of a token is u = beta (v - r) (or v), o = p + (k . q) u and the update S <- diag(a) S + k u^T, which is the order of the
-// recurrence: the read-out sees the current token's write. S stays in registers from token to token where the CTA's columns fit.
+// recurrence (o includes what the token itself wrote). S stays in registers from token to token where the CTA's columns fit.
 #include "key_decay.cuh"
 #include "sm100.cuh"
 #include <algorithm>
